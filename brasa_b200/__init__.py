@@ -5,7 +5,7 @@ The classes mirror the reference's Rust interfaces so that tests read like the r
   Context, Buffer, Command          crates/metal/src/runtime.rs
   Kernels, QMatrix, AttnShape,
   KvType, WeightType, RopeTable     crates/kernels/src/lib.rs
-  Qwen3, Limits, Config             crates/models/src/qwen3.rs
+  Model, Qwen3, Limits, Config      crates/models/src/qwen3.rs (Model: any family; MODELS is the registry)
   Session, SamplingParams, GenStats crates/runtime/src/{session,sampler}.rs
   planner                           crates/memory/src/planner.rs
 
@@ -52,9 +52,10 @@ class KvType(enum.IntEnum):
     F32 = 0
     F16 = 1
     Q8_0 = 2
+    BF16 = 3  # layer-stack families: bf16 products and caches (F32: everything in 32-bit)
 
     def block_bytes(self) -> int:
-        return {KvType.F32: 128, KvType.F16: 64, KvType.Q8_0: 34}[self]
+        return {KvType.F32: 128, KvType.F16: 64, KvType.Q8_0: 34, KvType.BF16: 64}[self]
 
     def bytes(self, n: int) -> int:
         if self == KvType.Q8_0:
@@ -64,7 +65,7 @@ class KvType(enum.IntEnum):
 
     @staticmethod
     def parse(s: str) -> "KvType | None":
-        return {"f32": KvType.F32, "f16": KvType.F16, "q8_0": KvType.Q8_0, "q8": KvType.Q8_0}.get(s)
+        return {"f32": KvType.F32, "f16": KvType.F16, "q8_0": KvType.Q8_0, "q8": KvType.Q8_0, "bf16": KvType.BF16}.get(s)
 
 
 class PrefillPrecision(enum.IntEnum):
@@ -671,6 +672,16 @@ class planner:
         return {n: getattr(p, n) for n, _ in _MemoryPlan._fields_}
 
     @staticmethod
+    def check_path(ctx: Context | None, path, limits: Limits, budget: int = 0) -> tuple[bool, dict, int]:
+        """(fits, plan, largest context that fits) of a session over the model at `path`, any family."""
+        p, mx = _MemoryPlan(), C.c_uint32()
+        s = _SessionShape(limits.ctx, limits.max_tokens, limits.max_logit_rows, int(limits.kv))
+        rc = lib().brasa_plan_file(ctx._h if ctx else None, str(path).encode(), C.byref(s), C.c_uint64(budget), C.byref(p), C.byref(mx))
+        if rc not in (0, EBUDGET):
+            raise BrasaError(rc, lib().brasa_last_error(ctx._h).decode(errors="replace") if ctx else "plan_file")
+        return rc == 0, {n: getattr(p, n) for n, _ in _MemoryPlan._fields_}, mx.value
+
+    @staticmethod
     def check(ctx: Context | None, shape: _ModelShape, limits: Limits, budget: int = 0) -> tuple[bool, dict, int]:
         """(fits, plan, largest context that fits)."""
         p, mx = _MemoryPlan(), C.c_uint32()
@@ -704,8 +715,9 @@ class planner:
         return n.value, pages.value, {k: getattr(p, k) for k, _ in _BatchPlan._fields_}
 
 
-class Qwen3:
-    """Model on the device with its KV cache and workspace (crates/models/src/qwen3.rs:301 Qwen3)."""
+class Model:
+    """A model on the device with its cache or state and its workspace, whatever its family
+    (crates/models/src/qwen3.rs:301 Qwen3)."""
 
     def __init__(self, ctx: Context, path, limits: Limits, _handle=None):
         self.ctx = ctx
@@ -720,26 +732,27 @@ class Qwen3:
         self.limits = Limits(l.ctx, l.max_tokens, l.max_logit_rows, KvType(l.kv))
 
     @classmethod
-    def load(cls, ctx: Context, path, limits: Limits) -> "Qwen3":
+    def load(cls, ctx: Context, path, limits: Limits) -> "Model":
         return cls(ctx, path, limits)
+
+    @classmethod
+    def load_in(cls, ctx: Context, path, dtype: str, ctx_len: int, max_tokens: int, max_logit_rows: int = 1) -> "Model":
+        """Loads with the cache type and product precision the family serves `dtype` ("bfloat16" or "float32") with."""
+        return cls(ctx, path, Limits(ctx=ctx_len, max_tokens=max_tokens, max_logit_rows=max_logit_rows, kv=cls.kv_type(dtype)))
+
+    @classmethod
+    def kv_type(cls, dtype: str) -> KvType:
+        raise NotImplementedError
 
     def free(self):
         if self._own and self._h and self.ctx._h:
             lib().brasa_model_free(self._h)
         self._h = C.c_void_p()
 
-    def set_tp(self, tp) -> None:
-        """Attaches a tensor-parallel exchange (brasa_b200.tp.TensorParallel) to this shard, before its first step."""
-        self.ctx._check(lib().brasa_model_set_tp(self._h, tp._h))
-        self._tp = tp
-
     def allocated(self) -> dict:
         a = _Allocated()
         self.ctx._check(lib().brasa_model_allocated(self._h, C.byref(a)))
         return {"weights": a.weights, "kv": a.kv, "workspace": a.workspace}
-
-    def set_prefill_precision(self, p: PrefillPrecision):
-        self.ctx._check(lib().brasa_model_set_prefill_precision(self._h, C.c_int32(int(p))))
 
     def forward(self, ids, pos0: int, logit_rows: int = 1, want_logits: bool = True):
         """Returns (logits [logit_rows, vocab] or None, device seconds); a tensor-parallel shard returns its own
@@ -751,6 +764,28 @@ class Qwen3:
                                                   C.c_uint32(logit_rows), logits.ctypes.data_as(C.c_void_p) if want_logits else None,
                                                   C.byref(secs)))
         return logits, secs.value
+
+    def forward_rows(self, ids, pos0: int, rows):
+        """One run of tokens; logits [len(rows), vocab] of the given places among them."""
+        ids, rows = np.ascontiguousarray(ids, dtype=np.uint32), np.ascontiguousarray(rows, dtype=np.uint32)
+        logits = np.empty((rows.size, self.cfg["head_rows"]), np.float32)
+        secs = C.c_double()
+        self.ctx._check(lib().brasa_model_forward_rows(self._h, ids.ctypes.data_as(C.c_void_p), C.c_uint32(ids.size), C.c_uint32(pos0),
+                                                       rows.ctypes.data_as(C.c_void_p), C.c_uint32(rows.size), logits.ctypes.data_as(C.c_void_p),
+                                                       C.byref(secs)))
+        return logits
+
+    def feed(self, ids, pos0: int, rows):
+        """forward_rows for any number of tokens and rows, in runs of at most max_tokens tokens and max_logit_rows rows."""
+        ids, rows, out, at = np.asarray(ids, np.uint32), sorted(int(r) for r in rows), [], 0
+        while at < ids.size:
+            n = min(self.limits.max_tokens, ids.size - at)
+            here = [r for r in rows if at <= r < at + n]
+            if len(here) > self.limits.max_logit_rows:
+                n, here = here[self.limits.max_logit_rows] - at, here[:self.limits.max_logit_rows]
+            out.append(self.forward_rows(ids[at:at + n], pos0 + at, [r - at for r in here]))
+            at += n
+        return np.concatenate(out) if out else np.empty((0, self.cfg["head_rows"]), np.float32)
 
     def run_layers(self, x, pos0: int, layers: range) -> np.ndarray:
         x = np.ascontiguousarray(x, dtype=np.float32).copy()
@@ -773,6 +808,28 @@ class Qwen3:
         self.ctx._check(lib().brasa_model_load_stats(self._h, C.byref(s), C.byref(n)))
         return {"seconds": s.value, "bytes": int(n.value), "gb_per_s": n.value / s.value / 1e9 if s.value > 0 else None}
 
+
+class Qwen3(Model):
+    """Qwen3 dense over `.brasa` weights (crates/models/src/qwen3.rs:301 Qwen3)."""
+
+    @classmethod
+    def load_in(cls, ctx, path, dtype, ctx_len, max_tokens, max_logit_rows=1):
+        m = super().load_in(ctx, path, dtype, ctx_len, max_tokens, max_logit_rows)
+        m.set_prefill_precision(PrefillPrecision.F32 if dtype == "float32" else PrefillPrecision.F16)
+        return m
+
+    @classmethod
+    def kv_type(cls, dtype):
+        return {"float32": KvType.F32, "bfloat16": KvType.F16}[dtype]
+
+    def set_tp(self, tp) -> None:
+        """Attaches a tensor-parallel exchange (brasa_b200.tp.TensorParallel) to this shard, before its first step."""
+        self.ctx._check(lib().brasa_model_set_tp(self._h, tp._h))
+        self._tp = tp
+
+    def set_prefill_precision(self, p: PrefillPrecision):
+        self.ctx._check(lib().brasa_model_set_prefill_precision(self._h, C.c_int32(int(p))))
+
     def read_kv(self, layer: int, which: str, pos_begin: int, pos_end: int) -> np.ndarray:
         kvd = self.cfg["kv_heads"] * self.cfg["head_dim"]
         n = self.limits.kv.bytes((pos_end - pos_begin) * kvd)
@@ -780,6 +837,27 @@ class Qwen3:
         self.ctx._check(lib().brasa_model_read_kv(self._h, C.c_uint32(layer), C.c_int32(1 if which == "v" else 0), C.c_uint32(pos_begin),
                                                   C.c_uint32(pos_end), out.ctypes.data_as(C.c_void_p), C.c_uint64(n)))
         return out
+
+
+class Dunuzen(Model):
+    """Layers of latent attention in a sliding window and of the gated delta rule, each beside a feed-forward, over bf16
+    safetensors. Its state goes forward only: a run starts at position 0 or where the one before it ended."""
+
+    @classmethod
+    def kv_type(cls, dtype):
+        return {"float32": KvType.F32, "bfloat16": KvType.BF16}[dtype]
+
+
+MODELS = {"qwen3": Qwen3, "Dunuzen": Dunuzen}
+
+
+def model_class(path) -> type[Model]:
+    """The class of the model at `path` (a `.brasa` file, or a folder with config.json and model.safetensors)."""
+    name = C.create_string_buffer(512)
+    rc = lib().brasa_model_family(str(path).encode(), name, C.c_uint64(512))
+    if rc != 0:
+        raise BrasaError(rc, name.value.decode(errors="replace"))
+    return MODELS[name.value.decode()]
 
 
 _STOP = {0: "Stop", 1: "MaxTokens", 2: "ContextFull", 3: "Cancelled"}
@@ -792,7 +870,7 @@ class Session:
         self.ctx = ctx
         self._h = C.c_void_p()
         ctx._check(lib().brasa_session_create(ctx._h, str(path).encode(), limits._c(), C.c_uint64(budget), C.byref(self._h)))
-        self.model = Qwen3(ctx, path, limits, _handle=lib().brasa_session_model(self._h))
+        self.model = model_class(path)(ctx, path, limits, _handle=lib().brasa_session_model(self._h))
 
     @classmethod
     def load_with_budget(cls, ctx, path, limits, budget) -> "Session":

@@ -852,6 +852,7 @@ void brasa_batch_free(brasa_batch *b) {
 int32_t brasa_batch_create(brasa_model *m, uint32_t max_seqs, uint32_t num_pages, uint32_t max_positions, brasa_batch **out) {
     if (!m || !out) return BRASA_EINVAL;
     brasa_ctx *ctx = m->ctx;
+    BRASA_REQUIRE(ctx, !m->stack, "batch: the %s family decodes one sequence at a time", m->family->name);
     BRASA_REQUIRE(ctx, max_seqs >= 1 && max_seqs <= m->limits.max_tokens, "batch: 1 to max_tokens (%u) sequences", m->limits.max_tokens);
     BRASA_REQUIRE(ctx, m->cfg.head_dim == 128 && m->cfg.heads % m->cfg.kv_heads == 0 && m->cfg.heads / m->cfg.kv_heads <= 8,
                   "batch: head_dim 128 and a GQA group of at most 8");

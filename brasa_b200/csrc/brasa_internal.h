@@ -156,6 +156,13 @@ static inline bool qm_fits(const brasa_qmatrix &m) {
 }
 
 int32_t brasa_post_launch(brasa_cmd *cmd, const char *name);
+
+// ops.cu. out[i] = layer norm of row x[rows ? rows[r] : r] times w[i] plus b[i], i < n_out (1 or 2), [n_rows][ldo] in f32 or bf16
+int32_t brasa_layer_norm_launch(brasa_cmd *cmd, const float *x, const uint32_t *rows, uint32_t n_rows, uint32_t n, float eps, const float *const *w,
+                                const float *const *b, void *const *out, uint32_t n_out, uint32_t ldo, bool f32);
+// out[t, :] = scale * table[ids[t], :] for a bf16 table
+int32_t brasa_embed_bf16_launch(brasa_cmd *cmd, const uint16_t *table, uint32_t ld, uint32_t rows, uint32_t n, float scale, const uint32_t *ids, float *out,
+                                uint32_t tokens);
 // Makes sure the context's split-K scratch holds at least this many floats / counters.
 int32_t brasa_gemv_scratch(brasa_ctx *ctx, size_t partial_floats, size_t counters);
 

@@ -317,7 +317,8 @@ int32_t brasa_gqa_supported(uint32_t hq, uint32_t hkv) {
 uint64_t brasa_kv_bytes(int32_t kv, uint64_t n) {
     switch (kv) {
     case BRASA_KV_F32: return n * 4;
-    case BRASA_KV_F16: return n * 2;
+    case BRASA_KV_F16:
+    case BRASA_KV_BF16: return n * 2;
     case BRASA_KV_Q8_0: return n / BRASA_KV_Q8_DIM * BRASA_KV_Q8_ROW;
     default: return 0;
     }
@@ -366,12 +367,6 @@ int32_t brasa_gemv_scratch(brasa_ctx *ctx, size_t partial_floats, size_t counter
     if (counters > ctx->gemv_counters_n) {
         BRASA_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
         cudaFree(ctx->gemv_counters);
-    cudaFree(ctx->argmax_scratch);
-    cudaFree(ctx->gemm_part);
-    cudaFree(ctx->kv_expand);
-    cudaFree(ctx->gemm_counters);
-    cudaFree(ctx->sample_scratch);
-    cudaFree(ctx->gemv_trace);
         ctx->gemv_counters = nullptr;
         ctx->gemv_counters_n = 0;
         BRASA_CUDA(ctx, cudaMalloc(&ctx->gemv_counters, counters * sizeof(uint32_t)));

@@ -224,9 +224,72 @@ uint64_t dtype_nbytes(const std::string &d, uint64_t n) {
     return q < 0 ? 0 : brasa_qtype_nbytes(q, n);
 }
 
-BrasaFile::~BrasaFile() {
+WeightFile::~WeightFile() {
     if (map_) munmap((void *)map_, size_);
     if (fd_ >= 0) close(fd_);
+}
+
+bool WeightFile::map_file(const std::string &path, std::string &err) {
+    fd_ = ::open(path.c_str(), O_RDONLY);
+    if (fd_ < 0) return err = path + ": cannot open", false;
+    struct stat st;
+    if (fstat(fd_, &st) != 0) return err = path + ": cannot stat", false;
+    size_ = (size_t)st.st_size;
+    if (size_ == 0) return err = path + ": empty file", false;
+    void *m = mmap(nullptr, size_, PROT_READ, MAP_PRIVATE, fd_, 0);
+    if (m == MAP_FAILED) return err = path + ": mmap failed", false;
+    map_ = (const uint8_t *)m;
+    return true;
+}
+
+std::unique_ptr<WeightFile> WeightFile::open_any(const std::string &path, std::string &err) {
+    struct stat st;
+    if (stat(path.c_str(), &st) == 0 && S_ISDIR(st.st_mode)) return SafeTensorsFolder::open(path, err);
+    return BrasaFile::open(path, err);
+}
+
+std::unique_ptr<SafeTensorsFolder> SafeTensorsFolder::open(const std::string &folder, std::string &err) {
+    std::unique_ptr<SafeTensorsFolder> f(new SafeTensorsFolder());
+    auto bad = [&](const std::string &m) {
+        err = folder + ": " + m;
+        return std::unique_ptr<SafeTensorsFolder>();
+    };
+    std::string text;
+    {
+        FILE *c = fopen((folder + "/config.json").c_str(), "rb");
+        if (!c) return bad("no config.json");
+        char buf[4096];
+        for (size_t n; (n = fread(buf, 1, sizeof buf, c)) > 0;) text.append(buf, n);
+        fclose(c);
+    }
+    std::string jerr;
+    if (!json_parse(text.data(), text.size(), f->config_json_, jerr)) return bad("config.json: " + jerr);
+    const Json *arch = f->config_json_.get("architecture");
+    if (!arch || arch->kind != Json::Str) return bad("config.json: no architecture");
+    f->config_ = &f->config_json_;
+    f->family_ = arch->str;
+    if (!f->map_file(folder + "/model.safetensors", err)) return nullptr;
+    uint64_t hlen = 0;
+    if (f->size_ < 8) return bad("model.safetensors: truncated");
+    memcpy(&hlen, f->map_, 8);
+    if (hlen > f->size_ - 8) return bad("model.safetensors: truncated header");
+    if (!json_parse((const char *)f->map_ + 8, (size_t)hlen, f->meta_, jerr) || f->meta_.kind != Json::Obj) return bad("model.safetensors: header: " + jerr);
+    for (auto &kv : f->meta_.obj) {
+        if (kv.first == "__metadata__") continue;
+        TensorInfo ti;
+        const Json *d = kv.second.get("dtype"), *s = kv.second.get("shape"), *o = kv.second.get("data_offsets");
+        if (!d || d->kind != Json::Str || !s || s->kind != Json::Arr || !o || o->kind != Json::Arr || o->arr.size() != 2) return bad(kv.first + ": bad header entry");
+        ti.name = kv.first;
+        ti.dtype = d->str == "BF16" ? "bf16" : (d->str == "F32" ? "f32" : (d->str == "I32" ? "i32" : ""));
+        if (ti.dtype.empty()) return bad(ti.name + ": unknown dtype " + d->str);
+        for (const Json &e : s->arr) ti.shape.push_back((uint64_t)e.inum);
+        const uint64_t at = (uint64_t)o->arr[0].inum, end = (uint64_t)o->arr[1].inum, room = f->size_ - 8 - hlen;
+        if (at > end || end > room || end - at != ti.numel() * (ti.dtype == "bf16" ? 2 : 4)) return bad(ti.name + ": outside the file");
+        ti.offset = 8 + hlen + at;
+        ti.nbytes = end - at;
+        f->tensors_.push_back(std::move(ti));
+    }
+    return f;
 }
 
 std::unique_ptr<BrasaFile> BrasaFile::open(const std::string &path, std::string &err) {
@@ -235,15 +298,8 @@ std::unique_ptr<BrasaFile> BrasaFile::open(const std::string &path, std::string 
         return std::unique_ptr<BrasaFile>();
     };
     std::unique_ptr<BrasaFile> f(new BrasaFile());
-    f->fd_ = ::open(path.c_str(), O_RDONLY);
-    if (f->fd_ < 0) return bad("cannot open");
-    struct stat st;
-    if (fstat(f->fd_, &st) != 0) return bad("cannot stat");
-    f->size_ = (size_t)st.st_size;
+    if (!f->map_file(path, err)) return nullptr;
     if (f->size_ < 16) return bad("not a .brasa file");
-    void *m = mmap(nullptr, f->size_, PROT_READ, MAP_PRIVATE, f->fd_, 0);
-    if (m == MAP_FAILED) return bad("mmap failed");
-    f->map_ = (const uint8_t *)m;
     const uint8_t *b = f->map_;
     if (memcmp(b, "BRSA", 4) != 0) return bad("not a .brasa file");
     uint32_t version;
@@ -288,7 +344,7 @@ std::unique_ptr<BrasaFile> BrasaFile::open(const std::string &path, std::string 
     return f;
 }
 
-const TensorInfo *BrasaFile::tensor(const std::string &name) const {
+const TensorInfo *WeightFile::tensor(const std::string &name) const {
     for (auto &t : tensors_)
         if (t.name == name) return &t;
     return nullptr;
@@ -437,35 +493,7 @@ int32_t brasa_plan(const brasa_model_shape *m, const brasa_session_shape *s, bra
 int32_t brasa_plan_check(brasa_ctx *ctx, const brasa_model_shape *m, const brasa_session_shape *s, uint64_t budget, brasa_memory_plan *out,
                          uint32_t *max_ctx_out) {
     if (!m || !s) return BRASA_EINVAL;
-    brasa_memory_plan plan;
-    BRASA_TRY(brasa_plan(m, s, &plan));
-    if (out) *out = plan;
-    if (budget == 0) {
-        if (!ctx) return BRASA_EINVAL;
-        uint64_t free_b = 0, total_b = 0;
-        BRASA_TRY(brasa_ctx_mem_info(ctx, &free_b, &total_b));
-        uint64_t reserve = 512ull << 20;
-        budget = free_b > reserve ? free_b - reserve : 0;
-        budget += plan.overhead;  // the context is already paid for inside `free`
-    }
-    if (max_ctx_out) *max_ctx_out = s->ctx;
-    if (plan.total <= budget) return BRASA_OK;
-    // largest context that fits: the plan grows monotonically with ctx
-    uint32_t lo = 0, hi = s->ctx;
-    while (lo < hi) {
-        uint32_t mid = lo + (hi - lo + 1) / 2;
-        brasa_session_shape t = *s;
-        t.ctx = mid;
-        if (t.max_tokens > mid) t.max_tokens = mid;
-        brasa_memory_plan p;
-        brasa_plan(m, &t, &p);
-        if (p.total <= budget) lo = mid;
-        else hi = mid - 1;
-    }
-    if (max_ctx_out) *max_ctx_out = lo;
-    return brasa_fail(ctx, BRASA_EBUDGET, "the model needs %.2f GiB (weights %.2f, KV %.2f, workspace %.2f, overhead %.2f) and the budget is %.2f GiB; the largest context that fits is %u",
-                      plan.total / 1073741824.0, plan.weights / 1073741824.0, plan.kv / 1073741824.0, plan.workspace / 1073741824.0,
-                      plan.overhead / 1073741824.0, budget / 1073741824.0, lo);
+    return brasa_plan_check_with(ctx, *s, budget, out, max_ctx_out, [m](const brasa_session_shape &t, brasa_memory_plan *p) { return brasa_plan(m, &t, p); });
 }
 
 int32_t brasa_file_check(const char *path, int32_t verify, char *err, uint64_t err_len) {
@@ -481,3 +509,36 @@ int32_t brasa_file_check(const char *path, int32_t verify, char *err, uint64_t e
 }
 
 }  // extern "C"
+
+int32_t brasa_plan_check_with(brasa_ctx *ctx, const brasa_session_shape &s, uint64_t budget, brasa_memory_plan *out, uint32_t *max_ctx_out,
+                              const std::function<int32_t(const brasa_session_shape &, brasa_memory_plan *)> &plan_of) {
+    brasa_memory_plan plan;
+    BRASA_TRY(plan_of(s, &plan));
+    if (out) *out = plan;
+    if (budget == 0) {
+        if (!ctx) return BRASA_EINVAL;
+        uint64_t free_b = 0, total_b = 0;
+        BRASA_TRY(brasa_ctx_mem_info(ctx, &free_b, &total_b));
+        uint64_t reserve = 512ull << 20;
+        budget = free_b > reserve ? free_b - reserve : 0;
+        budget += plan.overhead;  // the context is already paid for inside `free`
+    }
+    if (max_ctx_out) *max_ctx_out = s.ctx;
+    if (plan.total <= budget) return BRASA_OK;
+    // largest context that fits: the plan grows monotonically with ctx
+    uint32_t lo = 0, hi = s.ctx;
+    while (lo < hi) {
+        uint32_t mid = lo + (hi - lo + 1) / 2;
+        brasa_session_shape t = s;
+        t.ctx = mid;
+        if (t.max_tokens > mid) t.max_tokens = mid;
+        brasa_memory_plan p;
+        BRASA_TRY(plan_of(t, &p));
+        if (p.total <= budget) lo = mid;
+        else hi = mid - 1;
+    }
+    if (max_ctx_out) *max_ctx_out = lo;
+    return brasa_fail(ctx, BRASA_EBUDGET, "the model needs %.2f GiB (weights %.2f, KV %.2f, workspace %.2f, overhead %.2f) and the budget is %.2f GiB; the largest context that fits is %u",
+                      plan.total / 1073741824.0, plan.weights / 1073741824.0, plan.kv / 1073741824.0, plan.workspace / 1073741824.0,
+                      plan.overhead / 1073741824.0, budget / 1073741824.0, lo);
+}

@@ -3,10 +3,13 @@
 #pragma once
 #include <stdint.h>
 
+#include <functional>
 #include <map>
 #include <memory>
 #include <string>
 #include <vector>
+
+#include "../../include/brasa_cuda.h"
 
 namespace brasa {
 
@@ -41,13 +44,13 @@ struct TensorInfo {
     }
 };
 
-class BrasaFile {
+// A model on disk: a parsed configuration and named tensors in one mapped data file. Two containers: a `.brasa` file, and a
+// folder with config.json and model.safetensors.
+class WeightFile {
   public:
-    ~BrasaFile();
-    // Opens and validates structure: magic, version, bounds, page alignment, tensor sizes.
-    static std::unique_ptr<BrasaFile> open(const std::string &path, std::string &err);
-    // Checks every tensor's sha256 and data_sha256.
-    bool verify(std::string &err) const;
+    virtual ~WeightFile();
+    // A folder opens as config.json + model.safetensors, anything else as a `.brasa` file.
+    static std::unique_ptr<WeightFile> open_any(const std::string &path, std::string &err);
     const std::vector<TensorInfo> &tensors() const { return tensors_; }
     const TensorInfo *tensor(const std::string &name) const;
     const uint8_t *data(const TensorInfo &t) const { return map_ + t.offset; }
@@ -55,15 +58,37 @@ class BrasaFile {
     const Json &config() const { return *config_; }
     const std::string &family() const { return family_; }
 
-  private:
+  protected:
+    bool map_file(const std::string &path, std::string &err);
     const uint8_t *map_ = nullptr;
     size_t size_ = 0;
     int fd_ = -1;
     Json meta_;
     const Json *config_ = nullptr;
-    std::string family_, data_sha256_;
-    uint64_t page_ = 0;
+    std::string family_;
     std::vector<TensorInfo> tensors_;
+};
+
+class BrasaFile : public WeightFile {
+  public:
+    // Opens and validates structure: magic, version, bounds, page alignment, tensor sizes.
+    static std::unique_ptr<BrasaFile> open(const std::string &path, std::string &err);
+    // Checks every tensor's sha256 and data_sha256.
+    bool verify(std::string &err) const;
+
+  private:
+    std::string data_sha256_;
+    uint64_t page_ = 0;
+};
+
+// config.json (its "architecture" names the family) + model.safetensors: an 8-byte little-endian header length, the JSON
+// header name -> {dtype, shape, data_offsets}, the data. bf16, f32 and i32 tensors.
+class SafeTensorsFolder : public WeightFile {
+  public:
+    static std::unique_ptr<SafeTensorsFolder> open(const std::string &folder, std::string &err);
+
+  private:
+    Json config_json_;
 };
 
 int dtype_qtype(const std::string &dtype);  // "q4_0" -> BRASA_Q4_0 ...; -1 for f32 / unknown
@@ -91,3 +116,8 @@ class Sampler {
 };
 
 }  // namespace brasa
+
+// brasa_plan_check over any plan that grows with the context: budget 0 = the device's free memory minus a reserve; on a refusal
+// *max_ctx_out is the largest context that fits.
+int32_t brasa_plan_check_with(brasa_ctx *ctx, const brasa_session_shape &s, uint64_t budget, brasa_memory_plan *out, uint32_t *max_ctx_out,
+                              const std::function<int32_t(const brasa_session_shape &, brasa_memory_plan *)> &plan_of);

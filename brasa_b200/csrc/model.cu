@@ -1,7 +1,7 @@
-// Qwen3 dense model and generation session on the device
+// Model and session entry points, the table of model families, and the Qwen3 dense family
 // (crates/models/src/qwen3.rs, crates/runtime/src/session.rs).
 //
-// Per layer (T tokens from position pos0):
+// Qwen3, per layer (T tokens from position pos0):
 //   h = RMSNorm(x); q, k, v = W h; q, k = per-head RMSNorm then RoPE; K, V -> cache;
 //   o = attention(q, K, V); x += Wo o; h = RMSNorm(x); x += Wdown (silu(Wgate h) * Wup h)
 // Activations are f32. With more than GEMV_MAX_TOKENS tokens the projections run as GEMMs whose
@@ -143,7 +143,7 @@ int32_t alloc_buf(brasa_model *m, uint64_t bytes, brasa_buf **out, uint64_t *acc
     return BRASA_OK;
 }
 
-int32_t load_f32(brasa_model *m, const brasa::BrasaFile &f, const std::string &name, uint64_t n, brasa_buf **out) {
+int32_t load_f32(brasa_model *m, const brasa::WeightFile &f, const std::string &name, uint64_t n, brasa_buf **out) {
     brasa_ctx *ctx = m->ctx;
     const brasa::TensorInfo *t = f.tensor(name);
     if (!t) return brasa_fail(ctx, BRASA_EIO, "missing tensor %s", name.c_str());
@@ -153,7 +153,7 @@ int32_t load_f32(brasa_model *m, const brasa::BrasaFile &f, const std::string &n
 }
 
 // Uploads a quantised matrix and regroups it into the tiled layout when its shape allows.
-int32_t load_matrix(brasa_model *m, brasa_cmd *load_cmd, const brasa::BrasaFile &f, const std::string &name, uint32_t rows, uint32_t cols, brasa_buf *staging,
+int32_t load_matrix(brasa_model *m, brasa_cmd *load_cmd, const brasa::WeightFile &f, const std::string &name, uint32_t rows, uint32_t cols, brasa_buf *staging,
                     Matrix *out) {
     brasa_ctx *ctx = m->ctx;
     const brasa::TensorInfo *t = f.tensor(name);
@@ -336,15 +336,19 @@ int32_t check_tokens(brasa_model *m, uint32_t tokens, uint32_t pos0) {
     return BRASA_OK;
 }
 
-// One full decode step for the token in ws.ids[0] at position pos0: embed, layers, lm_head, argmax into
-// next_id, then "advance" (next_id -> ids[0] and the output list, position + 1). The first call runs the
-// kernels directly and records them; later calls replay the CUDA graph.
-int32_t decode_step_kernels(brasa_model *m, brasa_cmd *cmd) {
-    uint32_t *st = (uint32_t *)m->dev_state->ptr;
+// Embed, layers, lm_head and argmax of one token.
+int32_t qwen3_step(brasa_model *m, brasa_cmd *cmd) {
     BRASA_TRY(brasa_k_embed(cmd, m->embed.q, A(m->ids), A(m->x), 1));
     BRASA_TRY(encode_decode_token(m, cmd, 0, m->cfg.layers, true));
-    if (m->tp) BRASA_TRY(brasa_k_tp_argmax(cmd, m->tp, A(m->logits), m->cfg.head_rows, m->cfg.head_row0, A(m->next_id)));
-    else BRASA_TRY(brasa_argmax_launch(cmd, F(m->logits), m->cfg.head_rows, (uint32_t *)m->next_id->ptr));
+    if (m->tp) return brasa_k_tp_argmax(cmd, m->tp, A(m->logits), m->cfg.head_rows, m->cfg.head_row0, A(m->next_id));
+    return brasa_argmax_launch(cmd, F(m->logits), m->cfg.head_rows, (uint32_t *)m->next_id->ptr);
+}
+
+// One full decode step for the token in ws.ids[0] at the device's position: the family's layers, head and choice into
+// next_id, then "advance" (next_id -> ids[0] and the output list, position + 1).
+int32_t decode_step_kernels(brasa_model *m, brasa_cmd *cmd) {
+    uint32_t *st = (uint32_t *)m->dev_state->ptr;
+    BRASA_TRY(m->family->step(m, cmd));
     return brasa_advance_launch(cmd, (uint32_t *)m->ids->ptr, (const uint32_t *)m->next_id->ptr, (uint32_t *)m->out_ids->ptr, st + 1,
                                 m->limits.ctx, st);
 }
@@ -393,10 +397,14 @@ int32_t make_token_program(brasa_model *m) {
     return brasa_token_program_create(m->ctx, d, &m->token_prog);
 }
 
-// pos0 == UINT32_MAX keeps the position the device already holds (device-resident loop).
+bool is_qwen3(const brasa_model *m);
+bool decode_resident_ok(brasa_model *m) { return !is_qwen3(m) || decode_fused_ok(m); }
+
+// pos0 == UINT32_MAX keeps the position the device already holds (device-resident loop). The first call runs the kernels
+// directly and records them; later calls replay the CUDA graph.
 int32_t decode_step(brasa_model *m, brasa_cmd *cmd, uint32_t pos0) {
     if (pos0 != UINT32_MAX) BRASA_TRY(set_position(m, pos0));
-    if (!m->token_prog_tried) BRASA_TRY(make_token_program(m));
+    if (is_qwen3(m) && !m->token_prog_tried) BRASA_TRY(make_token_program(m));
     if (m->token_prog) return brasa_token_program_launch(cmd, m->token_prog);
     if (m->decode_graph) return brasa_graph_launch(cmd, m->decode_graph);
     BRASA_TRY(decode_step_kernels(m, cmd));
@@ -413,40 +421,177 @@ int32_t decode_step(brasa_model *m, brasa_cmd *cmd, uint32_t pos0) {
     return BRASA_OK;
 }
 
-// Enqueues a whole forward for ids already in ws.ids; logits of the last logit_rows positions end
-// up in ws.logits.
-int32_t encode_forward(brasa_model *m, brasa_cmd *cmd, uint32_t tokens, uint32_t pos0, uint32_t logit_rows) {
+int32_t qwen3_forward(brasa_model *m, brasa_cmd *cmd, uint32_t tokens, uint32_t pos0, const uint32_t *rows, uint32_t n_rows) {
     const brasa_config &c = m->cfg;
-    if (tokens == 1 && decode_fused_ok(m)) return decode_step(m, cmd, pos0);
     BRASA_TRY(brasa_k_embed(cmd, m->embed.q, A(m->ids), A(m->x), tokens));
     for (uint32_t li = 0; li < c.layers; ++li) BRASA_TRY(encode_layer_prefill(m, cmd, li, tokens, pos0));
-    uint32_t first = tokens - logit_rows;
-    BRASA_TRY(brasa_k_rms_norm(cmd, A(m->x, (uint64_t)first * c.hidden * 4), A(m->final_norm), A(m->norm_out), logit_rows, c.hidden, c.eps));
-    return brasa_k_gemv(cmd, m->head.q, A(m->norm_out), A(m->logits), logit_rows);
+    if (n_rows == 0) return BRASA_OK;
+    for (uint32_t i = 0, n; i < n_rows; i += n) {  // neighbouring places share a launch
+        for (n = 1; i + n < n_rows && rows[i + n] == rows[i] + n;) ++n;
+        BRASA_TRY(brasa_k_rms_norm(cmd, A(m->x, (uint64_t)rows[i] * c.hidden * 4), A(m->final_norm), A(m->norm_out, (uint64_t)i * c.hidden * 4), n, c.hidden, c.eps));
+    }
+    return brasa_k_gemv(cmd, m->head.q, A(m->norm_out), A(m->logits), n_rows);
+}
+
+// Enqueues a whole forward for ids already in ws.ids; logits of the given places among the tokens end up in ws.logits.
+int32_t encode_forward(brasa_model *m, brasa_cmd *cmd, uint32_t tokens, uint32_t pos0, const uint32_t *rows, uint32_t n_rows) {
+    if (m->family->begin) BRASA_TRY(m->family->begin(m, pos0, 0, m->cfg.layers));
+    if (tokens == 1 && decode_resident_ok(m) && n_rows <= 1) BRASA_TRY(decode_step(m, cmd, pos0));
+    else BRASA_TRY(m->family->forward(m, cmd, tokens, pos0, rows, n_rows));
+    if (m->family->finish) m->family->finish(m, pos0 + tokens, 0, m->cfg.layers);
+    return BRASA_OK;
+}
+
+bool qwen3_describe(const brasa::WeightFile &f, brasa_model_shape *shape, brasa_config *cfg, std::string &err) {
+    brasa_config c{};
+    if (!cfg_from_json(nullptr, f.config(), &c, err)) return false;
+    if (shape) {
+        uint64_t wb = 0;
+        for (auto &t : f.tensors()) wb += brasa_plan_buffer_bytes(t.nbytes);
+        *shape = brasa_model_shape{wb, c.layers, c.hidden, c.heads, c.kv_heads, c.head_dim, c.ffn, c.vocab};
+    }
+    if (cfg) *cfg = c;
+    return true;
+}
+
+int32_t qwen3_plan(brasa_ctx *ctx, const brasa::WeightFile &f, const brasa_session_shape &s, brasa_memory_plan *out) {
+    brasa_model_shape shape;
+    std::string err;
+    if (!qwen3_describe(f, &shape, nullptr, err)) return brasa_fail(ctx, BRASA_EIO, "%s", err.c_str());
+    return brasa_plan(&shape, &s, out);
+}
+
+int32_t qwen3_run_layers(brasa_model *m, brasa_cmd *cmd, const float *x, float *y, uint32_t tokens, uint32_t pos0, uint32_t l0, uint32_t l1) {
+    const uint64_t n = (uint64_t)tokens * m->cfg.hidden * 4;
+    BRASA_TRY(brasa_buf_upload(m->x, 0, x, n));
+    if (tokens == 1 && decode_fused_ok(m)) {
+        BRASA_TRY(set_position(m, pos0));
+        BRASA_TRY(encode_decode_token(m, cmd, l0, l1, false));
+    } else {
+        for (uint32_t li = l0; li < l1; ++li) BRASA_TRY(encode_layer_prefill(m, cmd, li, tokens, pos0));
+    }
+    return brasa_buf_download(m->x, 0, y, n);
+}
+
+int32_t qwen3_load(brasa_model *m, const brasa::WeightFile &file, brasa_cmd *load_cmd, brasa_buf *staging) {
+    brasa_ctx *ctx = m->ctx;
+    const brasa::WeightFile *f = &file;
+    const brasa_config &c = m->cfg;
+    const brasa_limits &limits = m->limits;
+    BRASA_REQUIRE(ctx, limits.kv >= BRASA_KV_F32 && limits.kv <= BRASA_KV_Q8_0, "unknown KV type %d", limits.kv);
+    BRASA_REQUIRE(ctx, c.head_dim == 128, "the kernels need head_dim 128 (got %u)", c.head_dim);
+    BRASA_REQUIRE(ctx, c.kv_heads > 0 && c.heads % c.kv_heads == 0, "heads must be a multiple of kv heads");
+    if (!c.tied && !f->tensor("lm_head.weight")) return brasa_fail(ctx, BRASA_EIO, "untied model without lm_head.weight");
+    const uint32_t H = c.hidden, qd = c.heads * c.head_dim, kvd = c.kv_heads * c.head_dim, ffn = c.ffn;
+    m->layers.resize(c.layers);
+    for (uint32_t i = 0; i < c.layers; ++i) {
+        auto n = [&](const char *s) { return "model.layers." + std::to_string(i) + "." + s; };
+        Layer &l = m->layers[i];
+        BRASA_TRY(load_f32(m, *f, n("input_layernorm.weight"), H, &l.attn_norm));
+        BRASA_TRY(load_matrix(m, load_cmd, *f, n("self_attn.q_proj.weight"), qd, H, staging, &l.wq));
+        BRASA_TRY(load_matrix(m, load_cmd, *f, n("self_attn.k_proj.weight"), kvd, H, staging, &l.wk));
+        BRASA_TRY(load_matrix(m, load_cmd, *f, n("self_attn.v_proj.weight"), kvd, H, staging, &l.wv));
+        BRASA_TRY(load_matrix(m, load_cmd, *f, n("self_attn.o_proj.weight"), H, qd, staging, &l.wo));
+        BRASA_TRY(load_f32(m, *f, n("self_attn.q_norm.weight"), c.head_dim, &l.q_norm));
+        BRASA_TRY(load_f32(m, *f, n("self_attn.k_norm.weight"), c.head_dim, &l.k_norm));
+        BRASA_TRY(load_f32(m, *f, n("post_attention_layernorm.weight"), H, &l.ffn_norm));
+        BRASA_TRY(load_matrix(m, load_cmd, *f, n("mlp.gate_proj.weight"), ffn, H, staging, &l.gate));
+        BRASA_TRY(load_matrix(m, load_cmd, *f, n("mlp.up_proj.weight"), ffn, H, staging, &l.up));
+        BRASA_TRY(load_matrix(m, load_cmd, *f, n("mlp.down_proj.weight"), H, ffn, staging, &l.down));
+    }
+    BRASA_TRY(load_matrix(m, load_cmd, *f, "model.embed_tokens.weight", c.vocab, H, staging, &m->embed));
+    if (m->embed.q.qtype != BRASA_Q8_0 && m->embed.q.qtype != BRASA_Q6_0)
+        return brasa_fail(ctx, BRASA_EIO, "the embedding table must be q8_0 or q6_0");
+    if (c.tied) m->head = m->embed;
+    else {
+        const brasa::TensorInfo *ht = f->tensor("lm_head.weight");
+        if (ht->shape.size() != 2 || ht->shape[0] == 0 || ht->shape[0] > c.vocab || m->cfg.head_row0 + ht->shape[0] > c.vocab)
+            return brasa_fail(ctx, BRASA_EIO, "lm_head.weight: unexpected shape");
+        m->cfg.head_rows = (uint32_t)ht->shape[0];
+        BRASA_TRY(load_matrix(m, load_cmd, *f, "lm_head.weight", m->cfg.head_rows, H, staging, &m->head));
+    }
+    BRASA_TRY(load_f32(m, *f, "model.norm.weight", H, &m->final_norm));
+    uint64_t *ws = &m->alloc.workspace;
+    std::vector<float> cs((size_t)limits.ctx * c.head_dim / 2), sn(cs.size());
+    BRASA_TRY(brasa_rope_table(c.rope_theta, c.head_dim, limits.ctx, cs.data(), sn.data()));
+    BRASA_TRY(alloc_buf(m, cs.size() * 4, &m->rope_cos, ws));
+    BRASA_TRY(alloc_buf(m, sn.size() * 4, &m->rope_sin, ws));
+    BRASA_TRY(brasa_buf_upload(m->rope_cos, 0, cs.data(), cs.size() * 4));
+    BRASA_TRY(brasa_buf_upload(m->rope_sin, 0, sn.data(), sn.size() * 4));
+
+    const uint64_t t = limits.max_tokens;
+    m->cap = (limits.ctx + BRASA_KV_ALIGN - 1) / BRASA_KV_ALIGN * BRASA_KV_ALIGN;
+    uint64_t kv_elems = (uint64_t)c.layers * m->cap * kvd;
+    BRASA_TRY(alloc_buf(m, brasa_kv_bytes(limits.kv, kv_elems), &m->kc, &m->alloc.kv));
+    BRASA_TRY(alloc_buf(m, brasa_kv_bytes(limits.kv, kv_elems), &m->vc, &m->alloc.kv));
+    BRASA_TRY(alloc_buf(m, t * H * 4, &m->x, ws));
+    BRASA_TRY(alloc_buf(m, t * H * 4, &m->h, ws));
+    BRASA_TRY(alloc_buf(m, t * H * 4, &m->norm_out, ws));
+    BRASA_TRY(alloc_buf(m, t * qd * 4, &m->q, ws));
+    BRASA_TRY(alloc_buf(m, t * qd * 4, &m->attn, ws));
+    BRASA_TRY(alloc_buf(m, t * kvd * 4, &m->k_new, ws));
+    BRASA_TRY(alloc_buf(m, t * kvd * 4, &m->v_new, ws));
+    BRASA_TRY(alloc_buf(m, t * ffn * 4, &m->gate, ws));
+    BRASA_TRY(alloc_buf(m, t * ffn * 4, &m->up, ws));
+    BRASA_TRY(alloc_buf(m, 2 * t * std::max<uint64_t>(ffn, std::max<uint64_t>(qd, H)), &m->xh, ws));
+    BRASA_TRY(alloc_buf(m, (uint64_t)brasa_norm_partials(H) * 4, &m->ss, ws));
+    m->partials_len = brasa_decode_partials_len(c.heads, limits.ctx);
+    BRASA_TRY(alloc_buf(m, m->partials_len * 4, &m->partials, ws));
+    return BRASA_OK;
+}
+
+const brasa_family qwen3_family = {"qwen3", qwen3_describe, qwen3_plan, qwen3_load, nullptr, qwen3_forward, qwen3_step, qwen3_run_layers, nullptr, nullptr, nullptr};
+bool is_qwen3(const brasa_model *m) { return m->family == &qwen3_family; }
+
+// The families this library runs.
+const brasa_family *const FAMILIES[] = {&qwen3_family, &brasa_stack::dunuzen_family};
+
+const brasa_family *family_of(const brasa::WeightFile &f, std::string &err) {
+    for (const brasa_family *fam : FAMILIES)
+        if (f.family() == fam->name) return fam;
+    err = "family " + f.family() + " is not supported";
+    return nullptr;
 }
 
 }  // namespace
+
+int32_t brasa_stage_upload(brasa_model *m, void *dst, const brasa::WeightFile &f, const brasa::TensorInfo &t) {
+    return m->stager->upload(dst, f.fd(), t.offset, f.data(t), t.nbytes);
+}
 
 extern "C" {
 
 int32_t brasa_model_shape_from_file(const char *path, brasa_model_shape *shape, brasa_config *cfg, char *err, uint64_t err_len) {
     std::string e;
-    auto f = brasa::BrasaFile::open(path ? path : "", e);
-    brasa_config c{};
-    if (f && f->family() != "qwen3") { e = "family " + f->family() + " is not supported"; f.reset(); }
-    if (f && !cfg_from_json(nullptr, f->config(), &c, e)) f.reset();
-    if (!f) {
+    auto f = brasa::WeightFile::open_any(path ? path : "", e);
+    const brasa_family *fam = f ? family_of(*f, e) : nullptr;
+    if (!fam || !fam->describe(*f, shape, cfg, e)) {
         if (err && err_len) snprintf(err, (size_t)err_len, "%s", e.c_str());
         return BRASA_EIO;
     }
-    if (shape) {
-        uint64_t wb = 0;
-        for (auto &t : f->tensors()) wb += brasa_plan_buffer_bytes(t.nbytes);
-        *shape = brasa_model_shape{wb, c.layers, c.hidden, c.heads, c.kv_heads, c.head_dim, c.ffn, c.vocab};
-    }
-    if (cfg) *cfg = c;
     if (err && err_len) err[0] = 0;
     return BRASA_OK;
+}
+
+int32_t brasa_model_family(const char *path, char *name, uint64_t name_len) {
+    std::string e;
+    auto f = brasa::WeightFile::open_any(path ? path : "", e);
+    if (!f || !family_of(*f, e)) {
+        if (name && name_len) snprintf(name, (size_t)name_len, "%s", e.c_str());
+        return BRASA_EIO;
+    }
+    if (name && name_len) snprintf(name, (size_t)name_len, "%s", f->family().c_str());
+    return BRASA_OK;
+}
+
+int32_t brasa_plan_file(brasa_ctx *ctx, const char *path, const brasa_session_shape *s, uint64_t budget, brasa_memory_plan *out, uint32_t *max_ctx_out) {
+    if (!path || !s) return BRASA_EINVAL;
+    std::string e;
+    auto f = brasa::WeightFile::open_any(path, e);
+    const brasa_family *fam = f ? family_of(*f, e) : nullptr;
+    if (!fam) return brasa_fail(ctx, BRASA_EIO, "%s", e.c_str());
+    return brasa_plan_check_with(ctx, *s, budget, out, max_ctx_out,
+                                 [&](const brasa_session_shape &t, brasa_memory_plan *p) { return fam->plan(ctx, *f, t, p); });
 }
 
 void brasa_model_free(brasa_model *m) {
@@ -455,6 +600,7 @@ void brasa_model_free(brasa_model *m) {
     brasa_token_program_free(m->token_prog);
     for (brasa_buf *b : m->owned) brasa_buf_free(b);
     if (m->pinned_id) cudaFreeHost(m->pinned_id);
+    if (m->family && m->family->release) m->family->release(m);
     delete m;
 }
 
@@ -462,24 +608,20 @@ int32_t brasa_model_load(brasa_ctx *ctx, const char *path, brasa_limits limits, 
     if (!ctx || !path || !out) return BRASA_EINVAL;
     *out = nullptr;
     std::string e;
-    auto f = brasa::BrasaFile::open(path, e);
+    auto f = brasa::WeightFile::open_any(path, e);
     if (!f) return brasa_fail(ctx, BRASA_EIO, "%s", e.c_str());
-    if (f->family() != "qwen3") return brasa_fail(ctx, BRASA_EIO, "family %s is not supported", f->family().c_str());
+    const brasa_family *fam = family_of(*f, e);
     brasa_config c{};
-    if (!cfg_from_json(ctx, f->config(), &c, e)) return brasa_fail(ctx, BRASA_EIO, "%s", e.c_str());
+    if (!fam || !fam->describe(*f, nullptr, &c, e)) return brasa_fail(ctx, BRASA_EIO, "%s", e.c_str());
     BRASA_REQUIRE(ctx, limits.ctx <= c.max_position, "context %u larger than the model's maximum (%u)", limits.ctx, c.max_position);
     BRASA_REQUIRE(ctx, limits.ctx > 0 && limits.max_tokens > 0 && limits.max_logit_rows > 0, "limits must be positive");
-    BRASA_REQUIRE(ctx, limits.kv >= BRASA_KV_F32 && limits.kv <= BRASA_KV_Q8_0, "unknown KV type %d", limits.kv);
-    BRASA_REQUIRE(ctx, c.head_dim == 128, "the kernels need head_dim 128 (got %u)", c.head_dim);
-    BRASA_REQUIRE(ctx, c.kv_heads > 0 && c.heads % c.kv_heads == 0, "heads must be a multiple of kv heads");
-    if (!c.tied && !f->tensor("lm_head.weight")) return brasa_fail(ctx, BRASA_EIO, "untied model without lm_head.weight");
 
     brasa_model *m = new brasa_model();
     m->ctx = ctx;
+    m->family = fam;
     m->cfg = c;
     m->limits = limits;
     int32_t rc = [&]() -> int32_t {
-        const uint32_t H = c.hidden, qd = c.heads * c.head_dim, kvd = c.kv_heads * c.head_dim, ffn = c.ffn;
         uint64_t biggest = 0;
         for (auto &t : f->tensors()) biggest = std::max<uint64_t>(biggest, t.nbytes);
         brasa_buf *staging = nullptr;
@@ -498,34 +640,7 @@ int32_t brasa_model_load(brasa_ctx *ctx, const char *path, brasa_limits limits, 
                 m->stager = nullptr;
             }
         } guard{load_cmd, m};
-        m->layers.resize(c.layers);
-        for (uint32_t i = 0; i < c.layers; ++i) {
-            auto n = [&](const char *s) { return "model.layers." + std::to_string(i) + "." + s; };
-            Layer &l = m->layers[i];
-            BRASA_TRY(load_f32(m, *f, n("input_layernorm.weight"), H, &l.attn_norm));
-            BRASA_TRY(load_matrix(m, load_cmd, *f, n("self_attn.q_proj.weight"), qd, H, staging, &l.wq));
-            BRASA_TRY(load_matrix(m, load_cmd, *f, n("self_attn.k_proj.weight"), kvd, H, staging, &l.wk));
-            BRASA_TRY(load_matrix(m, load_cmd, *f, n("self_attn.v_proj.weight"), kvd, H, staging, &l.wv));
-            BRASA_TRY(load_matrix(m, load_cmd, *f, n("self_attn.o_proj.weight"), H, qd, staging, &l.wo));
-            BRASA_TRY(load_f32(m, *f, n("self_attn.q_norm.weight"), c.head_dim, &l.q_norm));
-            BRASA_TRY(load_f32(m, *f, n("self_attn.k_norm.weight"), c.head_dim, &l.k_norm));
-            BRASA_TRY(load_f32(m, *f, n("post_attention_layernorm.weight"), H, &l.ffn_norm));
-            BRASA_TRY(load_matrix(m, load_cmd, *f, n("mlp.gate_proj.weight"), ffn, H, staging, &l.gate));
-            BRASA_TRY(load_matrix(m, load_cmd, *f, n("mlp.up_proj.weight"), ffn, H, staging, &l.up));
-            BRASA_TRY(load_matrix(m, load_cmd, *f, n("mlp.down_proj.weight"), H, ffn, staging, &l.down));
-        }
-        BRASA_TRY(load_matrix(m, load_cmd, *f, "model.embed_tokens.weight", c.vocab, H, staging, &m->embed));
-        if (m->embed.q.qtype != BRASA_Q8_0 && m->embed.q.qtype != BRASA_Q6_0)
-            return brasa_fail(ctx, BRASA_EIO, "the embedding table must be q8_0 or q6_0");
-        if (c.tied) m->head = m->embed;
-        else {
-            const brasa::TensorInfo *ht = f->tensor("lm_head.weight");
-            if (ht->shape.size() != 2 || ht->shape[0] == 0 || ht->shape[0] > c.vocab || m->cfg.head_row0 + ht->shape[0] > c.vocab)
-                return brasa_fail(ctx, BRASA_EIO, "lm_head.weight: unexpected shape");
-            m->cfg.head_rows = (uint32_t)ht->shape[0];
-            BRASA_TRY(load_matrix(m, load_cmd, *f, "lm_head.weight", m->cfg.head_rows, H, staging, &m->head));
-        }
-        BRASA_TRY(load_f32(m, *f, "model.norm.weight", H, &m->final_norm));
+        BRASA_TRY(fam->load(m, *f, load_cmd, staging));
         {
             brasa_cmd *c2 = load_cmd;
             load_cmd = nullptr;
@@ -534,37 +649,10 @@ int32_t brasa_model_load(brasa_ctx *ctx, const char *path, brasa_limits limits, 
         m->load_bytes = stager.bytes;
         m->load_seconds = std::chrono::duration<double>(std::chrono::steady_clock::now() - t_load).count();
         m->stager = nullptr;
-        // staging is not part of the steady-state footprint
-        m->owned.erase(std::remove(m->owned.begin(), m->owned.end(), staging), m->owned.end());
-        BRASA_TRY(brasa_buf_free(staging));
+        BRASA_TRY(brasa_buf_free(staging));  // not part of the steady-state footprint
 
-        uint64_t *ws = &m->alloc.workspace;
-        std::vector<float> cs((size_t)limits.ctx * c.head_dim / 2), sn(cs.size());
-        BRASA_TRY(brasa_rope_table(c.rope_theta, c.head_dim, limits.ctx, cs.data(), sn.data()));
-        BRASA_TRY(alloc_buf(m, cs.size() * 4, &m->rope_cos, ws));
-        BRASA_TRY(alloc_buf(m, sn.size() * 4, &m->rope_sin, ws));
-        BRASA_TRY(brasa_buf_upload(m->rope_cos, 0, cs.data(), cs.size() * 4));
-        BRASA_TRY(brasa_buf_upload(m->rope_sin, 0, sn.data(), sn.size() * 4));
-
-        const uint64_t t = limits.max_tokens;
-        m->cap = (limits.ctx + BRASA_KV_ALIGN - 1) / BRASA_KV_ALIGN * BRASA_KV_ALIGN;
-        uint64_t kv_elems = (uint64_t)c.layers * m->cap * kvd;
-        BRASA_TRY(alloc_buf(m, brasa_kv_bytes(limits.kv, kv_elems), &m->kc, &m->alloc.kv));
-        BRASA_TRY(alloc_buf(m, brasa_kv_bytes(limits.kv, kv_elems), &m->vc, &m->alloc.kv));
-        BRASA_TRY(alloc_buf(m, t * H * 4, &m->x, ws));
-        BRASA_TRY(alloc_buf(m, t * H * 4, &m->h, ws));
-        BRASA_TRY(alloc_buf(m, t * H * 4, &m->norm_out, ws));
-        BRASA_TRY(alloc_buf(m, t * qd * 4, &m->q, ws));
-        BRASA_TRY(alloc_buf(m, t * qd * 4, &m->attn, ws));
-        BRASA_TRY(alloc_buf(m, t * kvd * 4, &m->k_new, ws));
-        BRASA_TRY(alloc_buf(m, t * kvd * 4, &m->v_new, ws));
-        BRASA_TRY(alloc_buf(m, t * ffn * 4, &m->gate, ws));
-        BRASA_TRY(alloc_buf(m, t * ffn * 4, &m->up, ws));
-        BRASA_TRY(alloc_buf(m, 2 * t * std::max<uint64_t>(ffn, std::max<uint64_t>(qd, H)), &m->xh, ws));
-        BRASA_TRY(alloc_buf(m, t * 4, &m->ids, ws));
-        BRASA_TRY(alloc_buf(m, (uint64_t)brasa_norm_partials(H) * 4, &m->ss, ws));
-        m->partials_len = brasa_decode_partials_len(c.heads, limits.ctx);
-        BRASA_TRY(alloc_buf(m, m->partials_len * 4, &m->partials, ws));
+        uint64_t *ws = fam == &qwen3_family ? &m->alloc.workspace : nullptr;  // (other families have counted these)
+        BRASA_TRY(alloc_buf(m, (uint64_t)limits.max_tokens * 4, &m->ids, ws));
         BRASA_TRY(alloc_buf(m, (uint64_t)limits.max_logit_rows * m->cfg.head_rows * 4, &m->logits, ws));
         BRASA_TRY(alloc_buf(m, 64, &m->next_id, nullptr));
         BRASA_TRY(alloc_buf(m, (uint64_t)limits.ctx * 4, &m->out_ids, nullptr));
@@ -585,6 +673,7 @@ int32_t brasa_model_load(brasa_ctx *ctx, const char *path, brasa_limits limits, 
 int32_t brasa_model_set_tp(brasa_model *m, brasa_tp *tp) {
     if (!m || !tp) return BRASA_EINVAL;
     brasa_ctx *ctx = m->ctx;
+    BRASA_REQUIRE(ctx, is_qwen3(m), "set_tp: the %s family has no shards", m->family->name);
     BRASA_REQUIRE(ctx, !m->decode_graph && !m->token_prog, "set_tp: attach the exchange before the first decode step");
     BRASA_REQUIRE(ctx, m->cfg.hidden % 2 == 0, "set_tp: odd hidden size");
     BRASA_REQUIRE(ctx, m->cfg.head_row0 == 0 || brasa_tp_world(tp) > 1, "set_tp: a shard with a vocabulary offset needs its peers");
@@ -615,27 +704,38 @@ int32_t brasa_model_load_stats(brasa_model *m, double *seconds, uint64_t *bytes)
 }
 int32_t brasa_model_set_prefill_precision(brasa_model *m, int32_t precision) {
     if (!m) return BRASA_EINVAL;
+    BRASA_REQUIRE(m->ctx, is_qwen3(m), "the %s family takes its precision from the cache type", m->family->name);
     BRASA_REQUIRE(m->ctx, precision == BRASA_PREFILL_F16 || precision == BRASA_PREFILL_F32, "unknown precision %d", precision);
     m->prefill_precision = precision;
+    return BRASA_OK;
+}
+
+int32_t brasa_model_forward_rows(brasa_model *m, const uint32_t *ids, uint32_t tokens, uint32_t pos0, const uint32_t *rows, uint32_t n_rows, float *logits,
+                                 double *gpu_seconds) {
+    if (!m || !ids || (n_rows && !rows)) return BRASA_EINVAL;
+    brasa_ctx *ctx = m->ctx;
+    BRASA_TRY(check_tokens(m, tokens, pos0));
+    BRASA_REQUIRE(ctx, n_rows <= m->limits.max_logit_rows, "%u rows of logits per forward; the maximum is %u", n_rows, m->limits.max_logit_rows);
+    for (uint32_t i = 0; i < n_rows; ++i) BRASA_REQUIRE(ctx, rows[i] < tokens, "logits of token %u of %u", rows[i], tokens);
+    for (uint32_t i = 0; i < tokens; ++i) BRASA_REQUIRE(ctx, ids[i] < m->cfg.vocab, "token id %u outside the vocabulary", ids[i]);
+    BRASA_CUDA(ctx, cudaMemcpyAsync(m->ids->ptr, ids, (size_t)tokens * 4, cudaMemcpyHostToDevice, ctx->stream));
+    brasa_cmd *cmd;
+    BRASA_TRY(brasa_cmd_begin(ctx, &cmd));
+    int32_t rc = encode_forward(m, cmd, tokens, pos0, rows, n_rows);
+    int32_t rc2 = brasa_cmd_wait(cmd, gpu_seconds);
+    BRASA_TRY(rc);
+    BRASA_TRY(rc2);
+    if (logits && n_rows) BRASA_TRY(brasa_buf_download(m->logits, 0, logits, (uint64_t)n_rows * m->cfg.head_rows * 4));
     return BRASA_OK;
 }
 
 int32_t brasa_model_forward(brasa_model *m, const uint32_t *ids, uint32_t tokens, uint32_t pos0, uint32_t logit_rows, float *logits,
                             double *gpu_seconds) {
     if (!m || !ids) return BRASA_EINVAL;
-    brasa_ctx *ctx = m->ctx;
-    BRASA_TRY(check_tokens(m, tokens, pos0));
-    BRASA_REQUIRE(ctx, logit_rows >= 1 && logit_rows <= std::min(tokens, m->limits.max_logit_rows), "logit_rows %u is not valid", logit_rows);
-    for (uint32_t i = 0; i < tokens; ++i) BRASA_REQUIRE(ctx, ids[i] < m->cfg.vocab, "token id %u outside the vocabulary", ids[i]);
-    BRASA_CUDA(ctx, cudaMemcpyAsync(m->ids->ptr, ids, (size_t)tokens * 4, cudaMemcpyHostToDevice, ctx->stream));
-    brasa_cmd *cmd;
-    BRASA_TRY(brasa_cmd_begin(ctx, &cmd));
-    int32_t rc = encode_forward(m, cmd, tokens, pos0, logit_rows);
-    int32_t rc2 = brasa_cmd_wait(cmd, gpu_seconds);
-    BRASA_TRY(rc);
-    BRASA_TRY(rc2);
-    if (logits) BRASA_TRY(brasa_buf_download(m->logits, 0, logits, (uint64_t)logit_rows * m->cfg.head_rows * 4));
-    return BRASA_OK;
+    BRASA_REQUIRE(m->ctx, logit_rows >= 1 && logit_rows <= std::min(tokens, m->limits.max_logit_rows), "logit_rows %u is not valid", logit_rows);
+    std::vector<uint32_t> rows(logit_rows);
+    for (uint32_t i = 0; i < logit_rows; ++i) rows[i] = tokens - logit_rows + i;
+    return brasa_model_forward_rows(m, ids, tokens, pos0, rows.data(), logit_rows, logits, gpu_seconds);
 }
 
 int32_t brasa_model_run_layers(brasa_model *m, float *x, uint32_t tokens, uint32_t pos0, uint32_t layer_begin, uint32_t layer_end) {
@@ -643,21 +743,15 @@ int32_t brasa_model_run_layers(brasa_model *m, float *x, uint32_t tokens, uint32
     brasa_ctx *ctx = m->ctx;
     BRASA_TRY(check_tokens(m, tokens, pos0));
     BRASA_REQUIRE(ctx, layer_begin <= layer_end && layer_end <= m->cfg.layers, "layer range");
-    uint64_t n = (uint64_t)tokens * m->cfg.hidden * 4;
-    BRASA_TRY(brasa_buf_upload(m->x, 0, x, n));
+    if (m->family->begin) BRASA_TRY(m->family->begin(m, pos0, layer_begin, layer_end));
     brasa_cmd *cmd;
     BRASA_TRY(brasa_cmd_begin(ctx, &cmd));
-    int32_t rc = BRASA_OK;
-    if (tokens == 1 && decode_fused_ok(m)) {
-        rc = set_position(m, pos0);
-        if (rc == BRASA_OK) rc = encode_decode_token(m, cmd, layer_begin, layer_end, false);
-    }
-    else
-        for (uint32_t li = layer_begin; li < layer_end && rc == BRASA_OK; ++li) rc = encode_layer_prefill(m, cmd, li, tokens, pos0);
+    int32_t rc = m->family->run_layers(m, cmd, x, x, tokens, pos0, layer_begin, layer_end);
     int32_t rc2 = brasa_cmd_wait(cmd, nullptr);
     BRASA_TRY(rc);
     BRASA_TRY(rc2);
-    return brasa_buf_download(m->x, 0, x, n);
+    if (m->family->finish) m->family->finish(m, pos0 + tokens, layer_begin, layer_end);
+    return BRASA_OK;
 }
 
 int32_t brasa_model_decode_greedy(brasa_model *m, uint32_t first, uint32_t pos0, uint32_t steps, uint32_t *out_ids, double *gpu_seconds) {
@@ -665,7 +759,8 @@ int32_t brasa_model_decode_greedy(brasa_model *m, uint32_t first, uint32_t pos0,
     brasa_ctx *ctx = m->ctx;
     BRASA_REQUIRE(ctx, steps >= 1 && (uint64_t)pos0 + steps <= m->limits.ctx, "decode range outside the context");
     BRASA_REQUIRE(ctx, first < m->cfg.vocab, "token id %u outside the vocabulary", first);
-    BRASA_REQUIRE(ctx, decode_fused_ok(m), "the device-resident loop needs tiled q4_0 layers");
+    BRASA_REQUIRE(ctx, decode_resident_ok(m), "the device-resident loop needs tiled q4_0 layers");
+    if (m->family->begin) BRASA_TRY(m->family->begin(m, pos0, 0, m->cfg.layers));
     BRASA_TRY(brasa_buf_upload(m->ids, 0, &first, 4));
     uint32_t st[2] = {pos0, 0};  // position, output count
     BRASA_TRY(brasa_buf_upload(m->dev_state, 0, st, 8));
@@ -676,12 +771,14 @@ int32_t brasa_model_decode_greedy(brasa_model *m, uint32_t first, uint32_t pos0,
     int32_t rc2 = brasa_cmd_wait(cmd, gpu_seconds);
     BRASA_TRY(rc);
     BRASA_TRY(rc2);
+    if (m->family->finish) m->family->finish(m, pos0 + steps, 0, m->cfg.layers);
     return brasa_buf_download(m->out_ids, 0, out_ids, (uint64_t)steps * 4);
 }
 
 int32_t brasa_model_read_kv(brasa_model *m, uint32_t layer, int32_t which_v, uint32_t pos_begin, uint32_t pos_end, void *dst, uint64_t dst_bytes) {
     if (!m || !dst) return BRASA_EINVAL;
     brasa_ctx *ctx = m->ctx;
+    BRASA_REQUIRE(ctx, is_qwen3(m), "read_kv: the %s family has no K and V rows", m->family->name);
     BRASA_REQUIRE(ctx, layer < m->cfg.layers && pos_begin <= pos_end && pos_end <= m->limits.ctx, "read_kv: range");
     uint64_t kvd = (uint64_t)m->cfg.kv_heads * m->cfg.head_dim;
     uint64_t off = brasa_kv_bytes(m->limits.kv, ((uint64_t)layer * m->cap + pos_begin) * kvd);
@@ -708,13 +805,12 @@ extern "C" {
 int32_t brasa_session_create(brasa_ctx *ctx, const char *path, brasa_limits limits, uint64_t budget_bytes, brasa_session **out) {
     if (!ctx || !path || !out) return BRASA_EINVAL;
     *out = nullptr;
-    brasa_model_shape shape;
     brasa_config cfg;
     char err[512];
-    if (brasa_model_shape_from_file(path, &shape, &cfg, err, sizeof err) != BRASA_OK) return brasa_fail(ctx, BRASA_EIO, "%s", err);
+    if (brasa_model_shape_from_file(path, nullptr, &cfg, err, sizeof err) != BRASA_OK) return brasa_fail(ctx, BRASA_EIO, "%s", err);
     brasa_session_shape ss{limits.ctx, limits.max_tokens, limits.max_logit_rows, limits.kv};
     // the plan is checked before anything is loaded: a rejection allocates nothing
-    BRASA_TRY(brasa_plan_check(ctx, &shape, &ss, budget_bytes, nullptr, nullptr));
+    BRASA_TRY(brasa_plan_file(ctx, path, &ss, budget_bytes, nullptr, nullptr));
     BRASA_REQUIRE(ctx, cfg.head_row0 == 0, "a tensor-parallel shard cannot run as a session");
     brasa_model *m = nullptr;
     BRASA_TRY(brasa_model_load(ctx, path, limits, &m));
@@ -765,6 +861,8 @@ int32_t brasa_session_generate(brasa_session *s, const uint32_t *prompt, uint32_
     uint32_t common = 0;
     while (common < s->cached.size() && common < prompt_len && s->cached[common] == prompt[common]) ++common;
     common = std::min(common, prompt_len - 1);
+    // a state that cannot be rewound serves only prompts that go on from exactly where it stands
+    if (m->family->reached && (common != s->cached.size() || m->family->reached(m) != common)) common = 0;
     s->cached.resize(common);
 
     const bool greedy = params.temperature <= 0.0f;
@@ -799,7 +897,7 @@ int32_t brasa_session_generate(brasa_session *s, const uint32_t *prompt, uint32_
     auto t1 = clk::now();
     // Greedy with the fused decode path: the device keeps the position and feeds the chosen token back
     // itself; per token the host launches one graph and reads one id (pinned memory), nothing else.
-    const bool resident = device_pick && decode_fused_ok(m);
+    const bool resident = device_pick && decode_resident_ok(m);
     bool primed = false;  // device position and input token are set up
     // Resident decode keeps the device one step ahead of the host: the step that consumes token t + 1 (which the device
     // feeds itself) is queued before the host waits for the id of token t + 1, so the GPU never idles while the host
@@ -822,9 +920,13 @@ int32_t brasa_session_generate(brasa_session *s, const uint32_t *prompt, uint32_
         }
     } sev;
     uint32_t steps_launched = 0;  // resident steps queued so far; step i consumes the i-th token of this call and yields the next
+    std::vector<uint32_t> drawn;    // the tokens of this call
+    const uint32_t decode_pos0 = prompt_len;
     auto launch_step = [&]() -> int32_t {
         brasa_cmd step{ctx, nullptr, nullptr, false};
+        if (m->family->begin) BRASA_TRY(m->family->begin(m, decode_pos0 + steps_launched, 0, m->cfg.layers));
         BRASA_TRY(decode_step(m, &step, UINT32_MAX));
+        if (m->family->finish) m->family->finish(m, decode_pos0 + steps_launched + 1, 0, m->cfg.layers);
         const uint32_t slot = steps_launched & 1;
         BRASA_CUDA(ctx, cudaEventRecord(sev.done[slot], ctx->stream));
         BRASA_CUDA(ctx, cudaStreamWaitEvent(sev.copy, sev.done[slot], 0));
@@ -874,6 +976,7 @@ int32_t brasa_session_generate(brasa_session *s, const uint32_t *prompt, uint32_
         }
         if (generated == 0) ttft_ms = ms_since(t0);
         if (out_ids) out_ids[generated] = next;
+        drawn.push_back(next);
         ++generated;
         if (std::find(s->stop_ids.begin(), s->stop_ids.end(), next) != s->stop_ids.end()) {
             stop = 0;
@@ -903,6 +1006,10 @@ int32_t brasa_session_generate(brasa_session *s, const uint32_t *prompt, uint32_
         s->cached.push_back(next);
     }
     BRASA_TRY(brasa_ctx_sync(ctx));  // surfaces a device-side wait that gave up during the loop
+    // a step queued ahead has consumed a token the loop then ended on: where the state cannot be rewound it stays part of it
+    if (m->family->reached)
+        while (s->cached.size() < (size_t)prompt_len + steps_launched && s->cached.size() - prompt_len < drawn.size())
+            s->cached.push_back(drawn[s->cached.size() - prompt_len]);
     if (stats) {
         stats->prompt_tokens = prompt_len;
         stats->reused_tokens = common;

@@ -4,6 +4,7 @@
 
 #include "brasa_internal.h"
 #include "decode_token.h"
+#include "host_util.h"
 
 bool brasa_gemm_swiglu_fuses(const brasa_qmatrix &wg, const brasa_qmatrix &wu, uint32_t tokens);
 
@@ -30,8 +31,39 @@ struct Stager;
 
 using namespace brasa_model_detail;
 
+namespace brasa_stack {
+struct StackModel;
+}
+
+// What a model family provides to the model, session and planner entry points (model.cu holds the table of families).
+struct brasa_family {
+    const char *name;  // `.brasa` model family, or config.json "architecture"
+    bool (*describe)(const brasa::WeightFile &f, brasa_model_shape *shape, brasa_config *cfg, std::string &err);
+    int32_t (*plan)(brasa_ctx *ctx, const brasa::WeightFile &f, const brasa_session_shape &s, brasa_memory_plan *out);
+    // weights, per-sequence state and workspace of a model whose ctx, cfg and limits are set; staging holds the largest tensor
+    int32_t (*load)(brasa_model *m, const brasa::WeightFile &f, brasa_cmd *cmd, brasa_buf *staging);
+    void (*release)(brasa_model *m);
+    // ids in m->ids; logits of the given places among the tokens (host array) go to m->logits
+    int32_t (*forward)(brasa_model *m, brasa_cmd *cmd, uint32_t tokens, uint32_t pos0, const uint32_t *rows, uint32_t n_rows);
+    // one token m->ids[0] at the position in m->dev_state[0]: logits to m->logits, the greedy choice to m->next_id
+    int32_t (*step)(brasa_model *m, brasa_cmd *cmd);
+    int32_t (*run_layers)(brasa_model *m, brasa_cmd *cmd, const float *x, float *y, uint32_t tokens, uint32_t pos0, uint32_t l0, uint32_t l1);
+    // Families whose state cannot be rewound: begin checks that layers [l0, l1) can take a run at pos0 (their own position, or
+    // 0), finish notes the position they have reached, reached tells it. All null where any cached position can be continued from.
+    int32_t (*begin)(brasa_model *m, uint32_t pos0, uint32_t l0, uint32_t l1);
+    void (*finish)(brasa_model *m, uint32_t pos, uint32_t l0, uint32_t l1);
+    uint32_t (*reached)(brasa_model *m);
+};
+namespace brasa_stack {
+extern const brasa_family dunuzen_family;
+}
+// A tensor's bytes to dst on the device, through the loading model's pinned staging buffers.
+int32_t brasa_stage_upload(brasa_model *m, void *dst, const brasa::WeightFile &f, const brasa::TensorInfo &t);
+
 struct brasa_model {
     brasa_ctx *ctx = nullptr;
+    const brasa_family *family = nullptr;
+    brasa_stack::StackModel *stack = nullptr;  // families built on the layer stack (stack.cu); the Qwen3 members below stay empty
     brasa_tp *tp = nullptr;  // set for a tensor-parallel shard: residual adds are sums over ranks (not owned)
     brasa_config cfg{};
     brasa_limits limits{};

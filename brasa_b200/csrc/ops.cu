@@ -1,6 +1,7 @@
 // Element-wise, normalisation, RoPE, embedding and KV-store kernels
 // (crates/kernels/src/lib.rs:391-658, 976-1050 and the MSL files they dispatch).
 #include "brasa_internal.h"
+#include "tc_device.cuh"
 
 namespace {
 
@@ -138,6 +139,46 @@ __global__ void __launch_bounds__(128) rms_norm_block_kernel(const float *x, con
     }
 }
 
+// Layer norm: (x - mean) / sqrt(mean of squared deviations + eps) * w + b. One block per row; with NOUT = 2 one pass over the
+// row serves two consumers with their own weights. rows != nullptr picks the input rows.
+struct LayerNormParams {
+    const float *x;
+    const uint32_t *rows;
+    const float *w[2], *b[2];
+    void *out[2];
+    uint32_t n, ldo;
+    float eps;
+};
+template <int NOUT, typename T>
+__global__ void __launch_bounds__(256) layer_norm_kernel(LayerNormParams p) {
+    __shared__ float red[8];
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    const float *x = p.x + (size_t)(p.rows ? p.rows[blockIdx.x] : blockIdx.x) * p.n;
+    auto block_sum = [&](float v) {
+        for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+        if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+        __syncthreads();
+        v = ((red[0] + red[1]) + (red[2] + red[3])) + ((red[4] + red[5]) + (red[6] + red[7]));
+        __syncthreads();
+        return v;
+    };
+    float s = 0.0f;
+    for (uint32_t i = threadIdx.x; i < p.n; i += 256) s += x[i];
+    const float mean = block_sum(s) / (float)p.n;
+    s = 0.0f;
+    for (uint32_t i = threadIdx.x; i < p.n; i += 256) {
+        const float d = x[i] - mean;
+        s = fmaf(d, d, s);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(s) / (float)p.n + p.eps);
+    for (uint32_t i = threadIdx.x; i < p.n; i += 256) {
+        const float z = (x[i] - mean) * inv;
+#pragma unroll
+        for (int k = 0; k < NOUT; ++k) brasa_dev::elem_store(static_cast<T *>(p.out[k]) + (size_t)blockIdx.x * p.ldo + i, fmaf(z, p.w[k][i], p.b[k][i]));
+    }
+}
+
 __global__ void softmax_kernel(const float *x, float *out, uint32_t n) {
     __shared__ float red[32];
     const float *xr = x + (size_t)blockIdx.x * n;
@@ -200,6 +241,14 @@ __global__ void embed_kernel(const uint8_t *table, const uint32_t *ids, float *o
         q = (lo | (hi << 4)) - 32;
     }
     out[idx] = d * (float)q;
+}
+
+// Embedding gather out of a bf16 table, scaled: one thread per element.
+__global__ void embed_bf16_kernel(const uint16_t *table, uint32_t ld, uint32_t vocab, uint32_t n, float scale, const uint32_t *ids, float *out, uint32_t tokens) {
+    const uint64_t idx = (uint64_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (idx >= (uint64_t)tokens * n) return;
+    const uint32_t t = (uint32_t)(idx / n), col = (uint32_t)(idx % n), r = ids[t];
+    out[idx] = r < vocab ? __uint_as_float((uint32_t)table[(size_t)r * ld + col] << 16) * scale : 0.0f;
 }
 
 // x += h (optional); xw = x*w; ss[block] = sum of x^2 over this block's 256 elements
@@ -311,6 +360,26 @@ __global__ void store_kv_q8_kernel(const float *src, uint8_t *dst, uint64_t nblo
 inline unsigned blocks_for(uint64_t n, unsigned per) { return (unsigned)((n + per - 1) / per); }
 
 }  // namespace
+
+int32_t brasa_layer_norm_launch(brasa_cmd *cmd, const float *x, const uint32_t *rows, uint32_t n_rows, uint32_t n, float eps, const float *const *w,
+                                const float *const *b, void *const *out, uint32_t n_out, uint32_t ldo, bool f32) {
+    brasa_ctx *ctx = cmd->ctx;
+    if (n_rows == 0) return BRASA_OK;
+    LayerNormParams p{x, rows, {w[0], n_out > 1 ? w[1] : nullptr}, {b[0], n_out > 1 ? b[1] : nullptr}, {out[0], n_out > 1 ? out[1] : nullptr}, n, ldo, eps};
+    cudaError_t e;
+    if (f32) e = n_out > 1 ? brasa_launch_dependent(ctx, layer_norm_kernel<2, float>, dim3(n_rows), dim3(256), 0, p)
+                           : brasa_launch_dependent(ctx, layer_norm_kernel<1, float>, dim3(n_rows), dim3(256), 0, p);
+    else e = n_out > 1 ? brasa_launch_dependent(ctx, layer_norm_kernel<2, __nv_bfloat16>, dim3(n_rows), dim3(256), 0, p)
+                       : brasa_launch_dependent(ctx, layer_norm_kernel<1, __nv_bfloat16>, dim3(n_rows), dim3(256), 0, p);
+    BRASA_CUDA(ctx, e);
+    return brasa_post_launch(cmd, "layer_norm");
+}
+
+int32_t brasa_embed_bf16_launch(brasa_cmd *cmd, const uint16_t *table, uint32_t ld, uint32_t rows, uint32_t n, float scale, const uint32_t *ids, float *out,
+                                uint32_t tokens) {
+    embed_bf16_kernel<<<blocks_for((uint64_t)tokens * n, 256), 256, 0, cmd->ctx->stream>>>(table, ld, rows, n, scale, ids, out, tokens);
+    return brasa_post_launch(cmd, "embed_bf16");
+}
 
 extern "C" {
 

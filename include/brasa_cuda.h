@@ -39,7 +39,8 @@ extern "C" {
 /* crates/kernels/src/lib.rs:85-90 (discriminants in declaration order) */
 enum brasa_weight_type { BRASA_Q4_0 = 0, BRASA_Q8_0 = 1, BRASA_Q6_0 = 2 };
 /* crates/kernels/src/lib.rs:93-101 */
-enum brasa_kv_type { BRASA_KV_F32 = 0, BRASA_KV_F16 = 1, BRASA_KV_Q8_0 = 2 };
+/* (BF16: layer-stack families, whose cache type also names the precision of their products) */
+enum brasa_kv_type { BRASA_KV_F32 = 0, BRASA_KV_F16 = 1, BRASA_KV_Q8_0 = 2, BRASA_KV_BF16 = 3 };
 /* crates/kernels/src/lib.rs:1308-1314 */
 enum brasa_prefill_precision { BRASA_PREFILL_F16 = 0, BRASA_PREFILL_F32 = 1 };
 /* Byte layout of a quantised matrix in device memory.
@@ -266,6 +267,12 @@ typedef struct brasa_allocated { /* qwen3.rs:430 Allocated */
 
 /* BrasaFile::open + verify over a path: structure checks always, sha256 when verify != 0. */
 int32_t brasa_file_check(const char *path, int32_t verify, char *err, uint64_t err_len);
+/* path: a `.brasa` file, or a folder with config.json and model.safetensors (bf16 tensors), whose "architecture" names the
+ * family. Families: "qwen3", and the layer-stack family "Dunuzen". */
+int32_t brasa_model_family(const char *path, char *name, uint64_t name_len); /* the family's name, or the reason for BRASA_EIO */
+/* The plan of a session over the model at path, any family (brasa_plan_check for brasa_plan of that family). */
+int32_t brasa_plan_file(brasa_ctx *ctx, const char *path, const brasa_session_shape *s, uint64_t budget_bytes, brasa_memory_plan *out,
+                        uint32_t *max_ctx_out);
 int32_t brasa_model_shape_from_file(const char *path, brasa_model_shape *shape, brasa_config *cfg, char *err, uint64_t err_len); /* qwen3.rs:79 */
 
 int32_t brasa_model_load(brasa_ctx *ctx, const char *path, brasa_limits limits, brasa_model **out); /* Qwen3::load :345 */
@@ -280,6 +287,11 @@ int32_t brasa_model_set_prefill_precision(brasa_model *m, int32_t precision); /*
 /* Qwen3::forward :763. ids: host u32[tokens]; logits: host f32[logit_rows * vocab] (may be NULL to
  * leave them on the device); gpu_seconds: device time of the call (may be NULL). */
 int32_t brasa_model_forward(brasa_model *m, const uint32_t *ids, uint32_t tokens, uint32_t pos0, uint32_t logit_rows, float *logits, double *gpu_seconds);
+/* The same with logits of any places among the run's tokens: rows: host u32[n_rows], n_rows <= max_logit_rows (0: none).
+ * A family with recurrent state takes a run at position 0 (a new sequence) or where its state stands; anything else is
+ * BRASA_EINVAL. */
+int32_t brasa_model_forward_rows(brasa_model *m, const uint32_t *ids, uint32_t tokens, uint32_t pos0, const uint32_t *rows, uint32_t n_rows, float *logits,
+                                 double *gpu_seconds);
 /* Qwen3::run_layers :743. x: host f32[tokens*hidden], replaced by the output. */
 int32_t brasa_model_run_layers(brasa_model *m, float *x, uint32_t tokens, uint32_t pos0, uint32_t layer_begin, uint32_t layer_end);
 /* Device-resident decode: feeds the token chosen on the device back as the next input for `steps`
