@@ -23,6 +23,8 @@ tokens with an f16 KV cache, ctx 2048. One step = the 255 decode forwards that f
 `tp32b`   the Qwen3-32B architecture decoded tensor-parallel over all ranks of the job (batch 1 and batch 16), with a
           split-versus-unsplit parity check on a reduced model; at one rank the whole model runs on one GPU.
 
+--dunuzen times prefill and decode of Dunuzen models (bf16) at a few sizes beside Qwen3 models of equal size, and nothing else.
+
 With --gpus N > 1 (launched by torch.distributed.run) every rank serves its own replica: the path has
 no exchange step at batch 1, so the ranks share nothing and the aggregate is the sum ("replicas only").
 --impl reference times the reference's CPU path alone (rank 0 only): tools/qwen3_ref.py from oracle/_ref/ when that was
@@ -792,6 +794,81 @@ def kernel_roofline(B, ctx, K, cfg, peak, peak_kind, profile=False):
     return roof
 
 
+# --dunuzen: layers of a real model's size, random weights, beside a Qwen3 model of the same width, FFN, heads and depth
+DUNUZEN_SIZES = {"2048": dict(width=2048, ff=8192, heads=16, kv_heads=16, window=1024),
+                 "2560": dict(width=2560, ff=9728, heads=32, kv_heads=16, window=1024),
+                 "4096": dict(width=4096, ff=14336, heads=32, kv_heads=32, window=4096)}
+DUNUZEN_LAYERS, DUNUZEN_VOCAB = ["latent_attention", "channel_delta"] * 4, 32768
+
+
+def dunuzen_leg(B, ctx, tag: str, steps: int, warmup: int, tokens: int = 4096, decode: int = 128, models=("dunuzen", "qwen3"), chunk: int = 2048) -> dict:
+    """Prefill of `tokens` tokens and greedy decode behind them, for a Dunuzen model (bf16) and a Qwen3 model (q4_0, f16 cache)
+    of equal width, FFN width, heads and depth. Device time; every decode step reads more weights than L2 holds."""
+    from brasa_b200 import synth
+    size = DUNUZEN_SIZES[tag]
+    hbm, _ = measured_peaks()
+    tc = tensor_peak() or 1590.0
+    out = {"size": size, "layers": len(DUNUZEN_LAYERS), "vocab": DUNUZEN_VOCAB, "prompt_tokens": tokens}
+    ids = np.random.default_rng(SEED).integers(0, DUNUZEN_VOCAB, size=tokens).astype(np.uint32)
+    ctx_len = tokens + (warmup + steps + 1) * decode + 64
+    for name in models:
+        if name == "dunuzen":
+            cfg = synth.dunuzen_config(layers=DUNUZEN_LAYERS, vocab=DUNUZEN_VOCAB, **size)
+            path = model_path(f"dunuzen-{tag}").with_suffix("")
+            if not (path / "config.json").exists():
+                synth.write_synthetic_dunuzen(path, cfg, SEED)
+            flops = synth.dunuzen_prefill_flops(cfg, tokens)
+            step_bytes = lambda p: synth.dunuzen_decode_bytes(cfg, p)
+        else:
+            cfg = dict(synth.QWEN3_4B, hidden_size=size["width"], intermediate_size=size["ff"], num_attention_heads=size["heads"],
+                       num_hidden_layers=len(DUNUZEN_LAYERS), vocab_size=DUNUZEN_VOCAB)
+            path = model_path(f"qwen3-like-dunuzen-{tag}")
+            if not path.exists():
+                synth.write_synthetic_model(ctx, path, cfg, SEED)
+            mm = sum(2 * tokens * int(np.prod(sh)) for n, sh in synth.tensor_shapes(cfg).items() if len(sh) == 2 and "embed" not in n)
+            flops = {"matmul": mm, "attention": 4 * tokens * (tokens + 1) // 2 * cfg["num_attention_heads"] * 128 * cfg["num_hidden_layers"]}
+            step_bytes = lambda p: synth.weight_bytes_per_token(cfg) + synth.kv_bytes_per_position(cfg) * (p + 1)
+        m = B.model_class(path).load_in(ctx, path, "bfloat16", ctx_len, chunk)
+
+        def prefill():
+            return sum(m.forward(ids[o:o + chunk], o, want_logits=False)[1] for o in range(0, tokens, chunk))
+        for _ in range(max(3, warmup)):
+            prefill()
+        pre = [prefill() for _ in range(steps)]
+        first, pos, dec = int(np.argmax(m.forward(ids[:chunk], 0)[0][0])), chunk, []
+        for o in range(chunk, tokens, chunk):
+            m.forward(ids[o:o + chunk], o, want_logits=False)
+            pos = o + chunk
+        for i in range(max(3, warmup) + steps):
+            if pos + decode > ctx_len:
+                break
+            _, s = m.decode_greedy(first, pos, decode)
+            pos += decode
+            if i >= max(3, warmup):
+                dec.append(s)
+        p_s, t_s = statistics.median(pre), statistics.median(dec) / decode
+        total = flops["matmul"] + flops["attention"]
+        nbytes = step_bytes(pos - decode // 2)
+        out[name] = {"prefill_tok_s": tokens / p_s, "prefill_ms": p_s * 1e3, "prefill_tflops": total / p_s / 1e12, "prefill_frac_of_measured_bf16": total / p_s / 1e12 / tc,
+                     "decode_tok_s": 1.0 / t_s, "decode_us_per_token": t_s * 1e6, "decode_bytes_per_token": nbytes, "decode_gbs": nbytes / t_s / 1e9,
+                     "decode_frac_of_measured_hbm": nbytes / t_s / 1e9 / hbm}
+        m.free()
+    return out
+
+
+def run_dunuzen(args) -> None:
+    import brasa_b200 as B
+    ctx = B.Context(0)
+    tags = list(DUNUZEN_SIZES) if args.dunuzen == "all" else args.dunuzen.split(",")
+    models = tuple(args.dunuzen_models.split(","))
+    with ClockSampler(0) as clocks:
+        legs = {t: dunuzen_leg(B, ctx, t, args.steps, args.warmup, tokens=args.dunuzen_tokens, decode=min(128, args.decode_tokens), models=models) for t in tags}
+    first = legs[tags[0]].get("dunuzen") or legs[tags[0]]["qwen3"]
+    print(json.dumps({"metric": "dunuzen_decode_tok_s", "value": first["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+                      "higher_is_better": True, "data": "synthetic", "dtype": "bf16", "config": {"sizes": tags, "l2": "weights of a step exceed L2"},
+                      "clocks": clocks.summary(), "legs": legs}))
+
+
 def run_ours(args, rank: int, world: int, local_rank: int):
     import brasa_b200 as B
     from brasa_b200 import synth
@@ -1064,7 +1141,12 @@ def main():
     ap.add_argument("--serving-steps", type=int, default=512)
     ap.add_argument("--only-decode", action="store_true",
                     help="run only the device-resident decode loop (profiler captures): no end-to-end, kernel or CPU legs")
+    ap.add_argument("--dunuzen", default="", help="run only the Dunuzen legs: all, or some of " + ", ".join(DUNUZEN_SIZES) + " separated by commas")
+    ap.add_argument("--dunuzen-models", default="dunuzen,qwen3", help="which models those legs run (profiler captures take one)")
+    ap.add_argument("--dunuzen-tokens", type=int, default=4096)
     args = ap.parse_args()
+    if args.dunuzen:
+        return run_dunuzen(args)
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))

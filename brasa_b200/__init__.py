@@ -96,6 +96,17 @@ class _PagedKv(C.Structure):
                 ("num_pages", C.c_uint32), ("kv", C.c_int32)]
 
 
+class _Linear(C.Structure):
+    _fields_ = ([(n, _Arg) for n in ("w", "x", "w2", "x2", "y", "bias", "resid")] +
+                [(n, C.c_uint32) for n in ("cols", "ldw", "ldx", "cols2", "ldw2", "ldx2", "rows", "tokens", "ldy")] +
+                [("y_bf16", C.c_int32), ("act", C.c_int32), ("scale", C.c_float)])
+
+
+class _WindowAttn(C.Structure):
+    _fields_ = ([(n, _Arg) for n in ("q", "k", "v", "kr", "cos_t", "sin_t", "gate", "out")] +
+                [(n, C.c_uint32) for n in ("tokens", "heads", "dim", "rot", "rot_dims", "vdim", "pos0", "key0", "window")] + [("scale", C.c_float)])
+
+
 class _ModelShape(C.Structure):
     _fields_ = [("weight_bytes", C.c_uint64), ("layers", C.c_uint32), ("hidden", C.c_uint32), ("heads", C.c_uint32),
                 ("kv_heads", C.c_uint32), ("head_dim", C.c_uint32), ("ffn", C.c_uint32), ("vocab", C.c_uint32)]
@@ -565,6 +576,26 @@ class Kernels:
 
     def flash_attention_with(self, cmd, q, k, v, o, shape: AttnShape, precision):
         self._k(self.L.brasa_k_flash_attention_with(cmd._h, _arg(q), _arg(k), _arg(v), _arg(o), shape._c(), C.c_int32(int(precision))))
+
+    # bf16 operators of the layer-stack families
+    def layer_norm(self, cmd, x, w, b, out, rows, n, eps):
+        self._k(self.L.brasa_k_layer_norm(cmd._h, _arg(x), _arg(w), _arg(b), _arg(out), C.c_uint32(rows), C.c_uint32(n), C.c_float(eps)))
+
+    @staticmethod
+    def linear_problem(w, x, y, rows: int, cols: int, tokens: int, ldw=None, ldx=None, ldy=None, w2=None, x2=None, cols2=0, ldw2=0, ldx2=0, bias=None,
+                       resid=None, y_bf16=False, relu2=False, scale=1.0) -> _Linear:
+        return _Linear(_arg(w), _arg(x), _arg(w2), _arg(x2), _arg(y), _arg(bias), _arg(resid), cols, ldw or cols, ldx or cols, cols2, ldw2 or cols2,
+                       ldx2 or cols2, rows, tokens, ldy or rows, int(y_bf16), int(relu2), scale)
+
+    def linear(self, cmd, problems, f32_inputs: bool):
+        """Up to eight products with bf16 weights in one launch (linear_problem)."""
+        arr = (_Linear * len(problems))(*problems)
+        self._k(self.L.brasa_k_linear(cmd._h, arr, C.c_uint32(len(problems)), C.c_int32(int(f32_inputs))))
+
+    def window_attention(self, cmd, q, k, v, kr, table: RopeTable, gate, out, tokens, heads, dim, rot, vdim, pos0, key0, window, scale, f32: bool):
+        a = _WindowAttn(_arg(q), _arg(k), _arg(v), _arg(kr), _arg(table.cos), _arg(table.sin), _arg(gate), _arg(out), tokens, heads, dim, rot, table.dim, vdim,
+                        pos0, key0, window, scale)
+        self._k(self.L.brasa_k_window_attention(cmd._h, a, C.c_int32(int(f32))))
 
     def argmax(self, cmd, logits, n, out):
         self._k(self.L.brasa_k_argmax(cmd._h, _arg(logits), C.c_uint32(n), _arg(out)))

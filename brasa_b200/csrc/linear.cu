@@ -606,3 +606,31 @@ int32_t brasa_linear_gemv_launch(brasa_cmd *cmd, const GemvInput &in, const Gemv
 #undef GEMV_LAUNCH
     return brasa_post_launch(cmd, "linear_gemv");
 }
+
+extern "C" int32_t brasa_k_linear(brasa_cmd *cmd, const brasa_linear *ps, uint32_t count, int32_t f32_inputs) {
+    if (!cmd || !ps) return BRASA_EINVAL;
+    brasa_ctx *ctx = cmd->ctx;
+    BRASA_REQUIRE(ctx, count >= 1 && count <= LINEAR_MAX, "linear: 1 to %u products", LINEAR_MAX);
+    LinearProblem q[LINEAR_MAX];
+    const uint64_t xe = f32_inputs ? 4 : 2;
+    for (uint32_t i = 0; i < count; ++i) {
+        const brasa_linear &p = ps[i];
+        BRASA_REQUIRE(ctx, p.rows > 0 && p.tokens > 0 && p.cols > 0 && p.ldy >= p.rows, "linear: empty product");
+        BRASA_REQUIRE(ctx, arg_fits(p.w, (uint64_t)p.rows * p.ldw * 2) && arg_fits(p.x, (uint64_t)p.tokens * p.ldx * xe), "linear: w or x too small");
+        BRASA_REQUIRE(ctx, !p.cols2 || (arg_fits(p.w2, (uint64_t)p.rows * p.ldw2 * 2) && arg_fits(p.x2, (uint64_t)p.tokens * p.ldx2 * xe)), "linear: w2 or x2 too small");
+        BRASA_REQUIRE(ctx, arg_fits(p.y, (uint64_t)p.tokens * p.ldy * (p.y_bf16 ? 2 : 4)), "linear: y too small");
+        BRASA_REQUIRE(ctx, (!p.bias.buf || arg_fits(p.bias, (uint64_t)p.rows * 4)) && (!p.resid.buf || arg_fits(p.resid, (uint64_t)p.tokens * p.ldy * 4)), "linear: bias or resid too small");
+        q[i].seg[0] = LinearSeg{(const uint16_t *)arg_ptr(p.w), p.ldw, arg_ptr(p.x), p.ldx, p.cols};
+        if (p.cols2) q[i].seg[1] = LinearSeg{(const uint16_t *)arg_ptr(p.w2), p.ldw2, arg_ptr(p.x2), p.ldx2, p.cols2};
+        q[i].rows = p.rows;
+        q[i].tokens = p.tokens;
+        q[i].y = arg_ptr(p.y);
+        q[i].ldy = p.ldy;
+        q[i].y_bf16 = p.y_bf16 != 0;
+        q[i].bias = (const float *)arg_ptr(p.bias);
+        q[i].resid = (const float *)arg_ptr(p.resid);
+        q[i].act = p.act;
+        q[i].scale = p.scale;
+    }
+    return brasa_linear_launch(cmd, q, count, f32_inputs != 0);
+}

@@ -383,6 +383,16 @@ int32_t brasa_embed_bf16_launch(brasa_cmd *cmd, const uint16_t *table, uint32_t 
 
 extern "C" {
 
+int32_t brasa_k_layer_norm(brasa_cmd *cmd, brasa_arg x, brasa_arg w, brasa_arg b, brasa_arg out, uint32_t rows, uint32_t n, float eps) {
+    if (!cmd) return BRASA_EINVAL;
+    brasa_ctx *ctx = cmd->ctx;
+    BRASA_REQUIRE(ctx, n > 0 && arg_fits(x, (uint64_t)rows * n * 4) && arg_fits(out, (uint64_t)rows * n * 4) && arg_fits(w, (uint64_t)n * 4) && arg_fits(b, (uint64_t)n * 4),
+                  "layer_norm: a buffer is too small");
+    const float *ws[2] = {(const float *)arg_ptr(w), nullptr}, *bs[2] = {(const float *)arg_ptr(b), nullptr};
+    void *outs[2] = {arg_ptr(out), nullptr};
+    return brasa_layer_norm_launch(cmd, (const float *)arg_ptr(x), nullptr, rows, n, eps, ws, bs, outs, 1, n, true);
+}
+
 int32_t brasa_k_add(brasa_cmd *cmd, brasa_arg a, brasa_arg b, brasa_arg out, uint64_t n) {
     if (!cmd) return BRASA_EINVAL;
     brasa_ctx *ctx = cmd->ctx;

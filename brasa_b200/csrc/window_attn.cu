@@ -472,3 +472,35 @@ int32_t brasa_window_attention_launch(brasa_cmd *cmd, const WindowAttn &a, bool 
     }
     return launch_window_simt<__nv_bfloat16>(cmd, a);
 }
+
+extern "C" int32_t brasa_k_window_attention(brasa_cmd *cmd, brasa_window_attn p, int32_t f32) {
+    if (!cmd) return BRASA_EINVAL;
+    brasa_ctx *ctx = cmd->ctx;
+    BRASA_REQUIRE(ctx, p.tokens > 0 && p.heads > 0 && p.dim > 0 && p.rot > 0 && p.vdim > 0 && p.window > 0 && p.key0 <= p.pos0, "window attention: empty shape");
+    BRASA_REQUIRE(ctx, p.rot % 8 == 0 && (p.key0 == 0 || p.key0 + p.window <= p.pos0 + 1), "window attention: rot must be a multiple of 8 and every visible key present");
+    const uint64_t keys = (uint64_t)p.pos0 + p.tokens - p.key0, e = f32 ? 4 : 2, last = (uint64_t)p.pos0 + p.tokens;
+    BRASA_REQUIRE(ctx, arg_fits(p.q, (uint64_t)p.tokens * p.heads * (p.dim + p.rot) * 4) && arg_fits(p.k, keys * p.heads * p.dim * e) &&
+                           arg_fits(p.v, keys * p.heads * p.vdim * e) && arg_fits(p.kr, keys * p.rot * e) && arg_fits(p.gate, (uint64_t)p.tokens * p.heads * 4) &&
+                           arg_fits(p.out, (uint64_t)p.tokens * p.heads * p.vdim * e) && arg_fits(p.cos_t, last * (p.rot_dims / 2) * 4) &&
+                           arg_fits(p.sin_t, last * (p.rot_dims / 2) * 4),
+                  "window attention: a buffer is too small");
+    for (const brasa_arg *a : {&p.k, &p.v, &p.kr, &p.out}) BRASA_REQUIRE(ctx, a->offset % 16 == 0, "window attention: misaligned buffer");
+    WindowAttn a{};
+    a.q = (const float *)arg_ptr(p.q);
+    a.k = arg_ptr(p.k);
+    a.v = arg_ptr(p.v);
+    a.kr = arg_ptr(p.kr);
+    a.cos_t = (const float *)arg_ptr(p.cos_t);
+    a.sin_t = (const float *)arg_ptr(p.sin_t);
+    a.gate = (const float *)arg_ptr(p.gate);
+    a.out = arg_ptr(p.out);
+    a.ldq = p.heads * (p.dim + p.rot);
+    a.ldk = p.heads * p.dim;
+    a.ldv = a.ldo = p.heads * p.vdim;
+    a.ldr = p.rot;
+    a.ldg = p.heads;
+    a.tokens = p.tokens; a.heads = p.heads; a.dim = p.dim; a.rot = p.rot; a.rot_dims = p.rot_dims; a.vdim = p.vdim;
+    a.pos0 = p.pos0; a.key0 = p.key0; a.keys = (uint32_t)keys; a.window = p.window;
+    a.scale = p.scale;
+    return brasa_window_attention_launch(cmd, a, f32 != 0);
+}

@@ -134,3 +134,100 @@ def weight_bytes_per_token(cfg: dict) -> int:
 def kv_bytes_per_position(cfg: dict, kv: str = "f16") -> int:
     rows = 2 * cfg["num_hidden_layers"] * cfg["num_key_value_heads"]
     return rows * {"f32": 512, "f16": 256, "q8_0": 136}[kv]
+
+
+# ---- Dunuzen: config.json + model.safetensors with seeded bf16 weights, drawn on the host --------------------------------
+
+
+def dunuzen_config(width: int, ff: int, heads: int, kv_heads: int, layers: list[str], vocab: int, window: int, dim: int = 128, rot_dim: int = 64,
+                   vdim: int = 128, kv_rank: int = 512, conv: int = 4) -> dict:
+    """A configuration of uniform layers; `layers` names the mixer of each."""
+    mixers = {"latent_attention": {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "mask": {"size": window},
+                                   "rot": {"base": 10000.0, "dims": rot_dim}, "scale": (dim + rot_dim) ** -0.5},
+              "channel_delta": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}}
+    return {"architecture": "Dunuzen", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-5}, "logit_scale": 1.0,
+            "layers": [{"type": t, "mixer": mixers[t], "mlp": {"kind": "dense", "ff": ff}} for t in layers]}
+
+
+def dunuzen_shapes(cfg: dict, rank: int = 128) -> dict[str, list[int]]:
+    """name -> shape; rank: inner size of the decay's and the output gate's projections."""
+    w, t = cfg["width"], {"embed": [cfg["vocab"], cfg["width"]]}
+    for i, layer in enumerate(cfg["layers"]):
+        m, p, x = layer["mixer"], f"l{i}.", f"l{i}.mix."
+        for n in ("norm1", "norm2"):
+            t.update({p + n: [w], p + n + ".b": [w]})
+        if layer["type"] == "latent_attention":
+            h, kr = m["heads"], m["kv_rank"]
+            t.update({x + "q": [h * (m["dim"] + m["rot_dim"]), w], x + "dkv": [kr + m["rot_dim"], w], x + "dkv.norm": [kr], x + "uk": [h * m["dim"], kr],
+                      x + "uv": [h * m["vdim"], kr], x + "g": [h, w], x + "o": [w, h * m["vdim"]]})
+        else:
+            h, qk, vd = m["heads"], m["kv_heads"] * m["dim"], m["heads"] * m["vdim"]
+            t.update({x + "q": [qk, w], x + "q.conv": [qk, m["conv"]], x + "k": [qk, w], x + "k.conv": [qk, m["conv"]], x + "v": [vd, w],
+                      x + "v.conv": [vd, m["conv"]], x + "b": [h, w], x + "A_log": [h], x + "norm": [m["vdim"]], x + "a1": [rank, w],
+                      x + "a2": [h * m["dim"], rank], x + "dt_bias": [h * m["dim"]], x + "g1": [rank, w], x + "g2": [vd, rank], x + "o": [w, vd]})
+        f = layer["mlp"]["ff"]
+        t.update({p + "mlp.up": [f, w], p + "mlp.up.b": [f], p + "mlp.down": [w, f], p + "mlp.down.b": [w]})
+    t.update({"final.norm": [w], "final.norm.b": [w], "head": [cfg["vocab"], w]})
+    return t
+
+
+def write_synthetic_dunuzen(folder, cfg: dict, seed: int = 0, std: float = 0.02, rank: int = 128) -> None:
+    """Seeded N(0, std) matrices, norm weights of ones, biases of zeros; drawn and rounded tensor by tensor in parallel."""
+    import concurrent.futures
+    import os
+    folder = pathlib.Path(folder)
+    folder.mkdir(parents=True, exist_ok=True)
+    shapes = dunuzen_shapes(cfg, rank)
+    header, at = {}, 0
+    for name, shape in shapes.items():
+        n = 2 * int(np.prod(shape))
+        header[name] = {"dtype": "BF16", "shape": shape, "data_offsets": [at, at + n]}
+        at += n
+    js = json.dumps(header).encode()
+    js += b" " * (-len(js) % 8)
+
+    def draw(item):
+        i, (name, shape) = item
+        if len(shape) == 1:
+            w = np.full(shape, 1.0 if "norm" in name and not name.endswith(".b") else 0.0, np.float32)
+        else:
+            w = np.random.Generator(np.random.SFC64([seed, i])).standard_normal(shape, dtype=np.float32)
+            w *= np.float32(0.5 if name.endswith(".conv") else std)
+        b = w.view(np.uint32)
+        return name, ((b + np.uint32(0x8000)) >> np.uint32(16)).astype("<u2")
+
+    tmp = folder / f"model.safetensors.{os.getpid()}.tmp"
+    with open(tmp, "wb") as f, concurrent.futures.ThreadPoolExecutor(max_workers=min(16, os.cpu_count() or 1)) as ex:
+        f.write(struct.pack("<Q", len(js)) + js)
+        for name, data in ex.map(draw, enumerate(shapes.items())):
+            f.seek(8 + len(js) + header[name]["data_offsets"][0])
+            f.write(data.tobytes())
+    os.replace(tmp, folder / "model.safetensors")
+    (folder / "config.json").write_text(json.dumps(cfg))
+
+
+def dunuzen_decode_bytes(cfg: dict, pos: int, rank: int = 128) -> int:
+    """Bytes one bf16 decode step at position pos has to move: every matrix once, the states read and written, the visible rows."""
+    total = 2 * sum(int(np.prod(s)) for n, s in dunuzen_shapes(cfg, rank).items() if n != "embed") + 2 * cfg["width"]
+    for layer in cfg["layers"]:
+        m = layer["mixer"]
+        if layer["type"] == "latent_attention":
+            total += 2 * min(pos + 1, m["mask"]["size"]) * (m["kv_rank"] + m["rot_dim"])
+        else:
+            total += 8 * m["heads"] * m["dim"] * m["vdim"]
+    return total
+
+
+def dunuzen_prefill_flops(cfg: dict, tokens: int, rank: int = 128) -> dict:
+    """Operations of a prompt of `tokens` tokens: products with weights, attention inside the window, delta rule."""
+    mm = sum(2 * tokens * int(np.prod(s)) for n, s in dunuzen_shapes(cfg, rank).items() if len(s) == 2 and n not in ("embed", "head") and not n.endswith(".conv"))
+    attn = delta = 0
+    for layer in cfg["layers"]:
+        m = layer["mixer"]
+        if layer["type"] == "latent_attention":
+            w = min(m["mask"]["size"], tokens)
+            pairs = w * (w + 1) // 2 + (tokens - w) * w
+            attn += 2 * pairs * m["heads"] * (m["dim"] + m["rot_dim"] + m["vdim"])
+        else:
+            delta += 7 * tokens * m["heads"] * m["dim"] * m["vdim"]
+    return {"matmul": mm, "attention": attn, "delta": delta}

@@ -206,6 +206,34 @@ int32_t brasa_k_decode_attention_static(brasa_cmd *cmd, brasa_arg q, brasa_arg k
 int32_t brasa_k_flash_attention_with(brasa_cmd *cmd, brasa_arg q, brasa_arg k, brasa_arg v, brasa_arg o, brasa_attn_shape shape, int32_t precision);
 int32_t brasa_k_flash_attention(brasa_cmd *cmd, brasa_arg q, brasa_arg k, brasa_arg v, brasa_arg o_f16, brasa_attn_shape shape); /* :1169 */
 
+/* ---- bf16 operators of the layer-stack families (no counterpart in the reference, whose weights are quantised) ---- */
+
+/* out[r, :] = (x[r, :] - mean) / sqrt(mean square deviation + eps) * w + b, all f32 */
+int32_t brasa_k_layer_norm(brasa_cmd *cmd, brasa_arg x, brasa_arg w, brasa_arg b, brasa_arg out, uint32_t rows, uint32_t n, float eps);
+/* y[t, r] = resid[t, r] + scale * act(w[r, :] . x[t, :] (+ w2[r, :] . x2[t, :]) + bias[r]) with bf16 row-major weights. Leading
+ * dimensions in elements, multiples of 8. Optional parts have buf NULL (w2: cols2 = 0). */
+enum brasa_linear_act { BRASA_ACT_NONE = 0, BRASA_ACT_RELU2 = 1 /* relu(v)^2 */ };
+typedef struct brasa_linear {
+    brasa_arg w, x, w2, x2, y, bias, resid; /* bias f32[rows]; resid f32[tokens][ldy], may be y */
+    uint32_t cols, ldw, ldx, cols2, ldw2, ldx2, rows, tokens, ldy;
+    int32_t y_bf16; /* y in bf16 instead of f32 */
+    int32_t act;
+    float scale;
+} brasa_linear;
+/* up to 8 such products in one launch. f32_inputs 0: x in bf16, tcgen05 with f32 accumulation; 1: x in f32, f32 FMA. */
+int32_t brasa_k_linear(brasa_cmd *cmd, const brasa_linear *p, uint32_t count, int32_t f32_inputs);
+/* Attention of tokens queries at positions pos0 .. over keys at positions key0 .. pos0 + tokens - 1, each query seeing its own
+ * position and the window - 1 before it. A head's key has a part of its own (dim) and one shared by all heads (rot); q f32
+ * [tokens][heads][dim + rot] is rotated here (pairs i, i + rot_dims / 2 of the shared part; cos_t / sin_t f32
+ * [position][rot_dims / 2]), kr comes rotated. out = softmax(scale * score) v * sigmoid(gate). k [keys][heads][dim], v
+ * [keys][heads][vdim], kr [keys][rot], out [tokens][heads][vdim]: bf16, or f32 with f32 != 0; gate f32 [tokens][heads]. */
+typedef struct brasa_window_attn {
+    brasa_arg q, k, v, kr, cos_t, sin_t, gate, out;
+    uint32_t tokens, heads, dim, rot, rot_dims, vdim, pos0, key0, window;
+    float scale;
+} brasa_window_attn;
+int32_t brasa_k_window_attention(brasa_cmd *cmd, brasa_window_attn a, int32_t f32);
+
 /* ---- sampling on the device (crates/runtime/src/sampler.rs) --------------------------------- */
 
 /* first index of the maximum, NaN ignored, 0 when nothing exceeds -inf (:148-170); out: one u32 */
