@@ -4,11 +4,8 @@
 //   F = diag(g) S_old,  u = beta (v - F^T k),  S_new = F + k u^T,  o = S_new^T q
 // q, k and v come out of a short causal convolution and silu, q and k as unit vectors, g out of a softplus.
 //
-// Many tokens: delta_prep_kernel forms q, k, v, g and beta of every token side by side; delta_scan_kernel then walks the
-// tokens with the state in registers. 16 lanes share a state column (each a slice of the key channels), and because
-// S_new^T q = F^T q + u (k . q), both reductions of a token run together and a token costs one exchange between
-// lanes. Everything is f32 FMA in the order of the tokens, so a sequence cut into portions gives the same bits.
-// One token: delta_step_kernel does all of it, one block per head.
+// Many tokens: chunks of 16, everything that does not depend on the state for all chunks side by side, then the state through
+// the chunks (below). One token: delta_step_kernel does all of it, one block per head. Everything is f32 FMA.
 //
 // Per-sequence state: S [heads][dim][vdim] and the convolution's inputs as a ring of `taps` rows, position p in row p % taps
 // (one more row than needed, so that a step can store its own row while others still read the older ones). A sequence
@@ -58,87 +55,163 @@ __device__ __forceinline__ float conv_at(const float *x, uint32_t ldx, uint32_t 
     return s;
 }
 
-struct DeltaPrep {
+// ---- many tokens -------------------------------------------------------------------------------------------------------
+// Tokens go in chunks of CH. Inside a chunk write c_t for the product of the decays up to token t and let
+//   A[t][s] = sum k_t k_s c_t / c_s (s < t),  B[t][s] = sum q_t k_s c_t / c_s (s <= t)      (sums over key channels)
+// Unrolling the recurrence over the chunk gives, with the state S before it,
+//   U = T (V - K' S),  T = (I + diag(beta) A)^-1 diag(beta),  K'_t = c_t k_t
+//   O = Q' S + B U,  Q'_t = c_t q_t
+//   S_next = diag(c_last) S + K''^T U,  K''_s = k_s c_last / c_s
+// T and B do not depend on the state: delta_chunk_kernel forms them for all chunks side by side, together with q, k, v and g.
+// delta_scan_kernel then carries the state through the chunks with products instead of one reduction per token. The ratios
+// c_t / c_s are always formed as products of the decays between s and t, never by division.
+constexpr uint32_t CH = 16;
+
+struct DeltaChunk {
     DeltaShape s;
     ConvView cv;
-    const float *q, *k, *v, *b, *z;       // products [tokens][ld]
-    uint32_t ldqk, ldv, ldb, ldz;
+    const float *q, *k, *v, *b, *z;  // products [tokens][ld]
+    uint32_t ldqk, ldv, ldb, ldz, tokens;
     const float *wq, *wk, *wv, *a_log;
-    float *qn, *kn, *vn, *g, *beta, *kq;  // [tokens][qk], [qk], [vd], [heads * dim], [heads], [kv_heads]
+    float *qn, *kn, *vn, *g, *tb;    // [tokens][qk], [qk], [vd], [heads * dim]; [chunks][heads][T, B][CH][CH]
 };
 
-// One warp per kv head (q and k), head (v) or head (g and beta) of a token.
-__global__ void __launch_bounds__(256) delta_prep_kernel(DeltaPrep p) {
-    pdl_wait();
-    pdl_launch();
-    const DeltaShape s = p.s;
-    const uint32_t t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, items = s.kv_heads + 2 * s.heads;
-    for (uint32_t it = blockIdx.y * 8 + warp; it < items; it += gridDim.y * 8) {
-        if (it < s.kv_heads) {
-            float q[8], k[8], qq = 0.0f, kk = 0.0f, kq = 0.0f;
+// convolution and silu of one channel for the chunk's tokens, handed to put(t, value)
+template <typename Put>
+__device__ __forceinline__ void conv_chunk(const float *x, uint32_t ldx, uint32_t c, const float *w, uint32_t t0, uint32_t n, const ConvView &cv, uint32_t ch, Put put) {
+    if (cv.taps <= 4) {  // the window in registers
+        float wr[4], xr[4];
 #pragma unroll
-            for (int j = 0; j < 8; ++j) {
-                const uint32_t i = lane + 32 * j, c = it * s.dim + i;
-                q[j] = k[j] = 0.0f;
-                if (i < s.dim) {
-                    q[j] = silu_f(conv_at(p.q, p.ldqk, c, p.wq, t, p.cv, c));
-                    k[j] = silu_f(conv_at(p.k, p.ldqk, c, p.wk, t, p.cv, s.qk + c));
-                }
-                qq = fmaf(q[j], q[j], qq);
-                kk = fmaf(k[j], k[j], kk);
+        for (int i = 0; i < 4; ++i) {
+            const int tap = (int)cv.taps - 4 + i, back = 4 - i;  // xr[i]: `back` tokens before t0
+            wr[i] = tap >= 0 ? w[(size_t)c * cv.taps + tap] : 0.0f;
+            xr[i] = 0.0f;
+            if (i > 0 && tap > 0) {  // xr[1 .. 3] hold the three tokens ahead of the first one, where the window reaches them
+                const uint32_t bk = back;
+                if (bk <= t0) xr[i] = x[(size_t)(t0 - bk) * ldx + c];
+                else if (bk <= cv.pos0 + t0) xr[i] = cv.ring[(size_t)((cv.pos0 + t0 - bk) % cv.taps) * cv.channels + ch];
             }
-            qq = 1.0f / (sqrtf(warp_sum(qq) + UNIT_EPS) * sqrtf((float)s.dim));
-            kk = 1.0f / sqrtf(warp_sum(kk) + UNIT_EPS);
-#pragma unroll
-            for (int j = 0; j < 8; ++j) {
-                const uint32_t i = lane + 32 * j;
-                q[j] *= qq;
-                k[j] *= kk;
-                kq = fmaf(k[j], q[j], kq);
-                if (i < s.dim) {
-                    p.qn[(size_t)t * s.qk + it * s.dim + i] = q[j];
-                    p.kn[(size_t)t * s.qk + it * s.dim + i] = k[j];
-                }
-            }
-            kq = warp_sum(kq);
-            if (lane == 0) p.kq[(size_t)t * s.kv_heads + it] = kq;
-        } else if (it < s.kv_heads + s.heads) {
-            const uint32_t h = it - s.kv_heads;
-            for (uint32_t i = lane; i < s.vdim; i += 32) {
-                const uint32_t c = h * s.vdim + i;
-                p.vn[(size_t)t * s.vd + c] = silu_f(conv_at(p.v, p.ldv, c, p.wv, t, p.cv, 2 * s.qk + c));
-            }
-        } else {
-            const uint32_t h = it - s.kv_heads - s.heads;
-            const float a = expf(p.a_log[h]);
-            for (uint32_t i = lane; i < s.dim; i += 32)
-                p.g[(size_t)t * s.heads * s.dim + h * s.dim + i] = expf(-a * softplus_f(p.z[(size_t)t * p.ldz + h * s.dim + i]));
-            if (lane == 0) p.beta[(size_t)t * s.heads + h] = sigmoid_f(p.b[(size_t)t * p.ldb + h]);
         }
+        float in[CH];
+#pragma unroll
+        for (uint32_t t = 0; t < CH; ++t) in[t] = t < n ? x[(size_t)(t0 + t) * ldx + c] : 0.0f;
+#pragma unroll
+        for (uint32_t t = 0; t < CH; ++t) {
+            xr[0] = xr[1];
+            xr[1] = xr[2];
+            xr[2] = xr[3];
+            xr[3] = in[t];
+            if (t < n) put(t, silu_f(fmaf(xr[3], wr[3], fmaf(xr[2], wr[2], fmaf(xr[1], wr[1], xr[0] * wr[0])))));
+        }
+    } else {
+        for (uint32_t t = 0; t < n; ++t) put(t, silu_f(conv_at(x, ldx, c, w, t0 + t, cv, ch)));
     }
 }
 
-// The run's last inputs of the convolution into the ring.
-__global__ void __launch_bounds__(256) delta_ring_kernel(DeltaShape s, const float *q, const float *k, const float *v, uint32_t ldqk, uint32_t ldv,
-                                                         float *ring, uint32_t tokens, uint32_t pos0) {
+// Block: one chunk of one kv head and the heads that share it.
+__global__ void __launch_bounds__(256) delta_chunk_kernel(DeltaChunk p) {
+    extern __shared__ __align__(16) float sm[];
+    const DeltaShape s = p.s;
+    float *sq = sm, *sk = sq + CH * s.dim, *sg = sk + CH * s.dim;
+    __shared__ float A[CH][CH + 1], B[CH][CH], T[CH][CH + 1], beta[CH];
+    const uint32_t chunk = blockIdx.x, t0 = chunk * CH, n = min(CH, p.tokens - t0), kh = blockIdx.y, group = s.heads / s.kv_heads;
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     pdl_wait();
     pdl_launch();
-    const uint32_t channels = 2 * s.qk + s.vd, ch = blockIdx.x * 256 + threadIdx.x;
-    if (ch >= channels) return;
-    const uint32_t n = min(tokens, s.taps);
-    for (uint32_t t = tokens - n; t < tokens; ++t) {
-        const float x = ch < s.qk ? q[(size_t)t * ldqk + ch] : (ch < 2 * s.qk ? k[(size_t)t * ldqk + ch - s.qk] : v[(size_t)t * ldv + ch - 2 * s.qk]);
-        ring[(size_t)((pos0 + t) % s.taps) * channels + ch] = x;
+    for (uint32_t i = tid; i < 2 * s.dim; i += 256) {
+        const bool isk = i >= s.dim;
+        const uint32_t e = isk ? i - s.dim : i, c = kh * s.dim + e;
+        float *dst = (isk ? sk : sq) + e;
+        conv_chunk(isk ? p.k : p.q, p.ldqk, c, isk ? p.wk : p.wq, t0, n, p.cv, (isk ? s.qk : 0u) + c, [&](uint32_t t, float v) { dst[t * s.dim] = v; });
+        for (uint32_t t = n; t < CH; ++t) dst[t * s.dim] = 0.0f;
+    }
+    __syncthreads();
+    for (uint32_t i = warp; i < 2 * n; i += 8) {  // unit vectors; q also over the root of its size
+        float *v = (i & 1 ? sk : sq) + (i >> 1) * s.dim, *out = (i & 1 ? p.kn : p.qn) + (size_t)(t0 + (i >> 1)) * s.qk + kh * s.dim;
+        float ss = 0.0f;
+        for (uint32_t e = lane; e < s.dim; e += 32) ss = fmaf(v[e], v[e], ss);
+        ss = 1.0f / sqrtf(warp_sum(ss) + UNIT_EPS);
+        if (!(i & 1)) ss /= sqrtf((float)s.dim);
+        for (uint32_t e = lane; e < s.dim; e += 32) {
+            v[e] *= ss;
+            out[e] = v[e];
+        }
+    }
+    for (uint32_t hh = 0; hh < group; ++hh) {
+        const uint32_t h = kh * group + hh;
+        const float a = expf(p.a_log[h]);
+        for (uint32_t i = tid; i < s.vdim; i += 256) {
+            const uint32_t c = h * s.vdim + i;
+            conv_chunk(p.v, p.ldv, c, p.wv, t0, n, p.cv, 2 * s.qk + c, [&](uint32_t t, float v) { p.vn[(size_t)(t0 + t) * s.vd + c] = v; });
+        }
+        for (uint32_t t = warp; t < CH; t += 8)
+            for (uint32_t e = lane; e < s.dim; e += 32) {
+                float g = 1.0f;
+                if (t < n) {
+                    g = expf(-a * softplus_f(p.z[(size_t)(t0 + t) * p.ldz + h * s.dim + e]));
+                    p.g[((size_t)(t0 + t) * s.heads + h) * s.dim + e] = g;
+                }
+                sg[t * s.dim + e] = g;
+            }
+        if (tid < CH) beta[tid] = tid < n ? sigmoid_f(p.b[(size_t)(t0 + tid) * p.ldb + h]) : 0.0f;
+        __syncthreads();
+        // A and B: warp w takes the columns s = w and 15 - w; lanes run along the channels with the product of the decays so far
+        for (int half = 0; half < 2; ++half) {
+            const uint32_t col = half ? CH - 1 - warp : warp;
+            float ks[8], run[8];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                const uint32_t e = lane + 32 * j;
+                ks[j] = e < s.dim ? sk[col * s.dim + e] : 0.0f;
+            }
+#pragma unroll
+            for (int j = 0; j < 8; ++j) run[j] = ks[j];
+            for (uint32_t t = 0; t < col; ++t)
+                if (lane == 0) A[t][col] = B[t][col] = 0.0f;
+            for (uint32_t t = col; t < CH; ++t) {
+                float sa = 0.0f, sb = 0.0f;
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    const uint32_t e = lane + 32 * j;
+                    if (e < s.dim) {
+                        if (t > col) run[j] *= sg[t * s.dim + e];
+                        sa = fmaf(sk[t * s.dim + e], run[j], sa);
+                        sb = fmaf(sq[t * s.dim + e], run[j], sb);
+                    }
+                }
+                sa = warp_sum(sa);
+                sb = warp_sum(sb);
+                if (lane == 0) {
+                    A[t][col] = t > col ? sa : 0.0f;
+                    B[t][col] = sb;
+                }
+            }
+        }
+        __syncthreads();
+        if (tid < CH) {  // column tid of T by forward substitution
+            for (uint32_t t = 0; t < CH; ++t) {
+                float v = t == tid ? 1.0f : 0.0f;
+                for (uint32_t r = tid; r < t; ++r) v = fmaf(-A[t][r], T[r][tid], v);
+                T[t][tid] = t < tid ? 0.0f : beta[t] * v;
+            }
+        }
+        __syncthreads();
+        float *tb = p.tb + ((size_t)chunk * s.heads + h) * 2 * CH * CH;
+        tb[tid] = T[tid >> 4][tid & 15];
+        tb[CH * CH + tid] = B[tid >> 4][tid & 15];
+        __syncthreads();
     }
 }
 
 struct DeltaScan {
     DeltaShape s;
-    const float *qn, *kn, *vn, *g, *beta, *kq;
+    const float *qn, *kn, *vn, *g, *tb;
+    const float *q, *k, *v;  // the convolution's inputs, whose last rows go to the ring
+    uint32_t ldqk, ldv;
+    float *ring;
     float *state;  // [heads][dim][vdim]
     float *o;      // [tokens][vd]
-    uint32_t tokens;
-    int fresh;     // the sequence starts here: the state is zero, whatever is stored
+    uint32_t tokens, pos0;
 };
 
 __device__ __forceinline__ void cp4(float *dst, const float *src) {
@@ -148,121 +221,226 @@ __device__ __forceinline__ void cp16(float *dst, const float *src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
 
-// Block: one head, 16 * CPT state columns; thread = (lane of 16, column pair). Lane l of a column owns rows
-// 4 (l + 16 j) .. + 3, j < RPT / 4.
-template <int RPT, int CPT>
-__global__ void __launch_bounds__(256) delta_scan_kernel(DeltaScan p) {
-    constexpr int D = 16 * RPT, CB = 16 * CPT, SCAN_TOK = RPT > 8 ? 4 : 8;  // SCAN_TOK: tokens per stage
-    __shared__ __align__(16) float sq[2][SCAN_TOK][D], sk[2][SCAN_TOK][D], sg[2][SCAN_TOK][D], sv[2][SCAN_TOK][CB], sc[2][SCAN_TOK][2], so[SCAN_TOK][CB];
+// D: key channels rounded up to 64, 128 or 256; CB: state columns of a block, 16 or 32.
+template <int D, int CB>
+struct ScanShape {
+    static constexpr uint32_t IN = 3 * CH * D + CH * CB + 2 * CH * CH;  // a stage: q, k, g, v, T, B
+    static constexpr uint32_t LDA = 2 * CH + 4;                         // K' and Q' as [channel][32 rows], padded
+    static constexpr uint32_t FLOATS = 2 * IN + D * LDA + CH * D + D + D * CB + 8 * 2 * CH * CB + 2 * CH * CB;
+};
+
+template <int D, int CB>
+__global__ void __launch_bounds__(256, 1) delta_scan_kernel(DeltaScan p) {
+    using Sh = ScanShape<D, CB>;
+    constexpr uint32_t LDA = Sh::LDA, KW = D / 8, CPL = CB / 4, TILES = D / 4 * (CB / 4), TPT = (TILES + 255) / 256;
+    extern __shared__ __align__(16) float sm[];
+    float *in = sm, *at = in + 2 * Sh::IN, *kend = at + D * LDA, *cend = kend + CH * D, *S = cend + D, *red = S + D * CB, *X = red + 8 * 2 * CH * CB, *U = X + CH * CB;
     const DeltaShape s = p.s;
     const uint32_t h = blockIdx.x, kh = h / (s.heads / s.kv_heads), c0 = blockIdx.y * CB;
-    const int tid = threadIdx.x, l = tid & 15, cp = tid >> 4;
-    const uint32_t col = c0 + cp * CPT;
-    // rows past dim stay zero in every stage: zero k and q leave the padded rows of the state at zero
-    for (int i = tid; i < 2 * SCAN_TOK * D; i += 256) {
-        (&sq[0][0][0])[i] = 0.0f;
-        (&sk[0][0][0])[i] = 0.0f;
-        (&sg[0][0][0])[i] = 0.0f;
-    }
-    for (int i = tid; i < 2 * SCAN_TOK * CB; i += 256) (&sv[0][0][0])[i] = 0.0f;
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    for (uint32_t i = tid; i < 2 * Sh::IN; i += 256) in[i] = 0.0f;  // padding: zero k and q leave padded rows of the state at zero
     __syncthreads();
     pdl_wait();
     pdl_launch();
-    float S[RPT][CPT];
-#pragma unroll
-    for (int r = 0; r < RPT; ++r) {
-        const uint32_t row = 4 * (l + 16 * (r >> 2)) + (r & 3);
-#pragma unroll
-        for (int c = 0; c < CPT; ++c)
-            S[r][c] = (!p.fresh && row < s.dim && col + c < s.vdim) ? p.state[((size_t)h * s.dim + row) * s.vdim + col + c] : 0.0f;
+    {  // the run's last inputs of the convolution into the ring (the kernel that read the older ones has finished)
+        const uint32_t channels = 2 * s.qk + s.vd, n = min(p.tokens, s.taps), blocks = gridDim.x * gridDim.y;
+        for (uint32_t ch = (blockIdx.y * gridDim.x + blockIdx.x) * 256 + tid; ch < channels; ch += blocks * 256)
+            for (uint32_t t = p.tokens - n; t < p.tokens; ++t) {
+                const float x = ch < s.qk ? p.q[(size_t)t * p.ldqk + ch] : (ch < 2 * s.qk ? p.k[(size_t)t * p.ldqk + ch - s.qk] : p.v[(size_t)t * p.ldv + ch - 2 * s.qk]);
+                p.ring[(size_t)((p.pos0 + t) % s.taps) * channels + ch] = x;
+            }
     }
     const uint32_t ncol = min((uint32_t)CB, s.vdim - c0);
-    const bool vec = (s.dim & 3) == 0;
-    auto fetch = [&](uint32_t t0, int b) {
-        const uint32_t n = min((uint32_t)SCAN_TOK, p.tokens - t0);
+    // this thread's 4 x 4 tiles of the state, kept in registers; S in shared memory is what the products read
+    float st[TPT][4][4];
+#pragma unroll
+    for (uint32_t u = 0; u < TPT; ++u) {
+        const uint32_t tile = tid + 256 * u, r0 = tile / (CB / 4) * 4, k0 = tile % (CB / 4) * 4;
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const uint32_t row = r0 + i, col = c0 + k0 + j;
+                st[u][i][j] = (tile < TILES && p.pos0 != 0 && row < s.dim && col < s.vdim) ? p.state[((size_t)h * s.dim + row) * s.vdim + col] : 0.0f;
+                if (tile < TILES) S[(r0 + i) * CB + k0 + j] = st[u][i][j];
+            }
+    }
+    const bool vec = (s.dim & 3) == 0, vecv = (s.vdim & 3) == 0;
+    auto fetch = [&](uint32_t chunk) {
+        float *b = in + (chunk & 1) * Sh::IN;
+        const uint32_t t0 = chunk * CH, n = min(CH, p.tokens - t0);
         if (vec) {
-            const uint32_t d4 = s.dim / 4;
-            for (uint32_t i = tid; i < n * d4; i += 256) {
-                const uint32_t t = i / d4, e = (i - t * d4) * 4;
-                cp16(&sq[b][t][e], p.qn + (size_t)(t0 + t) * s.qk + kh * s.dim + e);
-                cp16(&sk[b][t][e], p.kn + (size_t)(t0 + t) * s.qk + kh * s.dim + e);
-                cp16(&sg[b][t][e], p.g + ((size_t)(t0 + t) * s.heads + h) * s.dim + e);
-            }
+            for (uint32_t t = warp; t < n; t += 8)
+                for (uint32_t e = lane * 4; e < s.dim; e += 128) {
+                    cp16(b + t * D + e, p.qn + (size_t)(t0 + t) * s.qk + kh * s.dim + e);
+                    cp16(b + (CH + t) * D + e, p.kn + (size_t)(t0 + t) * s.qk + kh * s.dim + e);
+                    cp16(b + (2 * CH + t) * D + e, p.g + ((size_t)(t0 + t) * s.heads + h) * s.dim + e);
+                }
         } else {
-            for (uint32_t i = tid; i < n * s.dim; i += 256) {
-                const uint32_t t = i / s.dim, e = i - t * s.dim;
-                cp4(&sq[b][t][e], p.qn + (size_t)(t0 + t) * s.qk + kh * s.dim + e);
-                cp4(&sk[b][t][e], p.kn + (size_t)(t0 + t) * s.qk + kh * s.dim + e);
-                cp4(&sg[b][t][e], p.g + ((size_t)(t0 + t) * s.heads + h) * s.dim + e);
-            }
+            for (uint32_t t = warp; t < n; t += 8)
+                for (uint32_t e = lane; e < s.dim; e += 32) {
+                    cp4(b + t * D + e, p.qn + (size_t)(t0 + t) * s.qk + kh * s.dim + e);
+                    cp4(b + (CH + t) * D + e, p.kn + (size_t)(t0 + t) * s.qk + kh * s.dim + e);
+                    cp4(b + (2 * CH + t) * D + e, p.g + ((size_t)(t0 + t) * s.heads + h) * s.dim + e);
+                }
         }
-        for (uint32_t i = tid; i < n * ncol; i += 256) {
-            const uint32_t t = i / ncol, e = i - t * ncol;
-            cp4(&sv[b][t][e], p.vn + (size_t)(t0 + t) * s.vd + h * s.vdim + c0 + e);
-        }
-        for (uint32_t t = tid; t < n; t += 256) {
-            cp4(&sc[b][t][0], p.beta + (size_t)(t0 + t) * s.heads + h);
-            cp4(&sc[b][t][1], p.kq + (size_t)(t0 + t) * s.kv_heads + kh);
-        }
+        float *bv = b + 3 * CH * D;
+        for (uint32_t t = warp; t < n; t += 8)
+            for (uint32_t e = lane; e < ncol; e += 32) cp4(bv + t * CB + e, p.vn + (size_t)(t0 + t) * s.vd + h * s.vdim + c0 + e);
+        if (tid < 2 * CH * CH / 4) cp16(bv + CH * CB + 4 * tid, p.tb + ((size_t)chunk * s.heads + h) * 2 * CH * CH + 4 * tid);
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    fetch(0, 0);
-    for (uint32_t t0 = 0, b = 0; t0 < p.tokens; t0 += SCAN_TOK, b ^= 1) {
-        if (t0 + SCAN_TOK < p.tokens) {
-            fetch(t0 + SCAN_TOK, b ^ 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();
-        const uint32_t n = min((uint32_t)SCAN_TOK, p.tokens - t0);
-        for (uint32_t t = 0; t < n; ++t) {
-            float k[RPT], rk[CPT] = {}, rq[CPT] = {};
+    const uint32_t chunks = (p.tokens + CH - 1) / CH;
+    fetch(0);
+    for (uint32_t chunk = 0; chunk < chunks; ++chunk) {
+        float *b = in + (chunk & 1) * Sh::IN, *bv = b + 3 * CH * D;
+        const float *bt = bv + CH * CB, *bb = bt + CH * CH;
+        const uint32_t t0 = chunk * CH, n = min(CH, p.tokens - t0);
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();  // the chunk's inputs have arrived; everything of the chunk before has been read
+        if (chunk + 1 < chunks) fetch(chunk + 1);
+        // K', Q', K'' and the chunk's whole decay, one channel per thread (tokens past the end: k = q = 0, no decay)
+        for (uint32_t c = tid; c < 2 * D; c += 256) {
+            const uint32_t e = c < D ? c : c - D;
+            if (c < D) {
+                float run = 1.0f;
 #pragma unroll
-            for (int j = 0; j < RPT / 4; ++j) {
-                const int e = 4 * (l + 16 * j);
-                const float4 k4 = *reinterpret_cast<const float4 *>(&sk[b][t][e]), q4 = *reinterpret_cast<const float4 *>(&sq[b][t][e]),
-                             g4 = *reinterpret_cast<const float4 *>(&sg[b][t][e]);
-                const float kk[4] = {k4.x, k4.y, k4.z, k4.w}, qq[4] = {q4.x, q4.y, q4.z, q4.w}, gg[4] = {g4.x, g4.y, g4.z, g4.w};
+                for (uint32_t t4 = 0; t4 < CH; t4 += 4) {
+                    float kk[4], qq[4];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    k[4 * j + i] = kk[i];
-#pragma unroll
-                    for (int c = 0; c < CPT; ++c) {
-                        S[4 * j + i][c] *= gg[i];
-                        rk[c] = fmaf(kk[i], S[4 * j + i][c], rk[c]);
-                        rq[c] = fmaf(qq[i], S[4 * j + i][c], rq[c]);
+                    for (int i = 0; i < 4; ++i) {
+                        const uint32_t t = t4 + i;
+                        if (t < n) run *= b[(2 * CH + t) * D + e];
+                        qq[i] = t < n ? b[t * D + e] * run : 0.0f;
+                        kk[i] = t < n ? b[(CH + t) * D + e] * run : 0.0f;
                     }
+                    *reinterpret_cast<float4 *>(at + e * LDA + t4) = make_float4(kk[0], kk[1], kk[2], kk[3]);
+                    *reinterpret_cast<float4 *>(at + e * LDA + CH + t4) = make_float4(qq[0], qq[1], qq[2], qq[3]);
                 }
-            }
+            } else {
+                float run = 1.0f;
 #pragma unroll
-            for (int o = 8; o > 0; o >>= 1)
-#pragma unroll
-                for (int c = 0; c < CPT; ++c) {
-                    rk[c] += __shfl_xor_sync(0xffffffffu, rk[c], o);
-                    rq[c] += __shfl_xor_sync(0xffffffffu, rq[c], o);
+                for (int t = CH - 1; t >= 0; --t) {
+                    const bool live = (uint32_t)t < n;
+                    kend[t * D + e] = live ? b[(CH + t) * D + e] * run : 0.0f;
+                    if (live) run *= b[(2 * CH + t) * D + e];
                 }
-            const float beta = sc[b][t][0], kq = sc[b][t][1];
-#pragma unroll
-            for (int c = 0; c < CPT; ++c) {
-                const float u = beta * (sv[b][t][cp * CPT + c] - rk[c]);
-#pragma unroll
-                for (int r = 0; r < RPT; ++r) S[r][c] = fmaf(k[r], u, S[r][c]);
-                if (l == 0) so[t][cp * CPT + c] = fmaf(u, kq, rq[c]);
+                cend[e] = run;
             }
         }
         __syncthreads();
-        for (uint32_t i = tid; i < n * ncol; i += 256) {
-            const uint32_t t = i / ncol, e = i - t * ncol;
-            p.o[(size_t)(t0 + t) * s.vd + h * s.vdim + c0 + e] = so[t][e];
+        {  // [K'; Q'] S: warp w sums over its share of the channels; lane = 4 of the 32 rows x CPL columns
+            float acc[4][CPL] = {};
+            const uint32_t r4 = (lane >> 2) * 4, cl = (lane & 3) * CPL;
+#pragma unroll 4
+            for (uint32_t k = warp * KW; k < (warp + 1) * KW; ++k) {
+                const float4 a = *reinterpret_cast<const float4 *>(at + k * LDA + r4);
+                const float av[4] = {a.x, a.y, a.z, a.w};
+                float sv[CPL];
+#pragma unroll
+                for (uint32_t j = 0; j < CPL; j += 4) {
+                    const float4 v = *reinterpret_cast<const float4 *>(S + k * CB + cl + j);
+                    sv[j] = v.x;
+                    sv[j + 1] = v.y;
+                    sv[j + 2] = v.z;
+                    sv[j + 3] = v.w;
+                }
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+#pragma unroll
+                    for (uint32_t j = 0; j < CPL; ++j) acc[i][j] = fmaf(av[i], sv[j], acc[i][j]);
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (uint32_t j = 0; j < CPL; j += 4)
+                    *reinterpret_cast<float4 *>(red + (warp * 2 * CH + r4 + i) * CB + cl + j) = make_float4(acc[i][j], acc[i][j + 1], acc[i][j + 2], acc[i][j + 3]);
+        }
+        __syncthreads();
+        // the sums over the warps: rows 0-15 become X = V - K' S, rows 16-31 stay with their thread (Q' S)
+        const uint32_t row = tid / (CB / 4), k4 = tid % (CB / 4) * 4;
+        const bool mine = row < 2 * CH;
+        float o[4] = {};
+        if (mine) {
+#pragma unroll
+            for (int w = 0; w < 8; ++w) {
+                const float4 v = *reinterpret_cast<const float4 *>(red + (w * 2 * CH + row) * CB + k4);
+                o[0] += v.x;
+                o[1] += v.y;
+                o[2] += v.z;
+                o[3] += v.w;
+            }
+            if (row < CH) {
+                const float4 v = *reinterpret_cast<const float4 *>(bv + row * CB + k4);
+                *reinterpret_cast<float4 *>(X + row * CB + k4) = row < n ? make_float4(v.x - o[0], v.y - o[1], v.z - o[2], v.w - o[3]) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+        }
+        __syncthreads();
+        if (mine && row < CH) {
+            float u[4] = {};
+#pragma unroll
+            for (uint32_t r = 0; r < CH; ++r) {
+                const float t = bt[row * CH + r];
+                const float4 x = *reinterpret_cast<const float4 *>(X + r * CB + k4);
+                u[0] = fmaf(t, x.x, u[0]);
+                u[1] = fmaf(t, x.y, u[1]);
+                u[2] = fmaf(t, x.z, u[2]);
+                u[3] = fmaf(t, x.w, u[3]);
+            }
+            *reinterpret_cast<float4 *>(U + row * CB + k4) = make_float4(u[0], u[1], u[2], u[3]);
+        }
+        __syncthreads();
+        if (mine && row >= CH && row - CH < n) {
+            const uint32_t t = row - CH;
+#pragma unroll
+            for (uint32_t r = 0; r < CH; ++r) {
+                const float w = bb[t * CH + r];
+                const float4 u = *reinterpret_cast<const float4 *>(U + r * CB + k4);
+                o[0] = fmaf(w, u.x, o[0]);
+                o[1] = fmaf(w, u.y, o[1]);
+                o[2] = fmaf(w, u.z, o[2]);
+                o[3] = fmaf(w, u.w, o[3]);
+            }
+            float *dst = p.o + (size_t)(t0 + t) * s.vd + h * s.vdim + c0 + k4;
+            if (vecv && k4 + 4 <= ncol) *reinterpret_cast<float4 *>(dst) = make_float4(o[0], o[1], o[2], o[3]);
+            else
+                for (uint32_t j = 0; j < 4; ++j)
+                    if (k4 + j < ncol) dst[j] = o[j];
+        }
+#pragma unroll
+        for (uint32_t u = 0; u < TPT; ++u) {
+            const uint32_t tile = tid + 256 * u, r0 = tile / (CB / 4) * 4, kc = tile % (CB / 4) * 4;
+            if (tile < TILES) {
+                const float4 ce = *reinterpret_cast<const float4 *>(cend + r0);
+                const float cv[4] = {ce.x, ce.y, ce.z, ce.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) st[u][i][j] *= cv[i];
+#pragma unroll
+                for (uint32_t r = 0; r < CH; ++r) {
+                    const float4 kv = *reinterpret_cast<const float4 *>(kend + r * D + r0), uv = *reinterpret_cast<const float4 *>(U + r * CB + kc);
+                    const float ka[4] = {kv.x, kv.y, kv.z, kv.w}, ua[4] = {uv.x, uv.y, uv.z, uv.w};
+#pragma unroll
+                    for (int i = 0; i < 4; ++i)
+#pragma unroll
+                        for (int j = 0; j < 4; ++j) st[u][i][j] = fmaf(ka[i], ua[j], st[u][i][j]);
+                }
+#pragma unroll
+                for (int i = 0; i < 4; ++i) *reinterpret_cast<float4 *>(S + (r0 + i) * CB + kc) = make_float4(st[u][i][0], st[u][i][1], st[u][i][2], st[u][i][3]);
+            }
         }
     }
 #pragma unroll
-    for (int r = 0; r < RPT; ++r) {
-        const uint32_t row = 4 * (l + 16 * (r >> 2)) + (r & 3);
+    for (uint32_t u = 0; u < TPT; ++u) {
+        const uint32_t tile = tid + 256 * u, r0 = tile / (CB / 4) * 4, kc = tile % (CB / 4) * 4;
 #pragma unroll
-        for (int c = 0; c < CPT; ++c)
-            if (row < s.dim && col + c < s.vdim) p.state[((size_t)h * s.dim + row) * s.vdim + col + c] = S[r][c];
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const uint32_t row = r0 + i, col = c0 + kc + j;
+                if (tile < TILES && row < s.dim && col < s.vdim) p.state[((size_t)h * s.dim + row) * s.vdim + col] = st[u][i][j];
+            }
     }
 }
 
@@ -532,15 +710,13 @@ class ChannelDelta : public Mixer {
         lp[1].ldy = ldv_;
         BRASA_TRY(brasa_linear_launch(r.cmd, lp, 2, r.f32));
         const uint32_t channels = 2 * s_.qk + s_.vd;
-        DeltaPrep pp{s_, ConvView{ring_, channels, s_.taps, r.pos0}, f(at_.q), f(at_.k), f(at_.v), f(at_.b), f(at_.z), ldqk_, ldv_, ldb_, ldz_, wq_, wk_, wv_, a_log_,
-                     f(at_.qn), f(at_.kn), f(at_.vn), f(at_.g), f(at_.beta), f(at_.kq)};
-        const uint32_t items = s_.kv_heads + 2 * s_.heads, gy = r.tokens < 512 ? (items + 7) / 8 : 1;
-        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_prep_kernel, dim3(r.tokens, gy), dim3(256), 0, pp));
-        BRASA_TRY(brasa_post_launch(r.cmd, "delta_prep"));
-        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_ring_kernel, dim3((channels + 255) / 256), dim3(256), 0, s_, f(at_.q), f(at_.k), f(at_.v), ldqk_, ldv_, ring_,
-                                               r.tokens, r.pos0));
-        BRASA_TRY(brasa_post_launch(r.cmd, "delta_ring"));
-        DeltaScan sp{s_, f(at_.qn), f(at_.kn), f(at_.vn), f(at_.g), f(at_.beta), f(at_.kq), state_, f(at_.o), r.tokens, r.pos0 == 0 ? 1 : 0};
+        DeltaChunk cp{s_, ConvView{ring_, channels, s_.taps, r.pos0}, f(at_.q), f(at_.k), f(at_.v), f(at_.b), f(at_.z), ldqk_, ldv_, ldb_, ldz_, r.tokens, wq_, wk_, wv_, a_log_,
+                      f(at_.qn), f(at_.kn), f(at_.vn), f(at_.g), f(at_.tb)};
+        const size_t csm = 3ull * CH * s_.dim * 4;
+        BRASA_TRY(brasa_smem_optin(ctx, (const void *)delta_chunk_kernel, csm));
+        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_chunk_kernel, dim3((r.tokens + CH - 1) / CH, s_.kv_heads), dim3(256), csm, cp));
+        BRASA_TRY(brasa_post_launch(r.cmd, "delta_chunk"));
+        DeltaScan sp{s_, f(at_.qn), f(at_.kn), f(at_.vn), f(at_.g), f(at_.tb), f(at_.q), f(at_.k), f(at_.v), ldqk_, ldv_, ring_, state_, f(at_.o), r.tokens, r.pos0};
         BRASA_TRY(scan(r.cmd, sp));
         const uint32_t blocks = (r.tokens * s_.heads + 7) / 8;
         if (r.f32) BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_out_kernel<float>, dim3(blocks), dim3(256), 0, f(at_.o), f(at_.gate), ldv_, norm_, (float *)r.out, r.ldo,
@@ -551,21 +727,20 @@ class ChannelDelta : public Mixer {
     }
 
   private:
-    int32_t scan(brasa_cmd *cmd, const DeltaScan &p) {
+    template <int D, int CB>
+    int32_t scan_as(brasa_cmd *cmd, const DeltaScan &p) {
         brasa_ctx *ctx = cmd->ctx;
-        // two columns per thread when that still fills the SMs
-        const bool two = s_.heads * ((s_.vdim + 31) / 32) >= (uint32_t)ctx->sm_count / 2;
-        const dim3 grid(s_.heads, (s_.vdim + (two ? 31 : 15)) / (two ? 32 : 16));
-#define SCAN(R)                                                                                                              \
-    do {                                                                                                                     \
-        if (two) BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_scan_kernel<R, 2>, grid, dim3(256), 0, p));               \
-        else BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_scan_kernel<R, 1>, grid, dim3(256), 0, p));                   \
-    } while (0)
-        if (s_.dim <= 64) SCAN(4);
-        else if (s_.dim <= 128) SCAN(8);
-        else BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_scan_kernel<16, 1>, dim3(s_.heads, (s_.vdim + 15) / 16), dim3(256), 0, p));
-#undef SCAN
+        const size_t smem = (size_t)ScanShape<D, CB>::FLOATS * 4;
+        BRASA_TRY(brasa_smem_optin(ctx, (const void *)delta_scan_kernel<D, CB>, smem));
+        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_scan_kernel<D, CB>, dim3(s_.heads, (s_.vdim + CB - 1) / CB), dim3(256), smem, p));
         return brasa_post_launch(cmd, "delta_scan");
+    }
+    int32_t scan(brasa_cmd *cmd, const DeltaScan &p) {
+        // wide blocks when they still cover most of the SMs
+        const bool wide = s_.heads * ((s_.vdim + 31) / 32) * 5 >= (uint32_t)cmd->ctx->sm_count * 4;
+        if (s_.dim <= 64) return wide ? scan_as<64, 32>(cmd, p) : scan_as<64, 16>(cmd, p);
+        if (s_.dim <= 128) return wide ? scan_as<128, 32>(cmd, p) : scan_as<128, 16>(cmd, p);
+        return scan_as<256, 16>(cmd, p);
     }
 
     void lay_out(uint64_t t, bool f32) {
@@ -589,8 +764,7 @@ class ChannelDelta : public Mixer {
         at_.kn = c.take(4 * t * s_.qk);
         at_.vn = c.take(4 * t * s_.vd);
         at_.g = c.take(4 * t * s_.heads * s_.dim);
-        at_.beta = c.take(4 * t * s_.heads);
-        at_.kq = c.take(4 * t * s_.kv_heads);
+        at_.tb = c.take(4ull * ((t + CH - 1) / CH) * s_.heads * 2 * CH * CH);
         at_.o = c.take(4 * t * s_.vd);
         at_.total = c.at;
     }
@@ -602,7 +776,7 @@ class ChannelDelta : public Mixer {
     const float *wq_ = nullptr, *wk_ = nullptr, *wv_ = nullptr, *a_log_ = nullptr, *dt_bias_ = nullptr, *norm_ = nullptr;
     float *ring_ = nullptr, *state_ = nullptr;
     struct {
-        uint64_t q, k, v, b, a1, g1, z, gate, qn, kn, vn, g, beta, kq, o, total;
+        uint64_t q, k, v, b, a1, g1, z, gate, qn, kn, vn, g, tb, o, total;
     } at_{};
 };
 
