@@ -108,98 +108,118 @@ __device__ __forceinline__ void conv_chunk(const float *x, uint32_t ldx, uint32_
     }
 }
 
-// Block: one chunk of one kv head and the heads that share it.
+// Block: one chunk of one head. E consecutive key channels per lane: dim up to 32 E.
+template <int E>
 __global__ void __launch_bounds__(256) delta_chunk_kernel(DeltaChunk p) {
+    constexpr uint32_t D = 32 * E;
     extern __shared__ __align__(16) float sm[];
     const DeltaShape s = p.s;
-    float *sq = sm, *sk = sq + CH * s.dim, *sg = sk + CH * s.dim;
-    __shared__ float A[CH][CH + 1], B[CH][CH], T[CH][CH + 1], beta[CH];
-    const uint32_t chunk = blockIdx.x, t0 = chunk * CH, n = min(CH, p.tokens - t0), kh = blockIdx.y, group = s.heads / s.kv_heads;
+    float *sq = sm, *sk = sq + CH * D, *sg = sk + CH * D;
+    __shared__ float B[CH][CH], beta[CH];
+    __shared__ __align__(16) float A[CH][CH];
+    const uint32_t chunk = blockIdx.x, t0 = chunk * CH, n = min(CH, p.tokens - t0), h = blockIdx.y, group = s.heads / s.kv_heads, kh = h / group;
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     pdl_wait();
     pdl_launch();
-    for (uint32_t i = tid; i < 2 * s.dim; i += 256) {
-        const bool isk = i >= s.dim;
-        const uint32_t e = isk ? i - s.dim : i, c = kh * s.dim + e;
+    for (uint32_t i = tid; i < 2 * D; i += 256) {
+        const bool isk = i >= D;
+        const uint32_t e = isk ? i - D : i, c = kh * s.dim + e;
         float *dst = (isk ? sk : sq) + e;
-        conv_chunk(isk ? p.k : p.q, p.ldqk, c, isk ? p.wk : p.wq, t0, n, p.cv, (isk ? s.qk : 0u) + c, [&](uint32_t t, float v) { dst[t * s.dim] = v; });
-        for (uint32_t t = n; t < CH; ++t) dst[t * s.dim] = 0.0f;
-    }
-    __syncthreads();
-    for (uint32_t i = warp; i < 2 * n; i += 8) {  // unit vectors; q also over the root of its size
-        float *v = (i & 1 ? sk : sq) + (i >> 1) * s.dim, *out = (i & 1 ? p.kn : p.qn) + (size_t)(t0 + (i >> 1)) * s.qk + kh * s.dim;
-        float ss = 0.0f;
-        for (uint32_t e = lane; e < s.dim; e += 32) ss = fmaf(v[e], v[e], ss);
-        ss = 1.0f / sqrtf(warp_sum(ss) + UNIT_EPS);
-        if (!(i & 1)) ss /= sqrtf((float)s.dim);
-        for (uint32_t e = lane; e < s.dim; e += 32) {
-            v[e] *= ss;
-            out[e] = v[e];
+        uint32_t t = 0;
+        if (e < s.dim) {
+            conv_chunk(isk ? p.k : p.q, p.ldqk, c, isk ? p.wk : p.wq, t0, n, p.cv, (isk ? s.qk : 0u) + c, [&](uint32_t tt, float v) { dst[tt * D] = v; });
+            t = n;
         }
+        for (; t < CH; ++t) dst[t * D] = 0.0f;
     }
-    for (uint32_t hh = 0; hh < group; ++hh) {
-        const uint32_t h = kh * group + hh;
+    {
         const float a = expf(p.a_log[h]);
-        for (uint32_t i = tid; i < s.vdim; i += 256) {
-            const uint32_t c = h * s.vdim + i;
-            conv_chunk(p.v, p.ldv, c, p.wv, t0, n, p.cv, 2 * s.qk + c, [&](uint32_t t, float v) { p.vn[(size_t)(t0 + t) * s.vd + c] = v; });
-        }
         for (uint32_t t = warp; t < CH; t += 8)
-            for (uint32_t e = lane; e < s.dim; e += 32) {
+#pragma unroll
+            for (int j = 0; j < E; ++j) {
+                const uint32_t e = lane + 32 * j;
                 float g = 1.0f;
-                if (t < n) {
+                if (t < n && e < s.dim) {
                     g = expf(-a * softplus_f(p.z[(size_t)(t0 + t) * p.ldz + h * s.dim + e]));
                     p.g[((size_t)(t0 + t) * s.heads + h) * s.dim + e] = g;
                 }
-                sg[t * s.dim + e] = g;
+                sg[t * D + e] = g;
             }
         if (tid < CH) beta[tid] = tid < n ? sigmoid_f(p.b[(size_t)(t0 + tid) * p.ldb + h]) : 0.0f;
-        __syncthreads();
-        // A and B: warp w takes the columns s = w and 15 - w; lanes run along the channels with the product of the decays so far
-        for (int half = 0; half < 2; ++half) {
-            const uint32_t col = half ? CH - 1 - warp : warp;
-            float ks[8], run[8];
+    }
+    __syncthreads();
+    for (uint32_t i = warp; i < 2 * n; i += 8) {  // unit vectors; q also over the root of its size
+        float *v = (i & 1 ? sk : sq) + (i >> 1) * D, *out = (i & 1 ? p.kn : p.qn) + (size_t)(t0 + (i >> 1)) * s.qk + kh * s.dim;
+        float x[E], ss = 0.0f;
 #pragma unroll
-            for (int j = 0; j < 8; ++j) {
-                const uint32_t e = lane + 32 * j;
-                ks[j] = e < s.dim ? sk[col * s.dim + e] : 0.0f;
-            }
+        for (int j = 0; j < E; ++j) {
+            x[j] = v[lane + 32 * j];
+            ss = fmaf(x[j], x[j], ss);
+        }
+        ss = 1.0f / sqrtf(warp_sum(ss) + UNIT_EPS);
+        if (!(i & 1)) ss /= sqrtf((float)s.dim);
 #pragma unroll
-            for (int j = 0; j < 8; ++j) run[j] = ks[j];
-            for (uint32_t t = 0; t < col; ++t)
-                if (lane == 0) A[t][col] = B[t][col] = 0.0f;
-            for (uint32_t t = col; t < CH; ++t) {
-                float sa = 0.0f, sb = 0.0f;
+        for (int j = 0; j < E; ++j) {
+            v[lane + 32 * j] = x[j] * ss;
+            if (h % group == 0 && lane + 32 * j < s.dim) out[lane + 32 * j] = x[j] * ss;
+        }
+    }
+    __syncthreads();
+    // A and B: warp w takes the columns s = w and 15 - w; a lane holds E channels of k_s times the decays so far, sums of all t
+    // are kept apart and reduced over the lanes together at the end
+#pragma unroll 1
+    for (int half = 0; half < 2; ++half) {
+        const uint32_t col = half ? CH - 1 - warp : warp;
+        float run[E], acc[2 * CH];
 #pragma unroll
-                for (int j = 0; j < 8; ++j) {
-                    const uint32_t e = lane + 32 * j;
-                    if (e < s.dim) {
-                        if (t > col) run[j] *= sg[t * s.dim + e];
-                        sa = fmaf(sk[t * s.dim + e], run[j], sa);
-                        sb = fmaf(sq[t * s.dim + e], run[j], sb);
-                    }
-                }
-                sa = warp_sum(sa);
-                sb = warp_sum(sb);
-                if (lane == 0) {
-                    A[t][col] = t > col ? sa : 0.0f;
-                    B[t][col] = sb;
+        for (int j = 0; j < E; ++j) run[j] = sk[col * D + lane * E + j];
+#pragma unroll
+        for (uint32_t t = 0; t < CH; ++t) {
+            acc[2 * t] = acc[2 * t + 1] = 0.0f;
+            if (t >= col) {
+#pragma unroll
+                for (int j = 0; j < E; ++j) {
+                    const uint32_t e = t * D + lane * E + j;
+                    if (t > col) run[j] *= sg[e];
+                    acc[2 * t] = fmaf(sk[e], run[j], acc[2 * t]);
+                    acc[2 * t + 1] = fmaf(sq[e], run[j], acc[2 * t + 1]);
                 }
             }
         }
-        __syncthreads();
-        if (tid < CH) {  // column tid of T by forward substitution
+        // 32 values over 32 lanes: lane i ends up with value i
+#pragma unroll
+        for (int w = CH; w >= 1; w >>= 1) {
+            const bool up = lane & w;
+#pragma unroll
+            for (int i = 0; i < w; ++i) {
+                const float give = up ? acc[i] : acc[i + w], keep = up ? acc[i + w] : acc[i];
+                acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, w);
+            }
+        }
+        const uint32_t t = lane >> 1;
+        if (lane & 1) B[t][col] = acc[0];
+        else A[t][col] = t > col ? acc[0] : 0.0f;
+    }
+    __syncthreads();
+    float *tb = p.tb + ((size_t)chunk * s.heads + h) * 2 * CH * CH;
+    if (warp == 0) {
+        if (lane < CH) {  // column `lane` of T by forward substitution
+            float T[CH];
+#pragma unroll
             for (uint32_t t = 0; t < CH; ++t) {
-                float v = t == tid ? 1.0f : 0.0f;
-                for (uint32_t r = tid; r < t; ++r) v = fmaf(-A[t][r], T[r][tid], v);
-                T[t][tid] = t < tid ? 0.0f : beta[t] * v;
+                float v = t == lane ? 1.0f : 0.0f;
+#pragma unroll
+                for (uint32_t r = 0; r < t; ++r) v = fmaf(-A[t][r], T[r], v);
+                T[t] = beta[t] * v;
+                tb[t * CH + lane] = T[t];
             }
         }
-        __syncthreads();
-        float *tb = p.tb + ((size_t)chunk * s.heads + h) * 2 * CH * CH;
-        tb[tid] = T[tid >> 4][tid & 15];
-        tb[CH * CH + tid] = B[tid >> 4][tid & 15];
-        __syncthreads();
+    } else {
+        for (uint32_t i = tid - 32; i < CH * CH; i += 224) tb[CH * CH + i] = B[i >> 4][i & 15];
+        for (uint32_t i = tid - 32; i < s.vdim; i += 224) {
+            const uint32_t c = h * s.vdim + i;
+            conv_chunk(p.v, p.ldv, c, p.wv, t0, n, p.cv, 2 * s.qk + c, [&](uint32_t t, float v) { p.vn[(size_t)(t0 + t) * s.vd + c] = v; });
+        }
     }
 }
 
@@ -221,7 +241,19 @@ __device__ __forceinline__ void cp16(float *dst, const float *src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
 
-// D: key channels rounded up to 64, 128 or 256; CB: state columns of a block, 16 or 32.
+// The run's last inputs of the convolution into the ring (the kernel that read the older ones has finished).
+__device__ __forceinline__ void store_ring(const DeltaScan &p, uint32_t threads) {
+    const DeltaShape &s = p.s;
+    const uint32_t channels = 2 * s.qk + s.vd, n = min(p.tokens, s.taps), step = gridDim.x * gridDim.y * threads;
+    for (uint32_t ch = (blockIdx.y * gridDim.x + blockIdx.x) * threads + threadIdx.x; ch < channels; ch += step)
+        for (uint32_t t = p.tokens - n; t < p.tokens; ++t) {
+            const float x = ch < s.qk ? p.q[(size_t)t * p.ldqk + ch] : (ch < 2 * s.qk ? p.k[(size_t)t * p.ldqk + ch - s.qk] : p.v[(size_t)t * p.ldv + ch - 2 * s.qk]);
+            p.ring[(size_t)((p.pos0 + t) % s.taps) * channels + ch] = x;
+        }
+}
+
+// The state through the chunks in f32 FMA (the 32-bit mode, and key sizes above 128). D: key channels rounded up to 64, 128 or
+// 256; CB: state columns of a block, 16 or 32.
 template <int D, int CB>
 struct ScanShape {
     static constexpr uint32_t IN = 3 * CH * D + CH * CB + 2 * CH * CH;  // a stage: q, k, g, v, T, B
@@ -242,14 +274,7 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(DeltaScan p) {
     __syncthreads();
     pdl_wait();
     pdl_launch();
-    {  // the run's last inputs of the convolution into the ring (the kernel that read the older ones has finished)
-        const uint32_t channels = 2 * s.qk + s.vd, n = min(p.tokens, s.taps), blocks = gridDim.x * gridDim.y;
-        for (uint32_t ch = (blockIdx.y * gridDim.x + blockIdx.x) * 256 + tid; ch < channels; ch += blocks * 256)
-            for (uint32_t t = p.tokens - n; t < p.tokens; ++t) {
-                const float x = ch < s.qk ? p.q[(size_t)t * p.ldqk + ch] : (ch < 2 * s.qk ? p.k[(size_t)t * p.ldqk + ch - s.qk] : p.v[(size_t)t * p.ldv + ch - 2 * s.qk]);
-                p.ring[(size_t)((p.pos0 + t) % s.taps) * channels + ch] = x;
-            }
-    }
+    store_ring(p, 256);
     const uint32_t ncol = min((uint32_t)CB, s.vdim - c0);
     // this thread's 4 x 4 tiles of the state, kept in registers; S in shared memory is what the products read
     float st[TPT][4][4];
@@ -444,6 +469,261 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(DeltaScan p) {
     }
 }
 
+// The same on tensor cores (bf16 mode, key sizes up to 128): every product with the state is formed from two-term tf32 splits,
+// x = hi + lo, as hi hi + hi lo + lo hi, which keeps 22 bits of each factor, with f32 accumulation; the state itself, the
+// factors and U stay f32.
+//
+// Four warps carry the state: warp = 16 columns x D / PARTS channels, as accumulators of the transposed state (rows = columns
+// of S). Those registers are at the same time the B operand of [K'; Q'] S when the eight channels of a step are taken in the
+// order 0 2 4 6 1 3 5 7, so the state never leaves them. Four more warps work one chunk ahead: they fetch q, k, g (two chunks
+// ahead) and form the split K', Q', K''.
+template <int D, int CB>
+struct MmaScanShape {
+    static constexpr uint32_t GROUPS = CB / 16, PARTS = 4 / GROUPS, NCH = D / PARTS, NK = NCH / 8;
+    static constexpr uint32_t IN = 3 * CH * D, LDF = D + 8, LDU = CB + 8;
+    static constexpr uint32_t FAC = 2 * 3 * CH * LDF + D;   // hi then lo of: K' (16 rows), Q' (16), K'' (16); the chunk's decay
+    static constexpr uint32_t VTB = CH * CB + 2 * CH * CH;  // v, T, B (three in flight)
+    static constexpr uint32_t FLOATS = 2 * IN + 2 * FAC + 3 * VTB + PARTS * 2 * CH * CB + 4 * CH * LDU;
+};
+
+__device__ __forceinline__ float tf32_hi(float x) {
+    uint32_t r;
+    asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(r) : "f"(x));
+    return __uint_as_float(r);
+}
+__device__ __forceinline__ void mma_tf32(float c[4], const float a[4], float b0, float b1) {
+    asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(__float_as_uint(a[0])), "r"(__float_as_uint(a[1])), "r"(__float_as_uint(a[2])), "r"(__float_as_uint(a[3])), "r"(__float_as_uint(b0)),
+                   "r"(__float_as_uint(b1)));
+}
+
+template <int D, int CB>
+__global__ void __launch_bounds__(256, 1) delta_scan_mma_kernel(DeltaScan p) {
+    using Sh = MmaScanShape<D, CB>;
+    constexpr uint32_t LDF = Sh::LDF, LDU = Sh::LDU, NK = Sh::NK, PARTS = Sh::PARTS, TPT = CH * CB / 128;
+    extern __shared__ __align__(16) float sm[];
+    float *in = sm, *fac = in + 2 * Sh::IN, *vtb = fac + 2 * Sh::FAC, *red = vtb + 3 * Sh::VTB, *X = red + PARTS * 2 * CH * CB, *U = X + CH * LDU, *Uh = U + CH * LDU, *Ul = Uh + CH * LDU;
+    const DeltaShape s = p.s;
+    const uint32_t h = blockIdx.x, kh = h / (s.heads / s.kv_heads), c0 = blockIdx.y * CB;
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    for (uint32_t i = tid; i < Sh::FLOATS; i += 256) sm[i] = 0.0f;  // padding: zero k and q leave padded rows of the state at zero
+    __syncthreads();
+    pdl_wait();
+    pdl_launch();
+    store_ring(p, 256);
+    const uint32_t ncol = min((uint32_t)CB, s.vdim - c0), chunks = (p.tokens + CH - 1) / CH;
+    if (warp >= 4) {  // ---- one chunk ahead ----
+        const uint32_t pt = tid - 128, pw = pt >> 5;
+        const bool vec = (s.dim & 3) == 0;
+        auto fetch = [&](uint32_t chunk) {
+            float *b = in + (chunk & 1) * Sh::IN, *bv = vtb + (chunk % 3) * Sh::VTB;
+            const uint32_t t0 = chunk * CH, n = min(CH, p.tokens - t0);
+            for (uint32_t t = pw; t < n; t += 4) {
+                const float *q = p.qn + (size_t)(t0 + t) * s.qk + kh * s.dim, *k = p.kn + (size_t)(t0 + t) * s.qk + kh * s.dim,
+                            *g = p.g + ((size_t)(t0 + t) * s.heads + h) * s.dim;
+                if (vec) {
+                    for (uint32_t e = lane * 4; e < s.dim; e += 128) {
+                        cp16(b + t * D + e, q + e);
+                        cp16(b + (CH + t) * D + e, k + e);
+                        cp16(b + (2 * CH + t) * D + e, g + e);
+                    }
+                } else {
+                    for (uint32_t e = lane; e < s.dim; e += 32) {
+                        cp4(b + t * D + e, q + e);
+                        cp4(b + (CH + t) * D + e, k + e);
+                        cp4(b + (2 * CH + t) * D + e, g + e);
+                    }
+                }
+                for (uint32_t e = lane; e < ncol; e += 32) cp4(bv + t * CB + e, p.vn + (size_t)(t0 + t) * s.vd + h * s.vdim + c0 + e);
+            }
+            cp16(bv + CH * CB + 4 * pt, p.tb + ((size_t)chunk * s.heads + h) * 2 * CH * CH + 4 * pt);
+            asm volatile("cp.async.commit_group;" ::: "memory");
+        };
+        auto form = [&](uint32_t chunk) {  // tokens past the end: k = q = 0, no decay
+            const float *b = in + (chunk & 1) * Sh::IN;
+            float *f = fac + (chunk & 1) * Sh::FAC;
+            const uint32_t n = min(CH, p.tokens - chunk * CH);
+            auto put = [&](uint32_t row, uint32_t e, float v) {
+                const float hi = tf32_hi(v);
+                f[row * LDF + e] = hi;
+                f[(3 * CH + row) * LDF + e] = tf32_hi(v - hi);
+            };
+            for (uint32_t e = pt; e < D; e += 128) {
+                float g[CH], k[CH], run = 1.0f;
+#pragma unroll
+                for (uint32_t t = 0; t < CH; ++t) {
+                    g[t] = t < n ? b[(2 * CH + t) * D + e] : 1.0f;
+                    k[t] = t < n ? b[(CH + t) * D + e] : 0.0f;
+                }
+#pragma unroll
+                for (uint32_t t = 0; t < CH; ++t) {
+                    run *= g[t];
+                    put(t, e, k[t] * run);
+                    put(CH + t, e, t < n ? b[t * D + e] * run : 0.0f);
+                }
+                f[2 * 3 * CH * LDF + e] = run;
+                run = 1.0f;
+#pragma unroll
+                for (int t = CH - 1; t >= 0; --t) {
+                    put(2 * CH + t, e, k[t] * run);
+                    run *= g[t];
+                }
+            }
+        };
+        fetch(0);
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        asm volatile("bar.sync 1, 128;" ::: "memory");
+        if (chunks > 1) fetch(1);
+        form(0);
+        __syncthreads();
+        for (uint32_t chunk = 0; chunk < chunks; ++chunk) {
+            if (chunk + 1 < chunks) {
+                asm volatile("cp.async.wait_group 0;" ::: "memory");
+                asm volatile("bar.sync 1, 128;" ::: "memory");
+                if (chunk + 2 < chunks) fetch(chunk + 2);
+                form(chunk + 1);
+            }
+            __syncthreads();
+        }
+        return;
+    }
+    // ---- the state ----
+    const uint32_t grp = warp % Sh::GROUPS, part = warp / Sh::GROUPS, g = lane >> 2, q = lane & 3;
+    const uint32_t ch0 = part * Sh::NCH, cg = 16 * grp;  // this warp's channels and columns
+    float S[NK][4];  // [tile of 8 channels]: columns g and g + 8 x channels 2 q and 2 q + 1
+#pragma unroll
+    for (uint32_t kt = 0; kt < NK; ++kt)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const uint32_t row = ch0 + 8 * kt + 2 * q + (i & 1), col = c0 + cg + g + 8 * (i >> 1);
+            S[kt][i] = (p.pos0 != 0 && row < s.dim && col < s.vdim) ? p.state[((size_t)h * s.dim + row) * s.vdim + col] : 0.0f;
+        }
+    __syncthreads();
+    for (uint32_t chunk = 0; chunk < chunks; ++chunk) {
+        const float *fh = fac + (chunk & 1) * Sh::FAC, *fl = fh + 3 * CH * LDF, *cend = fh + 2 * 3 * CH * LDF;
+        const float *bv = vtb + (chunk % 3) * Sh::VTB, *bt = bv + CH * CB, *bb = bt + CH * CH;
+        const uint32_t t0 = chunk * CH, n = min(CH, p.tokens - t0);
+        float big[2][2][4] = {}, small[2][2][4] = {};  // [K', Q'][columns 0-7, 8-15]
+#pragma unroll
+        for (uint32_t kt = 0; kt < NK; ++kt) {
+            float sh[4], sl[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                sh[i] = tf32_hi(S[kt][i]);
+                sl[i] = tf32_hi(S[kt][i] - sh[i]);
+            }
+#pragma unroll
+            for (uint32_t mt = 0; mt < 2; ++mt) {
+                const uint32_t at = (mt * CH + g) * LDF + ch0 + 8 * kt + 2 * q;
+                const float2 h0 = *reinterpret_cast<const float2 *>(fh + at), h1 = *reinterpret_cast<const float2 *>(fh + at + 8 * LDF);
+                const float2 l0 = *reinterpret_cast<const float2 *>(fl + at), l1 = *reinterpret_cast<const float2 *>(fl + at + 8 * LDF);
+                const float ah[4] = {h0.x, h1.x, h0.y, h1.y}, al[4] = {l0.x, l1.x, l0.y, l1.y};
+#pragma unroll
+                for (int nt = 0; nt < 2; ++nt) {
+                    mma_tf32(big[mt][nt], ah, sh[2 * nt], sh[2 * nt + 1]);
+                    mma_tf32(small[mt][nt], ah, sl[2 * nt], sl[2 * nt + 1]);
+                    mma_tf32(small[mt][nt], al, sh[2 * nt], sh[2 * nt + 1]);
+                }
+            }
+        }
+#pragma unroll
+        for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+                for (int i = 0; i < 4; i += 2)
+                    *reinterpret_cast<float2 *>(red + (part * 2 * CH + mt * CH + g + 4 * i) * CB + cg + 8 * nt + 2 * q) =
+                        make_float2(big[mt][nt][i] + small[mt][nt][i], big[mt][nt][i + 1] + small[mt][nt][i + 1]);
+        asm volatile("bar.sync 2, 128;" ::: "memory");
+        // thread: column uc, tokens ut .. ut + TPT - 1
+        const uint32_t uc = tid % CB, ut = tid / CB * TPT;
+        float o[TPT];
+#pragma unroll
+        for (uint32_t i = 0; i < TPT; ++i) {
+            const uint32_t t = ut + i;
+            float x = bv[t * CB + uc];
+            o[i] = 0.0f;
+#pragma unroll
+            for (uint32_t r = 0; r < PARTS; ++r) {
+                x -= red[(r * 2 * CH + t) * CB + uc];
+                o[i] += red[(r * 2 * CH + CH + t) * CB + uc];
+            }
+            X[t * LDU + uc] = t < n ? x : 0.0f;
+        }
+        asm volatile("bar.sync 2, 128;" ::: "memory");
+        {
+            float x[CH];
+#pragma unroll
+            for (uint32_t r = 0; r < CH; ++r) x[r] = X[r * LDU + uc];
+#pragma unroll
+            for (uint32_t i = 0; i < TPT; ++i) {
+                float u = 0.0f;
+#pragma unroll
+                for (uint32_t r = 0; r < CH; r += 4) {
+                    const float4 t = *reinterpret_cast<const float4 *>(bt + (ut + i) * CH + r);
+                    u = fmaf(t.x, x[r], fmaf(t.y, x[r + 1], fmaf(t.z, x[r + 2], fmaf(t.w, x[r + 3], u))));
+                }
+                const float hi = tf32_hi(u);
+                Uh[(ut + i) * LDU + uc] = hi;
+                Ul[(ut + i) * LDU + uc] = tf32_hi(u - hi);
+                U[(ut + i) * LDU + uc] = u;
+            }
+        }
+        asm volatile("bar.sync 2, 128;" ::: "memory");
+        {  // S <- diag(c) S + K''^T U, transposed: rows = columns of the state
+            float uh[2][4], ul[2][4];
+#pragma unroll
+            for (int ts = 0; ts < 2; ++ts)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const uint32_t at = (8 * ts + q + 4 * (i >> 1)) * LDU + cg + g + 8 * (i & 1);
+                    uh[ts][i] = Uh[at];
+                    ul[ts][i] = Ul[at];
+                }
+#pragma unroll
+            for (uint32_t kt = 0; kt < NK; ++kt) {
+                const float2 c = *reinterpret_cast<const float2 *>(cend + ch0 + 8 * kt + 2 * q);
+                S[kt][0] *= c.x;
+                S[kt][1] *= c.y;
+                S[kt][2] *= c.x;
+                S[kt][3] *= c.y;
+#pragma unroll
+                for (int ts = 0; ts < 2; ++ts) {
+                    const uint32_t at = (2 * CH + 8 * ts + q) * LDF + ch0 + 8 * kt + g;
+                    const float h0 = fh[at], h1 = fh[at + 4 * LDF], l0 = fl[at], l1 = fl[at + 4 * LDF];
+                    mma_tf32(S[kt], uh[ts], l0, l1);
+                    mma_tf32(S[kt], ul[ts], h0, h1);
+                    mma_tf32(S[kt], uh[ts], h0, h1);
+                }
+            }
+        }
+        {
+            float u[CH];
+#pragma unroll
+            for (uint32_t r = 0; r < CH; ++r) u[r] = U[r * LDU + uc];
+#pragma unroll
+            for (uint32_t i = 0; i < TPT; ++i) {
+                const uint32_t t = ut + i;
+#pragma unroll
+                for (uint32_t r = 0; r < CH; r += 4) {
+                    const float4 b = *reinterpret_cast<const float4 *>(bb + t * CH + r);
+                    o[i] = fmaf(b.x, u[r], fmaf(b.y, u[r + 1], fmaf(b.z, u[r + 2], fmaf(b.w, u[r + 3], o[i]))));
+                }
+                if (t < n && uc < ncol) p.o[(size_t)(t0 + t) * s.vd + h * s.vdim + c0 + uc] = o[i];
+            }
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (uint32_t kt = 0; kt < NK; ++kt)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const uint32_t row = ch0 + 8 * kt + 2 * q + (i & 1), col = c0 + cg + g + 8 * (i >> 1);
+            if (row < s.dim && col < s.vdim) p.state[((size_t)h * s.dim + row) * s.vdim + col] = S[kt][i];
+        }
+}
+
 // o / rms(o) * w * sigmoid(gate), per head; one warp per (token, head)
 template <typename T>
 __global__ void __launch_bounds__(256) delta_out_kernel(const float *o, const float *gate, uint32_t ldg, const float *w, T *out, uint32_t ldo, uint32_t heads,
@@ -474,20 +754,17 @@ struct DeltaStep {
 };
 constexpr int STEP_THREADS = 512, STEP_R = 8, STEP_C = 4;  // state kept in registers up to 128 x 128
 
-__device__ __forceinline__ float row_dot(const uint16_t *w, const float *x, uint32_t n, uint32_t lane) {
-    float s = 0.0f;
-    for (uint32_t c = lane * 8; c < n; c += 256) {
-        const uint4 q = *reinterpret_cast<const uint4 *>(w + c);
-        s = fmaf(bf16_lo(q.x), x[c], s);
-        s = fmaf(bf16_hi(q.x), x[c + 1], s);
-        s = fmaf(bf16_lo(q.y), x[c + 2], s);
-        s = fmaf(bf16_hi(q.y), x[c + 3], s);
-        s = fmaf(bf16_lo(q.z), x[c + 4], s);
-        s = fmaf(bf16_hi(q.z), x[c + 5], s);
-        s = fmaf(bf16_lo(q.w), x[c + 6], s);
-        s = fmaf(bf16_hi(q.w), x[c + 7], s);
-    }
-    return warp_sum(s);
+// eight weights times eight inputs
+__device__ __forceinline__ float dot8(const uint4 &q, const float *x, float s) {
+    const float4 a = *reinterpret_cast<const float4 *>(x), b = *reinterpret_cast<const float4 *>(x + 4);
+    s = fmaf(bf16_lo(q.x), a.x, s);
+    s = fmaf(bf16_hi(q.x), a.y, s);
+    s = fmaf(bf16_lo(q.y), a.z, s);
+    s = fmaf(bf16_hi(q.y), a.w, s);
+    s = fmaf(bf16_lo(q.z), b.x, s);
+    s = fmaf(bf16_hi(q.z), b.y, s);
+    s = fmaf(bf16_lo(q.w), b.z, s);
+    return fmaf(bf16_hi(q.w), b.w, s);
 }
 
 // Block = head. Warp w owns state rows w, w + 16, ..; lanes run along the columns.
@@ -500,16 +777,22 @@ __global__ void __launch_bounds__(STEP_THREADS, 1) delta_step_kernel(DeltaStep p
           *rq = rk + 16 * s.vdim, *red = rq + 16 * s.vdim, *a1 = red + 8 + ((0u - (3 * s.dim + 35 * s.vdim)) & 3u), *g1 = a1 + ra8;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     float *S = p.state + (size_t)h * s.dim * s.vdim;
-    float keep[STEP_R][STEP_C];
-    if (KEEP) {  // no kernel that may still be running writes the state
+    // Row i of the head's low-rank factors: the decay's rows, then the gate's. Warp w takes rows w, w + 16, .. in batches of
+    // eight; the first batch's weights and the state's cache lines are asked for ahead of the kernel before this one.
+    const uint32_t nrows = s.dim + s.vdim;
+    uint4 fw[8];
+    auto factor_load = [&](uint32_t r0, uint32_t c) {
 #pragma unroll
-        for (int r = 0; r < STEP_R; ++r)
-#pragma unroll
-            for (int c = 0; c < STEP_C; ++c) {
-                const uint32_t row = warp + 16 * r, col = lane + 32 * c;
-                keep[r][c] = (row < s.dim && col < s.vdim) ? S[(size_t)row * s.vdim + col] : 0.0f;
-            }
-    }
+        for (int j = 0; j < 8; ++j) {
+            const uint32_t i = r0 + 16 * j;
+            const bool decay = i < s.dim;
+            fw[j] = (i < nrows && c < (decay ? ra8 : rg8))
+                        ? *reinterpret_cast<const uint4 *>(decay ? p.wa2 + (size_t)(h * s.dim + i) * p.lda2 + c : p.wg2 + (size_t)(h * s.vdim + i - s.dim) * p.ldg2 + c)
+                        : make_uint4(0, 0, 0, 0);
+        }
+    };
+    factor_load(warp, lane * 8);
+    for (uint32_t i = tid; i < (s.dim * s.vdim + 31) / 32; i += STEP_THREADS) asm volatile("prefetch.global.L2 [%0];" ::"l"(S + (size_t)i * 32));
     pdl_wait();
     pdl_launch();
     const uint32_t pos = *p.pos;
@@ -530,14 +813,35 @@ __global__ void __launch_bounds__(STEP_THREADS, 1) delta_step_kernel(DeltaStep p
         p.ring[(size_t)(pos % s.taps) * cv.channels + ch] = x;
     }
     const float decay = expf(p.a_log[h]);
-    for (uint32_t i = warp; i < s.dim + s.vdim; i += 16) {
-        if (i < s.dim) {
-            const float z = row_dot(p.wa2 + (size_t)(h * s.dim + i) * p.lda2, a1, ra8, lane) + p.dt_bias[h * s.dim + i];
-            if (lane == 0) sg[i] = expf(-decay * softplus_f(z));
-        } else {
-            const float z = row_dot(p.wg2 + (size_t)(h * s.vdim + i - s.dim) * p.ldg2, g1, rg8, lane);
-            if (lane == 0) gate[i - s.dim] = sigmoid_f(z);
+    for (uint32_t r0 = warp; r0 < nrows; r0 += 128) {
+        float z[8] = {};
+        for (uint32_t c = lane * 8; c < max(ra8, rg8); c += 256) {
+            if (r0 != (uint32_t)warp || c != lane * 8) factor_load(r0, c);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                const bool dec = r0 + 16 * j < s.dim;
+                if (c < (dec ? ra8 : rg8)) z[j] = dot8(fw[j], (dec ? a1 : g1) + c, z[j]);
+            }
         }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const uint32_t i = r0 + 16 * j;
+            const float v = warp_sum(z[j]);
+            if (lane == 0 && i < nrows) {
+                if (i < s.dim) sg[i] = expf(-decay * softplus_f(v + p.dt_bias[h * s.dim + i]));
+                else gate[i - s.dim] = sigmoid_f(v);
+            }
+        }
+    }
+    float keep[STEP_R][STEP_C];
+    if (KEEP) {
+#pragma unroll
+        for (int r = 0; r < STEP_R; ++r)
+#pragma unroll
+            for (int c = 0; c < STEP_C; ++c) {
+                const uint32_t row = warp + 16 * r, col = lane + 32 * c;
+                keep[r][c] = (row < s.dim && col < s.vdim) ? S[(size_t)row * s.vdim + col] : 0.0f;
+            }
     }
     if (warp < 3) {  // |q|^2, |k|^2, k . q before the scaling
         float v = 0.0f;
@@ -712,12 +1016,11 @@ class ChannelDelta : public Mixer {
         const uint32_t channels = 2 * s_.qk + s_.vd;
         DeltaChunk cp{s_, ConvView{ring_, channels, s_.taps, r.pos0}, f(at_.q), f(at_.k), f(at_.v), f(at_.b), f(at_.z), ldqk_, ldv_, ldb_, ldz_, r.tokens, wq_, wk_, wv_, a_log_,
                       f(at_.qn), f(at_.kn), f(at_.vn), f(at_.g), f(at_.tb)};
-        const size_t csm = 3ull * CH * s_.dim * 4;
-        BRASA_TRY(brasa_smem_optin(ctx, (const void *)delta_chunk_kernel, csm));
-        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_chunk_kernel, dim3((r.tokens + CH - 1) / CH, s_.kv_heads), dim3(256), csm, cp));
-        BRASA_TRY(brasa_post_launch(r.cmd, "delta_chunk"));
+        if (s_.dim <= 64) BRASA_TRY(factors<2>(r.cmd, cp));
+        else if (s_.dim <= 128) BRASA_TRY(factors<4>(r.cmd, cp));
+        else BRASA_TRY(factors<8>(r.cmd, cp));
         DeltaScan sp{s_, f(at_.qn), f(at_.kn), f(at_.vn), f(at_.g), f(at_.tb), f(at_.q), f(at_.k), f(at_.v), ldqk_, ldv_, ring_, state_, f(at_.o), r.tokens, r.pos0};
-        BRASA_TRY(scan(r.cmd, sp));
+        BRASA_TRY(scan(r.cmd, sp, r.f32));
         const uint32_t blocks = (r.tokens * s_.heads + 7) / 8;
         if (r.f32) BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_out_kernel<float>, dim3(blocks), dim3(256), 0, f(at_.o), f(at_.gate), ldv_, norm_, (float *)r.out, r.ldo,
                                                           s_.heads, s_.vdim, r.tokens, eps_));
@@ -727,6 +1030,14 @@ class ChannelDelta : public Mixer {
     }
 
   private:
+    template <int E>
+    int32_t factors(brasa_cmd *cmd, const DeltaChunk &p) {
+        brasa_ctx *ctx = cmd->ctx;
+        const size_t smem = 3ull * CH * 32 * E * 4;
+        BRASA_TRY(brasa_smem_optin(ctx, (const void *)delta_chunk_kernel<E>, std::max<size_t>(smem, 48 * 1024)));
+        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_chunk_kernel<E>, dim3((p.tokens + CH - 1) / CH, s_.heads), dim3(256), smem, p));
+        return brasa_post_launch(cmd, "delta_chunk");
+    }
     template <int D, int CB>
     int32_t scan_as(brasa_cmd *cmd, const DeltaScan &p) {
         brasa_ctx *ctx = cmd->ctx;
@@ -735,9 +1046,19 @@ class ChannelDelta : public Mixer {
         BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_scan_kernel<D, CB>, dim3(s_.heads, (s_.vdim + CB - 1) / CB), dim3(256), smem, p));
         return brasa_post_launch(cmd, "delta_scan");
     }
-    int32_t scan(brasa_cmd *cmd, const DeltaScan &p) {
+    template <int D, int CB>
+    int32_t scan_mma(brasa_cmd *cmd, const DeltaScan &p) {
+        brasa_ctx *ctx = cmd->ctx;
+        const size_t smem = (size_t)MmaScanShape<D, CB>::FLOATS * 4;
+        BRASA_TRY(brasa_smem_optin(ctx, (const void *)delta_scan_mma_kernel<D, CB>, smem));
+        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_scan_mma_kernel<D, CB>, dim3(s_.heads, (s_.vdim + CB - 1) / CB), dim3(256), smem, p));
+        return brasa_post_launch(cmd, "delta_scan_mma");
+    }
+    int32_t scan(brasa_cmd *cmd, const DeltaScan &p, bool f32) {
         // wide blocks when they still cover most of the SMs
         const bool wide = s_.heads * ((s_.vdim + 31) / 32) * 5 >= (uint32_t)cmd->ctx->sm_count * 4;
+        if (!f32 && s_.dim <= 64) return wide ? scan_mma<64, 32>(cmd, p) : scan_mma<64, 16>(cmd, p);
+        if (!f32 && s_.dim <= 128) return wide ? scan_mma<128, 32>(cmd, p) : scan_mma<128, 16>(cmd, p);
         if (s_.dim <= 64) return wide ? scan_as<64, 32>(cmd, p) : scan_as<64, 16>(cmd, p);
         if (s_.dim <= 128) return wide ? scan_as<128, 32>(cmd, p) : scan_as<128, 16>(cmd, p);
         return scan_as<256, 16>(cmd, p);

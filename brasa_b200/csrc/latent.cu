@@ -146,15 +146,18 @@ __global__ void __launch_bounds__(256) latent_partial_kernel(LatentShape s, cons
     for (uint32_t k0 = beg; k0 < end; k0 += PK) {
         const uint32_t n = min(PK, end - k0);
         __syncthreads();
-        for (uint32_t i = tid; i < PK * (c16 + r16); i += 256) {
-            const uint32_t k = i / (c16 + r16), e = i - k * (c16 + r16);
-            uint4 v = make_uint4(0, 0, 0, 0);
-            if (k < n) {
-                const size_t slot = (k0 + k) % s.rows;
-                v = e < c16 ? *reinterpret_cast<const uint4 *>(c + slot * s.ldc + e * E) : *reinterpret_cast<const uint4 *>(r + slot * s.ldr + (e - c16) * E);
+#pragma unroll
+        for (uint32_t i = 0; i < PK / 8; ++i) {  // warp w: keys w, w + 8, ..
+            const uint32_t k = warp + 8 * i;
+            const size_t slot = (k0 + k) % s.rows;
+            for (uint32_t e = lane; e < c16 + r16; e += 32) {
+                T *dst = ks + (size_t)k * ldk + e * E;
+                const T *src = e < c16 ? c + slot * s.ldc + e * E : r + slot * s.ldr + (e - c16) * E;
+                if (k < n) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+                else *reinterpret_cast<uint4 *>(dst) = make_uint4(0, 0, 0, 0);
             }
-            *reinterpret_cast<uint4 *>(ks + (size_t)k * ldk + e * E) = v;
         }
+        asm volatile("cp.async.wait_all;" ::: "memory");
         __syncthreads();
         // scores: warp = head, lane = key
         float sc = 0.0f;
@@ -246,22 +249,35 @@ __global__ void __launch_bounds__(256) latent_partial_kernel(LatentShape s, cons
     }
 }
 
-// Block (h, y): head h's latent sum over all chunks, then value rows [y vper, (y + 1) vper) of the head, gated.
+// Block (h, y): head h's latent sum over all chunks, then value rows [y vper, (y + 1) vper) of the head, gated. A warp takes
+// rows warp, warp + 8, ..; the weights of its first four rows (latents up to 512 wide) are asked for ahead of the partial sums.
+constexpr uint32_t CR = 4;
 __global__ void __launch_bounds__(256) latent_combine_kernel(LatentShape s, const float *part, uint32_t chunks, const uint16_t *uv, uint32_t ldv, const float *gate,
                                                              float *out, uint32_t vper) {
     extern __shared__ __align__(16) float sm[];
     float *o = sm, *wt = sm + s.ldc;  // wt: [chunks]
     const uint32_t h = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const size_t ldp = s.ldc + 2;
+    const uint32_t v0 = blockIdx.y * vper + warp, v1 = min(s.vdim, (blockIdx.y + 1) * vper);
+    auto weights = [&](uint32_t v, uint32_t c) {
+        return v < v1 && c < ldv ? __ldcs(reinterpret_cast<const uint4 *>(uv + (size_t)(h * s.vdim + v) * ldv + c)) : make_uint4(0, 0, 0, 0);
+    };
+    uint4 pre[CR][2];
+#pragma unroll
+    for (uint32_t i = 0; i < CR; ++i)
+#pragma unroll
+        for (uint32_t j = 0; j < 2; ++j) pre[i][j] = weights(v0 + 8 * i, lane * 8 + 256 * j);
     pdl_wait();
     pdl_launch();
+    const float *ph = part + (size_t)h * ldp;
+    const size_t step = (size_t)s.heads * ldp;
     float m = -INFINITY;
-    for (uint32_t k = lane; k < chunks; k += 32) m = fmaxf(m, part[(k * (size_t)s.heads + h) * ldp + s.ldc]);
+    for (uint32_t k = lane; k < chunks; k += 32) m = fmaxf(m, ph[k * step + s.ldc]);
 #pragma unroll
     for (int i = 16; i > 0; i >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, i));
     float l = 0.0f;
     for (uint32_t k = lane; k < chunks; k += 32) {
-        const float *p = part + (k * (size_t)s.heads + h) * ldp + s.ldc;
+        const float *p = ph + k * step + s.ldc;
         const float w = p[0] == -INFINITY ? 0.0f : expf(p[0] - m);
         if (warp == 0) wt[k] = w;
         l = fmaf(w, p[1], l);
@@ -271,27 +287,42 @@ __global__ void __launch_bounds__(256) latent_combine_kernel(LatentShape s, cons
     const float g = 1.0f / (1.0f + expf(-gate[h])) / l;
     for (uint32_t c = tid; c < s.ldc; c += 256) {
         float a = 0.0f;
-        for (uint32_t k = 0; k < chunks; ++k)
-            if (wt[k] > 0.0f) a = fmaf(wt[k], part[(k * (size_t)s.heads + h) * ldp + c], a);  // (an empty chunk wrote no sums)
+        for (uint32_t k0 = 0; k0 < chunks; k0 += 8) {
+            float v[8];
+#pragma unroll
+            for (uint32_t k = 0; k < 8; ++k) v[k] = k0 + k < chunks && wt[k0 + k] > 0.0f ? ph[(k0 + k) * step + c] : 0.0f;  // (an empty chunk wrote no sums)
+#pragma unroll
+            for (uint32_t k = 0; k < 8; ++k)
+                if (k0 + k < chunks) a = fmaf(wt[k0 + k], v[k], a);
+        }
         o[c] = a;
     }
     __syncthreads();
-    const uint32_t v1 = min(s.vdim, (blockIdx.y + 1) * vper);
-    for (uint32_t v = blockIdx.y * vper + warp; v < v1; v += 8) {
-        const uint16_t *w = uv + (size_t)(h * s.vdim + v) * ldv;
+    auto dot8 = [&](const uint4 &q, uint32_t c, float a) {
+        const float4 x = *reinterpret_cast<const float4 *>(o + c), y = *reinterpret_cast<const float4 *>(o + c + 4);
+        a = fmaf(bf16_lo(q.x), x.x, a);
+        a = fmaf(bf16_hi(q.x), x.y, a);
+        a = fmaf(bf16_lo(q.y), x.z, a);
+        a = fmaf(bf16_hi(q.y), x.w, a);
+        a = fmaf(bf16_lo(q.z), y.x, a);
+        a = fmaf(bf16_hi(q.z), y.y, a);
+        a = fmaf(bf16_lo(q.w), y.z, a);
+        return fmaf(bf16_hi(q.w), y.w, a);
+    };
+#pragma unroll
+    for (uint32_t i = 0; i < CR; ++i) {
+        const uint32_t v = v0 + 8 * i;
         float a = 0.0f;
-        for (uint32_t c = lane * 8; c < ldv; c += 256) {
-            const uint4 q = *reinterpret_cast<const uint4 *>(w + c);
-            const float4 x = *reinterpret_cast<const float4 *>(o + c), y = *reinterpret_cast<const float4 *>(o + c + 4);
-            a = fmaf(bf16_lo(q.x), x.x, a);
-            a = fmaf(bf16_hi(q.x), x.y, a);
-            a = fmaf(bf16_lo(q.y), x.z, a);
-            a = fmaf(bf16_hi(q.y), x.w, a);
-            a = fmaf(bf16_lo(q.z), y.x, a);
-            a = fmaf(bf16_hi(q.z), y.y, a);
-            a = fmaf(bf16_lo(q.w), y.z, a);
-            a = fmaf(bf16_hi(q.w), y.w, a);
-        }
+#pragma unroll
+        for (uint32_t j = 0; j < 2; ++j)
+            if (lane * 8 + 256 * j < ldv) a = dot8(pre[i][j], lane * 8 + 256 * j, a);
+        for (uint32_t c = lane * 8 + 512; c < ldv; c += 256) a = dot8(weights(v, c), c, a);
+        a = warp_sum(a);
+        if (lane == 0 && v < v1) out[h * s.vdim + v] = a * g;
+    }
+    for (uint32_t v = v0 + 8 * CR; v < v1; v += 8) {
+        float a = 0.0f;
+        for (uint32_t c = lane * 8; c < ldv; c += 256) a = dot8(weights(v, c), c, a);
         a = warp_sum(a);
         if (lane == 0) out[h * s.vdim + v] = a * g;
     }
@@ -442,7 +473,7 @@ class LatentAttention : public Mixer {
         BRASA_CUDA(ctx, brasa_launch_dependent(ctx, latent_partial_kernel<T>, dim3(chunks_, (s_.heads + PH - 1) / PH), dim3(256), smem, s_, f(at_.qa), c, kr, f(at_.part), per_,
                                                r.dev_pos));
         BRASA_TRY(brasa_post_launch(r.cmd, "latent_partial"));
-        const uint32_t split = std::max(1u, std::min((s_.vdim + 7) / 8, 296u / s_.heads)), vper = (s_.vdim + split - 1) / split;
+        const uint32_t split = std::max(1u, std::min((s_.vdim + 7) / 8, 148u / s_.heads)), vper = (s_.vdim + split - 1) / split;
         const size_t csm = (size_t)(s_.ldc + chunks_) * 4;
         BRASA_TRY(brasa_smem_optin(ctx, (const void *)latent_combine_kernel, std::max<size_t>(csm, 48 * 1024)));
         BRASA_CUDA(ctx, brasa_launch_dependent(ctx, latent_combine_kernel, dim3(s_.heads, (s_.vdim + vper - 1) / vper), dim3(256), csm, s_, f(at_.part), chunks_, uv_.p, uv_.ld,

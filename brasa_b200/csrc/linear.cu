@@ -116,22 +116,46 @@ __global__ void __launch_bounds__(32 * GV_WARPS, 1) linear_gemv_kernel(const __g
     constexpr uint32_t TEAMS = GV_WARPS / S;
     const uint32_t team = blockIdx.x * TEAMS + warp / S, teams = gridDim.x * TEAMS, sub = warp % S;
     const uint32_t half = gp.x_floats / 2;
-    auto locate = [&](uint32_t row, uint32_t &pi) {
-        pi = 0;
-        while (pi + 1 < gp.n && row >= gp.row_end[pi]) ++pi;
-        return row - (pi ? gp.row_end[pi - 1] : 0u);
+    // A warp's work is a list of batches of up to GV_UNROLL x 16 bytes per lane: along a row's first segment, its second, the
+    // team's next row, .. The next batch's weights are in flight while this one is multiplied.
+    struct Cursor {
+        uint32_t row, pi, r, seg, c0;
     };
-    // the first weights of this warp's first row
-    uint4 pre[GV_UNROLL];
-    {
-        uint32_t pi;
-        const uint32_t r = locate(min(team, gp.total_rows - 1), pi);
-        const uint16_t *w = gp.p[pi].w[0] + (size_t)r * gp.p[pi].ldw[0];
+    auto place = [&](Cursor &c) {  // problem and row of c.row
+        c.pi = 0;
+        while (c.pi + 1 < gp.n && c.row >= gp.row_end[c.pi]) ++c.pi;
+        c.r = c.row - (c.pi ? gp.row_end[c.pi - 1] : 0u);
+    };
+    auto load = [&](const Cursor &c, uint4 *q) {
+        const GemvDevProblem &p = gp.p[c.pi];
+        const uint32_t cols = p.cols8[c.seg];
+        const uint16_t *w = p.w[c.seg] + (size_t)c.r * p.ldw[c.seg];
 #pragma unroll
         for (int u = 0; u < GV_UNROLL; ++u) {
-            const uint32_t c = (sub * 32 + lane) * 8 + u * 256 * S;
-            pre[u] = c < gp.p[pi].cols8[0] ? __ldcs(reinterpret_cast<const uint4 *>(w + c)) : make_uint4(0, 0, 0, 0);
+            const uint32_t k = c.c0 + (sub * 32 + lane) * 8 + u * 256 * S;
+            q[u] = k < cols ? __ldcs(reinterpret_cast<const uint4 *>(w + k)) : make_uint4(0, 0, 0, 0);
         }
+    };
+    auto advance = [&](Cursor &c) {  // false at the end; a new row has seg == 0 and c0 == 0
+        c.c0 += GV_UNROLL * 256 * S;
+        if (c.c0 < gp.p[c.pi].cols8[c.seg]) return true;
+        c.c0 = 0;
+        if (c.seg == 0 && gp.p[c.pi].cols8[1]) {
+            c.seg = 1;
+            return true;
+        }
+        c.seg = 0;
+        c.row += teams;
+        if (c.row >= gp.total_rows) return false;
+        place(c);
+        return true;
+    };
+    Cursor cur{team, 0, 0, 0, 0};
+    bool more = team < gp.total_rows;
+    uint4 q[GV_UNROLL];
+    if (more) {
+        place(cur);
+        load(cur, q);
     }
     pdl_wait();
     pdl_launch();
@@ -158,64 +182,53 @@ __global__ void __launch_bounds__(32 * GV_WARPS, 1) linear_gemv_kernel(const __g
             for (uint32_t i = tid; i < gp.len[k]; i += 32 * GV_WARPS) xs[gv_plane(gp.off[k] + i, half)] = gp.v[k][i];
     }
     __syncthreads();
-    // ---- rows ----
-    const uint32_t iters = (gp.total_rows + teams - 1) / teams;
-    for (uint32_t it = 0; it < iters; ++it) {
-        const uint32_t row = team + it * teams;
-        float acc = 0.0f;
-        uint32_t pi = 0, r = 0;
-        if (row < gp.total_rows) {
-            r = locate(row, pi);
-            const GemvDevProblem &p = gp.p[pi];
-#pragma unroll 1
-            for (int s = 0; s < 2; ++s) {
-                const uint32_t cols = p.cols8[s];
-                const uint16_t *w = p.w[s] + (size_t)r * p.ldw[s];
-                const float *x = xs + (p.xoff[s] >> 1);
-                for (uint32_t c0 = (sub * 32 + lane) * 8; c0 < cols; c0 += GV_UNROLL * 256 * S) {
-                    uint4 q[GV_UNROLL];
-                    if (it == 0 && s == 0 && c0 < 256 * S) {
+    // ---- batches ----
+    float acc = 0.0f;
+    uint32_t parity = 0;
+    while (more) {
+        Cursor nxt = cur;
+        const bool go_on = advance(nxt);
+        uint4 qn[GV_UNROLL];
+        if (go_on) load(nxt, qn);
+        const GemvDevProblem &p = gp.p[cur.pi];
+        const float *x = xs + (p.xoff[cur.seg] >> 1);
+        const uint32_t cols = p.cols8[cur.seg];
 #pragma unroll
-                        for (int u = 0; u < GV_UNROLL; ++u) q[u] = pre[u];
-                    } else {
-#pragma unroll
-                        for (int u = 0; u < GV_UNROLL; ++u) {
-                            const uint32_t c = c0 + u * 256 * S;
-                            q[u] = c < cols ? __ldcs(reinterpret_cast<const uint4 *>(w + c)) : make_uint4(0, 0, 0, 0);
-                        }
-                    }
-#pragma unroll
-                    for (int u = 0; u < GV_UNROLL; ++u) {
-                        const uint32_t c = c0 + u * 256 * S;
-                        if (c < cols) {
-                            const float4 a = *reinterpret_cast<const float4 *>(x + (c >> 1)), b = *reinterpret_cast<const float4 *>(x + half + (c >> 1));
-                            acc = fmaf(bf16_lo(q[u].x), a.x, acc);
-                            acc = fmaf(bf16_hi(q[u].x), a.y, acc);
-                            acc = fmaf(bf16_lo(q[u].y), a.z, acc);
-                            acc = fmaf(bf16_hi(q[u].y), a.w, acc);
-                            acc = fmaf(bf16_lo(q[u].z), b.x, acc);
-                            acc = fmaf(bf16_hi(q[u].z), b.y, acc);
-                            acc = fmaf(bf16_lo(q[u].w), b.z, acc);
-                            acc = fmaf(bf16_hi(q[u].w), b.w, acc);
-                        }
-                    }
-                }
+        for (int u = 0; u < GV_UNROLL; ++u) {
+            const uint32_t c = cur.c0 + (sub * 32 + lane) * 8 + u * 256 * S;
+            if (c < cols) {
+                const float4 a = *reinterpret_cast<const float4 *>(x + (c >> 1)), b = *reinterpret_cast<const float4 *>(x + half + (c >> 1));
+                acc = fmaf(bf16_lo(q[u].x), a.x, acc);
+                acc = fmaf(bf16_hi(q[u].x), a.y, acc);
+                acc = fmaf(bf16_lo(q[u].y), a.z, acc);
+                acc = fmaf(bf16_hi(q[u].y), a.w, acc);
+                acc = fmaf(bf16_lo(q[u].z), b.x, acc);
+                acc = fmaf(bf16_hi(q[u].z), b.y, acc);
+                acc = fmaf(bf16_lo(q[u].w), b.z, acc);
+                acc = fmaf(bf16_hi(q[u].w), b.w, acc);
             }
+        }
+        if (!go_on || (nxt.seg == 0 && nxt.c0 == 0)) {  // the row is complete
 #pragma unroll
             for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+            if (S > 1) {  // (the warps of a team walk the same batches)
+                if (lane == 0) part[parity][warp] = acc;
+                asm volatile("bar.sync %0, %1;" ::"r"(warp / S), "r"(32 * S) : "memory");
+                if (sub == 0 && lane == 0)
+                    for (int k = 1; k < S; ++k) acc += part[parity][warp + k];
+                parity ^= 1;
+            }
+            if (sub == 0 && lane == 0) {
+                float v = activate(acc + (p.bias ? p.bias[cur.r] : 0.0f), p.act) * p.scale;
+                if (p.resid) v += p.resid[cur.r];
+                p.y[cur.r] = v;
+            }
+            acc = 0.0f;
         }
-        if (S > 1) {
-            if (lane == 0) part[it & 1][warp] = acc;
-            __syncthreads();
-            if (sub == 0 && lane == 0)
-                for (int k = 1; k < S; ++k) acc += part[it & 1][warp + k];
-        }
-        if (row < gp.total_rows && sub == 0 && lane == 0) {
-            const GemvDevProblem &p = gp.p[pi];
-            float v = activate(acc + (p.bias ? p.bias[r] : 0.0f), p.act) * p.scale;
-            if (p.resid) v += p.resid[r];
-            p.y[r] = v;
-        }
+        more = go_on;
+        cur = nxt;
+#pragma unroll
+        for (int u = 0; u < GV_UNROLL; ++u) q[u] = qn[u];
     }
 }
 
@@ -550,7 +563,7 @@ int32_t brasa_linear_gemv_launch(brasa_cmd *cmd, const GemvInput &in, const Gemv
     }
     g.x_floats = off;
     BRASA_REQUIRE(ctx, g.nin >= 1 && (g.nin == 1 || g.len[0] > 0), "gemv: no input");
-    uint32_t rows = 0, widest = 0;
+    uint32_t rows = 0;
     for (uint32_t i = 0; i < n; ++i) {
         const LinearProblem &q = ps[i].p;
         GemvDevProblem &d = g.p[i];
@@ -563,7 +576,6 @@ int32_t brasa_linear_gemv_launch(brasa_cmd *cmd, const GemvInput &in, const Gemv
             d.ldw[s] = sg.ldw;
             d.cols8[s] = up8(sg.cols);
             d.xoff[s] = g.off[k];
-            widest = std::max(widest, d.cols8[s]);
         }
         if (!d.w[1]) d.w[1] = d.w[0];
         d.rows = q.rows;
@@ -579,15 +591,15 @@ int32_t brasa_linear_gemv_launch(brasa_cmd *cmd, const GemvInput &in, const Gemv
     g.total_rows = rows;
     const size_t smem = (size_t)g.x_floats * 4;
     BRASA_REQUIRE(ctx, rows > 0 && smem + 4096 <= ctx->smem_optin, "gemv: input of %u values is too long", g.x_floats);
-    // how many warps share a row: the fewest that keep the last round of rows nearly full
-    uint32_t best = 1;
-    double best_eff = 0.0;
+    // how many warps share a row: what leaves the busiest warp the fewest batches
+    uint32_t best = 1, best_cost = UINT32_MAX;
     for (uint32_t s = 1; s <= 8; s *= 2) {
-        if (s > 1 && widest < 256 * s) break;
-        const uint32_t teams = (uint32_t)ctx->sm_count * GV_WARPS / s;
-        const double eff = (double)rows / ((double)((rows + teams - 1) / teams) * teams) - 0.02 * (s - 1);
-        if (eff > best_eff + 0.01) {
-            best_eff = eff;
+        const uint32_t teams = (uint32_t)ctx->sm_count * GV_WARPS / s, step = GV_UNROLL * 256 * s;
+        uint64_t batches = 0;
+        for (uint32_t i = 0; i < n; ++i) batches += (uint64_t)g.p[i].rows * ((g.p[i].cols8[0] + step - 1) / step + (g.p[i].cols8[1] + step - 1) / step);
+        const uint32_t rounds = (rows + teams - 1) / teams, cost = (uint32_t)(rounds * ((batches + rows - 1) / rows) * 16 + rounds * (s > 1 ? 4 : 1));
+        if (cost < best_cost) {
+            best_cost = cost;
             best = s;
         }
     }

@@ -149,6 +149,7 @@ struct LayerNormParams {
     uint32_t n, ldo;
     float eps;
 };
+constexpr int LN_VEC = 5;  // float4s of a row per thread
 template <int NOUT, typename T>
 __global__ void __launch_bounds__(256) layer_norm_kernel(LayerNormParams p) {
     __shared__ float red[8];
@@ -164,6 +165,39 @@ __global__ void __launch_bounds__(256) layer_norm_kernel(LayerNormParams p) {
         return v;
     };
     float s = 0.0f;
+    if ((p.n & 3) == 0 && p.n <= 256 * 4 * LN_VEC && (p.ldo & 3) == 0) {  // the row in registers, four values at a time
+        const float4 *x4 = reinterpret_cast<const float4 *>(x);
+        float4 v[LN_VEC];
+#pragma unroll
+        for (int c = 0; c < LN_VEC; ++c) {
+            const uint32_t i = threadIdx.x + 256 * c;
+            v[c] = i < p.n / 4 ? x4[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+            s += (v[c].x + v[c].y) + (v[c].z + v[c].w);
+        }
+        const float mean = block_sum(s) / (float)p.n;
+        s = 0.0f;
+#pragma unroll
+        for (int c = 0; c < LN_VEC; ++c)
+            if (threadIdx.x + 256 * c < p.n / 4) {
+                v[c] = make_float4(v[c].x - mean, v[c].y - mean, v[c].z - mean, v[c].w - mean);
+                s += (v[c].x * v[c].x + v[c].y * v[c].y) + (v[c].z * v[c].z + v[c].w * v[c].w);
+            }
+        const float inv = 1.0f / sqrtf(block_sum(s) / (float)p.n + p.eps);
+#pragma unroll
+        for (int c = 0; c < LN_VEC; ++c) {
+            const uint32_t i = threadIdx.x + 256 * c;
+            if (i < p.n / 4)
+#pragma unroll
+                for (int k = 0; k < NOUT; ++k) {
+                    const float4 w = reinterpret_cast<const float4 *>(p.w[k])[i], b = reinterpret_cast<const float4 *>(p.b[k])[i];
+                    const float4 o = make_float4(fmaf(v[c].x * inv, w.x, b.x), fmaf(v[c].y * inv, w.y, b.y), fmaf(v[c].z * inv, w.z, b.z), fmaf(v[c].w * inv, w.w, b.w));
+                    T *dst = static_cast<T *>(p.out[k]) + (size_t)blockIdx.x * p.ldo + 4 * i;
+                    if (sizeof(T) == 4) *reinterpret_cast<float4 *>(dst) = o;
+                    else *reinterpret_cast<uint2 *>(dst) = make_uint2(brasa_dev::bf16_pack(o.x, o.y), brasa_dev::bf16_pack(o.z, o.w));
+                }
+        }
+        return;
+    }
     for (uint32_t i = threadIdx.x; i < p.n; i += 256) s += x[i];
     const float mean = block_sum(s) / (float)p.n;
     s = 0.0f;

@@ -155,7 +155,7 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
     const uint32_t lo = max(a.key0, qfirst + 1 > a.window ? qfirst + 1 - a.window : 0u);
     const uint32_t jbeg = (lo - a.key0) / 128, nkt = (qlast - a.key0) / 128 + 1 - jbeg;
 
-    if (tid == 0) {
+    if (tid == 256) {  // the issuing thread, which asks for the first tiles before the block meets
         for (int i = 0; i < 2; ++i) {
             mbar_init(&bar_s[i], 1);
             mbar_init(&bar_k[i], 1);
@@ -171,8 +171,31 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
     }
     pdl_wait();
     pdl_launch();
+    uint32_t inflight = 0;  // issuing thread: bit b = a K copy into buffer b, bit 2 + b = a V copy, not yet waited for
+    auto fetch_k = [&](uint32_t j) {
+        const uint32_t b = KBUF == 2 ? (j & 1) : 0u;
+        const int row = (int)((jbeg + j) * 128);
+        mbar_expect_tx(&bar_k[b], NQ * BLK);
+#pragma unroll
+        for (int i = 0; i < NU; ++i) tma_load_3d(KB(j) + i * BLK, &maps.k, i * 64, (int)h, row, &bar_k[b]);
+#pragma unroll
+        for (int i = 0; i < NR; ++i) tma_load_2d(KB(j) + (NU + i) * BLK, &maps.kr, i * 64, row, &bar_k[b]);
+        inflight |= 1u << b;
+    };
+    auto fetch_v = [&](uint32_t j) {
+        mbar_expect_tx(&bar_v[j & 1], NV * BLK);
+#pragma unroll
+        for (int i = 0; i < NV; ++i) tma_load_3d(VB(j) + i * BLK, &maps.v, i * 64, (int)h, (int)((jbeg + j) * 128), &bar_v[j & 1]);
+        inflight |= 4u << (j & 1);
+    };
+    if (tid == 256) {
+        fetch_k(0);
+        fetch_v(0);
+        if (KBUF == 2 && nkt > 1) fetch_k(1);
+    }
     // Q tile: rotated, rounded to bf16, swizzled K-major; rows past the last query and columns past the sizes are zeros
     const uint32_t half = a.rot_dims / 2;
+    const bool qvec = ((a.ldq | dq | a.dim) & 3) == 0;
     for (uint32_t i = tid; i < 128 * NQ * 8; i += 288) {
         const uint32_t r = i / (NQ * 8), c = i - r * (NQ * 8), blk = c >> 3, c8 = (c & 7) * 8;
         uint32_t w[4] = {0, 0, 0, 0};
@@ -181,6 +204,11 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
             const uint32_t p = qfirst + r;
             const float *ct = a.cos_t + (size_t)p * half, *st = a.sin_t + (size_t)p * half;
             float v[8];
+            if (qvec && blk < NU && blk * 64 + c8 + 8 <= a.dim) {
+                const float4 x = *reinterpret_cast<const float4 *>(q + blk * 64 + c8), y = *reinterpret_cast<const float4 *>(q + blk * 64 + c8 + 4);
+                v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+                v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
+            } else
 #pragma unroll
             for (int e = 0; e < 8; ++e) {
                 const uint32_t col = (blk < NU ? blk : blk - NU) * 64 + c8 + e;
@@ -206,23 +234,6 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
         atomicExch(status, 7u);
         *abort_flag = 1;
         return false;
-    };
-    uint32_t inflight = 0;  // issuing thread: bit b = a K copy into buffer b, bit 2 + b = a V copy, not yet waited for
-    auto fetch_k = [&](uint32_t j) {
-        const uint32_t b = KBUF == 2 ? (j & 1) : 0u;
-        const int row = (int)((jbeg + j) * 128);
-        mbar_expect_tx(&bar_k[b], NQ * BLK);
-#pragma unroll
-        for (int i = 0; i < NU; ++i) tma_load_3d(KB(j) + i * BLK, &maps.k, i * 64, (int)h, row, &bar_k[b]);
-#pragma unroll
-        for (int i = 0; i < NR; ++i) tma_load_2d(KB(j) + (NU + i) * BLK, &maps.kr, i * 64, row, &bar_k[b]);
-        inflight |= 1u << b;
-    };
-    auto fetch_v = [&](uint32_t j) {
-        mbar_expect_tx(&bar_v[j & 1], NV * BLK);
-#pragma unroll
-        for (int i = 0; i < NV; ++i) tma_load_3d(VB(j) + i * BLK, &maps.v, i * 64, (int)h, (int)((jbeg + j) * 128), &bar_v[j & 1]);
-        inflight |= 4u << (j & 1);
     };
     constexpr uint32_t idesc_s = tc_idesc_bf16(128, 128), idesc_o = tc_idesc_bf16(128, NV * 64) | (1u << 16);  // V: an MN-major B operand
     auto issue_s = [&](uint32_t j) {
@@ -256,9 +267,6 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
         return r;
     };
     if (issuer) {
-        fetch_k(0);
-        fetch_v(0);
-        if (KBUF == 2 && nkt > 1) fetch_k(1);
         if (wait_k(0)) {
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             issue_s(0);
