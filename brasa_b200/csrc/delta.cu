@@ -108,6 +108,25 @@ __device__ __forceinline__ void conv_chunk(const float *x, uint32_t ldx, uint32_
     }
 }
 
+// E consecutive floats of shared memory
+template <int E>
+__device__ __forceinline__ void load_run(const float *p, float v[E]) {
+    if (E == 2) {
+        const float2 a = *reinterpret_cast<const float2 *>(p);
+        v[0] = a.x;
+        v[1] = a.y;
+    } else {
+#pragma unroll
+        for (int j = 0; j < E; j += 4) {
+            const float4 a = *reinterpret_cast<const float4 *>(p + j);
+            v[j] = a.x;
+            v[j + 1] = a.y;
+            v[j + 2] = a.z;
+            v[j + 3] = a.w;
+        }
+    }
+}
+
 // Block: one chunk of one head. E consecutive key channels per lane: dim up to 32 E.
 template <int E>
 __global__ void __launch_bounds__(256) delta_chunk_kernel(DeltaChunk p) {
@@ -171,18 +190,24 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(DeltaChunk p) {
     for (int half = 0; half < 2; ++half) {
         const uint32_t col = half ? CH - 1 - warp : warp;
         float run[E], acc[2 * CH];
-#pragma unroll
-        for (int j = 0; j < E; ++j) run[j] = sk[col * D + lane * E + j];
+        load_run<E>(sk + col * D + lane * E, run);
 #pragma unroll
         for (uint32_t t = 0; t < CH; ++t) {
             acc[2 * t] = acc[2 * t + 1] = 0.0f;
             if (t >= col) {
+                float kk[E], qq[E];
+                load_run<E>(sk + t * D + lane * E, kk);
+                load_run<E>(sq + t * D + lane * E, qq);
+                if (t > col) {
+                    float gg[E];
+                    load_run<E>(sg + t * D + lane * E, gg);
+#pragma unroll
+                    for (int j = 0; j < E; ++j) run[j] *= gg[j];
+                }
 #pragma unroll
                 for (int j = 0; j < E; ++j) {
-                    const uint32_t e = t * D + lane * E + j;
-                    if (t > col) run[j] *= sg[e];
-                    acc[2 * t] = fmaf(sk[e], run[j], acc[2 * t]);
-                    acc[2 * t + 1] = fmaf(sq[e], run[j], acc[2 * t + 1]);
+                    acc[2 * t] = fmaf(kk[j], run[j], acc[2 * t]);
+                    acc[2 * t + 1] = fmaf(qq[j], run[j], acc[2 * t + 1]);
                 }
             }
         }
@@ -473,24 +498,21 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(DeltaScan p) {
 // x = hi + lo, as hi hi + hi lo + lo hi, which keeps 22 bits of each factor, with f32 accumulation; the state itself, the
 // factors and U stay f32.
 //
-// Four warps carry the state: warp = 16 columns x D / PARTS channels, as accumulators of the transposed state (rows = columns
+// Eight warps carry the state: warp = 16 columns x D / PARTS channels, as accumulators of the transposed state (rows = columns
 // of S). Those registers are at the same time the B operand of [K'; Q'] S when the eight channels of a step are taken in the
-// order 0 2 4 6 1 3 5 7, so the state never leaves them. Four more warps work one chunk ahead: they fetch q, k, g (two chunks
+// order 0 2 4 6 1 3 5 7, so the state never leaves them. Eight more warps work one chunk ahead: they fetch q, k, g (three chunks
 // ahead) and form the split K', Q', K''.
 template <int D, int CB>
 struct MmaScanShape {
-    static constexpr uint32_t GROUPS = CB / 16, PARTS = 4 / GROUPS, NCH = D / PARTS, NK = NCH / 8;
+    static constexpr uint32_t GROUPS = CB / 16, PARTS = 8 / GROUPS, NCH = D / PARTS, NK = NCH / 8;
     static constexpr uint32_t IN = 3 * CH * D, LDF = D + 8, LDU = CB + 8;
     static constexpr uint32_t FAC = 2 * 3 * CH * LDF + D;   // hi then lo of: K' (16 rows), Q' (16), K'' (16); the chunk's decay
-    static constexpr uint32_t VTB = CH * CB + 2 * CH * CH;  // v, T, B (three in flight)
-    static constexpr uint32_t FLOATS = 2 * IN + 2 * FAC + 3 * VTB + PARTS * 2 * CH * CB + 4 * CH * LDU;
+    static constexpr uint32_t VTB = CH * CB + 2 * CH * CH;  // v, T, B (four in flight)
+    static constexpr uint32_t FLOATS = 3 * IN + 2 * FAC + 4 * VTB + PARTS * 2 * CH * CB + 4 * CH * LDU;
 };
 
-__device__ __forceinline__ float tf32_hi(float x) {
-    uint32_t r;
-    asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(r) : "f"(x));
-    return __uint_as_float(r);
-}
+// the part of x a tf32 operand holds (x - tf32_hi(x) is exact; of that remainder the tensor core reads the leading bits)
+__device__ __forceinline__ float tf32_hi(float x) { return __uint_as_float(__float_as_uint(x) & 0xFFFFE000u); }
 __device__ __forceinline__ void mma_tf32(float c[4], const float a[4], float b0, float b1) {
     asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
@@ -499,27 +521,27 @@ __device__ __forceinline__ void mma_tf32(float c[4], const float a[4], float b0,
 }
 
 template <int D, int CB>
-__global__ void __launch_bounds__(256, 1) delta_scan_mma_kernel(DeltaScan p) {
+__global__ void __launch_bounds__(512, 1) delta_scan_mma_kernel(DeltaScan p) {
     using Sh = MmaScanShape<D, CB>;
-    constexpr uint32_t LDF = Sh::LDF, LDU = Sh::LDU, NK = Sh::NK, PARTS = Sh::PARTS, TPT = CH * CB / 128;
+    constexpr uint32_t LDF = Sh::LDF, LDU = Sh::LDU, NK = Sh::NK, PARTS = Sh::PARTS, TPT = CH * CB / 256;
     extern __shared__ __align__(16) float sm[];
-    float *in = sm, *fac = in + 2 * Sh::IN, *vtb = fac + 2 * Sh::FAC, *red = vtb + 3 * Sh::VTB, *X = red + PARTS * 2 * CH * CB, *U = X + CH * LDU, *Uh = U + CH * LDU, *Ul = Uh + CH * LDU;
+    float *in = sm, *fac = in + 3 * Sh::IN, *vtb = fac + 2 * Sh::FAC, *red = vtb + 4 * Sh::VTB, *X = red + PARTS * 2 * CH * CB, *U = X + CH * LDU, *Uh = U + CH * LDU, *Ul = Uh + CH * LDU;
     const DeltaShape s = p.s;
     const uint32_t h = blockIdx.x, kh = h / (s.heads / s.kv_heads), c0 = blockIdx.y * CB;
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    for (uint32_t i = tid; i < Sh::FLOATS; i += 256) sm[i] = 0.0f;  // padding: zero k and q leave padded rows of the state at zero
+    for (uint32_t i = tid; i < Sh::FLOATS; i += 512) sm[i] = 0.0f;  // padding: zero k and q leave padded rows of the state at zero
     __syncthreads();
     pdl_wait();
     pdl_launch();
-    store_ring(p, 256);
+    store_ring(p, 512);
     const uint32_t ncol = min((uint32_t)CB, s.vdim - c0), chunks = (p.tokens + CH - 1) / CH;
-    if (warp >= 4) {  // ---- one chunk ahead ----
-        const uint32_t pt = tid - 128, pw = pt >> 5;
+    if (warp >= 8) {  // ---- one chunk ahead ----
+        const uint32_t pt = tid - 256, pw = pt >> 5;
         const bool vec = (s.dim & 3) == 0;
         auto fetch = [&](uint32_t chunk) {
-            float *b = in + (chunk & 1) * Sh::IN, *bv = vtb + (chunk % 3) * Sh::VTB;
+            float *b = in + (chunk % 3) * Sh::IN, *bv = vtb + (chunk & 3) * Sh::VTB;
             const uint32_t t0 = chunk * CH, n = min(CH, p.tokens - t0);
-            for (uint32_t t = pw; t < n; t += 4) {
+            for (uint32_t t = pw; t < n; t += 8) {
                 const float *q = p.qn + (size_t)(t0 + t) * s.qk + kh * s.dim, *k = p.kn + (size_t)(t0 + t) * s.qk + kh * s.dim,
                             *g = p.g + ((size_t)(t0 + t) * s.heads + h) * s.dim;
                 if (vec) {
@@ -537,51 +559,58 @@ __global__ void __launch_bounds__(256, 1) delta_scan_mma_kernel(DeltaScan p) {
                 }
                 for (uint32_t e = lane; e < ncol; e += 32) cp4(bv + t * CB + e, p.vn + (size_t)(t0 + t) * s.vd + h * s.vdim + c0 + e);
             }
-            cp16(bv + CH * CB + 4 * pt, p.tb + ((size_t)chunk * s.heads + h) * 2 * CH * CH + 4 * pt);
+            if (pt < 128) cp16(bv + CH * CB + 4 * pt, p.tb + ((size_t)chunk * s.heads + h) * 2 * CH * CH + 4 * pt);
             asm volatile("cp.async.commit_group;" ::: "memory");
         };
         auto form = [&](uint32_t chunk) {  // tokens past the end: k = q = 0, no decay
-            const float *b = in + (chunk & 1) * Sh::IN;
+            const float *b = in + (chunk % 3) * Sh::IN;
             float *f = fac + (chunk & 1) * Sh::FAC;
             const uint32_t n = min(CH, p.tokens - chunk * CH);
             auto put = [&](uint32_t row, uint32_t e, float v) {
                 const float hi = tf32_hi(v);
                 f[row * LDF + e] = hi;
-                f[(3 * CH + row) * LDF + e] = tf32_hi(v - hi);
+                f[(3 * CH + row) * LDF + e] = v - hi;
             };
-            for (uint32_t e = pt; e < D; e += 128) {
-                float g[CH], k[CH], run = 1.0f;
+            const uint32_t e = pt & 127;  // 128 threads for K' and Q', 128 for K''
+            if (e >= D) return;
+            float g[CH], k[CH], run = 1.0f;
 #pragma unroll
-                for (uint32_t t = 0; t < CH; ++t) {
-                    g[t] = t < n ? b[(2 * CH + t) * D + e] : 1.0f;
-                    k[t] = t < n ? b[(CH + t) * D + e] : 0.0f;
-                }
+            for (uint32_t t = 0; t < CH; ++t) {
+                g[t] = t < n ? b[(2 * CH + t) * D + e] : 1.0f;
+                k[t] = t < n ? b[(CH + t) * D + e] : 0.0f;
+            }
+            if (pt < 128) {
 #pragma unroll
                 for (uint32_t t = 0; t < CH; ++t) {
                     run *= g[t];
                     put(t, e, k[t] * run);
                     put(CH + t, e, t < n ? b[t * D + e] * run : 0.0f);
                 }
-                f[2 * 3 * CH * LDF + e] = run;
-                run = 1.0f;
+            } else {
 #pragma unroll
                 for (int t = CH - 1; t >= 0; --t) {
                     put(2 * CH + t, e, k[t] * run);
                     run *= g[t];
                 }
+                f[2 * 3 * CH * LDF + e] = run;
             }
         };
+        auto fetch_or_none = [&](uint32_t chunk) {  // (a group per chunk, empty past the end: the waits below count groups)
+            if (chunk < chunks) fetch(chunk);
+            else asm volatile("cp.async.commit_group;" ::: "memory");
+        };
         fetch(0);
-        asm volatile("cp.async.wait_group 0;" ::: "memory");
-        asm volatile("bar.sync 1, 128;" ::: "memory");
-        if (chunks > 1) fetch(1);
+        fetch_or_none(1);
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        fetch_or_none(2);
         form(0);
         __syncthreads();
         for (uint32_t chunk = 0; chunk < chunks; ++chunk) {
             if (chunk + 1 < chunks) {
-                asm volatile("cp.async.wait_group 0;" ::: "memory");
-                asm volatile("bar.sync 1, 128;" ::: "memory");
-                if (chunk + 2 < chunks) fetch(chunk + 2);
+                asm volatile("cp.async.wait_group 1;" ::: "memory");  // chunk + 1 is here
+                asm volatile("bar.sync 1, 256;" ::: "memory");
+                fetch_or_none(chunk + 3);
                 form(chunk + 1);
             }
             __syncthreads();
@@ -602,7 +631,7 @@ __global__ void __launch_bounds__(256, 1) delta_scan_mma_kernel(DeltaScan p) {
     __syncthreads();
     for (uint32_t chunk = 0; chunk < chunks; ++chunk) {
         const float *fh = fac + (chunk & 1) * Sh::FAC, *fl = fh + 3 * CH * LDF, *cend = fh + 2 * 3 * CH * LDF;
-        const float *bv = vtb + (chunk % 3) * Sh::VTB, *bt = bv + CH * CB, *bb = bt + CH * CH;
+        const float *bv = vtb + (chunk & 3) * Sh::VTB, *bt = bv + CH * CB, *bb = bt + CH * CH;
         const uint32_t t0 = chunk * CH, n = min(CH, p.tokens - t0);
         float big[2][2][4] = {}, small[2][2][4] = {};  // [K', Q'][columns 0-7, 8-15]
 #pragma unroll
@@ -611,7 +640,7 @@ __global__ void __launch_bounds__(256, 1) delta_scan_mma_kernel(DeltaScan p) {
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 sh[i] = tf32_hi(S[kt][i]);
-                sl[i] = tf32_hi(S[kt][i] - sh[i]);
+                sl[i] = S[kt][i] - sh[i];
             }
 #pragma unroll
             for (uint32_t mt = 0; mt < 2; ++mt) {
@@ -635,7 +664,7 @@ __global__ void __launch_bounds__(256, 1) delta_scan_mma_kernel(DeltaScan p) {
                 for (int i = 0; i < 4; i += 2)
                     *reinterpret_cast<float2 *>(red + (part * 2 * CH + mt * CH + g + 4 * i) * CB + cg + 8 * nt + 2 * q) =
                         make_float2(big[mt][nt][i] + small[mt][nt][i], big[mt][nt][i + 1] + small[mt][nt][i + 1]);
-        asm volatile("bar.sync 2, 128;" ::: "memory");
+        asm volatile("bar.sync 2, 256;" ::: "memory");
         // thread: column uc, tokens ut .. ut + TPT - 1
         const uint32_t uc = tid % CB, ut = tid / CB * TPT;
         float o[TPT];
@@ -651,7 +680,7 @@ __global__ void __launch_bounds__(256, 1) delta_scan_mma_kernel(DeltaScan p) {
             }
             X[t * LDU + uc] = t < n ? x : 0.0f;
         }
-        asm volatile("bar.sync 2, 128;" ::: "memory");
+        asm volatile("bar.sync 2, 256;" ::: "memory");
         {
             float x[CH];
 #pragma unroll
@@ -666,11 +695,11 @@ __global__ void __launch_bounds__(256, 1) delta_scan_mma_kernel(DeltaScan p) {
                 }
                 const float hi = tf32_hi(u);
                 Uh[(ut + i) * LDU + uc] = hi;
-                Ul[(ut + i) * LDU + uc] = tf32_hi(u - hi);
+                Ul[(ut + i) * LDU + uc] = u - hi;
                 U[(ut + i) * LDU + uc] = u;
             }
         }
-        asm volatile("bar.sync 2, 128;" ::: "memory");
+        asm volatile("bar.sync 2, 256;" ::: "memory");
         {  // S <- diag(c) S + K''^T U, transposed: rows = columns of the state
             float uh[2][4], ul[2][4];
 #pragma unroll
@@ -1051,7 +1080,7 @@ class ChannelDelta : public Mixer {
         brasa_ctx *ctx = cmd->ctx;
         const size_t smem = (size_t)MmaScanShape<D, CB>::FLOATS * 4;
         BRASA_TRY(brasa_smem_optin(ctx, (const void *)delta_scan_mma_kernel<D, CB>, smem));
-        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_scan_mma_kernel<D, CB>, dim3(s_.heads, (s_.vdim + CB - 1) / CB), dim3(256), smem, p));
+        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_scan_mma_kernel<D, CB>, dim3(s_.heads, (s_.vdim + CB - 1) / CB), dim3(512), smem, p));
         return brasa_post_launch(cmd, "delta_scan_mma");
     }
     int32_t scan(brasa_cmd *cmd, const DeltaScan &p, bool f32) {

@@ -195,7 +195,7 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
     }
     // Q tile: rotated, rounded to bf16, swizzled K-major; rows past the last query and columns past the sizes are zeros
     const uint32_t half = a.rot_dims / 2;
-    const bool qvec = ((a.ldq | dq | a.dim) & 3) == 0;
+    const bool qvec = ((a.ldq | dq | a.dim) & 3) == 0, rvec = (half & 7) == 0;
     for (uint32_t i = tid; i < 128 * NQ * 8; i += 288) {
         const uint32_t r = i / (NQ * 8), c = i - r * (NQ * 8), blk = c >> 3, c8 = (c & 7) * 8;
         uint32_t w[4] = {0, 0, 0, 0};
@@ -208,6 +208,20 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
                 const float4 x = *reinterpret_cast<const float4 *>(q + blk * 64 + c8), y = *reinterpret_cast<const float4 *>(q + blk * 64 + c8 + 4);
                 v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
                 v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
+            } else if (qvec && rvec && blk >= NU && (blk - NU) * 64 + c8 + 8 <= a.rot_dims) {
+                // eight neighbours of one half of the pairs
+                const uint32_t e0 = (blk - NU) * 64 + c8, f0 = e0 < half ? e0 : e0 - half;
+                const float *own = q + a.dim + e0, *other = e0 < half ? own + half : own - half;
+                const float sign = e0 < half ? -1.0f : 1.0f;
+#pragma unroll
+                for (int u = 0; u < 8; u += 4) {
+                    const float4 x = *reinterpret_cast<const float4 *>(own + u), y = *reinterpret_cast<const float4 *>(other + u);
+                    const float4 cc = *reinterpret_cast<const float4 *>(ct + f0 + u), ss = *reinterpret_cast<const float4 *>(st + f0 + u);
+                    v[u] = fmaf(sign * y.x, ss.x, x.x * cc.x);
+                    v[u + 1] = fmaf(sign * y.y, ss.y, x.y * cc.y);
+                    v[u + 2] = fmaf(sign * y.z, ss.z, x.z * cc.z);
+                    v[u + 3] = fmaf(sign * y.w, ss.w, x.w * cc.w);
+                }
             } else
 #pragma unroll
             for (int e = 0; e < 8; ++e) {
