@@ -56,12 +56,31 @@ __device__ __forceinline__ void store_row(const LatentShape &s, const float *d, 
         elem_store(r + (size_t)slot * s.ldr + i, rot_elem(d + s.kr, i, s.rot_dims, cos_t + (size_t)pos * half, sin_t + (size_t)pos * half));
 }
 
+// Many tokens: one warp per token, its latent in registers (up to 1024 wide).
 template <typename T>
-__global__ void __launch_bounds__(256) latent_store_kernel(LatentShape s, const float *down, uint32_t ldd, uint32_t pos0, const float *w, const float *cos_t,
+__global__ void __launch_bounds__(256) latent_store_kernel(LatentShape s, const float *down, uint32_t ldd, uint32_t tokens, uint32_t pos0, const float *w, const float *cos_t,
                                                            const float *sin_t, T *c, T *r) {
     pdl_wait();
     pdl_launch();
-    store_row<T>(s, down + (size_t)blockIdx.x * ldd, pos0 + blockIdx.x, w, cos_t, sin_t, c, r);
+    const uint32_t t = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (t >= tokens) return;
+    const float *d = down + (size_t)t * ldd;
+    const uint32_t pos = pos0 + t, slot = pos % s.rows, half = s.rot_dims / 2;
+    float v[32], ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < 32; ++j) {
+        const uint32_t i = lane + 32 * j;
+        v[j] = i < s.kr ? d[i] : 0.0f;
+        ss = fmaf(v[j], v[j], ss);
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)s.kr + s.eps);
+#pragma unroll
+    for (int j = 0; j < 32; ++j) {
+        const uint32_t i = lane + 32 * j;
+        if (i < s.kr) elem_store(c + (size_t)slot * s.ldc + i, v[j] * inv * w[i]);
+    }
+    for (uint32_t i = lane; i < s.rot; i += 32)
+        elem_store(r + (size_t)slot * s.ldr + i, rot_elem(d + s.kr, i, s.rot_dims, cos_t + (size_t)pos * half, sin_t + (size_t)pos * half));
 }
 
 // the shared key part of positions key0 .. out of the ring, in order
@@ -418,7 +437,7 @@ class LatentAttention : public Mixer {
         brasa_ctx *ctx = r.cmd->ctx;
         auto f = [&](uint64_t at) { return (float *)(r.scratch + at); };
         T *c = (T *)c_, *kr = (T *)r_, *krow = (T *)(r.scratch + at_.kr);
-        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, latent_store_kernel<T>, dim3(r.tokens), dim3(256), 0, s_, f(at_.down), ldd_, r.pos0, norm_, cos_, sin_, c, kr));
+        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, latent_store_kernel<T>, dim3((r.tokens + 7) / 8), dim3(256), 0, s_, f(at_.down), ldd_, r.tokens, r.pos0, norm_, cos_, sin_, c, kr));
         BRASA_TRY(brasa_post_launch(r.cmd, "latent_store"));
         // every position some query of the run sees, in order; the ring holds them in at most two pieces
         const uint32_t key0 = r.pos0 + 1 > s_.window ? r.pos0 + 1 - s_.window : 0u, keys = r.pos0 + r.tokens - key0;
