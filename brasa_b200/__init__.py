@@ -99,12 +99,14 @@ class _PagedKv(C.Structure):
 class _Linear(C.Structure):
     _fields_ = ([(n, _Arg) for n in ("w", "x", "w2", "x2", "y", "bias", "resid")] +
                 [(n, C.c_uint32) for n in ("cols", "ldw", "ldx", "cols2", "ldw2", "ldx2", "rows", "tokens", "ldy")] +
-                [("y_bf16", C.c_int32), ("act", C.c_int32), ("scale", C.c_float)])
+                [("y_bf16", C.c_int32), ("act", C.c_int32), ("scale", C.c_float), ("cap", C.c_float), ("mul", _Arg), ("mul_ids", _Arg), ("ldm", C.c_uint32),
+                 ("mul_rows", C.c_uint32)])
 
 
 class _WindowAttn(C.Structure):
     _fields_ = ([(n, _Arg) for n in ("q", "k", "v", "kr", "cos_t", "sin_t", "gate", "out")] +
-                [(n, C.c_uint32) for n in ("tokens", "heads", "dim", "rot", "rot_dims", "vdim", "pos0", "key0", "window")] + [("scale", C.c_float)])
+                [(n, C.c_uint32) for n in ("tokens", "heads", "dim", "rot", "rot_dims", "vdim", "pos0", "key0", "window")] +
+                [("scale", C.c_float), ("kv_heads", C.c_uint32), ("ring", C.c_uint32), ("softcap", C.c_float), ("out_scale", C.c_float)])
 
 
 class _ModelShape(C.Structure):
@@ -581,20 +583,29 @@ class Kernels:
     def layer_norm(self, cmd, x, w, b, out, rows, n, eps):
         self._k(self.L.brasa_k_layer_norm(cmd._h, _arg(x), _arg(w), _arg(b), _arg(out), C.c_uint32(rows), C.c_uint32(n), C.c_float(eps)))
 
+    def add_rms_norm(self, cmd, x, y, wy, x_out, w, out, rows, n, eps):
+        """x' = x + y / rms(y) * wy, x_out = x', out = x' / rms(x') * w; y (with wy), x_out, w and out may be None."""
+        self._k(self.L.brasa_k_add_rms_norm(cmd._h, _arg(x), _arg(y), _arg(wy), _arg(x_out), _arg(w), _arg(out), C.c_uint32(rows), C.c_uint32(n), C.c_float(eps)))
+
+    ACT_NONE, ACT_RELU2, ACT_GELU_TANH, ACT_SWIGLU = range(4)
+
     @staticmethod
     def linear_problem(w, x, y, rows: int, cols: int, tokens: int, ldw=None, ldx=None, ldy=None, w2=None, x2=None, cols2=0, ldw2=0, ldx2=0, bias=None,
-                       resid=None, y_bf16=False, relu2=False, scale=1.0) -> _Linear:
+                       resid=None, y_bf16=False, relu2=False, scale=1.0, act=None, cap=0.0, mul=None, mul_ids=None, ldm=0, mul_rows=0) -> _Linear:
+        """act: one of ACT_NONE, ACT_RELU2, ACT_GELU_TANH, ACT_SWIGLU (relu2 is short for ACT_RELU2)."""
         return _Linear(_arg(w), _arg(x), _arg(w2), _arg(x2), _arg(y), _arg(bias), _arg(resid), cols, ldw or cols, ldx or cols, cols2, ldw2 or cols2,
-                       ldx2 or cols2, rows, tokens, ldy or rows, int(y_bf16), int(relu2), scale)
+                       ldx2 or cols2, rows, tokens, ldy or rows, int(y_bf16), int(relu2) if act is None else act, scale, cap, _arg(mul), _arg(mul_ids), ldm, mul_rows)
 
     def linear(self, cmd, problems, f32_inputs: bool):
         """Up to eight products with bf16 weights in one launch (linear_problem)."""
         arr = (_Linear * len(problems))(*problems)
         self._k(self.L.brasa_k_linear(cmd._h, arr, C.c_uint32(len(problems)), C.c_int32(int(f32_inputs))))
 
-    def window_attention(self, cmd, q, k, v, kr, table: RopeTable, gate, out, tokens, heads, dim, rot, vdim, pos0, key0, window, scale, f32: bool):
+    def window_attention(self, cmd, q, k, v, kr, table: RopeTable, gate, out, tokens, heads, dim, rot, vdim, pos0, key0, window, scale, f32: bool, kv_heads=0, ring=0,
+                         softcap=0.0, out_scale=1.0):
+        """kv_heads 0: as many as heads; kr and gate may be None (rot 0)."""
         a = _WindowAttn(_arg(q), _arg(k), _arg(v), _arg(kr), _arg(table.cos), _arg(table.sin), _arg(gate), _arg(out), tokens, heads, dim, rot, table.dim, vdim,
-                        pos0, key0, window, scale)
+                        pos0, key0, window, scale, kv_heads or heads, ring, softcap, out_scale)
         self._k(self.L.brasa_k_window_attention(cmd._h, a, C.c_int32(int(f32))))
 
     def argmax(self, cmd, logits, n, out):
@@ -818,11 +829,14 @@ class Model:
             at += n
         return np.concatenate(out) if out else np.empty((0, self.cfg["head_rows"]), np.float32)
 
-    def run_layers(self, x, pos0: int, layers: range) -> np.ndarray:
+    def run_layers(self, x, pos0: int, layers: range, ids=None) -> np.ndarray:
+        """ids: of the tokens, for models whose layers read them too."""
         x = np.ascontiguousarray(x, dtype=np.float32).copy()
         tokens = x.size // self.cfg["hidden"]
-        self.ctx._check(lib().brasa_model_run_layers(self._h, x.ctypes.data_as(C.c_void_p), C.c_uint32(tokens), C.c_uint32(pos0),
-                                                     C.c_uint32(layers.start), C.c_uint32(layers.stop)))
+        ids = None if ids is None else np.ascontiguousarray(ids, dtype=np.uint32)
+        assert ids is None or ids.size == tokens
+        self.ctx._check(lib().brasa_model_run_layers_ids(self._h, None if ids is None else ids.ctypes.data_as(C.c_void_p), x.ctypes.data_as(C.c_void_p),
+                                                         C.c_uint32(tokens), C.c_uint32(pos0), C.c_uint32(layers.start), C.c_uint32(layers.stop)))
         return x
 
     def decode_greedy(self, first: int, pos0: int, steps: int):
@@ -870,16 +884,25 @@ class Qwen3(Model):
         return out
 
 
-class Dunuzen(Model):
-    """Layers of latent attention in a sliding window and of the gated delta rule, each beside a feed-forward, over bf16
-    safetensors. Its state goes forward only: a run starts at position 0 or where the one before it ended."""
+class LayerStack(Model):
+    """Layers listed one by one in the configuration, over bf16 safetensors. The state goes forward only: a run starts at
+    position 0 or where the one before it ended."""
 
     @classmethod
     def kv_type(cls, dtype):
         return {"float32": KvType.F32, "bfloat16": KvType.BF16}[dtype]
 
 
-MODELS = {"qwen3": Qwen3, "Dunuzen": Dunuzen}
+class Dunuzen(LayerStack):
+    """Layers of latent attention in a sliding window and of the gated delta rule, each beside a feed-forward."""
+
+
+class Gugedra(LayerStack):
+    """Layers of the gated delta rule, and of windowed attention and a state-space mixer side by side, with norms around every
+    sublayer and a gated input per token and layer."""
+
+
+MODELS = {"qwen3": Qwen3, "Dunuzen": Dunuzen, "Gugedra": Gugedra}
 
 
 def model_class(path) -> type[Model]:

@@ -160,6 +160,10 @@ int32_t brasa_post_launch(brasa_cmd *cmd, const char *name);
 // ops.cu. out[i] = layer norm of row x[rows ? rows[r] : r] times w[i] plus b[i], i < n_out (1 or 2), [n_rows][ldo] in f32 or bf16
 int32_t brasa_layer_norm_launch(brasa_cmd *cmd, const float *x, const uint32_t *rows, uint32_t n_rows, uint32_t n, float eps, const float *const *w,
                                 const float *const *b, void *const *out, uint32_t n_out, uint32_t ldo, bool f32);
+// x' = x + y / rms(y) * wy (y null: x), x_out = x' (null: not stored; may be x), out = x' / rms(x') * w in f32 or bf16 (w null: x'
+// itself; out null: none), of row rows[r] or r
+int32_t brasa_add_rms_norm_launch(brasa_cmd *cmd, const float *x, const float *y, const float *wy, float *x_out, const float *w, void *out, const uint32_t *rows,
+                                  uint32_t n_rows, uint32_t n, uint32_t ldo, float eps, bool f32);
 // out[t, :] = scale * table[ids[t], :] for a bf16 table
 int32_t brasa_embed_bf16_launch(brasa_cmd *cmd, const uint16_t *table, uint32_t ld, uint32_t rows, uint32_t n, float scale, const uint32_t *ids, float *out,
                                 uint32_t tokens);

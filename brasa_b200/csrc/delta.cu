@@ -1,8 +1,10 @@
-// Gated delta rule with one decay per key channel ("channel_delta"), a recurrent mixer. A head keeps a matrix S [dim][vdim] of
-// what each key direction stands for. A token fades the rows of S by its decays g, reads what its key k finds there, moves that
-// towards its value v by the fraction beta, and its query q reads the result:
+// Gated delta rule, a recurrent mixer. A head keeps a matrix S [dim][vdim] of what each key direction stands for. A token fades
+// the rows of S by its decays g, reads what its key k finds there, moves that towards its value v by the fraction beta, and its
+// query q reads the result:
 //   F = diag(g) S_old,  u = beta (v - F^T k),  S_new = F + k u^T,  o = S_new^T q
 // q, k and v come out of a short causal convolution and silu, q and k as unit vectors, g out of a softplus.
+// Two forms: "channel_delta" has one decay per key channel and a sigmoid output gate, both out of low-rank projections; "delta"
+// has one decay per head (HD below) and a silu output gate, both out of plain projections.
 //
 // Many tokens: chunks of 16, everything that does not depend on the state for all chunks side by side, then the state through
 // the chunks (below). One token: delta_step_kernel does all of it, one block per head. Everything is f32 FMA.
@@ -12,6 +14,7 @@
 // starts at position 0 by ignoring both.
 #include <cuda_bf16.h>
 
+#include "conv_device.cuh"
 #include "stack.h"
 #include "tc_device.cuh"
 
@@ -21,39 +24,11 @@ namespace {
 
 constexpr float UNIT_EPS = 1e-6f;
 
-__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
-__device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
-__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
-__device__ __forceinline__ float warp_sum(float v) {
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    return v;
-}
-
 struct DeltaShape {
     uint32_t heads, kv_heads, dim, vdim, taps;
     uint32_t qk;  // kv_heads * dim
     uint32_t vd;  // heads * vdim
 };
-
-// The convolution of one channel at token t: x f32 [tokens][ldx] holds this run's inputs, the ring the ones before it.
-// ch: the channel in the ring (q channels, then k's, then v's).
-struct ConvView {
-    const float *ring;
-    uint32_t channels, taps, pos0;
-};
-__device__ __forceinline__ float conv_at(const float *x, uint32_t ldx, uint32_t c, const float *w, uint32_t t, const ConvView &cv, uint32_t ch) {
-    float s = 0.0f;
-    for (uint32_t i = 0; i < cv.taps; ++i) {
-        const uint32_t back = cv.taps - 1 - i;  // tokens before this one
-        float v;
-        if (back <= t) v = x[(size_t)(t - back) * ldx + c];
-        else if (back <= cv.pos0 + t) v = cv.ring[(size_t)((cv.pos0 + t - back) % cv.taps) * cv.channels + ch];
-        else v = 0.0f;
-        s = fmaf(v, w[(size_t)c * cv.taps + i], s);
-    }
-    return s;
-}
 
 // ---- many tokens -------------------------------------------------------------------------------------------------------
 // Tokens go in chunks of CH. Inside a chunk write c_t for the product of the decays up to token t and let
@@ -73,40 +48,8 @@ struct DeltaChunk {
     const float *q, *k, *v, *b, *z;  // products [tokens][ld]
     uint32_t ldqk, ldv, ldb, ldz, tokens;
     const float *wq, *wk, *wv, *a_log;
-    float *qn, *kn, *vn, *g, *tb;    // [tokens][qk], [qk], [vd], [heads * dim]; [chunks][heads][T, B][CH][CH]
+    float *qn, *kn, *vn, *g, *tb;    // [tokens][qk], [qk], [vd], [heads * dim] (HD: [heads]); [chunks][heads][T, B][CH][CH]
 };
-
-// convolution and silu of one channel for the chunk's tokens, handed to put(t, value)
-template <typename Put>
-__device__ __forceinline__ void conv_chunk(const float *x, uint32_t ldx, uint32_t c, const float *w, uint32_t t0, uint32_t n, const ConvView &cv, uint32_t ch, Put put) {
-    if (cv.taps <= 4) {  // the window in registers
-        float wr[4], xr[4];
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const int tap = (int)cv.taps - 4 + i, back = 4 - i;  // xr[i]: `back` tokens before t0
-            wr[i] = tap >= 0 ? w[(size_t)c * cv.taps + tap] : 0.0f;
-            xr[i] = 0.0f;
-            if (i > 0 && tap > 0) {  // xr[1 .. 3] hold the three tokens ahead of the first one, where the window reaches them
-                const uint32_t bk = back;
-                if (bk <= t0) xr[i] = x[(size_t)(t0 - bk) * ldx + c];
-                else if (bk <= cv.pos0 + t0) xr[i] = cv.ring[(size_t)((cv.pos0 + t0 - bk) % cv.taps) * cv.channels + ch];
-            }
-        }
-        float in[CH];
-#pragma unroll
-        for (uint32_t t = 0; t < CH; ++t) in[t] = t < n ? x[(size_t)(t0 + t) * ldx + c] : 0.0f;
-#pragma unroll
-        for (uint32_t t = 0; t < CH; ++t) {
-            xr[0] = xr[1];
-            xr[1] = xr[2];
-            xr[2] = xr[3];
-            xr[3] = in[t];
-            if (t < n) put(t, silu_f(fmaf(xr[3], wr[3], fmaf(xr[2], wr[2], fmaf(xr[1], wr[1], xr[0] * wr[0])))));
-        }
-    } else {
-        for (uint32_t t = 0; t < n; ++t) put(t, silu_f(conv_at(x, ldx, c, w, t0 + t, cv, ch)));
-    }
-}
 
 // E consecutive floats of shared memory
 template <int E>
@@ -128,13 +71,13 @@ __device__ __forceinline__ void load_run(const float *p, float v[E]) {
 }
 
 // Block: one chunk of one head. E consecutive key channels per lane: dim up to 32 E.
-template <int E>
+template <int E, bool HD>
 __global__ void __launch_bounds__(256) delta_chunk_kernel(DeltaChunk p) {
     constexpr uint32_t D = 32 * E;
     extern __shared__ __align__(16) float sm[];
     const DeltaShape s = p.s;
     float *sq = sm, *sk = sq + CH * D, *sg = sk + CH * D;
-    __shared__ float B[CH][CH], beta[CH];
+    __shared__ float B[CH][CH], beta[CH], gh[CH];
     __shared__ __align__(16) float A[CH][CH];
     const uint32_t chunk = blockIdx.x, t0 = chunk * CH, n = min(CH, p.tokens - t0), h = blockIdx.y, group = s.heads / s.kv_heads, kh = h / group;
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -146,13 +89,19 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(DeltaChunk p) {
         float *dst = (isk ? sk : sq) + e;
         uint32_t t = 0;
         if (e < s.dim) {
-            conv_chunk(isk ? p.k : p.q, p.ldqk, c, isk ? p.wk : p.wq, t0, n, p.cv, (isk ? s.qk : 0u) + c, [&](uint32_t tt, float v) { dst[tt * D] = v; });
+            conv_chunk(isk ? p.k : p.q, p.ldqk, c, isk ? p.wk : p.wq, 0.0f, t0, n, p.cv, (isk ? s.qk : 0u) + c, [&](uint32_t tt, float v) { dst[tt * D] = v; });
             t = n;
         }
         for (; t < CH; ++t) dst[t * D] = 0.0f;
     }
     {
         const float a = expf(p.a_log[h]);
+        if (HD) {
+            if (tid < CH) {
+                gh[tid] = tid < n ? expf(-a * softplus_f(p.z[(size_t)(t0 + tid) * p.ldz + h])) : 1.0f;
+                if (tid < n) p.g[(size_t)(t0 + tid) * s.heads + h] = gh[tid];
+            }
+        } else
         for (uint32_t t = warp; t < CH; t += 8)
 #pragma unroll
             for (int j = 0; j < E; ++j) {
@@ -198,7 +147,11 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(DeltaChunk p) {
                 float kk[E], qq[E];
                 load_run<E>(sk + t * D + lane * E, kk);
                 load_run<E>(sq + t * D + lane * E, qq);
-                if (t > col) {
+                if (HD) {
+                    if (t > col)
+#pragma unroll
+                        for (int j = 0; j < E; ++j) run[j] *= gh[t];
+                } else if (t > col) {
                     float gg[E];
                     load_run<E>(sg + t * D + lane * E, gg);
 #pragma unroll
@@ -243,7 +196,7 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(DeltaChunk p) {
         for (uint32_t i = tid - 32; i < CH * CH; i += 224) tb[CH * CH + i] = B[i >> 4][i & 15];
         for (uint32_t i = tid - 32; i < s.vdim; i += 224) {
             const uint32_t c = h * s.vdim + i;
-            conv_chunk(p.v, p.ldv, c, p.wv, t0, n, p.cv, 2 * s.qk + c, [&](uint32_t t, float v) { p.vn[(size_t)(t0 + t) * s.vd + c] = v; });
+            conv_chunk(p.v, p.ldv, c, p.wv, 0.0f, t0, n, p.cv, 2 * s.qk + c, [&](uint32_t t, float v) { p.vn[(size_t)(t0 + t) * s.vd + c] = v; });
         }
     }
 }
@@ -258,13 +211,6 @@ struct DeltaScan {
     float *o;      // [tokens][vd]
     uint32_t tokens, pos0;
 };
-
-__device__ __forceinline__ void cp4(float *dst, const float *src) {
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp16(float *dst, const float *src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
 
 // The run's last inputs of the convolution into the ring (the kernel that read the older ones has finished).
 __device__ __forceinline__ void store_ring(const DeltaScan &p, uint32_t threads) {
@@ -286,7 +232,7 @@ struct ScanShape {
     static constexpr uint32_t FLOATS = 2 * IN + D * LDA + CH * D + D + D * CB + 8 * 2 * CH * CB + 2 * CH * CB;
 };
 
-template <int D, int CB>
+template <int D, int CB, bool HD>
 __global__ void __launch_bounds__(256, 1) delta_scan_kernel(DeltaScan p) {
     using Sh = ScanShape<D, CB>;
     constexpr uint32_t LDA = Sh::LDA, KW = D / 8, CPL = CB / 4, TILES = D / 4 * (CB / 4), TPT = (TILES + 255) / 256;
@@ -324,16 +270,17 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(DeltaScan p) {
                 for (uint32_t e = lane * 4; e < s.dim; e += 128) {
                     cp16(b + t * D + e, p.qn + (size_t)(t0 + t) * s.qk + kh * s.dim + e);
                     cp16(b + (CH + t) * D + e, p.kn + (size_t)(t0 + t) * s.qk + kh * s.dim + e);
-                    cp16(b + (2 * CH + t) * D + e, p.g + ((size_t)(t0 + t) * s.heads + h) * s.dim + e);
+                    if (!HD) cp16(b + (2 * CH + t) * D + e, p.g + ((size_t)(t0 + t) * s.heads + h) * s.dim + e);
                 }
         } else {
             for (uint32_t t = warp; t < n; t += 8)
                 for (uint32_t e = lane; e < s.dim; e += 32) {
                     cp4(b + t * D + e, p.qn + (size_t)(t0 + t) * s.qk + kh * s.dim + e);
                     cp4(b + (CH + t) * D + e, p.kn + (size_t)(t0 + t) * s.qk + kh * s.dim + e);
-                    cp4(b + (2 * CH + t) * D + e, p.g + ((size_t)(t0 + t) * s.heads + h) * s.dim + e);
+                    if (!HD) cp4(b + (2 * CH + t) * D + e, p.g + ((size_t)(t0 + t) * s.heads + h) * s.dim + e);
                 }
         }
+        if (HD && tid < n) cp4(b + 2 * CH * D + tid, p.g + (size_t)(t0 + tid) * s.heads + h);
         float *bv = b + 3 * CH * D;
         for (uint32_t t = warp; t < n; t += 8)
             for (uint32_t e = lane; e < ncol; e += 32) cp4(bv + t * CB + e, p.vn + (size_t)(t0 + t) * s.vd + h * s.vdim + c0 + e);
@@ -360,7 +307,7 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(DeltaScan p) {
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
                         const uint32_t t = t4 + i;
-                        if (t < n) run *= b[(2 * CH + t) * D + e];
+                        if (t < n) run *= b[HD ? 2 * CH * D + t : (2 * CH + t) * D + e];
                         qq[i] = t < n ? b[t * D + e] * run : 0.0f;
                         kk[i] = t < n ? b[(CH + t) * D + e] * run : 0.0f;
                     }
@@ -373,7 +320,7 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(DeltaScan p) {
                 for (int t = CH - 1; t >= 0; --t) {
                     const bool live = (uint32_t)t < n;
                     kend[t * D + e] = live ? b[(CH + t) * D + e] * run : 0.0f;
-                    if (live) run *= b[(2 * CH + t) * D + e];
+                    if (live) run *= b[HD ? 2 * CH * D + t : (2 * CH + t) * D + e];
                 }
                 cend[e] = run;
             }
@@ -520,7 +467,7 @@ __device__ __forceinline__ void mma_tf32(float c[4], const float a[4], float b0,
                    "r"(__float_as_uint(b1)));
 }
 
-template <int D, int CB>
+template <int D, int CB, bool HD>
 __global__ void __launch_bounds__(512, 1) delta_scan_mma_kernel(DeltaScan p) {
     using Sh = MmaScanShape<D, CB>;
     constexpr uint32_t LDF = Sh::LDF, LDU = Sh::LDU, NK = Sh::NK, PARTS = Sh::PARTS, TPT = CH * CB / 256;
@@ -543,18 +490,19 @@ __global__ void __launch_bounds__(512, 1) delta_scan_mma_kernel(DeltaScan p) {
             const uint32_t t0 = chunk * CH, n = min(CH, p.tokens - t0);
             for (uint32_t t = pw; t < n; t += 8) {
                 const float *q = p.qn + (size_t)(t0 + t) * s.qk + kh * s.dim, *k = p.kn + (size_t)(t0 + t) * s.qk + kh * s.dim,
-                            *g = p.g + ((size_t)(t0 + t) * s.heads + h) * s.dim;
+                            *g = p.g + ((size_t)(t0 + t) * s.heads + h) * (HD ? 1 : s.dim);
+                if (HD && lane == 0) cp4(b + 2 * CH * D + t, g);
                 if (vec) {
                     for (uint32_t e = lane * 4; e < s.dim; e += 128) {
                         cp16(b + t * D + e, q + e);
                         cp16(b + (CH + t) * D + e, k + e);
-                        cp16(b + (2 * CH + t) * D + e, g + e);
+                        if (!HD) cp16(b + (2 * CH + t) * D + e, g + e);
                     }
                 } else {
                     for (uint32_t e = lane; e < s.dim; e += 32) {
                         cp4(b + t * D + e, q + e);
                         cp4(b + (CH + t) * D + e, k + e);
-                        cp4(b + (2 * CH + t) * D + e, g + e);
+                        if (!HD) cp4(b + (2 * CH + t) * D + e, g + e);
                     }
                 }
                 for (uint32_t e = lane; e < ncol; e += 32) cp4(bv + t * CB + e, p.vn + (size_t)(t0 + t) * s.vd + h * s.vdim + c0 + e);
@@ -576,7 +524,7 @@ __global__ void __launch_bounds__(512, 1) delta_scan_mma_kernel(DeltaScan p) {
             float g[CH], k[CH], run = 1.0f;
 #pragma unroll
             for (uint32_t t = 0; t < CH; ++t) {
-                g[t] = t < n ? b[(2 * CH + t) * D + e] : 1.0f;
+                g[t] = t < n ? b[HD ? 2 * CH * D + t : (2 * CH + t) * D + e] : 1.0f;
                 k[t] = t < n ? b[(CH + t) * D + e] : 0.0f;
             }
             if (pt < 128) {
@@ -753,8 +701,8 @@ __global__ void __launch_bounds__(512, 1) delta_scan_mma_kernel(DeltaScan p) {
         }
 }
 
-// o / rms(o) * w * sigmoid(gate), per head; one warp per (token, head)
-template <typename T>
+// o / rms(o) * w * sigmoid(gate) (SILU: silu(gate)), per head; one warp per (token, head)
+template <typename T, bool SILU>
 __global__ void __launch_bounds__(256) delta_out_kernel(const float *o, const float *gate, uint32_t ldg, const float *w, T *out, uint32_t ldo, uint32_t heads,
                                                         uint32_t vdim, uint32_t tokens, float eps) {
     pdl_wait();
@@ -767,7 +715,10 @@ __global__ void __launch_bounds__(256) delta_out_kernel(const float *o, const fl
     for (uint32_t e = lane; e < vdim; e += 32) ss = fmaf(x[e], x[e], ss);
     const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + eps);
     for (uint32_t e = lane; e < vdim; e += 32)
-        elem_store(out + (size_t)t * ldo + h * vdim + e, x[e] * inv * w[e] * sigmoid_f(gate[(size_t)t * ldg + h * vdim + e]));
+    {
+        const float z = gate[(size_t)t * ldg + h * vdim + e];
+        elem_store(out + (size_t)t * ldo + h * vdim + e, x[e] * inv * w[e] * (SILU ? silu_f(z) : sigmoid_f(z)));
+    }
 }
 
 // ---- one token ---------------------------------------------------------------------------------------------------------
@@ -775,7 +726,7 @@ struct DeltaStep {
     DeltaShape s;
     const float *q, *k, *v, *b, *a1, *g1;        // products of this token
     const float *wq, *wk, *wv, *a_log, *dt_bias, *norm;
-    const uint16_t *wa2, *wg2;
+    const uint16_t *wa2, *wg2;  // null: a1 is the decay's projection with its bias, one per head, and g1 the silu gate's, one per value
     uint32_t ra, rg, lda2, ldg2;
     float *ring, *state, *out;
     const uint32_t *pos;
@@ -808,7 +759,7 @@ __global__ void __launch_bounds__(STEP_THREADS, 1) delta_step_kernel(DeltaStep p
     float *S = p.state + (size_t)h * s.dim * s.vdim;
     // Row i of the head's low-rank factors: the decay's rows, then the gate's. Warp w takes rows w, w + 16, .. in batches of
     // eight; the first batch's weights and the state's cache lines are asked for ahead of the kernel before this one.
-    const uint32_t nrows = s.dim + s.vdim;
+    const uint32_t nrows = p.wa2 ? s.dim + s.vdim : 0u;
     uint4 fw[8];
     auto factor_load = [&](uint32_t r0, uint32_t c) {
 #pragma unroll
@@ -842,6 +793,10 @@ __global__ void __launch_bounds__(STEP_THREADS, 1) delta_step_kernel(DeltaStep p
         p.ring[(size_t)(pos % s.taps) * cv.channels + ch] = x;
     }
     const float decay = expf(p.a_log[h]);
+    if (!p.wa2) {
+        for (uint32_t i = tid; i < s.dim; i += STEP_THREADS) sg[i] = expf(-decay * softplus_f(p.a1[h]));
+        for (uint32_t i = tid; i < s.vdim; i += STEP_THREADS) gate[i] = silu_f(p.g1[h * s.vdim + i]);
+    }
     for (uint32_t r0 = warp; r0 < nrows; r0 += 128) {
         float z[8] = {};
         for (uint32_t c = lane * 8; c < max(ra8, rg8); c += 256) {
@@ -955,19 +910,20 @@ size_t step_smem(const DeltaShape &s, uint32_t ra, uint32_t rg) {
 namespace brasa_stack {
 namespace {
 
-class ChannelDelta : public Mixer {
+class DeltaRule : public Mixer {
   public:
+    explicit DeltaRule(bool per_head) : hd_(per_head), name_(per_head ? "delta" : "channel_delta") {}
+
     bool configure(const brasa::Json &c, uint32_t width, float eps, std::string &err) override {
         if (!read_u32(c, "heads", &s_.heads, err) || !read_u32(c, "kv_heads", &s_.kv_heads, err) || !read_u32(c, "dim", &s_.dim, err) ||
             !read_u32(c, "vdim", &s_.vdim, err) || !read_u32(c, "conv", &s_.taps, err))
             return false;
-        if (s_.heads % s_.kv_heads != 0) return err = "channel_delta: heads must be a multiple of kv_heads", false;
-        if (s_.dim > 256 || s_.vdim > 1024) return err = "channel_delta: dim up to 256 and vdim up to 1024", false;
+        if (s_.heads % s_.kv_heads != 0) return err = name_ + ": heads must be a multiple of kv_heads", false;
+        if (s_.dim > 256 || s_.vdim > 1024) return err = name_ + ": dim up to 256 and vdim up to 1024", false;
         s_.qk = s_.kv_heads * s_.dim;
         s_.vd = s_.heads * s_.vdim;
         width_ = width;
         eps_ = eps;
-        out_width = s_.vd;
         return true;
     }
 
@@ -976,16 +932,22 @@ class ChannelDelta : public Mixer {
         BRASA_TRY(b.matrix(x + "k", s_.qk, width_, &k_));
         BRASA_TRY(b.matrix(x + "v", s_.vd, width_, &v_));
         BRASA_TRY(b.matrix(x + "b", s_.heads, width_, &b_));
-        BRASA_TRY(b.matrix(x + "a1", 0, width_, &a1_));
-        BRASA_TRY(b.matrix(x + "a2", s_.heads * s_.dim, a1_.rows, &a2_));
-        BRASA_TRY(b.matrix(x + "g1", 0, width_, &g1_));
-        BRASA_TRY(b.matrix(x + "g2", s_.vd, g1_.rows, &g2_));
-        BRASA_TRY(b.matrix(x + "o", width_, s_.vd, &wo));
+        if (hd_) {
+            BRASA_TRY(b.matrix(x + "a", s_.heads, width_, &a1_));
+            BRASA_TRY(b.matrix(x + "g", s_.vd, width_, &g1_));
+        } else {
+            BRASA_TRY(b.matrix(x + "a1", 0, width_, &a1_));
+            BRASA_TRY(b.matrix(x + "a2", s_.heads * s_.dim, a1_.rows, &a2_));
+            BRASA_TRY(b.matrix(x + "g1", 0, width_, &g1_));
+            BRASA_TRY(b.matrix(x + "g2", s_.vd, g1_.rows, &g2_));
+        }
+        outs.resize(1);
+        BRASA_TRY(b.matrix(x + "o", width_, s_.vd, &outs[0]));
         BRASA_TRY(b.vector(x + "q.conv", (uint64_t)s_.qk * s_.taps, &wq_));
         BRASA_TRY(b.vector(x + "k.conv", (uint64_t)s_.qk * s_.taps, &wk_));
         BRASA_TRY(b.vector(x + "v.conv", (uint64_t)s_.vd * s_.taps, &wv_));
         BRASA_TRY(b.vector(x + "A_log", s_.heads, &a_log_));
-        BRASA_TRY(b.vector(x + "dt_bias", (uint64_t)s_.heads * s_.dim, &dt_bias_));
+        BRASA_TRY(b.vector(x + "dt_bias", (uint64_t)s_.heads * (hd_ ? 1 : s_.dim), &dt_bias_));
         BRASA_TRY(b.vector(x + "norm", s_.vdim, &norm_));
         BRASA_TRY(b.get(Builder::STATE, 4ull * s_.taps * (2 * s_.qk + s_.vd), (void **)&ring_));
         BRASA_TRY(b.get(Builder::STATE, 4ull * s_.heads * s_.dim * s_.vdim, (void **)&state_));
@@ -993,7 +955,7 @@ class ChannelDelta : public Mixer {
         return BRASA_OK;
     }
 
-    uint64_t scratch_bytes(const Builder &) const override { return at_.total; }
+    uint64_t scratch_bytes() const override { return at_.total; }
 
     void project(const Run &r, std::vector<GemvProblem> &out) override {
         auto add = [&](const Weight &w, uint64_t at, uint32_t ld, bool low) {
@@ -1010,16 +972,22 @@ class ChannelDelta : public Mixer {
         add(k_, at_.k, ldqk_, false);
         add(v_, at_.v, ldv_, false);
         add(b_, at_.b, ldb_, false);
-        add(a1_, at_.a1, lda_, true);  // inputs of a product: bf16 where products take bf16
-        add(g1_, at_.g1, ldg_, true);
+        if (hd_) {
+            add(a1_, at_.z, ldz_, false);
+            out.back().p.bias = dt_bias_;
+            add(g1_, at_.gate, ldv_, false);
+        } else {
+            add(a1_, at_.a1, lda_, true);  // inputs of a product: bf16 where products take bf16
+            add(g1_, at_.g1, ldg_, true);
+        }
     }
 
     int32_t mix(const Run &r) override {
         brasa_ctx *ctx = r.cmd->ctx;
         auto f = [&](uint64_t at) { return (float *)(r.scratch + at); };
         if (r.dev_pos) {
-            DeltaStep p{s_, f(at_.q), f(at_.k), f(at_.v), f(at_.b), f(at_.a1), f(at_.g1), wq_, wk_, wv_, a_log_, dt_bias_, norm_, a2_.p, g2_.p,
-                        a2_.cols, g2_.cols, a2_.ld, g2_.ld, ring_, state_, (float *)r.out, r.dev_pos, eps_};
+            DeltaStep p{s_, f(at_.q), f(at_.k), f(at_.v), f(at_.b), hd_ ? f(at_.z) : f(at_.a1), hd_ ? f(at_.gate) : f(at_.g1), wq_, wk_, wv_, a_log_, dt_bias_, norm_,
+                        a2_.p, g2_.p, a2_.cols, g2_.cols, a2_.ld, g2_.ld, ring_, state_, (float *)r.out[0], r.dev_pos, eps_};
             const size_t smem = step_smem(s_, a2_.cols, g2_.cols);
             const bool keep = s_.dim <= 16 * STEP_R && s_.vdim <= 32 * STEP_C;
             const void *fn = keep ? (const void *)delta_step_kernel<true> : (const void *)delta_step_kernel<false>;
@@ -1028,69 +996,78 @@ class ChannelDelta : public Mixer {
             else BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_step_kernel<false>, dim3(s_.heads), dim3(STEP_THREADS), smem, p));
             return brasa_post_launch(r.cmd, "delta_step");
         }
-        // the second factors of the decay's and the gate's projections
-        LinearProblem lp[2];
-        lp[0].seg[0] = segment(a2_, r.scratch + at_.a1, lda_);
-        lp[0].rows = a2_.rows;
-        lp[0].tokens = r.tokens;
-        lp[0].y = r.scratch + at_.z;
-        lp[0].ldy = ldz_;
-        lp[0].bias = dt_bias_;
-        lp[1].seg[0] = segment(g2_, r.scratch + at_.g1, ldg_);
-        lp[1].rows = g2_.rows;
-        lp[1].tokens = r.tokens;
-        lp[1].y = r.scratch + at_.gate;
-        lp[1].ldy = ldv_;
-        BRASA_TRY(brasa_linear_launch(r.cmd, lp, 2, r.f32));
+        if (!hd_) {  // the second factors of the decay's and the gate's projections
+            LinearProblem lp[2];
+            lp[0].seg[0] = segment(a2_, r.scratch + at_.a1, lda_);
+            lp[0].rows = a2_.rows;
+            lp[0].tokens = r.tokens;
+            lp[0].y = r.scratch + at_.z;
+            lp[0].ldy = ldz_;
+            lp[0].bias = dt_bias_;
+            lp[1].seg[0] = segment(g2_, r.scratch + at_.g1, ldg_);
+            lp[1].rows = g2_.rows;
+            lp[1].tokens = r.tokens;
+            lp[1].y = r.scratch + at_.gate;
+            lp[1].ldy = ldv_;
+            BRASA_TRY(brasa_linear_launch(r.cmd, lp, 2, r.f32));
+        }
         const uint32_t channels = 2 * s_.qk + s_.vd;
         DeltaChunk cp{s_, ConvView{ring_, channels, s_.taps, r.pos0}, f(at_.q), f(at_.k), f(at_.v), f(at_.b), f(at_.z), ldqk_, ldv_, ldb_, ldz_, r.tokens, wq_, wk_, wv_, a_log_,
                       f(at_.qn), f(at_.kn), f(at_.vn), f(at_.g), f(at_.tb)};
-        if (s_.dim <= 64) BRASA_TRY(factors<2>(r.cmd, cp));
-        else if (s_.dim <= 128) BRASA_TRY(factors<4>(r.cmd, cp));
-        else BRASA_TRY(factors<8>(r.cmd, cp));
+        if (hd_) BRASA_TRY(factors_any<true>(r.cmd, cp));
+        else BRASA_TRY(factors_any<false>(r.cmd, cp));
         DeltaScan sp{s_, f(at_.qn), f(at_.kn), f(at_.vn), f(at_.g), f(at_.tb), f(at_.q), f(at_.k), f(at_.v), ldqk_, ldv_, ring_, state_, f(at_.o), r.tokens, r.pos0};
-        BRASA_TRY(scan(r.cmd, sp, r.f32));
+        if (hd_) BRASA_TRY(scan<true>(r.cmd, sp, r.f32));
+        else BRASA_TRY(scan<false>(r.cmd, sp, r.f32));
         const uint32_t blocks = (r.tokens * s_.heads + 7) / 8;
-        if (r.f32) BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_out_kernel<float>, dim3(blocks), dim3(256), 0, f(at_.o), f(at_.gate), ldv_, norm_, (float *)r.out, r.ldo,
-                                                          s_.heads, s_.vdim, r.tokens, eps_));
-        else BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_out_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, f(at_.o), f(at_.gate), ldv_, norm_,
-                                                    (__nv_bfloat16 *)r.out, r.ldo, s_.heads, s_.vdim, r.tokens, eps_));
+        auto out = [&](auto kernel, auto *dst) {
+            return brasa_launch_dependent(ctx, kernel, dim3(blocks), dim3(256), 0, f(at_.o), f(at_.gate), ldv_, norm_, dst, r.ldo[0], s_.heads, s_.vdim, r.tokens, eps_);
+        };
+        if (r.f32) BRASA_CUDA(ctx, hd_ ? out(delta_out_kernel<float, true>, (float *)r.out[0]) : out(delta_out_kernel<float, false>, (float *)r.out[0]));
+        else BRASA_CUDA(ctx, hd_ ? out(delta_out_kernel<__nv_bfloat16, true>, (__nv_bfloat16 *)r.out[0]) : out(delta_out_kernel<__nv_bfloat16, false>, (__nv_bfloat16 *)r.out[0]));
         return brasa_post_launch(r.cmd, "delta_out");
     }
 
   private:
-    template <int E>
+    template <bool HD>
+    int32_t factors_any(brasa_cmd *cmd, const DeltaChunk &p) {
+        if (s_.dim <= 64) return factors<2, HD>(cmd, p);
+        if (s_.dim <= 128) return factors<4, HD>(cmd, p);
+        return factors<8, HD>(cmd, p);
+    }
+    template <int E, bool HD>
     int32_t factors(brasa_cmd *cmd, const DeltaChunk &p) {
         brasa_ctx *ctx = cmd->ctx;
         const size_t smem = 3ull * CH * 32 * E * 4;
-        BRASA_TRY(brasa_smem_optin(ctx, (const void *)delta_chunk_kernel<E>, std::max<size_t>(smem, 48 * 1024)));
-        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_chunk_kernel<E>, dim3((p.tokens + CH - 1) / CH, s_.heads), dim3(256), smem, p));
+        BRASA_TRY(brasa_smem_optin(ctx, (const void *)delta_chunk_kernel<E, HD>, std::max<size_t>(smem, 48 * 1024)));
+        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_chunk_kernel<E, HD>, dim3((p.tokens + CH - 1) / CH, s_.heads), dim3(256), smem, p));
         return brasa_post_launch(cmd, "delta_chunk");
     }
-    template <int D, int CB>
+    template <int D, int CB, bool HD>
     int32_t scan_as(brasa_cmd *cmd, const DeltaScan &p) {
         brasa_ctx *ctx = cmd->ctx;
         const size_t smem = (size_t)ScanShape<D, CB>::FLOATS * 4;
-        BRASA_TRY(brasa_smem_optin(ctx, (const void *)delta_scan_kernel<D, CB>, smem));
-        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_scan_kernel<D, CB>, dim3(s_.heads, (s_.vdim + CB - 1) / CB), dim3(256), smem, p));
+        BRASA_TRY(brasa_smem_optin(ctx, (const void *)delta_scan_kernel<D, CB, HD>, smem));
+        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_scan_kernel<D, CB, HD>, dim3(s_.heads, (s_.vdim + CB - 1) / CB), dim3(256), smem, p));
         return brasa_post_launch(cmd, "delta_scan");
     }
-    template <int D, int CB>
+    template <int D, int CB, bool HD>
     int32_t scan_mma(brasa_cmd *cmd, const DeltaScan &p) {
         brasa_ctx *ctx = cmd->ctx;
         const size_t smem = (size_t)MmaScanShape<D, CB>::FLOATS * 4;
-        BRASA_TRY(brasa_smem_optin(ctx, (const void *)delta_scan_mma_kernel<D, CB>, smem));
-        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_scan_mma_kernel<D, CB>, dim3(s_.heads, (s_.vdim + CB - 1) / CB), dim3(512), smem, p));
+        BRASA_TRY(brasa_smem_optin(ctx, (const void *)delta_scan_mma_kernel<D, CB, HD>, smem));
+        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, delta_scan_mma_kernel<D, CB, HD>, dim3(s_.heads, (s_.vdim + CB - 1) / CB), dim3(512), smem, p));
         return brasa_post_launch(cmd, "delta_scan_mma");
     }
+    template <bool HD>
     int32_t scan(brasa_cmd *cmd, const DeltaScan &p, bool f32) {
         // wide blocks when they still cover most of the SMs
         const bool wide = s_.heads * ((s_.vdim + 31) / 32) * 5 >= (uint32_t)cmd->ctx->sm_count * 4;
-        if (!f32 && s_.dim <= 64) return wide ? scan_mma<64, 32>(cmd, p) : scan_mma<64, 16>(cmd, p);
-        if (!f32 && s_.dim <= 128) return wide ? scan_mma<128, 32>(cmd, p) : scan_mma<128, 16>(cmd, p);
-        if (s_.dim <= 64) return wide ? scan_as<64, 32>(cmd, p) : scan_as<64, 16>(cmd, p);
-        if (s_.dim <= 128) return wide ? scan_as<128, 32>(cmd, p) : scan_as<128, 16>(cmd, p);
-        return scan_as<256, 16>(cmd, p);
+        if (!f32 && s_.dim <= 64) return wide ? scan_mma<64, 32, HD>(cmd, p) : scan_mma<64, 16, HD>(cmd, p);
+        if (!f32 && s_.dim <= 128) return wide ? scan_mma<128, 32, HD>(cmd, p) : scan_mma<128, 16, HD>(cmd, p);
+        if (s_.dim <= 64) return wide ? scan_as<64, 32, HD>(cmd, p) : scan_as<64, 16, HD>(cmd, p);
+        if (s_.dim <= 128) return wide ? scan_as<128, 32, HD>(cmd, p) : scan_as<128, 16, HD>(cmd, p);
+        return scan_as<256, 16, HD>(cmd, p);
     }
 
     void lay_out(uint64_t t, bool f32) {
@@ -1099,26 +1076,28 @@ class ChannelDelta : public Mixer {
         ldb_ = up8(s_.heads);
         lda_ = up8(a1_.rows);
         ldg_ = up8(g1_.rows);
-        ldz_ = up8(s_.heads * s_.dim);
+        ldz_ = up8(s_.heads * (hd_ ? 1 : s_.dim));
         (void)f32;
         Carver c;
         at_.q = c.take(4 * t * ldqk_);
         at_.k = c.take(4 * t * ldqk_);
         at_.v = c.take(4 * t * ldv_);
         at_.b = c.take(4 * t * ldb_);
-        at_.a1 = c.take(4 * t * lda_);
-        at_.g1 = c.take(4 * t * ldg_);
+        at_.a1 = c.take(hd_ ? 0 : 4 * t * lda_);
+        at_.g1 = c.take(hd_ ? 0 : 4 * t * ldg_);
         at_.z = c.take(4 * t * ldz_);
         at_.gate = c.take(4 * t * ldv_);
         at_.qn = c.take(4 * t * s_.qk);
         at_.kn = c.take(4 * t * s_.qk);
         at_.vn = c.take(4 * t * s_.vd);
-        at_.g = c.take(4 * t * s_.heads * s_.dim);
+        at_.g = c.take(4 * t * s_.heads * (hd_ ? 1 : s_.dim));
         at_.tb = c.take(4ull * ((t + CH - 1) / CH) * s_.heads * 2 * CH * CH);
         at_.o = c.take(4 * t * s_.vd);
         at_.total = c.at;
     }
 
+    const bool hd_;  // one decay per head
+    const std::string name_;
     DeltaShape s_{};
     uint32_t width_ = 0, ldqk_ = 0, ldv_ = 0, ldb_ = 0, lda_ = 0, ldg_ = 0, ldz_ = 0;
     float eps_ = 0.0f;
@@ -1132,6 +1111,7 @@ class ChannelDelta : public Mixer {
 
 }  // namespace
 
-std::unique_ptr<Mixer> make_channel_delta() { return std::unique_ptr<Mixer>(new ChannelDelta()); }
+std::unique_ptr<Mixer> make_channel_delta() { return std::unique_ptr<Mixer>(new DeltaRule(false)); }
+std::unique_ptr<Mixer> make_delta() { return std::unique_ptr<Mixer>(new DeltaRule(true)); }
 
 }  // namespace brasa_stack

@@ -369,7 +369,6 @@ class LatentAttention : public Mixer {
         s_.ldc = up8(s_.kr);
         s_.ldr = up8(s_.rot);
         width_ = width;
-        out_width = s_.heads * s_.vdim;
         return true;
     }
 
@@ -379,7 +378,8 @@ class LatentAttention : public Mixer {
         BRASA_TRY(b.matrix(x + "uk", s_.heads * s_.dim, s_.kr, &uk_));
         BRASA_TRY(b.matrix(x + "uv", s_.heads * s_.vdim, s_.kr, &uv_));
         BRASA_TRY(b.matrix(x + "g", s_.heads, width_, &g_));
-        BRASA_TRY(b.matrix(x + "o", width_, s_.heads * s_.vdim, &wo));
+        outs.resize(1);
+        BRASA_TRY(b.matrix(x + "o", width_, s_.heads * s_.vdim, &outs[0]));
         BRASA_TRY(b.vector(x + "dkv.norm", s_.kr, &norm_));
         BRASA_TRY(b.rope(base_, s_.rot_dims, &cos_, &sin_));
         const uint64_t t = b.limits.max_tokens, span = std::min<uint64_t>(b.limits.ctx, t + s_.window - 1);
@@ -409,7 +409,7 @@ class LatentAttention : public Mixer {
         return BRASA_OK;
     }
 
-    uint64_t scratch_bytes(const Builder &) const override { return at_.total; }
+    uint64_t scratch_bytes() const override { return at_.total; }
 
     void project(const Run &r, std::vector<GemvProblem> &out) override {
         auto add = [&](const Weight &w, uint64_t at, uint32_t ld) {
@@ -469,11 +469,13 @@ class LatentAttention : public Mixer {
         a.cos_t = cos_;
         a.sin_t = sin_;
         a.gate = f(at_.gate);
-        a.out = r.out;
-        a.ldq = ldq_; a.ldk = ldk_; a.ldv = ldv_; a.ldr = s_.ldr; a.ldg = ldg_; a.ldo = r.ldo;
+        a.out = r.out[0];
+        a.ldq = ldq_; a.ldk = ldk_; a.ldv = ldv_; a.ldr = s_.ldr; a.ldg = ldg_; a.ldo = r.ldo[0];
         a.tokens = r.tokens; a.heads = s_.heads; a.dim = s_.dim; a.rot = s_.rot; a.rot_dims = s_.rot_dims; a.vdim = s_.vdim;
         a.pos0 = r.pos0; a.key0 = key0; a.keys = keys; a.window = s_.window;
         a.scale = s_.scale;
+        a.kv_heads = s_.heads; a.kstep = s_.dim; a.vstep = s_.vdim;
+        a.out_scale = 1.0f;
         return brasa_window_attention_launch(r.cmd, a, r.f32);
     }
 
@@ -496,7 +498,7 @@ class LatentAttention : public Mixer {
         const size_t csm = (size_t)(s_.ldc + chunks_) * 4;
         BRASA_TRY(brasa_smem_optin(ctx, (const void *)latent_combine_kernel, std::max<size_t>(csm, 48 * 1024)));
         BRASA_CUDA(ctx, brasa_launch_dependent(ctx, latent_combine_kernel, dim3(s_.heads, (s_.vdim + vper - 1) / vper), dim3(256), csm, s_, f(at_.part), chunks_, uv_.p, uv_.ld,
-                                               f(at_.gate), (float *)r.out, vper));
+                                               f(at_.gate), (float *)r.out[0], vper));
         return brasa_post_launch(r.cmd, "latent_combine");
     }
 

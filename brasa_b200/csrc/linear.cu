@@ -9,12 +9,23 @@ using namespace brasa_dev;
 
 namespace {
 
+__device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float activate(float v, int act) {
     if (act == LINEAR_ACT_RELU2) {
         v = fmaxf(v, 0.0f);
         v *= v;
+    } else if (act == LINEAR_ACT_GELU_TANH) {
+        v = 0.5f * v * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * v * v, v, v)));
     }
     return v;
+}
+// the epilogue behind the sum and its bias, up to the residual
+__device__ __forceinline__ float finish(float v, int act, float scale, float cap) {
+    v = activate(v, act) * scale;
+    return cap > 0.0f ? cap * tanhf(v / cap) : v;
+}
+__device__ __forceinline__ float mul_at(const uint16_t *mul, uint32_t ldm, uint32_t id, uint32_t r) {
+    return __uint_as_float((uint32_t)mul[(size_t)id * ldm + r] << 16);
 }
 
 // ---- f32: inputs f32 (or bf16), weights bf16, f32 FMA. Block 16 x 16 threads, each 4 tokens x 4 rows. -----------------
@@ -57,12 +68,14 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const __grid_constant__
             __syncthreads();
         }
     }
+    const bool glu = p.act == LINEAR_ACT_SWIGLU;  // tile rows 0-31 are gate rows, 32-63 their up rows
     for (int i = 0; i < 4; ++i)
-        for (int j = 0; j < 4; ++j) {
-            const uint32_t tok = tok0 + ty + 16 * i, r = row0 + tx + 16 * j;
-            if (tok >= p.tokens || r >= p.rows) continue;
+        for (int j = 0; j < (glu ? 2 : 4); ++j) {
+            const uint32_t tok = tok0 + ty + 16 * i, r = (glu ? row0 / 2 : row0) + tx + 16 * j;
+            if (tok >= p.tokens || r >= (glu ? p.rows / 2 : p.rows)) continue;
             const size_t at = (size_t)tok * p.ldy + r;
-            float v = activate(acc[i][j] + (p.bias ? p.bias[r] : 0.0f), p.act) * p.scale;
+            float v = glu ? silu_f(acc[i][j]) * acc[i][j + 2] : finish(acc[i][j] + (p.bias ? p.bias[r] : 0.0f), p.act, p.scale, p.cap);
+            if (p.mul) v *= mul_at(p.mul, p.ldm, p.mul_ids[tok], r);
             if (p.resid) v += p.resid[at];
             if (p.y_bf16) static_cast<__nv_bfloat16 *>(p.y)[at] = __float2bfloat16_rn(v);
             else static_cast<float *>(p.y)[at] = v;
@@ -80,17 +93,24 @@ struct GemvDevProblem {
     float *y;
     const float *bias, *resid;
     int act;
-    float scale;
+    float scale, cap;
+    const uint16_t *mul;
+    const uint32_t *mul_id;
+    uint32_t ldm;
 };
 struct GemvDevParams {
     GemvDevProblem p[LINEAR_MAX];
     uint32_t row_end[LINEAR_MAX];
     uint32_t n, total_rows;
-    const float *ln_x;
+    const float *x, *y, *wy;
+    float *x_out;
+    int norm;
     uint32_t width, nin;
     float eps;
-    const float *w[2], *b[2], *v[2];
-    uint32_t len[2], off[2], x_floats;
+    const float *w[2], *b[2], *v[2], *vw[2];
+    float vscale[2];
+    uint32_t len[2], off[2], parts[2], x_floats;
+    bool gated;
 };
 constexpr int GV_WARPS = 32, GV_UNROLL = 4;
 
@@ -162,24 +182,74 @@ __global__ void __launch_bounds__(32 * GV_WARPS, 1) linear_gemv_kernel(const __g
     // ---- the input vectors ----
     for (uint32_t i = tid; i < gp.x_floats; i += 32 * GV_WARPS) xs[i] = 0.0f;  // (padding)
     __syncthreads();
-    if (gp.ln_x) {
-        float s = 0.0f;
-        for (uint32_t i = tid; i < gp.width; i += 32 * GV_WARPS) s += gp.ln_x[i];
-        const float mean = block_sum_1024(s, red) / (float)gp.width;
+    if (gp.x) {
+        // the residual stream, with the pending sublayer's normed result added; every thread keeps to its own elements
+        float s = 0.0f, sy = 0.0f;
+        if (gp.y) {
+            for (uint32_t i = tid; i < gp.width; i += 32 * GV_WARPS) s = fmaf(gp.y[i], gp.y[i], s);
+            sy = 1.0f / sqrtf(block_sum_1024(s, red) / (float)gp.width + gp.eps);
+        }
         s = 0.0f;
         for (uint32_t i = tid; i < gp.width; i += 32 * GV_WARPS) {
-            const float d = gp.ln_x[i] - mean;
-            s = fmaf(d, d, s);
+            float v = gp.x[i];
+            if (gp.y) {
+                v = fmaf(gp.y[i] * sy, gp.wy[i], v);
+                if (blockIdx.x == 0 && gp.x_out) gp.x_out[i] = v;
+            }
+            xs[gv_plane(gp.off[0] + i, half)] = v;
+            s += gp.norm == GEMV_LAYER_NORM ? v : v * v;
         }
-        const float inv = 1.0f / sqrtf(block_sum_1024(s, red) / (float)gp.width + gp.eps);
-        for (uint32_t i = tid; i < gp.width; i += 32 * GV_WARPS) {
-            const float z = (gp.ln_x[i] - mean) * inv;
-            xs[gv_plane(gp.off[0] + i, half)] = fmaf(z, gp.w[0][i], gp.b[0][i]);
-            if (gp.nin > 1) xs[gv_plane(gp.off[1] + i, half)] = fmaf(z, gp.w[1][i], gp.b[1][i]);
+        if (gp.norm == GEMV_LAYER_NORM) {
+            const float mean = block_sum_1024(s, red) / (float)gp.width;
+            s = 0.0f;
+            for (uint32_t i = tid; i < gp.width; i += 32 * GV_WARPS) {
+                const float d = xs[gv_plane(gp.off[0] + i, half)] - mean;
+                s = fmaf(d, d, s);
+            }
+            const float inv = 1.0f / sqrtf(block_sum_1024(s, red) / (float)gp.width + gp.eps);
+            for (uint32_t i = tid; i < gp.width; i += 32 * GV_WARPS) {
+                const float z = (xs[gv_plane(gp.off[0] + i, half)] - mean) * inv;
+                xs[gv_plane(gp.off[0] + i, half)] = fmaf(z, gp.w[0][i], gp.b[0][i]);
+                if (gp.nin > 1) xs[gv_plane(gp.off[1] + i, half)] = fmaf(z, gp.w[1][i], gp.b[1][i]);
+            }
+        } else if (gp.norm == GEMV_RMS_NORM) {
+            const float inv = 1.0f / sqrtf(block_sum_1024(s, red) / (float)gp.width + gp.eps);
+            for (uint32_t i = tid; i < gp.width; i += 32 * GV_WARPS) {
+                const uint32_t at = gv_plane(gp.off[0] + i, half);
+                xs[at] = xs[at] * inv * gp.w[0][i];
+            }
         }
     } else {
-        for (uint32_t k = 0; k < gp.nin; ++k)
-            for (uint32_t i = tid; i < gp.len[k]; i += 32 * GV_WARPS) xs[gv_plane(gp.off[k] + i, half)] = gp.v[k][i];
+        for (uint32_t k = 0; k < gp.nin; ++k) {
+            if (gp.gated && k == 0) {
+                for (uint32_t i = tid; i < gp.len[0]; i += 32 * GV_WARPS) {
+                    const float *g = gp.v[0] + (size_t)(i >> 5) * 64 + (i & 31);
+                    xs[gv_plane(gp.off[0] + i, half)] = silu_f(g[0]) * g[32];
+                }
+            } else if (gp.parts[k]) {
+                // a warp takes parts warp, warp + 32, .. where there are many; otherwise a part is the block's
+                const uint32_t n = gp.len[k] / gp.parts[k];
+                if (gp.parts[k] >= GV_WARPS / 2) {
+                    for (uint32_t part = warp; part < gp.parts[k]; part += GV_WARPS) {
+                        float s = 0.0f;
+                        for (uint32_t i = lane; i < n; i += 32) s = fmaf(gp.v[k][part * n + i], gp.v[k][part * n + i], s);
+#pragma unroll
+                        for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+                        const float inv = gp.vscale[k] / sqrtf(s / (float)n + gp.eps);
+                        for (uint32_t i = lane; i < n; i += 32) xs[gv_plane(gp.off[k] + part * n + i, half)] = gp.v[k][part * n + i] * inv * gp.vw[k][part * n + i];
+                    }
+                } else {
+                    for (uint32_t part = 0; part < gp.parts[k]; ++part) {
+                        float s = 0.0f;
+                        for (uint32_t i = tid; i < n; i += 32 * GV_WARPS) s = fmaf(gp.v[k][part * n + i], gp.v[k][part * n + i], s);
+                        const float inv = gp.vscale[k] / sqrtf(block_sum_1024(s, red) / (float)n + gp.eps);
+                        for (uint32_t i = tid; i < n; i += 32 * GV_WARPS) xs[gv_plane(gp.off[k] + part * n + i, half)] = gp.v[k][part * n + i] * inv * gp.vw[k][part * n + i];
+                    }
+                }
+            } else {
+                for (uint32_t i = tid; i < gp.len[k]; i += 32 * GV_WARPS) xs[gv_plane(gp.off[k] + i, half)] = gp.v[k][i];
+            }
+        }
     }
     __syncthreads();
     // ---- batches ----
@@ -219,7 +289,8 @@ __global__ void __launch_bounds__(32 * GV_WARPS, 1) linear_gemv_kernel(const __g
                 parity ^= 1;
             }
             if (sub == 0 && lane == 0) {
-                float v = activate(acc + (p.bias ? p.bias[cur.r] : 0.0f), p.act) * p.scale;
+                float v = finish(acc + (p.bias ? p.bias[cur.r] : 0.0f), p.act, p.scale, p.cap);
+                if (p.mul) v *= mul_at(p.mul, p.ldm, *p.mul_id, cur.r);
                 if (p.resid) v += p.resid[cur.r];
                 p.y[cur.r] = v;
             }
@@ -248,7 +319,10 @@ struct TcProblem {
     uint32_t ldy, y_bf16;
     const float *bias, *resid;
     int act;
-    float scale;
+    float scale, cap;
+    const uint16_t *mul;
+    const uint32_t *mul_ids;
+    uint32_t ldm;
 };
 struct TcParams {
     CUtensorMap x[LINEAR_MAX][2], w[LINEAR_MAX][2];
@@ -376,28 +450,37 @@ __global__ void __launch_bounds__(256, 1) linear_tc_kernel(const __grid_constant
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const uint32_t ncol = min((uint32_t)BN, p.rows - row0);
-            const bool live = tok0 + 32 * q < p.tokens;
-            for (uint32_t c0 = 0; c0 < ncol && live; c0 += 32) {
+            const bool live = tok0 + 32 * q < p.tokens, glu = p.act == LINEAR_ACT_SWIGLU;
+            const uint32_t out_rows = glu ? p.rows / 2 : p.rows;
+            for (uint32_t c0 = 0; c0 < ncol && live; c0 += glu ? 64 : 32) {
                 uint32_t v[32];
                 tc_ld32(tmem + buf * BN + ((q * 32u) << 16) + c0, v);
+                if (glu) {
+                    uint32_t u[32];
+                    tc_ld32(tmem + buf * BN + ((q * 32u) << 16) + c0 + 32, u);
+#pragma unroll
+                    for (int e = 0; e < 32; ++e) v[e] = __float_as_uint(silu_f(__uint_as_float(v[e])) * __uint_as_float(u[e]));
+                }
 #pragma unroll
                 for (int g = 0; g < 8; ++g)
                     *reinterpret_cast<float4 *>(stage + lane * EPI_LD + 4 * g) =
                         make_float4(__uint_as_float(v[4 * g]), __uint_as_float(v[4 * g + 1]), __uint_as_float(v[4 * g + 2]), __uint_as_float(v[4 * g + 3]));
                 __syncwarp();
-                const uint32_t r = row0 + c0 + tc;
+                const uint32_t r = (glu ? (row0 + c0) / 2 : row0 + c0) + tc;
                 float bias[4];
 #pragma unroll
-                for (int e = 0; e < 4; ++e) bias[e] = (p.bias && r + e < p.rows) ? p.bias[r + e] : 0.0f;
-                const bool vec = r + 4 <= p.rows && (p.ldy & 3) == 0;
+                for (int e = 0; e < 4; ++e) bias[e] = (p.bias && r + e < out_rows) ? p.bias[r + e] : 0.0f;
+                const bool vec = r + 4 <= out_rows && (p.ldy & 3) == 0;
 #pragma unroll
                 for (int i = 0; i < 8; ++i) {
                     const uint32_t tok = tok0 + 32 * q + 4 * i + tr;
-                    if (tok < p.tokens && r < p.rows) {
+                    if (tok < p.tokens && r < out_rows) {
                         const float4 a = *reinterpret_cast<const float4 *>(stage + (4 * i + tr) * EPI_LD + tc);
                         float o[4] = {a.x, a.y, a.z, a.w};
 #pragma unroll
-                        for (int e = 0; e < 4; ++e) o[e] = activate(o[e] + bias[e], p.act) * p.scale;
+                        for (int e = 0; e < 4; ++e) o[e] = glu ? o[e] : finish(o[e] + bias[e], p.act, p.scale, p.cap);
+                        if (p.mul)
+                            for (int e = 0; e < 4 && r + e < out_rows; ++e) o[e] *= mul_at(p.mul, p.ldm, p.mul_ids[tok], r + e);
                         const size_t at = (size_t)tok * p.ldy + r;
                         if (vec) {
                             if (p.resid) {
@@ -407,7 +490,7 @@ __global__ void __launch_bounds__(256, 1) linear_tc_kernel(const __grid_constant
                             if (p.y_bf16) *reinterpret_cast<uint2 *>(static_cast<__nv_bfloat16 *>(p.y) + at) = make_uint2(bf16_pack(o[0], o[1]), bf16_pack(o[2], o[3]));
                             else *reinterpret_cast<float4 *>(static_cast<float *>(p.y) + at) = make_float4(o[0], o[1], o[2], o[3]);
                         } else {
-                            for (int e = 0; e < 4 && r + e < p.rows; ++e) {
+                            for (int e = 0; e < 4 && r + e < out_rows; ++e) {
                                 if (p.resid) o[e] += p.resid[at + e];
                                 if (p.y_bf16) static_cast<__nv_bfloat16 *>(p.y)[at + e] = __float2bfloat16_rn(o[e]);
                                 else static_cast<float *>(p.y)[at + e] = o[e];
@@ -455,6 +538,10 @@ int32_t launch_tc(brasa_cmd *cmd, const LinearProblem *p, uint32_t n) {
         d.resid = q.resid;
         d.act = q.act;
         d.scale = q.scale;
+        d.cap = q.cap;
+        d.mul = q.mul;
+        d.mul_ids = q.mul_ids;
+        d.ldm = q.ldm;
         for (int s = 0; s < 2; ++s) {
             const LinearSeg &g = q.seg[s].cols ? q.seg[s] : q.seg[0];
             const uint64_t xd[2] = {g.cols, q.tokens}, xst[1] = {(uint64_t)g.ldx * 2}, wd[2] = {g.cols, q.rows}, wst[1] = {(uint64_t)g.ldw * 2};
@@ -506,7 +593,9 @@ int32_t brasa_linear_launch(brasa_cmd *cmd, const LinearProblem *ps, uint32_t co
     for (uint32_t i = 0; i < count; ++i) {
         const LinearProblem &q = ps[i];
         if (q.tokens == 0 || q.rows == 0) continue;
-        BRASA_REQUIRE(ctx, q.seg[0].cols > 0 && q.y && q.seg[0].x && q.seg[0].w && q.ldy >= q.rows, "linear: empty or short product");
+        BRASA_REQUIRE(ctx, q.seg[0].cols > 0 && q.y && q.seg[0].x && q.seg[0].w && q.ldy >= q.out_rows(), "linear: empty or short product");
+        BRASA_REQUIRE(ctx, q.act != LINEAR_ACT_SWIGLU || (q.rows % 64 == 0 && !q.bias && q.scale == 1.0f && q.cap == 0.0f), "linear: gated rows come in pairs of 32, without bias, scale and cap");
+        BRASA_REQUIRE(ctx, !q.mul || q.mul_ids, "linear: a factor's rows need token ids");
         for (int s = 0; s < 2; ++s) {
             const LinearSeg &g = q.seg[s];
             if (!g.cols) continue;
@@ -546,23 +635,33 @@ int32_t brasa_linear_gemv_launch(brasa_cmd *cmd, const GemvInput &in, const Gemv
     GemvDevParams g;
     memset(&g, 0, sizeof g);
     auto up8 = [](uint32_t v) { return (v + 7) / 8 * 8; };
-    g.ln_x = in.ln_x;
+    BRASA_REQUIRE(ctx, !in.y || (in.x && in.wy && in.x_out != in.x), "gemv: a pending sum needs its weights and a place of its own");
+    g.x = in.x;
+    g.y = in.y;
+    g.wy = in.wy;
+    g.x_out = in.x_out;
+    g.norm = in.norm;
+    g.gated = in.gated;
     g.width = in.width;
     g.eps = in.eps;
     uint32_t off = 0;
     for (int i = 0; i < 2; ++i) {
-        const bool used = in.ln_x ? in.w[i] != nullptr : in.v[i] != nullptr;
+        const bool used = in.x ? in.w[i] != nullptr || (in.norm == GEMV_PLAIN && i == 0) : in.v[i] != nullptr;
         if (!used) continue;
+        BRASA_REQUIRE(ctx, !in.parts[i] || in.x || (in.vw[i] && in.len[i] % in.parts[i] == 0), "gemv: an input that does not divide into its parts");
+        g.parts[i] = in.x ? 0u : in.parts[i];
+        g.vw[i] = in.vw[i];
+        g.vscale[i] = in.vscale[i];
         g.w[i] = in.w[i];
         g.b[i] = in.b[i];
         g.v[i] = in.v[i];
-        g.len[i] = in.ln_x ? in.width : in.len[i];
+        g.len[i] = in.x ? in.width : in.len[i];
         g.off[i] = off;
         off += up8(g.len[i]);
         g.nin = i + 1;
     }
     g.x_floats = off;
-    BRASA_REQUIRE(ctx, g.nin >= 1 && (g.nin == 1 || g.len[0] > 0), "gemv: no input");
+    BRASA_REQUIRE(ctx, g.nin >= 1 && (g.nin == 1 || g.len[0] > 0) && (g.nin == 1 || !in.x || in.norm == GEMV_LAYER_NORM), "gemv: no input, or two forms of an RMS norm");
     uint32_t rows = 0;
     for (uint32_t i = 0; i < n; ++i) {
         const LinearProblem &q = ps[i].p;
@@ -584,6 +683,11 @@ int32_t brasa_linear_gemv_launch(brasa_cmd *cmd, const GemvInput &in, const Gemv
         d.resid = q.resid;
         d.act = q.act;
         d.scale = q.scale;
+        d.cap = q.cap;
+        d.mul = q.mul;
+        d.mul_id = q.mul_ids;
+        d.ldm = q.ldm;
+        BRASA_REQUIRE(ctx, q.act != LINEAR_ACT_SWIGLU && (!q.mul || q.mul_ids), "gemv: gated rows are formed by the next product; a factor needs the token's id");
         rows += q.rows;
         g.row_end[i] = rows;
     }
@@ -627,7 +731,11 @@ extern "C" int32_t brasa_k_linear(brasa_cmd *cmd, const brasa_linear *ps, uint32
     const uint64_t xe = f32_inputs ? 4 : 2;
     for (uint32_t i = 0; i < count; ++i) {
         const brasa_linear &p = ps[i];
-        BRASA_REQUIRE(ctx, p.rows > 0 && p.tokens > 0 && p.cols > 0 && p.ldy >= p.rows, "linear: empty product");
+        BRASA_REQUIRE(ctx, p.rows > 0 && p.tokens > 0 && p.cols > 0 && p.ldy >= (p.act == BRASA_ACT_SWIGLU ? p.rows / 2 : p.rows), "linear: empty product");
+        BRASA_REQUIRE(ctx, p.act >= BRASA_ACT_NONE && p.act <= BRASA_ACT_SWIGLU && p.cap >= 0.0f, "linear: unknown activation or negative cap");
+        BRASA_REQUIRE(ctx, !p.mul.buf || (arg_fits(p.mul_ids, (uint64_t)p.tokens * 4) && p.ldm >= (p.act == BRASA_ACT_SWIGLU ? p.rows / 2 : p.rows) &&
+                                          arg_fits(p.mul, (uint64_t)p.mul_rows * p.ldm * 2)),
+                      "linear: mul or its ids too small");
         BRASA_REQUIRE(ctx, arg_fits(p.w, (uint64_t)p.rows * p.ldw * 2) && arg_fits(p.x, (uint64_t)p.tokens * p.ldx * xe), "linear: w or x too small");
         BRASA_REQUIRE(ctx, !p.cols2 || (arg_fits(p.w2, (uint64_t)p.rows * p.ldw2 * 2) && arg_fits(p.x2, (uint64_t)p.tokens * p.ldx2 * xe)), "linear: w2 or x2 too small");
         BRASA_REQUIRE(ctx, arg_fits(p.y, (uint64_t)p.tokens * p.ldy * (p.y_bf16 ? 2 : 4)), "linear: y too small");
@@ -643,6 +751,10 @@ extern "C" int32_t brasa_k_linear(brasa_cmd *cmd, const brasa_linear *ps, uint32
         q[i].resid = (const float *)arg_ptr(p.resid);
         q[i].act = p.act;
         q[i].scale = p.scale;
+        q[i].cap = p.cap;
+        q[i].mul = (const uint16_t *)arg_ptr(p.mul);
+        q[i].ldm = p.ldm;
+        q[i].mul_ids = (const uint32_t *)arg_ptr(p.mul_ids);
     }
     return brasa_linear_launch(cmd, q, count, f32_inputs != 0);
 }

@@ -461,7 +461,7 @@ int32_t qwen3_plan(brasa_ctx *ctx, const brasa::WeightFile &f, const brasa_sessi
     return brasa_plan(&shape, &s, out);
 }
 
-int32_t qwen3_run_layers(brasa_model *m, brasa_cmd *cmd, const float *x, float *y, uint32_t tokens, uint32_t pos0, uint32_t l0, uint32_t l1) {
+int32_t qwen3_run_layers(brasa_model *m, brasa_cmd *cmd, const uint32_t *, const float *x, float *y, uint32_t tokens, uint32_t pos0, uint32_t l0, uint32_t l1) {
     const uint64_t n = (uint64_t)tokens * m->cfg.hidden * 4;
     BRASA_TRY(brasa_buf_upload(m->x, 0, x, n));
     if (tokens == 1 && decode_fused_ok(m)) {
@@ -544,7 +544,7 @@ const brasa_family qwen3_family = {"qwen3", qwen3_describe, qwen3_plan, qwen3_lo
 bool is_qwen3(const brasa_model *m) { return m->family == &qwen3_family; }
 
 // The families this library runs.
-const brasa_family *const FAMILIES[] = {&qwen3_family, &brasa_stack::dunuzen_family};
+const brasa_family *const FAMILIES[] = {&qwen3_family, &brasa_stack::dunuzen_family, &brasa_stack::gugedra_family};
 
 const brasa_family *family_of(const brasa::WeightFile &f, std::string &err) {
     for (const brasa_family *fam : FAMILIES)
@@ -739,14 +739,20 @@ int32_t brasa_model_forward(brasa_model *m, const uint32_t *ids, uint32_t tokens
 }
 
 int32_t brasa_model_run_layers(brasa_model *m, float *x, uint32_t tokens, uint32_t pos0, uint32_t layer_begin, uint32_t layer_end) {
+    return brasa_model_run_layers_ids(m, nullptr, x, tokens, pos0, layer_begin, layer_end);
+}
+
+int32_t brasa_model_run_layers_ids(brasa_model *m, const uint32_t *ids, float *x, uint32_t tokens, uint32_t pos0, uint32_t layer_begin, uint32_t layer_end) {
     if (!m || !x) return BRASA_EINVAL;
     brasa_ctx *ctx = m->ctx;
     BRASA_TRY(check_tokens(m, tokens, pos0));
     BRASA_REQUIRE(ctx, layer_begin <= layer_end && layer_end <= m->cfg.layers, "layer range");
+    BRASA_REQUIRE(ctx, ids || !brasa_stack::layers_read_ids(m), "run_layers: the layers of this model read the tokens' ids too");
+    for (uint32_t i = 0; ids && i < tokens; ++i) BRASA_REQUIRE(ctx, ids[i] < m->cfg.vocab, "token id %u outside the vocabulary", ids[i]);
     if (m->family->begin) BRASA_TRY(m->family->begin(m, pos0, layer_begin, layer_end));
     brasa_cmd *cmd;
     BRASA_TRY(brasa_cmd_begin(ctx, &cmd));
-    int32_t rc = m->family->run_layers(m, cmd, x, x, tokens, pos0, layer_begin, layer_end);
+    int32_t rc = m->family->run_layers(m, cmd, ids, x, x, tokens, pos0, layer_begin, layer_end);
     int32_t rc2 = brasa_cmd_wait(cmd, nullptr);
     BRASA_TRY(rc);
     BRASA_TRY(rc2);

@@ -47,7 +47,8 @@ struct brasa_family {
     int32_t (*forward)(brasa_model *m, brasa_cmd *cmd, uint32_t tokens, uint32_t pos0, const uint32_t *rows, uint32_t n_rows);
     // one token m->ids[0] at the position in m->dev_state[0]: logits to m->logits, the greedy choice to m->next_id
     int32_t (*step)(brasa_model *m, brasa_cmd *cmd);
-    int32_t (*run_layers)(brasa_model *m, brasa_cmd *cmd, const float *x, float *y, uint32_t tokens, uint32_t pos0, uint32_t l0, uint32_t l1);
+    // ids: of the tokens; may be null where the layers do not read them
+    int32_t (*run_layers)(brasa_model *m, brasa_cmd *cmd, const uint32_t *ids, const float *x, float *y, uint32_t tokens, uint32_t pos0, uint32_t l0, uint32_t l1);
     // Families whose state cannot be rewound: begin checks that layers [l0, l1) can take a run at pos0 (their own position, or
     // 0), finish notes the position they have reached, reached tells it. All null where any cached position can be continued from.
     int32_t (*begin)(brasa_model *m, uint32_t pos0, uint32_t l0, uint32_t l1);
@@ -55,7 +56,8 @@ struct brasa_family {
     uint32_t (*reached)(brasa_model *m);
 };
 namespace brasa_stack {
-extern const brasa_family dunuzen_family;
+extern const brasa_family dunuzen_family, gugedra_family;
+bool layers_read_ids(const brasa_model *m);
 }
 // A tensor's bytes to dst on the device, through the loading model's pinned staging buffers.
 int32_t brasa_stage_upload(brasa_model *m, void *dst, const brasa::WeightFile &f, const brasa::TensorInfo &t);

@@ -213,6 +213,97 @@ __global__ void __launch_bounds__(256) layer_norm_kernel(LayerNormParams p) {
     }
 }
 
+// Pre- and post-norms of a residual stream in one pass over a row: x' = x + y / rms(y) * wy (y != nullptr; a sublayer's result),
+// x_out = x' (x itself or another buffer; may be null), out = x' / rms(x') * w, or x' as it is without w. rows != nullptr picks
+// the input rows. One block per row.
+struct AddRmsNormParams {
+    const float *x, *y, *wy, *w;
+    float *x_out;
+    void *out;
+    const uint32_t *rows;
+    uint32_t n, ldo;
+    float eps;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) add_rms_norm_kernel(AddRmsNormParams p) {
+    __shared__ float red[8];
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    const size_t row = (size_t)(p.rows ? p.rows[blockIdx.x] : blockIdx.x) * p.n;
+    const float *x = p.x + row, *y = p.y + row;
+    auto block_sum = [&](float v) {
+        for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+        if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+        __syncthreads();
+        v = ((red[0] + red[1]) + (red[2] + red[3])) + ((red[4] + red[5]) + (red[6] + red[7]));
+        __syncthreads();
+        return v;
+    };
+    float s = 0.0f;
+    if ((p.n & 3) == 0 && p.n <= 256 * 4 * LN_VEC && (p.ldo & 3) == 0) {  // the row in registers, four values at a time
+        const float4 *x4 = reinterpret_cast<const float4 *>(x);
+        float4 v[LN_VEC], u[LN_VEC];
+#pragma unroll
+        for (int c = 0; c < LN_VEC; ++c) {
+            const uint32_t i = threadIdx.x + 256 * c;
+            v[c] = i < p.n / 4 ? x4[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+            if (p.y) u[c] = i < p.n / 4 ? reinterpret_cast<const float4 *>(y)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+        if (p.y) {
+#pragma unroll
+            for (int c = 0; c < LN_VEC; ++c) s += (u[c].x * u[c].x + u[c].y * u[c].y) + (u[c].z * u[c].z + u[c].w * u[c].w);
+            const float inv = 1.0f / sqrtf(block_sum(s) / (float)p.n + p.eps);
+#pragma unroll
+            for (int c = 0; c < LN_VEC; ++c) {
+                const uint32_t i = threadIdx.x + 256 * c;
+                if (i < p.n / 4) {
+                    const float4 w = reinterpret_cast<const float4 *>(p.wy)[i];
+                    v[c] = make_float4(fmaf(u[c].x * inv, w.x, v[c].x), fmaf(u[c].y * inv, w.y, v[c].y), fmaf(u[c].z * inv, w.z, v[c].z), fmaf(u[c].w * inv, w.w, v[c].w));
+                    if (p.x_out) reinterpret_cast<float4 *>(p.x_out + row)[i] = v[c];
+                }
+            }
+        }
+        if (!p.out) return;
+        float inv = 1.0f;
+        if (p.w) {
+            s = 0.0f;
+#pragma unroll
+            for (int c = 0; c < LN_VEC; ++c) s += (v[c].x * v[c].x + v[c].y * v[c].y) + (v[c].z * v[c].z + v[c].w * v[c].w);
+            inv = 1.0f / sqrtf(block_sum(s) / (float)p.n + p.eps);
+        }
+#pragma unroll
+        for (int c = 0; c < LN_VEC; ++c) {
+            const uint32_t i = threadIdx.x + 256 * c;
+            if (i < p.n / 4) {
+                const float4 w = p.w ? reinterpret_cast<const float4 *>(p.w)[i] : make_float4(1.f, 1.f, 1.f, 1.f);
+                const float4 o = make_float4(v[c].x * inv * w.x, v[c].y * inv * w.y, v[c].z * inv * w.z, v[c].w * inv * w.w);
+                T *dst = static_cast<T *>(p.out) + (size_t)blockIdx.x * p.ldo + 4 * i;
+                if (sizeof(T) == 4) *reinterpret_cast<float4 *>(dst) = o;
+                else *reinterpret_cast<uint2 *>(dst) = make_uint2(brasa_dev::bf16_pack(o.x, o.y), brasa_dev::bf16_pack(o.z, o.w));
+            }
+        }
+        return;
+    }
+    float iy = 0.0f;
+    if (p.y) {
+        for (uint32_t i = threadIdx.x; i < p.n; i += 256) s = fmaf(y[i], y[i], s);
+        iy = 1.0f / sqrtf(block_sum(s) / (float)p.n + p.eps);
+    }
+    auto value = [&](uint32_t i) { return p.y ? fmaf(y[i] * iy, p.wy[i], x[i]) : x[i]; };
+    float inv = 1.0f;
+    if (p.out && p.w) {
+        s = 0.0f;
+        for (uint32_t i = threadIdx.x; i < p.n; i += 256) s = fmaf(value(i), value(i), s);
+        inv = 1.0f / sqrtf(block_sum(s) / (float)p.n + p.eps);
+    }
+    for (uint32_t i = threadIdx.x; i < p.n; i += 256) {
+        const float v = value(i);
+        if (p.out) brasa_dev::elem_store(static_cast<T *>(p.out) + (size_t)blockIdx.x * p.ldo + i, p.w ? v * inv * p.w[i] : v);
+        if (p.y && p.x_out) p.x_out[row + i] = v;
+    }
+}
+
 __global__ void softmax_kernel(const float *x, float *out, uint32_t n) {
     __shared__ float red[32];
     const float *xr = x + (size_t)blockIdx.x * n;
@@ -409,6 +500,16 @@ int32_t brasa_layer_norm_launch(brasa_cmd *cmd, const float *x, const uint32_t *
     return brasa_post_launch(cmd, "layer_norm");
 }
 
+int32_t brasa_add_rms_norm_launch(brasa_cmd *cmd, const float *x, const float *y, const float *wy, float *x_out, const float *w, void *out, const uint32_t *rows,
+                                  uint32_t n_rows, uint32_t n, uint32_t ldo, float eps, bool f32) {
+    brasa_ctx *ctx = cmd->ctx;
+    if (n_rows == 0) return BRASA_OK;
+    AddRmsNormParams p{x, y, wy, w, x_out, out, rows, n, ldo, eps};
+    if (f32) BRASA_CUDA(ctx, brasa_launch_dependent(ctx, add_rms_norm_kernel<float>, dim3(n_rows), dim3(256), 0, p));
+    else BRASA_CUDA(ctx, brasa_launch_dependent(ctx, add_rms_norm_kernel<__nv_bfloat16>, dim3(n_rows), dim3(256), 0, p));
+    return brasa_post_launch(cmd, "add_rms_norm");
+}
+
 int32_t brasa_embed_bf16_launch(brasa_cmd *cmd, const uint16_t *table, uint32_t ld, uint32_t rows, uint32_t n, float scale, const uint32_t *ids, float *out,
                                 uint32_t tokens) {
     embed_bf16_kernel<<<blocks_for((uint64_t)tokens * n, 256), 256, 0, cmd->ctx->stream>>>(table, ld, rows, n, scale, ids, out, tokens);
@@ -425,6 +526,19 @@ int32_t brasa_k_layer_norm(brasa_cmd *cmd, brasa_arg x, brasa_arg w, brasa_arg b
     const float *ws[2] = {(const float *)arg_ptr(w), nullptr}, *bs[2] = {(const float *)arg_ptr(b), nullptr};
     void *outs[2] = {arg_ptr(out), nullptr};
     return brasa_layer_norm_launch(cmd, (const float *)arg_ptr(x), nullptr, rows, n, eps, ws, bs, outs, 1, n, true);
+}
+
+int32_t brasa_k_add_rms_norm(brasa_cmd *cmd, brasa_arg x, brasa_arg y, brasa_arg wy, brasa_arg x_out, brasa_arg w, brasa_arg out, uint32_t rows, uint32_t n,
+                             float eps) {
+    if (!cmd) return BRASA_EINVAL;
+    brasa_ctx *ctx = cmd->ctx;
+    const uint64_t all = (uint64_t)rows * n * 4, one = (uint64_t)n * 4;
+    BRASA_REQUIRE(ctx, n > 0 && arg_fits(x, all) && (!y.buf || (arg_fits(y, all) && arg_fits(wy, one))) && (!x_out.buf || arg_fits(x_out, all)) &&
+                           (!w.buf || arg_fits(w, one)) && (!out.buf || arg_fits(out, all)),
+                  "add_rms_norm: a buffer is too small");
+    for (const brasa_arg *a : {&x, &y, &wy, &x_out, &w, &out}) BRASA_REQUIRE(ctx, a->offset % 16 == 0, "add_rms_norm: misaligned buffer");
+    return brasa_add_rms_norm_launch(cmd, (const float *)arg_ptr(x), (const float *)arg_ptr(y), (const float *)arg_ptr(wy), (float *)arg_ptr(x_out), (const float *)arg_ptr(w),
+                                     arg_ptr(out), nullptr, rows, n, n, eps, true);
 }
 
 int32_t brasa_k_add(brasa_cmd *cmd, brasa_arg a, brasa_arg b, brasa_arg out, uint64_t n) {

@@ -1,11 +1,12 @@
-// Prefill attention inside a sliding window over keys in two parts (window_attn.h): score = (q_u . k_head + rot(q_r) . k_shared)
-// * scale, softmax over the visible keys, output times sigmoid(gate of the head).
+// Prefill attention inside a sliding window (window_attn.h): score = (q_own . k_head + q_shared . k_shared) * scale, optionally
+// softcapped, softmax over the visible keys, output times sigmoid(gate of the head).
 //
 // window_tc_kernel (bf16, tcgen05): one CTA = 128 queries of one head, 128-key tiles from the first tile its window touches.
 // Warp 8 (one lane) fetches K, shared-K and V tiles by TMA and issues every product; warps 0-7 are the softmax, two threads
 // per query row. S of tile j + 1 is computed while the probabilities of tile j are formed. The probabilities enter P V out
 // of tensor memory as two bf16 terms (hi + lo), so the weights keep 16 significant bits and more. One sweep over the keys: a row's
-// reference value moves only when a tile exceeds it by more than 8 ln 2, as in the causal kernel of flash_tc.cu.
+// reference value moves only when a tile exceeds it by more than 8 ln 2, as in the causal kernel of flash_tc.cu. Softcapped
+// scores are bounded, so their reference value is 0 throughout: one look at the scores, no maxima, nothing is ever rescaled.
 // window_simt_kernel<T>: the same in f32 FMA, for the 32-bit mode and for sizes TMA cannot address.
 #include "tc_device.cuh"
 #include "window_attn.h"
@@ -42,25 +43,28 @@ __global__ void __launch_bounds__(256) window_simt_kernel(WindowAttn a) {
         if (t0 + t < a.tokens) {
             const float *q = a.q + (size_t)(t0 + t) * a.ldq + h * dq;
             const uint32_t p = a.pos0 + t0 + t;
-            v = e < a.dim ? q[e] : rotated(q + a.dim, e - a.dim, a.rot_dims, a.cos_t + (size_t)p * half, a.sin_t + (size_t)p * half);
+            const float *ct = a.cos_t + (size_t)p * half, *st = a.sin_t + (size_t)p * half;
+            if (a.rot == 0) v = rotated(q, e, a.rot_dims, ct, st);
+            else v = e < a.dim ? q[e] : rotated(q + a.dim, e - a.dim, a.rot_dims, ct, st);
         }
         qs[i] = v;
     }
     float acc[SIMT_VMAX] = {}, m = -INFINITY, lsum = 0.0f;
     const uint32_t first = a.pos0 + t0, last = a.pos0 + min(t0 + SQ, a.tokens) - 1, lo = max(a.key0, first + 1 > a.window ? first + 1 - a.window : 0u);
-    const uint32_t pos = a.pos0 + t0 + qi;
+    const uint32_t pos = a.pos0 + t0 + qi, kvh = h / (a.heads / a.kv_heads);
+    auto row_of = [&](uint32_t p) { return (size_t)(a.ring ? p % a.ring : p - a.key0); };
     for (uint32_t j0 = lo; j0 <= last; j0 += SKT) {
         __syncthreads();
         for (uint32_t i = tid; i < SKT * dq; i += 256) {
-            const uint32_t j = i / dq, e = i - j * dq, row = j0 + j - a.key0;
+            const uint32_t j = i / dq, e = i - j * dq;
             float v = 0.0f;
-            if (row < a.keys)
-                v = e < a.dim ? elem_load((const T *)a.k + (size_t)row * a.ldk + h * a.dim + e) : elem_load((const T *)a.kr + (size_t)row * a.ldr + e - a.dim);
+            if (j0 + j <= last)
+                v = e < a.dim ? elem_load((const T *)a.k + row_of(j0 + j) * a.ldk + kvh * a.kstep + e) : elem_load((const T *)a.kr + row_of(j0 + j) * a.ldr + e - a.dim);
             ks[j * ldk + e] = v;
         }
         for (uint32_t i = tid; i < SKT * a.vdim; i += 256) {
-            const uint32_t j = i / a.vdim, e = i - j * a.vdim, row = j0 + j - a.key0;
-            vs[i] = row < a.keys ? elem_load((const T *)a.v + (size_t)row * a.ldv + h * a.vdim + e) : 0.0f;
+            const uint32_t j = i / a.vdim, e = i - j * a.vdim;
+            vs[i] = j0 + j <= last ? elem_load((const T *)a.v + row_of(j0 + j) * a.ldv + kvh * a.vstep + e) : 0.0f;
         }
         __syncthreads();
         float s[2] = {0.0f, 0.0f};
@@ -72,7 +76,9 @@ __global__ void __launch_bounds__(256) window_simt_kernel(WindowAttn a) {
         float mx = -INFINITY;
         for (int u = 0; u < 2; ++u) {
             const uint32_t j = j0 + l + 16 * u;
-            s[u] = (j <= pos && pos - j < a.window) ? s[u] * a.scale : -INFINITY;
+            s[u] *= a.scale;
+            if (a.softcap > 0.0f) s[u] = a.softcap * tanhf(s[u] / a.softcap);
+            if (j > pos || pos - j >= a.window) s[u] = -INFINITY;
             mx = fmaxf(mx, s[u]);
         }
 #pragma unroll
@@ -101,7 +107,7 @@ __global__ void __launch_bounds__(256) window_simt_kernel(WindowAttn a) {
         __syncwarp();
     }
     if (t0 + qi < a.tokens) {
-        const float g = 1.0f / (1.0f + expf(-a.gate[(size_t)(t0 + qi) * a.ldg + h])) / lsum;
+        const float g = (a.gate ? 1.0f / (1.0f + expf(-a.gate[(size_t)(t0 + qi) * a.ldg + h])) : 1.0f) * a.out_scale / lsum;
 #pragma unroll
         for (int i = 0; i < SIMT_VMAX; ++i) {
             const uint32_t e = l + 16 * i;
@@ -129,7 +135,24 @@ __device__ __forceinline__ void split_bf16(float p0, float p1, uint32_t &hi, uin
     lo = bf16_pack(p0 - bf16_lo(hi), p1 - bf16_hi(hi));
 }
 
-// NU, NR: 64-column blocks of the unrotated and the rotated key part; NV: of the values
+// The exponential of four softcapped scores, in powers of two: with u = s * c2 (c2 = 2 log2(e) scale / cap) it is
+// 2^(capl (1 - 2 / (1 + 2^u))), capl = cap log2(e). One reciprocal serves all four; past u = 29 the tanh is 1 in f32.
+__device__ __forceinline__ void capped_exp4(float s[4], float c2, float capl) {
+    float a[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) a[i] = 1.0f + ex2(fminf(s[i] * c2, 29.0f));
+    const float p01 = a[0] * a[1], p23 = a[2] * a[3];
+    float r;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(p01 * p23));
+    const float r01 = r * p23, r23 = r * p01, m = -2.0f * capl;
+    s[0] = ex2(fmaf(m, r01 * a[1], capl));
+    s[1] = ex2(fmaf(m, r01 * a[0], capl));
+    s[2] = ex2(fmaf(m, r23 * a[3], capl));
+    s[3] = ex2(fmaf(m, r23 * a[2], capl));
+}
+constexpr float CAP_MAX = 64.0f;  // e^cap times the number of keys stays inside f32 up to here
+
+// NU, NR: 64-column blocks of a key's own and its shared part (0: none); NV: of the values
 template <int NU, int NR, int NV>
 struct WinShape {
     static constexpr uint32_t NQ = NU + NR;
@@ -137,7 +160,7 @@ struct WinShape {
     static constexpr size_t SMEM = (size_t)(NQ + KBUF * NQ + 2 * NV) * BLK + 1024;
 };
 
-template <int NU, int NR, int NV>
+template <int NU, int NR, int NV, bool CAP>
 __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant__ WinMaps maps, WindowAttn a, uint32_t *status) {
     constexpr uint32_t NQ = NU + NR, KBUF = WinShape<NU, NR, NV>::KBUF;
     extern __shared__ __align__(1024) uint8_t smem_raw[];
@@ -153,7 +176,8 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
     const uint32_t qfirst = a.pos0 + q0, qlast = qfirst + nq - 1;
     // key tiles count from key0; the first visible position of the first query opens the sweep
     const uint32_t lo = max(a.key0, qfirst + 1 > a.window ? qfirst + 1 - a.window : 0u);
-    const uint32_t jbeg = (lo - a.key0) / 128, nkt = (qlast - a.key0) / 128 + 1 - jbeg;
+    const uint32_t jbeg = (lo - a.key0) / 128, nkt = (qlast - a.key0) / 128 + 1 - jbeg, kvh = h / (a.heads / a.kv_heads);
+    auto tile_row = [&](uint32_t j) { return (int)(a.ring ? (a.key0 + (jbeg + j) * 128) % a.ring : (jbeg + j) * 128); };
 
     if (tid == 256) {  // the issuing thread, which asks for the first tiles before the block meets
         for (int i = 0; i < 2; ++i) {
@@ -174,10 +198,10 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
     uint32_t inflight = 0;  // issuing thread: bit b = a K copy into buffer b, bit 2 + b = a V copy, not yet waited for
     auto fetch_k = [&](uint32_t j) {
         const uint32_t b = KBUF == 2 ? (j & 1) : 0u;
-        const int row = (int)((jbeg + j) * 128);
+        const int row = tile_row(j);
         mbar_expect_tx(&bar_k[b], NQ * BLK);
 #pragma unroll
-        for (int i = 0; i < NU; ++i) tma_load_3d(KB(j) + i * BLK, &maps.k, i * 64, (int)h, row, &bar_k[b]);
+        for (int i = 0; i < NU; ++i) tma_load_3d(KB(j) + i * BLK, &maps.k, i * 64, (int)kvh, row, &bar_k[b]);
 #pragma unroll
         for (int i = 0; i < NR; ++i) tma_load_2d(KB(j) + (NU + i) * BLK, &maps.kr, i * 64, row, &bar_k[b]);
         inflight |= 1u << b;
@@ -185,7 +209,7 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
     auto fetch_v = [&](uint32_t j) {
         mbar_expect_tx(&bar_v[j & 1], NV * BLK);
 #pragma unroll
-        for (int i = 0; i < NV; ++i) tma_load_3d(VB(j) + i * BLK, &maps.v, i * 64, (int)h, (int)((jbeg + j) * 128), &bar_v[j & 1]);
+        for (int i = 0; i < NV; ++i) tma_load_3d(VB(j) + i * BLK, &maps.v, i * 64, (int)kvh, tile_row(j), &bar_v[j & 1]);
         inflight |= 4u << (j & 1);
     };
     if (tid == 256) {
@@ -196,6 +220,7 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
     // Q tile: rotated, rounded to bf16, swizzled K-major; rows past the last query and columns past the sizes are zeros
     const uint32_t half = a.rot_dims / 2;
     const bool qvec = ((a.ldq | dq | a.dim) & 3) == 0, rvec = (half & 7) == 0;
+    const uint32_t own_rot = NR == 0 ? a.rot_dims : 0u;  // rotated columns of the own part
     for (uint32_t i = tid; i < 128 * NQ * 8; i += 288) {
         const uint32_t r = i / (NQ * 8), c = i - r * (NQ * 8), blk = c >> 3, c8 = (c & 7) * 8;
         uint32_t w[4] = {0, 0, 0, 0};
@@ -204,14 +229,14 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
             const uint32_t p = qfirst + r;
             const float *ct = a.cos_t + (size_t)p * half, *st = a.sin_t + (size_t)p * half;
             float v[8];
-            if (qvec && blk < NU && blk * 64 + c8 + 8 <= a.dim) {
+            if (qvec && blk < NU && blk * 64 + c8 >= own_rot && blk * 64 + c8 + 8 <= a.dim) {
                 const float4 x = *reinterpret_cast<const float4 *>(q + blk * 64 + c8), y = *reinterpret_cast<const float4 *>(q + blk * 64 + c8 + 4);
                 v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
                 v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
-            } else if (qvec && rvec && blk >= NU && (blk - NU) * 64 + c8 + 8 <= a.rot_dims) {
+            } else if (qvec && rvec && (blk >= NU || NR == 0) && (blk - (NR ? NU : 0)) * 64 + c8 + 8 <= a.rot_dims) {
                 // eight neighbours of one half of the pairs
-                const uint32_t e0 = (blk - NU) * 64 + c8, f0 = e0 < half ? e0 : e0 - half;
-                const float *own = q + a.dim + e0, *other = e0 < half ? own + half : own - half;
+                const uint32_t e0 = (blk - (NR ? NU : 0)) * 64 + c8, f0 = e0 < half ? e0 : e0 - half;
+                const float *own = q + (NR ? a.dim : 0) + e0, *other = e0 < half ? own + half : own - half;
                 const float sign = e0 < half ? -1.0f : 1.0f;
 #pragma unroll
                 for (int u = 0; u < 8; u += 4) {
@@ -226,7 +251,8 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
 #pragma unroll
             for (int e = 0; e < 8; ++e) {
                 const uint32_t col = (blk < NU ? blk : blk - NU) * 64 + c8 + e;
-                if (blk < NU) v[e] = col < a.dim ? q[col] : 0.0f;
+                if (NR == 0) v[e] = col < a.dim ? rotated(q, col, a.rot_dims, ct, st) : 0.0f;
+                else if (blk < NU) v[e] = col < a.dim ? q[col] : 0.0f;
                 else v[e] = col < a.rot ? rotated(q + a.dim, col, a.rot_dims, ct, st) : 0.0f;
             }
 #pragma unroll
@@ -262,7 +288,7 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
     const bool issuer = tid == 256, softmax = tid < 256;
     const uint32_t row = (warp & 3) * 32 + lane, cgrp = (warp >> 2) & 1, c0 = cgrp * 64, trow = ((warp & 3) * 32u) << 16;
     const uint32_t qpos = qfirst + row;
-    const float sl = a.scale * LOG2E;
+    const float sl = a.scale * LOG2E, c2 = CAP ? 2.0f * sl / a.softcap : 0.0f, capl = a.softcap * LOG2E;
     float m = -INFINITY, l = 0.0f;  // reference value and row sum, in powers of two of the scaled score
     uint32_t phs = 0, phk = 0, phv = 0, ph_o = 0;  // bit b: parity of buffer b's barrier
     bool ok = true;
@@ -311,6 +337,27 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
             const bool free_tile = k0 + 127 <= qfirst && k0 + a.window > qfirst + 127;
             // a key of column c is visible when lob <= c <= hib
             const int hib = (int)qpos - (int)(k0 + c0), lob = hib - (int)a.window + 1;
+            if constexpr (CAP) {
+#pragma unroll
+                for (int cc = 0; cc < 2; ++cc) {
+                    uint32_t v[32];
+                    tc_ld32(ts + 32 * cc, v);
+#pragma unroll
+                    for (int i = 0; i < 32; i += 4) {
+                        float p[4];
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) p[e] = __uint_as_float(v[i + e]);
+                        capped_exp4(p, c2, capl);
+                        if (!free_tile)
+#pragma unroll
+                            for (int e = 0; e < 4; ++e)
+                                if (32 * cc + i + e > hib || 32 * cc + i + e < lob) p[e] = 0.0f;
+                        l += (p[0] + p[1]) + (p[2] + p[3]);
+                        split_bf16(p[0], p[1], hi[16 * cc + i / 2], lo_[16 * cc + i / 2]);
+                        split_bf16(p[2], p[3], hi[16 * cc + i / 2 + 1], lo_[16 * cc + i / 2 + 1]);
+                    }
+                }
+            } else {
             float tmax = -INFINITY;
 #pragma unroll
             for (int cc = 0; cc < 2; ++cc) {
@@ -351,6 +398,7 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
                     split_bf16(p0, p1, hi[16 * cc + i / 2], lo_[16 * cc + i / 2]);
                 }
             }
+            }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
         }
         if (ok && j > 0) {  // P and the other V buffer are free once P V of tile j - 1 has finished
@@ -361,7 +409,7 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
         if (ok && issuer && j + 1 < nkt) fetch_v(j + 1);
         if (ok && softmax) {
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            if (j > 0 && __any_sync(0xffffffffu, move)) {
+            if (!CAP && j > 0 && __any_sync(0xffffffffu, move)) {
                 // a row's reference moved: what O holds for it was accumulated against the old one; each thread of the pair
                 // scales its half of the value columns
 #pragma unroll 1
@@ -408,7 +456,7 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
         if (softmax) {
             const float total = pair_max[0][row] + pair_max[1][row];
             float g = 0.0f;
-            if (row < nq) g = 1.0f / (1.0f + expf(-a.gate[(size_t)(q0 + row) * a.ldg + h])) / total;
+            if (row < nq) g = (a.gate ? 1.0f / (1.0f + expf(-a.gate[(size_t)(q0 + row) * a.ldg + h])) : 1.0f) * a.out_scale / total;
             __nv_bfloat16 *dst = (__nv_bfloat16 *)a.out + (size_t)(q0 + row) * a.ldo + h * a.vdim;
             const bool vec = ((a.ldo | a.vdim) & 7) == 0;
 #pragma unroll 1
@@ -448,21 +496,32 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
     }
 }
 
-template <int NU, int NR, int NV>
+template <int NU, int NR, int NV, bool CAP>
 int32_t launch_window_tc(brasa_cmd *cmd, const WindowAttn &a) {
     brasa_ctx *ctx = cmd->ctx;
     WinMaps maps;
-    const uint64_t kd[3] = {a.dim, a.heads, a.keys}, kst[2] = {(uint64_t)a.dim * 2, (uint64_t)a.ldk * 2};
-    const uint64_t vd[3] = {a.vdim, a.heads, a.keys}, vst[2] = {(uint64_t)a.vdim * 2, (uint64_t)a.ldv * 2};
-    const uint64_t rd[2] = {a.rot, a.keys}, rst[1] = {(uint64_t)a.ldr * 2};
+    // (columns between a head's size and its step are never read: they lie outside the map, or the query tile has zeros there
+    // and the output leaves them out)
+    const uint64_t rows = a.ring ? a.ring : a.keys;
+    const uint64_t kd[3] = {(a.dim + 7) / 8 * 8, a.kv_heads, rows}, kst[2] = {(uint64_t)a.kstep * 2, (uint64_t)a.ldk * 2};
+    const uint64_t vd[3] = {(a.vdim + 7) / 8 * 8, a.kv_heads, rows}, vst[2] = {(uint64_t)a.vstep * 2, (uint64_t)a.ldv * 2};
     const uint32_t box3[3] = {64, 1, 128}, box2[2] = {64, 128};
     BRASA_TRY(brasa_tmap_bf16(ctx, &maps.k, 3, a.k, kd, kst, box3));
     BRASA_TRY(brasa_tmap_bf16(ctx, &maps.v, 3, a.v, vd, vst, box3));
-    BRASA_TRY(brasa_tmap_bf16(ctx, &maps.kr, 2, a.kr, rd, rst, box2));
+    maps.kr = maps.k;
+    if (NR) {
+        const uint64_t rd[2] = {a.rot, rows}, rst[1] = {(uint64_t)a.ldr * 2};
+        BRASA_TRY(brasa_tmap_bf16(ctx, &maps.kr, 2, a.kr, rd, rst, box2));
+    }
     const size_t smem = WinShape<NU, NR, NV>::SMEM;
-    BRASA_TRY(brasa_smem_optin(ctx, (const void *)window_tc_kernel<NU, NR, NV>, smem));
-    BRASA_CUDA(ctx, brasa_launch_dependent(ctx, window_tc_kernel<NU, NR, NV>, dim3((a.tokens + 127) / 128, a.heads), dim3(288), smem, maps, a, ctx->status));
+    BRASA_TRY(brasa_smem_optin(ctx, (const void *)window_tc_kernel<NU, NR, NV, CAP>, smem));
+    BRASA_CUDA(ctx, brasa_launch_dependent(ctx, window_tc_kernel<NU, NR, NV, CAP>, dim3((a.tokens + 127) / 128, a.heads), dim3(288), smem, maps, a, ctx->status));
     return brasa_post_launch(cmd, "window_tc");
+}
+
+template <int NU, int NV>
+int32_t launch_window_own(brasa_cmd *cmd, const WindowAttn &a) {
+    return a.softcap > 0.0f ? launch_window_tc<NU, 0, NV, true>(cmd, a) : launch_window_tc<NU, 0, NV, false>(cmd, a);
 }
 
 template <typename T>
@@ -479,18 +538,31 @@ int32_t launch_window_simt(brasa_cmd *cmd, const WindowAttn &a) {
 }  // namespace
 
 int32_t brasa_window_attention_launch(brasa_cmd *cmd, const WindowAttn &a, bool f32) {
-    BRASA_REQUIRE(cmd->ctx, a.tokens > 0 && a.heads > 0 && a.window > 0 && a.key0 <= a.pos0 && a.key0 + a.keys == a.pos0 + a.tokens && a.rot_dims <= a.rot &&
+    BRASA_REQUIRE(cmd->ctx, a.tokens > 0 && a.heads > 0 && a.window > 0 && a.key0 <= a.pos0 && a.key0 + a.keys == a.pos0 + a.tokens && (a.rot == 0 || a.rot_dims <= a.rot) &&
                                 a.rot_dims % 2 == 0,
                   "window attention: bad range or sizes");
+    BRASA_REQUIRE(cmd->ctx, a.kv_heads > 0 && a.heads % a.kv_heads == 0 && a.kstep >= a.dim && a.vstep >= a.vdim && (a.rot > 0 || a.rot_dims <= a.dim) && a.softcap >= 0.0f,
+                  "window attention: bad heads or steps");
+    BRASA_REQUIRE(cmd->ctx, !a.ring || (a.ring % 128 == 0 && a.key0 % 128 == 0), "window attention: a ring and its first key are multiples of 128");
     if (f32) return launch_window_simt<float>(cmd, a);
     const uint32_t nu = (a.dim + 63) / 64, nr = (a.rot + 63) / 64, nv = (a.vdim + 63) / 64;
-    if (((a.dim | a.vdim | a.ldk | a.ldv | a.ldr) & 7) == 0 && nr == 1) {
-        if (nu == 1 && nv == 1) return launch_window_tc<1, 1, 1>(cmd, a);
-        if (nu == 1 && nv == 2) return launch_window_tc<1, 1, 2>(cmd, a);
-        if (nu == 2 && nv == 1) return launch_window_tc<2, 1, 1>(cmd, a);
-        if (nu == 2 && nv == 2) return launch_window_tc<2, 1, 2>(cmd, a);
-        if (nu == 3 && nv == 1) return launch_window_tc<3, 1, 1>(cmd, a);
-        if (nu == 3 && nv == 2) return launch_window_tc<3, 1, 2>(cmd, a);
+    if (((a.kstep | a.vstep | a.ldk | a.ldv | a.ldr) & 7) == 0) {
+        if (nr == 1 && a.softcap == 0.0f) {
+            if (nu == 1 && nv == 1) return launch_window_tc<1, 1, 1, false>(cmd, a);
+            if (nu == 1 && nv == 2) return launch_window_tc<1, 1, 2, false>(cmd, a);
+            if (nu == 2 && nv == 1) return launch_window_tc<2, 1, 1, false>(cmd, a);
+            if (nu == 2 && nv == 2) return launch_window_tc<2, 1, 2, false>(cmd, a);
+            if (nu == 3 && nv == 1) return launch_window_tc<3, 1, 1, false>(cmd, a);
+            if (nu == 3 && nv == 2) return launch_window_tc<3, 1, 2, false>(cmd, a);
+        }
+        if (nr == 0 && a.softcap <= CAP_MAX) {
+            if (nu == 1 && nv == 1) return launch_window_own<1, 1>(cmd, a);
+            if (nu == 1 && nv == 2) return launch_window_own<1, 2>(cmd, a);
+            if (nu == 2 && nv == 1) return launch_window_own<2, 1>(cmd, a);
+            if (nu == 2 && nv == 2) return launch_window_own<2, 2>(cmd, a);
+            if (nu == 3 && nv == 1) return launch_window_own<3, 1>(cmd, a);
+            if (nu == 3 && nv == 2) return launch_window_own<3, 2>(cmd, a);
+        }
     }
     return launch_window_simt<__nv_bfloat16>(cmd, a);
 }
@@ -498,13 +570,16 @@ int32_t brasa_window_attention_launch(brasa_cmd *cmd, const WindowAttn &a, bool 
 extern "C" int32_t brasa_k_window_attention(brasa_cmd *cmd, brasa_window_attn p, int32_t f32) {
     if (!cmd) return BRASA_EINVAL;
     brasa_ctx *ctx = cmd->ctx;
-    BRASA_REQUIRE(ctx, p.tokens > 0 && p.heads > 0 && p.dim > 0 && p.rot > 0 && p.vdim > 0 && p.window > 0 && p.key0 <= p.pos0, "window attention: empty shape");
-    BRASA_REQUIRE(ctx, p.rot % 8 == 0 && (p.key0 == 0 || p.key0 + p.window <= p.pos0 + 1), "window attention: rot must be a multiple of 8 and every visible key present");
-    const uint64_t keys = (uint64_t)p.pos0 + p.tokens - p.key0, e = f32 ? 4 : 2, last = (uint64_t)p.pos0 + p.tokens;
-    BRASA_REQUIRE(ctx, arg_fits(p.q, (uint64_t)p.tokens * p.heads * (p.dim + p.rot) * 4) && arg_fits(p.k, keys * p.heads * p.dim * e) &&
-                           arg_fits(p.v, keys * p.heads * p.vdim * e) && arg_fits(p.kr, keys * p.rot * e) && arg_fits(p.gate, (uint64_t)p.tokens * p.heads * 4) &&
-                           arg_fits(p.out, (uint64_t)p.tokens * p.heads * p.vdim * e) && arg_fits(p.cos_t, last * (p.rot_dims / 2) * 4) &&
-                           arg_fits(p.sin_t, last * (p.rot_dims / 2) * 4),
+    BRASA_REQUIRE(ctx, p.tokens > 0 && p.heads > 0 && p.dim > 0 && p.vdim > 0 && p.window > 0 && p.key0 <= p.pos0 && p.kv_heads > 0 && p.heads % p.kv_heads == 0,
+                  "window attention: empty shape");
+    BRASA_REQUIRE(ctx, p.rot % 8 == 0 && p.rot_dims <= (p.rot ? p.rot : p.dim) && (p.key0 == 0 || p.key0 + p.window <= p.pos0 + 1),
+                  "window attention: rot must be a multiple of 8 and every visible key present");
+    const uint64_t keys = (uint64_t)p.pos0 + p.tokens - p.key0, e = f32 ? 4 : 2, last = (uint64_t)p.pos0 + p.tokens, rows = p.ring ? p.ring : keys;
+    BRASA_REQUIRE(ctx, !p.ring || std::min<uint64_t>(p.window - 1, p.pos0) + p.tokens <= p.ring, "window attention: the ring is shorter than the window and the run");
+    BRASA_REQUIRE(ctx, arg_fits(p.q, (uint64_t)p.tokens * p.heads * (p.dim + p.rot) * 4) && arg_fits(p.k, rows * p.kv_heads * p.dim * e) &&
+                           arg_fits(p.v, rows * p.kv_heads * p.vdim * e) && (!p.rot || arg_fits(p.kr, rows * p.rot * e)) &&
+                           (!p.gate.buf || arg_fits(p.gate, (uint64_t)p.tokens * p.heads * 4)) && arg_fits(p.out, (uint64_t)p.tokens * p.heads * p.vdim * e) &&
+                           arg_fits(p.cos_t, last * (p.rot_dims / 2) * 4) && arg_fits(p.sin_t, last * (p.rot_dims / 2) * 4),
                   "window attention: a buffer is too small");
     for (const brasa_arg *a : {&p.k, &p.v, &p.kr, &p.out}) BRASA_REQUIRE(ctx, a->offset % 16 == 0, "window attention: misaligned buffer");
     WindowAttn a{};
@@ -517,12 +592,17 @@ extern "C" int32_t brasa_k_window_attention(brasa_cmd *cmd, brasa_window_attn p,
     a.gate = (const float *)arg_ptr(p.gate);
     a.out = arg_ptr(p.out);
     a.ldq = p.heads * (p.dim + p.rot);
-    a.ldk = p.heads * p.dim;
-    a.ldv = a.ldo = p.heads * p.vdim;
+    a.ldk = p.kv_heads * p.dim;
+    a.ldv = p.kv_heads * p.vdim;
+    a.ldo = p.heads * p.vdim;
     a.ldr = p.rot;
     a.ldg = p.heads;
     a.tokens = p.tokens; a.heads = p.heads; a.dim = p.dim; a.rot = p.rot; a.rot_dims = p.rot_dims; a.vdim = p.vdim;
     a.pos0 = p.pos0; a.key0 = p.key0; a.keys = (uint32_t)keys; a.window = p.window;
     a.scale = p.scale;
+    a.kv_heads = p.kv_heads; a.kstep = p.dim; a.vstep = p.vdim;
+    a.ring = p.ring;
+    a.softcap = p.softcap;
+    a.out_scale = p.out_scale;
     return brasa_window_attention_launch(cmd, a, f32 != 0);
 }

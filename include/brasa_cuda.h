@@ -210,27 +210,40 @@ int32_t brasa_k_flash_attention(brasa_cmd *cmd, brasa_arg q, brasa_arg k, brasa_
 
 /* out[r, :] = (x[r, :] - mean) / sqrt(mean square deviation + eps) * w + b, all f32 */
 int32_t brasa_k_layer_norm(brasa_cmd *cmd, brasa_arg x, brasa_arg w, brasa_arg b, brasa_arg out, uint32_t rows, uint32_t n, float eps);
-/* y[t, r] = resid[t, r] + scale * act(w[r, :] . x[t, :] (+ w2[r, :] . x2[t, :]) + bias[r]) with bf16 row-major weights. Leading
- * dimensions in elements, multiples of 8. Optional parts have buf NULL (w2: cols2 = 0). */
-enum brasa_linear_act { BRASA_ACT_NONE = 0, BRASA_ACT_RELU2 = 1 /* relu(v)^2 */ };
+/* x' = x + y / rms(y) * wy (without y: x), x_out = x', out = x' / rms(x') * w (without w: x'), all f32, rows of n; rms(v) =
+ * sqrt(mean square + eps). Optional parts have buf NULL; x_out may be x. */
+int32_t brasa_k_add_rms_norm(brasa_cmd *cmd, brasa_arg x, brasa_arg y, brasa_arg wy, brasa_arg x_out, brasa_arg w, brasa_arg out, uint32_t rows, uint32_t n,
+                             float eps);
+/* y[t, r] = resid[t, r] + mul[mul_ids[t], r] * softcap(scale * act(w[r, :] . x[t, :] (+ w2[r, :] . x2[t, :]) + bias[r])) with bf16
+ * row-major weights; softcap(v) = cap tanh(v / cap), cap 0: none. Leading dimensions in elements, multiples of 8 (ldm: any).
+ * Optional parts have buf NULL (w2: cols2 = 0). SWIGLU: the rows are alternating blocks of 32 gate and 32 up rows, y has rows / 2
+ * columns silu(gate) * up (no bias, scale or cap). The ids must lie inside mul's mul_rows rows. */
+enum brasa_linear_act { BRASA_ACT_NONE = 0, BRASA_ACT_RELU2 = 1 /* relu(v)^2 */, BRASA_ACT_GELU_TANH = 2, BRASA_ACT_SWIGLU = 3 };
 typedef struct brasa_linear {
     brasa_arg w, x, w2, x2, y, bias, resid; /* bias f32[rows]; resid f32[tokens][ldy], may be y */
     uint32_t cols, ldw, ldx, cols2, ldw2, ldx2, rows, tokens, ldy;
     int32_t y_bf16; /* y in bf16 instead of f32 */
     int32_t act;
-    float scale;
+    float scale, cap;
+    brasa_arg mul, mul_ids; /* mul bf16 [mul_rows][ldm]; mul_ids u32[tokens] */
+    uint32_t ldm, mul_rows;
 } brasa_linear;
 /* up to 8 such products in one launch. f32_inputs 0: x in bf16, tcgen05 with f32 accumulation; 1: x in f32, f32 FMA. */
 int32_t brasa_k_linear(brasa_cmd *cmd, const brasa_linear *p, uint32_t count, int32_t f32_inputs);
 /* Attention of tokens queries at positions pos0 .. over keys at positions key0 .. pos0 + tokens - 1, each query seeing its own
- * position and the window - 1 before it. A head's key has a part of its own (dim) and one shared by all heads (rot); q f32
- * [tokens][heads][dim + rot] is rotated here (pairs i, i + rot_dims / 2 of the shared part; cos_t / sin_t f32
- * [position][rot_dims / 2]), kr comes rotated. out = softmax(scale * score) v * sigmoid(gate). k [keys][heads][dim], v
- * [keys][heads][vdim], kr [keys][rot], out [tokens][heads][vdim]: bf16, or f32 with f32 != 0; gate f32 [tokens][heads]. */
+ * position and the window - 1 before it. A head's key has a part of its own (dim) and one shared by all heads (rot, may be 0); q
+ * f32 [tokens][heads][dim + rot] is rotated here (pairs i, i + rot_dims / 2 of the shared part, or of the own part when rot is 0;
+ * cos_t / sin_t f32 [position][rot_dims / 2]), k and kr come rotated. out = softmax(cap(scale * score)) v * out_scale *
+ * sigmoid(gate), cap(s) = softcap tanh(s / softcap) (softcap 0: none; gate may have buf NULL). k [keys][kv_heads][dim], v
+ * [keys][kv_heads][vdim] (head h reads key head h / (heads / kv_heads)), kr [keys][rot], out [tokens][heads][vdim]: bf16, or f32
+ * with f32 != 0; gate f32 [tokens][heads]. ring > 0 (a multiple of 128): position p lies in row p % ring of k, v (and kr), whose
+ * other rows hold finite values. */
 typedef struct brasa_window_attn {
     brasa_arg q, k, v, kr, cos_t, sin_t, gate, out;
     uint32_t tokens, heads, dim, rot, rot_dims, vdim, pos0, key0, window;
     float scale;
+    uint32_t kv_heads, ring;
+    float softcap, out_scale;
 } brasa_window_attn;
 int32_t brasa_k_window_attention(brasa_cmd *cmd, brasa_window_attn a, int32_t f32);
 
@@ -296,7 +309,7 @@ typedef struct brasa_allocated { /* qwen3.rs:430 Allocated */
 /* BrasaFile::open + verify over a path: structure checks always, sha256 when verify != 0. */
 int32_t brasa_file_check(const char *path, int32_t verify, char *err, uint64_t err_len);
 /* path: a `.brasa` file, or a folder with config.json and model.safetensors (bf16 tensors), whose "architecture" names the
- * family. Families: "qwen3", and the layer-stack family "Dunuzen". */
+ * family. Families: "qwen3", and the layer-stack families "Dunuzen" and "Gugedra". */
 int32_t brasa_model_family(const char *path, char *name, uint64_t name_len); /* the family's name, or the reason for BRASA_EIO */
 /* The plan of a session over the model at path, any family (brasa_plan_check for brasa_plan of that family). */
 int32_t brasa_plan_file(brasa_ctx *ctx, const char *path, const brasa_session_shape *s, uint64_t budget_bytes, brasa_memory_plan *out,
@@ -322,6 +335,8 @@ int32_t brasa_model_forward_rows(brasa_model *m, const uint32_t *ids, uint32_t t
                                  double *gpu_seconds);
 /* Qwen3::run_layers :743. x: host f32[tokens*hidden], replaced by the output. */
 int32_t brasa_model_run_layers(brasa_model *m, float *x, uint32_t tokens, uint32_t pos0, uint32_t layer_begin, uint32_t layer_end);
+/* The same with the tokens' ids, for families whose layers read them too (the other call refuses those). */
+int32_t brasa_model_run_layers_ids(brasa_model *m, const uint32_t *ids, float *x, uint32_t tokens, uint32_t pos0, uint32_t layer_begin, uint32_t layer_end);
 /* Device-resident decode: feeds the token chosen on the device back as the next input for `steps`
  * greedy steps starting from `first` at position pos0, without host round trips; out_ids: host
  * u32[steps] read once at the end. Used for the HBM-resident throughput figure. */
