@@ -23,7 +23,8 @@ tokens with an f16 KV cache, ctx 2048. One step = the 255 decode forwards that f
 `tp32b`   the Qwen3-32B architecture decoded tensor-parallel over all ranks of the job (batch 1 and batch 16), with a
           split-versus-unsplit parity check on a reduced model; at one rank the whole model runs on one GPU.
 
---dunuzen times prefill and decode of Dunuzen models (bf16) at a few sizes beside Qwen3 models of equal size, and nothing else.
+--dunuzen and --gugedra time prefill and decode of those models (bf16) at a few sizes beside Qwen3 and Dunuzen models of equal
+size, and nothing else.
 
 With --gpus N > 1 (launched by torch.distributed.run) every rank serves its own replica: the path has
 no exchange step at batch 1, so the ranks share nothing and the aggregate is the sum ("replicas only").
@@ -794,40 +795,47 @@ def kernel_roofline(B, ctx, K, cfg, peak, peak_kind, profile=False):
     return roof
 
 
-# --dunuzen: layers of a real model's size, random weights, beside a Qwen3 model of the same width, FFN, heads and depth
-DUNUZEN_SIZES = {"2048": dict(width=2048, ff=8192, heads=16, kv_heads=16, window=1024),
-                 "2560": dict(width=2560, ff=9728, heads=32, kv_heads=16, window=1024),
-                 "4096": dict(width=4096, ff=14336, heads=32, kv_heads=32, window=4096)}
-DUNUZEN_LAYERS, DUNUZEN_VOCAB = ["latent_attention", "channel_delta"] * 4, 32768
+# --dunuzen, --gugedra: layer-stack models with layers of a real model's size and random weights, beside a model of the same width,
+# FFN width, heads, window and depth: Dunuzen beside Qwen3, Gugedra beside Dunuzen
+STACK_SIZES = {"2048": dict(width=2048, ff=8192, heads=16, kv_heads=16, window=1024),
+               "2560": dict(width=2560, ff=9728, heads=32, kv_heads=16, window=1024),
+               "4096": dict(width=4096, ff=14336, heads=32, kv_heads=32, window=4096)}
+STACK_VOCAB = 32768
+STACK_LAYERS = {"dunuzen": ["latent_attention", "channel_delta"] * 4, "gugedra": ["parallel", "delta"] * 4}
 
 
-def dunuzen_leg(B, ctx, tag: str, steps: int, warmup: int, tokens: int = 4096, decode: int = 128, models=("dunuzen", "qwen3"), chunk: int = 2048) -> dict:
-    """Prefill of `tokens` tokens and greedy decode behind them, for a Dunuzen model (bf16) and a Qwen3 model (q4_0, f16 cache)
-    of equal width, FFN width, heads and depth. Device time; every decode step reads more weights than L2 holds."""
+def stack_model(ctx, name: str, tag: str, tokens: int):
+    """(path, operations of the prompt, bytes of a decode step as a function of its position) of a synthetic model."""
     from brasa_b200 import synth
-    size = DUNUZEN_SIZES[tag]
+    size = STACK_SIZES[tag]
+    if name == "qwen3":
+        cfg = dict(synth.QWEN3_4B, hidden_size=size["width"], intermediate_size=size["ff"], num_attention_heads=size["heads"],
+                   num_hidden_layers=len(STACK_LAYERS["dunuzen"]), vocab_size=STACK_VOCAB)
+        path = model_path(f"qwen3-like-dunuzen-{tag}")
+        if not path.exists():
+            synth.write_synthetic_model(ctx, path, cfg, SEED)
+        mm = sum(2 * tokens * int(np.prod(sh)) for n, sh in synth.tensor_shapes(cfg).items() if len(sh) == 2 and "embed" not in n)
+        flops = {"matmul": mm, "attention": 4 * tokens * (tokens + 1) // 2 * cfg["num_attention_heads"] * 128 * cfg["num_hidden_layers"]}
+        return path, flops, lambda p: synth.weight_bytes_per_token(cfg) + synth.kv_bytes_per_position(cfg) * (p + 1)
+    make, shapes, fl, by = {"dunuzen": (synth.dunuzen_config, synth.dunuzen_shapes, synth.dunuzen_prefill_flops, synth.dunuzen_decode_bytes),
+                            "gugedra": (synth.gugedra_config, synth.gugedra_shapes, synth.gugedra_prefill_flops, synth.gugedra_decode_bytes)}[name]
+    cfg = make(layers=STACK_LAYERS[name], vocab=STACK_VOCAB, **size)
+    path = model_path(f"{name}-{tag}").with_suffix("")
+    if not (path / "config.json").exists():
+        synth.write_synthetic_stack(path, cfg, shapes(cfg), SEED)
+    return path, fl(cfg, tokens), lambda p: by(cfg, p)
+
+
+def stack_leg(B, ctx, tag: str, steps: int, warmup: int, models, tokens: int = 4096, decode: int = 128, chunk: int = 2048) -> dict:
+    """Prefill of `tokens` tokens and greedy decode behind them, for each of `models` (stack models in bf16, Qwen3 in q4_0 with an
+    f16 cache). Device time; every decode step reads more weights than L2 holds."""
     hbm, _ = measured_peaks()
     tc = tensor_peak() or 1590.0
-    out = {"size": size, "layers": len(DUNUZEN_LAYERS), "vocab": DUNUZEN_VOCAB, "prompt_tokens": tokens}
-    ids = np.random.default_rng(SEED).integers(0, DUNUZEN_VOCAB, size=tokens).astype(np.uint32)
+    out = {"size": STACK_SIZES[tag], "layers": len(STACK_LAYERS["dunuzen"]), "vocab": STACK_VOCAB, "prompt_tokens": tokens}
+    ids = np.random.default_rng(SEED).integers(0, STACK_VOCAB, size=tokens).astype(np.uint32)
     ctx_len = tokens + (warmup + steps + 1) * decode + 64
     for name in models:
-        if name == "dunuzen":
-            cfg = synth.dunuzen_config(layers=DUNUZEN_LAYERS, vocab=DUNUZEN_VOCAB, **size)
-            path = model_path(f"dunuzen-{tag}").with_suffix("")
-            if not (path / "config.json").exists():
-                synth.write_synthetic_dunuzen(path, cfg, SEED)
-            flops = synth.dunuzen_prefill_flops(cfg, tokens)
-            step_bytes = lambda p: synth.dunuzen_decode_bytes(cfg, p)
-        else:
-            cfg = dict(synth.QWEN3_4B, hidden_size=size["width"], intermediate_size=size["ff"], num_attention_heads=size["heads"],
-                       num_hidden_layers=len(DUNUZEN_LAYERS), vocab_size=DUNUZEN_VOCAB)
-            path = model_path(f"qwen3-like-dunuzen-{tag}")
-            if not path.exists():
-                synth.write_synthetic_model(ctx, path, cfg, SEED)
-            mm = sum(2 * tokens * int(np.prod(sh)) for n, sh in synth.tensor_shapes(cfg).items() if len(sh) == 2 and "embed" not in n)
-            flops = {"matmul": mm, "attention": 4 * tokens * (tokens + 1) // 2 * cfg["num_attention_heads"] * 128 * cfg["num_hidden_layers"]}
-            step_bytes = lambda p: synth.weight_bytes_per_token(cfg) + synth.kv_bytes_per_position(cfg) * (p + 1)
+        path, flops, step_bytes = stack_model(ctx, name, tag, tokens)
         m = B.model_class(path).load_in(ctx, path, "bfloat16", ctx_len, chunk)
 
         def prefill():
@@ -856,15 +864,14 @@ def dunuzen_leg(B, ctx, tag: str, steps: int, warmup: int, tokens: int = 4096, d
     return out
 
 
-def run_dunuzen(args) -> None:
+def run_stack(args, name: str, which: str, models) -> None:
     import brasa_b200 as B
     ctx = B.Context(0)
-    tags = list(DUNUZEN_SIZES) if args.dunuzen == "all" else args.dunuzen.split(",")
-    models = tuple(args.dunuzen_models.split(","))
+    tags = list(STACK_SIZES) if which == "all" else which.split(",")
     with ClockSampler(0) as clocks:
-        legs = {t: dunuzen_leg(B, ctx, t, args.steps, args.warmup, tokens=args.dunuzen_tokens, decode=min(128, args.decode_tokens), models=models) for t in tags}
-    first = legs[tags[0]].get("dunuzen") or legs[tags[0]]["qwen3"]
-    print(json.dumps({"metric": "dunuzen_decode_tok_s", "value": first["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+        legs = {t: stack_leg(B, ctx, t, args.steps, args.warmup, models, tokens=args.stack_tokens, decode=min(128, args.decode_tokens)) for t in tags}
+    first = legs[tags[0]].get(name) or legs[tags[0]][models[0]]
+    print(json.dumps({"metric": f"{name}_decode_tok_s", "value": first["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
                       "higher_is_better": True, "data": "synthetic", "dtype": "bf16", "config": {"sizes": tags, "l2": "weights of a step exceed L2"},
                       "clocks": clocks.summary(), "legs": legs}))
 
@@ -1141,12 +1148,15 @@ def main():
     ap.add_argument("--serving-steps", type=int, default=512)
     ap.add_argument("--only-decode", action="store_true",
                     help="run only the device-resident decode loop (profiler captures): no end-to-end, kernel or CPU legs")
-    ap.add_argument("--dunuzen", default="", help="run only the Dunuzen legs: all, or some of " + ", ".join(DUNUZEN_SIZES) + " separated by commas")
-    ap.add_argument("--dunuzen-models", default="dunuzen,qwen3", help="which models those legs run (profiler captures take one)")
-    ap.add_argument("--dunuzen-tokens", type=int, default=4096)
+    sizes = ", ".join(STACK_SIZES) + " separated by commas"
+    ap.add_argument("--dunuzen", default="", help="run only the Dunuzen legs, beside Qwen3: all, or some of " + sizes)
+    ap.add_argument("--gugedra", default="", help="run only the Gugedra legs, beside Dunuzen: all, or some of " + sizes)
+    ap.add_argument("--stack-models", default="", help="which models those legs run, separated by commas (profiler captures take one)")
+    ap.add_argument("--stack-tokens", type=int, default=4096)
     args = ap.parse_args()
-    if args.dunuzen:
-        return run_dunuzen(args)
+    for name, which, beside in (("dunuzen", args.dunuzen, "qwen3"), ("gugedra", args.gugedra, "dunuzen")):
+        if which:
+            return run_stack(args, name, which, args.stack_models.split(",") if args.stack_models else [name, beside])
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))

@@ -136,7 +136,7 @@ def kv_bytes_per_position(cfg: dict, kv: str = "f16") -> int:
     return rows * {"f32": 512, "f16": 256, "q8_0": 136}[kv]
 
 
-# ---- Dunuzen: config.json + model.safetensors with seeded bf16 weights, drawn on the host --------------------------------
+# ---- layer-stack models: config.json + model.safetensors with seeded bf16 weights, drawn on the host ---------------------
 
 
 def dunuzen_config(width: int, ff: int, heads: int, kv_heads: int, layers: list[str], vocab: int, window: int, dim: int = 128, rot_dim: int = 64,
@@ -171,13 +171,12 @@ def dunuzen_shapes(cfg: dict, rank: int = 128) -> dict[str, list[int]]:
     return t
 
 
-def write_synthetic_dunuzen(folder, cfg: dict, seed: int = 0, std: float = 0.02, rank: int = 128) -> None:
+def write_synthetic_stack(folder, cfg: dict, shapes: dict[str, list[int]], seed: int = 0, std: float = 0.02) -> None:
     """Seeded N(0, std) matrices, norm weights of ones, biases of zeros; drawn and rounded tensor by tensor in parallel."""
     import concurrent.futures
     import os
     folder = pathlib.Path(folder)
     folder.mkdir(parents=True, exist_ok=True)
-    shapes = dunuzen_shapes(cfg, rank)
     header, at = {}, 0
     for name, shape in shapes.items():
         n = 2 * int(np.prod(shape))
@@ -189,7 +188,7 @@ def write_synthetic_dunuzen(folder, cfg: dict, seed: int = 0, std: float = 0.02,
     def draw(item):
         i, (name, shape) = item
         if len(shape) == 1:
-            w = np.full(shape, 1.0 if "norm" in name and not name.endswith(".b") else 0.0, np.float32)
+            w = np.full(shape, 1.0 if "norm" in name and not name.endswith(".b") else (-1.0 if name.endswith("dt_bias") else 0.0), np.float32)
         else:
             w = np.random.Generator(np.random.SFC64([seed, i])).standard_normal(shape, dtype=np.float32)
             w *= np.float32(0.5 if name.endswith(".conv") else std)
@@ -231,3 +230,70 @@ def dunuzen_prefill_flops(cfg: dict, tokens: int, rank: int = 128) -> dict:
         else:
             delta += 7 * tokens * m["heads"] * m["dim"] * m["vdim"]
     return {"matmul": mm, "attention": attn, "delta": delta}
+
+
+def gugedra_config(width: int, ff: int, heads: int, kv_heads: int, layers: list[str], vocab: int, window: int, dim: int = 128, rot_dims: int = 64, vdim: int = 128,
+                   state: int = 128, ssm_vdim: int = 64, conv: int = 4, side: int = 256) -> dict:
+    """A configuration of uniform layers; `layers` names the mixer of each. The state-space side is twice as wide as the model."""
+    ssm_heads = 2 * width // ssm_vdim
+    mixers = {"parallel": {"left": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": dim, "vdim": vdim, "mask": {"size": window},
+                                    "rot": {"base": 10000.0, "dims": rot_dims}, "scale": dim ** -0.5, "softcap": 50.0},
+                           "right": {"heads": ssm_heads, "vdim": ssm_vdim, "state": state, "groups": 1, "norm_groups": 1, "conv": conv},
+                           "left_scale": 1.0, "right_scale": 1.0},
+              "delta": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}}
+    return {"architecture": "Gugedra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "token_side": {"dim": side}, "logit_softcap": 30.0,
+            "layers": [{"type": t, "mixer": mixers[t], "mlp": {"kind": "dense", "ff": ff}} for t in layers]}
+
+
+def gugedra_shapes(cfg: dict) -> dict[str, list[int]]:
+    w, side = cfg["width"], cfg["token_side"]["dim"]
+    t = {"embed": [cfg["vocab"], w], "side.embed": [cfg["vocab"], side * len(cfg["layers"])]}
+    for i, layer in enumerate(cfg["layers"]):
+        m, p, x = layer["mixer"], f"l{i}.", f"l{i}.mix."
+        t.update({p + n: [w] for n in ("norm1", "norm1b", "norm2", "norm2b")})
+        if layer["type"] == "parallel":
+            a, r = m["left"], m["right"]
+            inner, gn = r["heads"] * r["vdim"], r["groups"] * r["state"]
+            t.update({x + "left.q": [a["heads"] * a["dim"], w], x + "left.k": [a["kv_heads"] * a["dim"], w], x + "left.v": [a["kv_heads"] * a["vdim"], w],
+                      x + "left.o": [w, a["heads"] * a["vdim"]], x + "right.in": [2 * inner + 2 * gn + r["heads"], w], x + "right.conv": [inner + 2 * gn, r["conv"]],
+                      x + "right.conv.b": [inner + 2 * gn], x + "right.dt_bias": [r["heads"]], x + "right.A_log": [r["heads"]], x + "right.D": [r["heads"]],
+                      x + "right.norm": [inner], x + "right.o": [w, inner]})
+        else:
+            h, qk, vd = m["heads"], m["kv_heads"] * m["dim"], m["heads"] * m["vdim"]
+            t.update({x + "q": [qk, w], x + "q.conv": [qk, m["conv"]], x + "k": [qk, w], x + "k.conv": [qk, m["conv"]], x + "v": [vd, w],
+                      x + "v.conv": [vd, m["conv"]], x + "b": [h, w], x + "a": [h, w], x + "dt_bias": [h], x + "A_log": [h], x + "norm": [m["vdim"]],
+                      x + "g": [vd, w], x + "o": [w, vd]})
+        f = layer["mlp"]["ff"]
+        t.update({p + "mlp.gate": [f, w], p + "mlp.up": [f, w], p + "mlp.down": [w, f], p + "side.gate": [side, w], p + "side.proj": [w, side], p + "side.norm": [w]})
+    t.update({"final.norm": [w], "head": [cfg["vocab"], w]})
+    return t
+
+
+def gugedra_decode_bytes(cfg: dict, pos: int) -> int:
+    """Bytes one bf16 decode step at position pos has to move: every matrix once, the states read and written, the visible keys."""
+    total = 2 * sum(int(np.prod(s)) for n, s in gugedra_shapes(cfg).items() if n not in ("embed", "side.embed")) + 2 * cfg["width"]
+    for layer in cfg["layers"]:
+        m = layer["mixer"]
+        if layer["type"] == "parallel":
+            a, r = m["left"], m["right"]
+            total += 2 * min(pos + 1, a["mask"]["size"]) * a["kv_heads"] * (a["dim"] + a["vdim"]) + 8 * r["heads"] * r["state"] * r["vdim"]
+        else:
+            total += 8 * m["heads"] * m["dim"] * m["vdim"]
+    return total
+
+
+def gugedra_prefill_flops(cfg: dict, tokens: int) -> dict:
+    """Operations of a prompt of `tokens` tokens: products with weights, attention inside the window, the recurrences."""
+    skip = ("embed", "side.embed", "head")
+    mm = sum(2 * tokens * int(np.prod(s)) for n, s in gugedra_shapes(cfg).items() if len(s) == 2 and n not in skip and not n.endswith(".conv"))
+    attn = rec = 0
+    for layer in cfg["layers"]:
+        m = layer["mixer"]
+        if layer["type"] == "parallel":
+            a, r = m["left"], m["right"]
+            w = min(a["mask"]["size"], tokens)
+            attn += 2 * (w * (w + 1) // 2 + (tokens - w) * w) * a["heads"] * (a["dim"] + a["vdim"])
+            rec += 5 * tokens * r["heads"] * r["state"] * r["vdim"]
+        else:
+            rec += 7 * tokens * m["heads"] * m["dim"] * m["vdim"]
+    return {"matmul": mm, "attention": attn, "recurrence": rec}

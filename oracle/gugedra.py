@@ -2,7 +2,9 @@
 a recurrence, whole score matrices where it is an attention. It shares no code with the product path.
 
 A model is (config, weights): the parsed config.json and a dict name -> float array. `forward` takes the whole token
-sequence of one request and returns logits for every position and the residual stream after every layer."""
+sequence of one request and returns logits for every position and the residual stream after every layer. `r` rounds what a
+16-bit implementation may keep in 16 bits (the products' inputs, keys, values, convolved values); with bf16_round it tells how far
+rounding alone carries a model."""
 
 from __future__ import annotations
 
@@ -33,18 +35,22 @@ def attention_scores(q, k, scale, cap):
     return softcap(q @ k.T * scale, cap)
 
 
-def window_attention(h, W, m):
+def exact(x):
+    return x
+
+
+def window_attention(h, W, m, r=exact):
     n, H, G, d, dv = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
     pos, dims, base = np.arange(n), m["rot"]["dims"], m["rot"]["base"]
-    q = rope_half((h @ W("q").T).reshape(n, H, d), pos, dims, base)
-    k = rope_half((h @ W("k").T).reshape(n, G, d), pos, dims, base)
-    v = (h @ W("v").T).reshape(n, G, dv)
+    q = r(rope_half((h @ W("q").T).reshape(n, H, d), pos, dims, base))
+    k = r(rope_half((h @ W("k").T).reshape(n, G, d), pos, dims, base))
+    v = r((h @ W("v").T).reshape(n, G, dv))
     seen = window_visible(n, m["mask"]["size"])
     out = np.zeros((n, H, dv))
     for head in range(H):
         g = head // (H // G)
         out[:, head] = softmax_rows(attention_scores(q[:, head], k[:, g], m["scale"], m["softcap"]), seen) @ v[:, g]
-    return out.reshape(n, H * dv) @ W("o").T
+    return r(out.reshape(n, H * dv)) @ W("o").T
 
 
 def state_space_scan(x, B, C, dt, a_log, D, state):
@@ -56,12 +62,12 @@ def state_space_scan(x, B, C, dt, a_log, D, state):
     return np.array(out).reshape(x.shape), S
 
 
-def state_space(h, W, m, eps):
+def state_space(h, W, m, eps, r=exact):
     n, H, dv, N, G = h.shape[0], m["heads"], m["vdim"], m["state"], m["groups"]
     inner = H * dv
     p = h @ W("in").T
     z, conv_in, dt = p[:, :inner], p[:, inner:2 * inner + 2 * G * N], p[:, 2 * inner + 2 * G * N:]
-    c = silu(causal_conv(conv_in, W("conv")) + W("conv.b"))
+    c = r(silu(causal_conv(conv_in, W("conv")) + W("conv.b")))
     x, B, C = c[:, :inner].reshape(n, H, dv), c[:, inner:inner + G * N].reshape(n, G, N), c[:, inner + G * N:].reshape(n, G, N)
     dt = softplus(dt + W("dt_bias"))
     y = np.zeros((n, H, dv))
@@ -69,15 +75,15 @@ def state_space(h, W, m, eps):
         g = head // (H // G)
         y[:, head], _ = state_space_scan(x[:, head], B[:, g], C[:, g], dt[:, head], W("A_log")[head], W("D")[head], np.zeros((N, dv)))
     y = y.reshape(n, inner) * silu(z)
-    return (grouped_rms(y, m["norm_groups"], eps) * W("norm")) @ W("o").T
+    return r(grouped_rms(y, m["norm_groups"], eps) * W("norm")) @ W("o").T
 
 
-def parallel(h, W, m, eps):
-    return (m["left_scale"] * window_attention(h, lambda s: W("left." + s), m["left"])
-            + m["right_scale"] * state_space(h, lambda s: W("right." + s), m["right"], eps))
+def parallel(h, W, m, eps, r=exact):
+    return (m["left_scale"] * window_attention(h, lambda s: W("left." + s), m["left"], r)
+            + m["right_scale"] * state_space(h, lambda s: W("right." + s), m["right"], eps, r))
 
 
-def delta(h, W, m, eps):
+def delta(h, W, m, eps, r=exact):
     n, H, KH, d, dv = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
     q = silu(causal_conv(h @ W("q").T, W("q.conv"))).reshape(n, KH, d)
     k = silu(causal_conv(h @ W("k").T, W("k.conv"))).reshape(n, KH, d)
@@ -91,42 +97,42 @@ def delta(h, W, m, eps):
         decay = np.repeat(g[:, head, None], d, axis=1)
         o[:, head], _ = delta_scan(q[:, kh], k[:, kh], v[:, head], decay, beta[:, head], np.zeros((d, dv)))
     o = rms(o, eps) * W("norm") * silu((h @ W("g").T).reshape(n, H, dv))
-    return o.reshape(n, H * dv) @ W("o").T
+    return r(o.reshape(n, H * dv)) @ W("o").T
 
 
-def feed_forward(h, W):
-    return (silu(h @ W("gate").T) * (h @ W("up").T)) @ W("down").T
+def feed_forward(h, W, r=exact):
+    return r(silu(h @ W("gate").T) * (h @ W("up").T)) @ W("down").T
 
 
-def token_side(x, e, W, eps):
+def token_side(x, e, W, eps, r=exact):
     """x [tokens, width], e [tokens, dim]: this layer's part of the tokens' second embedding."""
-    y = (gelu_tanh(x @ W("gate").T) * e) @ W("proj").T
+    y = r(gelu_tanh(r(x) @ W("gate").T) * e) @ W("proj").T
     return rms_norm(y, W("norm"), eps)
 
 
 MIXERS = {"parallel": parallel, "delta": delta}
 
 
-def layer(x, e, cfg, entry, W):
+def layer(x, e, cfg, entry, W, r=exact):
     """One layer on the residual stream x; W(name) returns a tensor of this layer."""
     eps = cfg["norm"]["eps"]
-    y = MIXERS[entry["type"]](rms_norm(x, W("norm1"), eps), lambda s: W("mix." + s), entry["mixer"], eps)
+    y = MIXERS[entry["type"]](r(rms_norm(x, W("norm1"), eps)), lambda s: W("mix." + s), entry["mixer"], eps, r)
     x = x + rms_norm(y, W("norm1b"), eps)
     if entry["mlp"] is not None:
-        x = x + rms_norm(feed_forward(rms_norm(x, W("norm2"), eps), lambda s: W("mlp." + s)), W("norm2b"), eps)
-    return x + token_side(x, e, lambda s: W("side." + s), eps)
+        x = x + rms_norm(feed_forward(r(rms_norm(x, W("norm2"), eps)), lambda s: W("mlp." + s), r), W("norm2b"), eps)
+    return x + token_side(x, e, lambda s: W("side." + s), eps, r)
 
 
-def forward(config, weights, tokens):
+def forward(config, weights, tokens, r=exact):
     """Returns (logits [tokens, vocab], residual stream after every layer [layers, tokens, width])."""
     T = {k: np.asarray(v, np.float64) for k, v in weights.items()}
     ids, dim, after = np.asarray(tokens), config["token_side"]["dim"], []
     x = T["embed"][ids]
     for i, entry in enumerate(config["layers"]):
-        x = layer(x, T["side.embed"][ids][:, i * dim:(i + 1) * dim], config, entry, lambda s: T[f"l{i}." + s])
+        x = layer(x, T["side.embed"][ids][:, i * dim:(i + 1) * dim], config, entry, lambda s: T[f"l{i}." + s], r)
         after.append(x)
     x = rms_norm(x, T["final.norm"], config["norm"]["eps"])
-    return softcap(x @ T["head"].T, config["logit_softcap"]), np.array(after)
+    return softcap(r(x) @ T["head"].T, config["logit_softcap"]), np.array(after)
 
 
 def tensor_shapes(config):

@@ -14,6 +14,7 @@ import brasa_b200 as B
 from oracle import dunuzen as D
 
 from dunuzen_cases import CASES, LA, build, config, delta, latent, off, tokens
+from stack_helpers import follows, pad, portions
 
 pytestmark = pytest.mark.gpu
 ROOT = pathlib.Path(__file__).resolve().parent.parent
@@ -57,16 +58,6 @@ def load(ctx, path, dtype, ctx_len=512, max_tokens=512, rows=512):
     return B.Dunuzen.load_in(ctx, path, dtype, ctx_len, max_tokens, rows)
 
 
-def portions(model, ids, sizes):
-    """Logits of every position, fed in portions of the given sizes over and over."""
-    out, at, i = [], 0, 0
-    while at < len(ids):
-        n = min(sizes[i % len(sizes)], len(ids) - at)
-        out.append(model.feed(ids[at:at + n], at, range(n)))
-        at, i = at + n, i + 1
-    return np.concatenate(out)
-
-
 # ---- operators -------------------------------------------------------------------------------------------------------------
 
 
@@ -80,12 +71,6 @@ def test_layer_norm(ctx, rows, n):
     cmd.wait()
     want = D.layer_norm(x.astype(np.float64), w, b, 1e-3)
     assert np.abs(out.download(np.float32).reshape(rows, n) - want).max() <= 2e-5 * np.abs(want).max()
-
-
-def pad(a, ld):
-    out = np.zeros((a.shape[0], ld), a.dtype)
-    out[:, :a.shape[1]] = a
-    return out
 
 
 @pytest.mark.parametrize("f32", [False, True])
@@ -375,11 +360,7 @@ def test_plan_is_what_is_allocated(ctx, folders, name, dtype):
 
 
 def follow(cfg, w, prompt, ids, tol):
-    """Every generated token is the oracle's best for the sequence so far, or within rounding of it."""
-    lg, _ = D.forward(cfg, w, np.concatenate([prompt, ids]))
-    for i, t in enumerate(ids):
-        row = lg[len(prompt) - 1 + i]
-        assert row.max() - row[t] <= tol * np.std(row), i
+    follows(D.forward, cfg, w, prompt, ids, tol)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
