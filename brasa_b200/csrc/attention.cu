@@ -6,7 +6,7 @@
 // contiguous. Heads lie up8(dim) and up8(vdim) elements apart. The rings are cleared once: tiles read rows nothing was stored in.
 // Many tokens: attn_store_kernel, then window_attn.cu over the rings as they are.
 // One token: attn_step_kernel, one cluster of blocks per key head (and per eight of its query heads), the keys dealt out to the
-// cluster's warps in tiles of 32, each warp with softmax sums of its own, merged through distributed shared memory.
+// cluster's warps eight at a time, each warp with softmax sums of its own, merged through distributed shared memory.
 #include <cooperative_groups.h>
 #include <cuda_bf16.h>
 
@@ -50,58 +50,108 @@ __global__ void __launch_bounds__(256) attn_store_kernel(AttnShape s, const floa
     for (uint32_t e = lane; e < s.vdim; e += 32) elem_store(vc + (slot * s.kv_heads + g) * s.vstep + e, vr[e]);
 }
 
-constexpr uint32_t PH = 8, PW = 8, VMAX = 8;  // query heads of a block, warps of a block, value columns of a lane (vdim up to 256)
+constexpr uint32_t PH = 8, PW = 16, PK = 8, VMAX = 8;  // query heads of a block, warps of a block, keys of a tile, value columns of a lane (vdim up to 256)
 
-// Grid (splits, groups): cluster = one group's splits; group = key head g and its query heads [8 sub, 8 sub + 8).
-template <typename T, int V>
-__global__ void __launch_bounds__(256) attn_step_kernel(AttnShape s, const float *q, const float *k, const float *v, const float *cos_t, const float *sin_t, T *kc, T *vc,
-                                                        float *out, const uint32_t *pos_p) {
+// Shared memory of a step's block, in floats: parts [PW][heads][ldp] and the block's merged sums [heads][ldp] (ldp: value columns,
+// then maximum and sum of weights), weights of the parts [heads][PW], rotated queries [heads][kstep], this token's key and value.
+struct StepPlan {
+    uint32_t heads, ldp, own, wt, qs, now, bytes;
+    __host__ __device__ StepPlan(const AttnShape &s, uint32_t elem) {
+        const uint32_t share = s.heads / s.kv_heads;
+        heads = share < PH ? share : PH;
+        ldp = s.vdim + 2;
+        own = PW * heads * ldp;
+        wt = own + heads * ldp;
+        qs = (wt + heads * PW + 3) / 4 * 4;
+        now = qs + heads * s.kstep;
+        bytes = now * 4 + (s.kstep + s.vstep) * elem;
+    }
+};
+
+// Grid (splits, groups): cluster = one group's splits; group = key head g and its query heads [8 sub, 8 sub + 8). A tile of eight
+// keys: lane = key lane / 4 and every fourth 16-byte piece of its row from piece lane % 4 on; then value columns lane, lane + 32, ..
+// V: value columns of a lane; HM: the most query heads of a block.
+template <typename T, int V, uint32_t HM>
+__global__ void __launch_bounds__(32 * PW, 1) attn_step_kernel(AttnShape s, const float *q, const float *k, const float *v, const float *cos_t, const float *sin_t, T *kc,
+                                                               T *vc, float *out, const uint32_t *pos_p) {
     extern __shared__ __align__(16) float sm[];
     constexpr uint32_t E = 16 / sizeof(T);  // elements of a 16-byte access
+    const StepPlan pl(s, sizeof(T));
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, splits = gridDim.x, rank = blockIdx.x;
     const uint32_t share = s.heads / s.kv_heads, subs = (share + PH - 1) / PH, g = blockIdx.y / subs, h0 = g * share + blockIdx.y % subs * PH;
-    const uint32_t nh = min(PH, (g + 1) * share - h0), ldp = s.vdim + 2, half = s.rot_dims / 2;
-    // own [PH][ldp]: the block's merged sums; parts [PW][PH][ldp]; qs [PH][kstep]; this token's key and value as the rings hold them
-    float *own = sm, *parts = own + PH * ldp, *qs = parts + PW * PH * ldp;
-    T *k_now = reinterpret_cast<T *>(qs + PH * s.kstep), *v_now = k_now + s.kstep;
+    const uint32_t nh = min(PH, (g + 1) * share - h0), ldp = pl.ldp, half = s.rot_dims / 2;
+    float *parts = sm, *own = sm + pl.own, *wt = sm + pl.wt, *qs = sm + pl.qs;
+    T *k_now = reinterpret_cast<T *>(sm + pl.now), *v_now = k_now + s.kstep;
+    // The position and the older keys and values were written several kernels ago: the first tile is asked for ahead of the wait.
+    const uint32_t pos = *pos_p, beg = pos + 1 > s.window ? pos + 1 - s.window : 0u, slot0 = beg % s.rows;
+    const float *ct = cos_t + (size_t)pos * half, *st = sin_t + (size_t)pos * half;
+    auto slot_of = [&](uint32_t key) {  // of a visible position
+        const uint32_t r = slot0 + key - beg;
+        return (size_t)(r >= s.rows ? r - s.rows : r) * s.kv_heads + g;
+    };
+    constexpr uint32_t KR = 4;  // 16-byte pieces of a lane's key kept ahead
+    uint4 kk4[KR];
+    float vv[PK][V];
+    auto load = [&](uint32_t t0) {  // positions before this token's
+        const uint32_t key = t0 + (lane >> 2);
+        const T *kp = kc + slot_of(key < pos ? key : beg) * s.kstep;
+#pragma unroll
+        for (uint32_t i = 0; i < KR; ++i) {
+            const uint32_t e = ((lane & 3) + 4 * i) * E;
+            kk4[i] = key < pos && e < s.kstep ? *reinterpret_cast<const uint4 *>(kp + e) : make_uint4(0, 0, 0, 0);
+        }
+#pragma unroll
+        for (uint32_t j = 0; j < PK; ++j) {
+            const T *vp = vc + slot_of(t0 + j < pos ? t0 + j : beg) * s.vstep;
+#pragma unroll
+            for (int c = 0; c < V; ++c) vv[j][c] = t0 + j < pos && lane + 32 * c < s.vdim ? elem_load(vp + lane + 32 * c) : 0.0f;
+        }
+    };
+    const uint32_t first = beg + PK * (rank * PW + warp);
+    load(first);
     pdl_wait();
     pdl_launch();
-    const uint32_t pos = *pos_p, beg = pos + 1 > s.window ? pos + 1 - s.window : 0u;
-    const float *ct = cos_t + (size_t)pos * half, *st = sin_t + (size_t)pos * half;
-    for (uint32_t i = tid; i < PH * s.kstep; i += 256) {
-        const uint32_t h = i / s.kstep, e = i - h * s.kstep;
-        qs[i] = h < nh && e < s.dim ? rot_elem(q + (size_t)(h0 + h) * s.dim, e, s.rot_dims, ct, st) * s.scale : 0.0f;
-    }
-    const size_t slot = pos % s.rows;
     const bool keeper = rank == 0 && blockIdx.y % subs == 0;  // stores this token's rows (nobody reads them there in this step)
-    for (uint32_t e = tid; e < s.kstep; e += 256) {
-        elem_store(k_now + e, e < s.dim ? rot_elem(k + g * s.dim, e, s.rot_dims, ct, st) : 0.0f);
-        if (keeper && e < s.dim) kc[(slot * s.kv_heads + g) * s.kstep + e] = k_now[e];
-    }
-    for (uint32_t e = tid; e < s.vstep; e += 256) {
-        elem_store(v_now + e, e < s.vdim ? v[g * s.vdim + e] : 0.0f);
-        if (keeper && e < s.vdim) vc[(slot * s.kv_heads + g) * s.vstep + e] = v_now[e];
+    for (uint32_t i = warp; i < nh + 2; i += PW) {
+        if (i < nh) {
+            for (uint32_t e = lane; e < s.kstep; e += 32) qs[i * s.kstep + e] = e < s.dim ? rot_elem(q + (size_t)(h0 + i) * s.dim, e, s.rot_dims, ct, st) * s.scale : 0.0f;
+        } else {
+            const bool key = i == nh;
+            const uint32_t n = key ? s.dim : s.vdim, step = key ? s.kstep : s.vstep;
+            T *now = key ? k_now : v_now, *keep = (key ? kc : vc) + slot_of(pos) * step;
+            for (uint32_t e = lane; e < step; e += 32) {
+                elem_store(now + e, e >= n ? 0.0f : (key ? rot_elem(k + g * s.dim, e, s.rot_dims, ct, st) : v[g * s.vdim + e]));
+                if (keeper && e < n) keep[e] = now[e];
+            }
+        }
     }
     __syncthreads();
-    float m[PH], l[PH], acc[PH][V];
+    float m[HM], l[HM], acc[HM][V];
 #pragma unroll
-    for (uint32_t h = 0; h < PH; ++h) {
+    for (uint32_t h = 0; h < HM; ++h) {
         m[h] = -INFINITY;
         l[h] = 0.0f;
 #pragma unroll
         for (int c = 0; c < V; ++c) acc[h][c] = 0.0f;
     }
-    for (uint32_t t0 = beg + 32 * (rank * PW + warp); t0 <= pos; t0 += 32 * PW * splits) {
-        const uint32_t key = t0 + lane;
+    for (uint32_t t0 = first; t0 <= pos; t0 += PK * PW * splits) {
+        const uint32_t key = t0 + (lane >> 2);
         const bool live = key <= pos;
-        const size_t row = (size_t)((live ? key : pos) % s.rows) * s.kv_heads + g;
-        const T *kp = key >= pos ? k_now : kc + row * s.kstep;
-        float sc[PH];
+        const T *kp = key >= pos ? k_now : kc + slot_of(key) * s.kstep;
+        if (t0 != first) load(t0);
+        if (key == pos)
 #pragma unroll
-        for (uint32_t h = 0; h < PH; ++h) sc[h] = 0.0f;
-#pragma unroll 4
-        for (uint32_t e = 0; e < s.kstep; e += E) {
-            const uint4 kv = *reinterpret_cast<const uint4 *>(kp + e);
+            for (uint32_t i = 0; i < KR; ++i)
+                if (((lane & 3) + 4 * i) * E < s.kstep) kk4[i] = *reinterpret_cast<const uint4 *>(k_now + ((lane & 3) + 4 * i) * E);
+#pragma unroll
+        for (uint32_t j = 0; j < PK; ++j)
+            if (t0 + j == pos)
+#pragma unroll
+                for (int c = 0; c < V; ++c) vv[j][c] = lane + 32 * c < s.vdim ? elem_load(v_now + lane + 32 * c) : 0.0f;
+        float sc[HM];
+#pragma unroll
+        for (uint32_t h = 0; h < HM; ++h) sc[h] = 0.0f;
+        auto dots = [&](const uint4 &kv, uint32_t e) {
             float kk[E];
             if (sizeof(T) == 2) {
                 kk[0] = bf16_lo(kv.x); kk[1] = bf16_hi(kv.x); kk[2] = bf16_lo(kv.y); kk[3] = bf16_hi(kv.y);
@@ -110,52 +160,48 @@ __global__ void __launch_bounds__(256) attn_step_kernel(AttnShape s, const float
                 kk[0] = __uint_as_float(kv.x); kk[1] = __uint_as_float(kv.y); kk[2] = __uint_as_float(kv.z); kk[3] = __uint_as_float(kv.w);
             }
 #pragma unroll
-            for (uint32_t h = 0; h < PH; ++h)
+            for (uint32_t h = 0; h < HM; ++h)
                 if (h < nh)
 #pragma unroll
                     for (uint32_t i = 0; i < E; i += 4) {
                         const float4 qv = *reinterpret_cast<const float4 *>(qs + h * s.kstep + e + i);
                         sc[h] = fmaf(kk[i], qv.x, fmaf(kk[i + 1], qv.y, fmaf(kk[i + 2], qv.z, fmaf(kk[i + 3], qv.w, sc[h]))));
                     }
-        }
-        const uint32_t n = min(32u, pos + 1 - t0);
+        };
 #pragma unroll
-        for (uint32_t h = 0; h < PH; ++h)
+        for (uint32_t i = 0; i < KR; ++i)
+            if (((lane & 3) + 4 * i) * E < s.kstep) dots(kk4[i], ((lane & 3) + 4 * i) * E);
+        for (uint32_t e = ((lane & 3) + 4 * KR) * E; e < s.kstep; e += 4 * E) dots(*reinterpret_cast<const uint4 *>(kp + e), e);
+#pragma unroll
+        for (uint32_t h = 0; h < HM; ++h)
             if (h < nh) {
                 float x = sc[h];
+                x += __shfl_xor_sync(0xffffffffu, x, 1);
+                x += __shfl_xor_sync(0xffffffffu, x, 2);
                 if (s.softcap > 0.0f) x = s.softcap * tanhf(x / s.softcap);
                 if (!live) x = -INFINITY;
                 float mx = x;
 #pragma unroll
-                for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+                for (int o = 16; o > 2; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
                 mx = fmaxf(mx, m[h]);  // finite: a tile has at least one visible key
-                const float p = expf(x - mx), r = expf(m[h] - mx);
-                l[h] = l[h] * r + warp_sum(p);
+                float p = expf(x - mx), r = expf(m[h] - mx);
                 m[h] = mx;
-                sc[h] = p;
 #pragma unroll
                 for (int c = 0; c < V; ++c) acc[h][c] *= r;
-            }
-#pragma unroll 8
-        for (uint32_t j = 0; j < n; ++j) {
-            const uint32_t kj = t0 + j;
-            const T *vp = kj == pos ? v_now : vc + ((size_t)(kj % s.rows) * s.kv_heads + g) * s.vstep;
-            float vv[V];
+                l[h] *= r;
 #pragma unroll
-            for (int c = 0; c < V; ++c) vv[c] = lane + 32 * c < s.vdim ? elem_load(vp + lane + 32 * c) : 0.0f;
+                for (uint32_t j = 0; j < PK; ++j) {
+                    const float w = __shfl_sync(0xffffffffu, p, 4 * j);
+                    l[h] += w;
 #pragma unroll
-            for (uint32_t h = 0; h < PH; ++h)
-                if (h < nh) {
-                    const float p = __shfl_sync(0xffffffffu, sc[h], j);
-#pragma unroll
-                    for (int c = 0; c < V; ++c) acc[h][c] = fmaf(p, vv[c], acc[h][c]);
+                    for (int c = 0; c < V; ++c) acc[h][c] = fmaf(w, vv[j][c], acc[h][c]);
                 }
-        }
+            }
     }
 #pragma unroll
-    for (uint32_t h = 0; h < PH; ++h)
+    for (uint32_t h = 0; h < HM; ++h)
         if (h < nh) {
-            float *p = parts + (warp * PH + h) * ldp;
+            float *p = parts + (warp * pl.heads + h) * ldp;
 #pragma unroll
             for (int c = 0; c < V; ++c)
                 if (lane + 32 * c < s.vdim) p[lane + 32 * c] = acc[h][c];
@@ -165,45 +211,53 @@ __global__ void __launch_bounds__(256) attn_step_kernel(AttnShape s, const float
             }
         }
     __syncthreads();
-    // sums of n parts, `step` floats apart, of head h: column e
-    for (uint32_t i = tid; i < nh * s.vdim; i += 256) {
-        const uint32_t h = i / s.vdim, e = i - h * s.vdim;
-        const float *p = parts + h * ldp;
-        float mx = -INFINITY, a = 0.0f, ls = 0.0f;
-        for (uint32_t w = 0; w < PW; ++w) mx = fmaxf(mx, p[w * PH * ldp + s.vdim]);
-        for (uint32_t w = 0; w < PW; ++w) {
-            const float f = p[w * PH * ldp + s.vdim];
-            const float r = f == -INFINITY ? 0.0f : expf(f - mx);
-            a = fmaf(r, p[w * PH * ldp + e], a);
-            ls = fmaf(r, p[w * PH * ldp + s.vdim + 1], ls);
-        }
-        own[h * ldp + e] = a;
-        if (e == 0) {
-            own[h * ldp + s.vdim] = mx;
-            own[h * ldp + s.vdim + 1] = ls;
+    // The block's sums: head `warp`, lane = part; then all columns. (A warp that had no tile: maximum -inf, weight 0.)
+    if (warp < nh) {
+        const float *p = parts + (lane * pl.heads + warp) * ldp + s.vdim;
+        const float f = lane < PW ? p[0] : -INFINITY;
+        float mx = f;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        const float r = f == -INFINITY ? 0.0f : expf(f - mx);
+        if (lane < PW) wt[warp * PW + lane] = r;
+        const float ls = warp_sum(lane < PW ? r * p[1] : 0.0f);
+        if (lane == 0) {
+            own[warp * ldp + s.vdim] = mx;
+            own[warp * ldp + s.vdim + 1] = ls;
         }
     }
+    __syncthreads();
+    for (uint32_t h = 0; h < nh; ++h)
+        for (uint32_t e = tid; e < s.vdim; e += 32 * PW) {
+            float a = 0.0f;
+#pragma unroll
+            for (uint32_t w = 0; w < PW; ++w) a = fmaf(wt[h * PW + w], parts[(w * pl.heads + h) * ldp + e], a);
+            own[h * ldp + e] = a;
+        }
     cg::cluster_group cluster = cg::this_cluster();
     cluster.sync();
-    for (uint32_t i = rank * 256 + tid; i < nh * s.vdim; i += 256 * splits) {
-        const uint32_t h = i / s.vdim, e = i - h * s.vdim;
-        float mx = -INFINITY, a = 0.0f, ls = 0.0f;
-        for (uint32_t b = 0; b < splits; ++b) mx = fmaxf(mx, cluster.map_shared_rank(own, b)[h * ldp + s.vdim]);
-        for (uint32_t b = 0; b < splits; ++b) {
-            const float *p = cluster.map_shared_rank(own, b) + h * ldp;
-            const float r = p[s.vdim] == -INFINITY ? 0.0f : expf(p[s.vdim] - mx);
-            a = fmaf(r, p[e], a);
-            ls = fmaf(r, p[s.vdim + 1], ls);
+    // The cluster's sums: block `rank` takes heads rank, rank + splits, ..
+    for (uint32_t h = rank; h < nh; h += splits) {
+        float mx = -INFINITY, ls = 0.0f, r[8];
+#pragma unroll
+        for (uint32_t b = 0; b < 8; ++b) {
+            r[b] = b < splits ? cluster.map_shared_rank(own, b)[h * ldp + s.vdim] : -INFINITY;
+            mx = fmaxf(mx, r[b]);
         }
-        out[(size_t)(h0 + h) * s.vdim + e] = a / ls * s.out_scale;
+#pragma unroll
+        for (uint32_t b = 0; b < 8; ++b) {
+            r[b] = r[b] == -INFINITY ? 0.0f : expf(r[b] - mx);
+            if (b < splits) ls = fmaf(r[b], cluster.map_shared_rank(own, b)[h * ldp + s.vdim + 1], ls);
+        }
+        for (uint32_t e = tid; e < s.vdim; e += 32 * PW) {
+            float a = 0.0f;
+#pragma unroll
+            for (uint32_t b = 0; b < 8; ++b)
+                if (b < splits) a = fmaf(r[b], cluster.map_shared_rank(own, b)[h * ldp + e], a);
+            out[(size_t)(h0 + h) * s.vdim + e] = a / ls * s.out_scale;
+        }
     }
     cluster.sync();  // nobody leaves while its sums are being read
-}
-
-template <typename T>
-size_t step_smem(const AttnShape &s) {
-    const size_t ldp = s.vdim + 2;
-    return (PH * ldp + PW * PH * ldp + PH * s.kstep) * 4 + (s.kstep + s.vstep) * sizeof(T);
 }
 
 }  // namespace
@@ -310,24 +364,25 @@ class WindowAttention : public Mixer {
 
     template <typename T>
     int32_t step_as(const Run &r) {
-        if (s_.vdim <= 64) return step<T, 2>(r);
-        if (s_.vdim <= 128) return step<T, 4>(r);
-        return step<T, (int)VMAX>(r);
+        const bool few = s_.heads / s_.kv_heads <= 4;
+        if (s_.vdim <= 64) return few ? step<T, 2, 4>(r) : step<T, 2, PH>(r);
+        if (s_.vdim <= 128) return few ? step<T, 4, 4>(r) : step<T, 4, PH>(r);
+        return few ? step<T, (int)VMAX, 4>(r) : step<T, (int)VMAX, PH>(r);
     }
-    template <typename T, int V>
+    template <typename T, int V, uint32_t HM>
     int32_t step(const Run &r) {
         brasa_ctx *ctx = r.cmd->ctx;
         auto f = [&](uint64_t at) { return (const float *)(r.scratch + at); };
         const uint32_t share = s_.heads / s_.kv_heads, groups = s_.kv_heads * ((share + PH - 1) / PH);
         uint32_t splits = 1;  // a cluster of at most eight blocks, no more than there are tiles for
-        while (splits < 8 && splits * 32 * PW < seen_) splits *= 2;
-        const size_t smem = step_smem<T>(s_);
+        while (splits < 8 && splits * PK * PW < seen_) splits *= 2;
+        const size_t smem = StepPlan(s_, sizeof(T)).bytes;
         BRASA_REQUIRE(ctx, smem + 1024 <= ctx->smem_optin, "attention: head sizes too large");
-        auto kernel = attn_step_kernel<T, V>;
+        auto kernel = attn_step_kernel<T, V, HM>;
         BRASA_TRY(brasa_smem_optin(ctx, (const void *)kernel, std::max<size_t>(smem, 48 * 1024)));
         cudaLaunchConfig_t cfg{};
         cfg.gridDim = dim3(splits, groups);
-        cfg.blockDim = dim3(256);
+        cfg.blockDim = dim3(32 * PW);
         cfg.dynamicSmemBytes = smem;
         cfg.stream = ctx->stream;
         cudaLaunchAttribute attr[2];

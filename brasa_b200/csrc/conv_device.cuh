@@ -9,6 +9,8 @@ namespace brasa_dev {
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
+// for results that are rounded to bf16
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
@@ -35,9 +37,22 @@ __device__ __forceinline__ float conv_at(const float *x, uint32_t ldx, uint32_t 
     return s;
 }
 
+// The same for one token (x its inputs, slot = pos0 % taps); up to four taps with every load on its way at once.
+__device__ __forceinline__ float conv_step(const float *x, uint32_t c, const float *w, const ConvView &cv, uint32_t slot, uint32_t ch) {
+    if (cv.taps > 4) return conv_at(x, 0, c, w, 0, cv, ch);
+    float v[4], k[4];
+#pragma unroll
+    for (uint32_t b = 0; b < 4; ++b) {  // b tokens before this one
+        const bool live = b < cv.taps && b <= cv.pos0;
+        v[b] = !live ? 0.0f : (b == 0 ? x[c] : cv.ring[(size_t)(slot >= b ? slot - b : slot + cv.taps - b) * cv.channels + ch]);
+        k[b] = b < cv.taps ? w[(size_t)c * cv.taps + cv.taps - 1 - b] : 0.0f;
+    }
+    return fmaf(v[0], k[0], fmaf(v[1], k[1], fmaf(v[2], k[2], v[3] * k[3])));
+}
+
 // convolution, bias and silu of one channel for tokens t0 .. t0 + n - 1 (n up to CONV_RUN), handed to put(t, value)
 constexpr uint32_t CONV_RUN = 16;
-template <typename Put>
+template <bool FAST = false, typename Put>
 __device__ __forceinline__ void conv_chunk(const float *x, uint32_t ldx, uint32_t c, const float *w, float bias, uint32_t t0, uint32_t n, const ConvView &cv, uint32_t ch, Put put) {
     if (cv.taps <= 4) {  // the window in registers
         float wr[4], xr[4];
@@ -61,7 +76,8 @@ __device__ __forceinline__ void conv_chunk(const float *x, uint32_t ldx, uint32_
             xr[1] = xr[2];
             xr[2] = xr[3];
             xr[3] = in[t];
-            if (t < n) put(t, silu_f(fmaf(xr[3], wr[3], fmaf(xr[2], wr[2], fmaf(xr[1], wr[1], fmaf(xr[0], wr[0], bias))))));
+            const float z = fmaf(xr[3], wr[3], fmaf(xr[2], wr[2], fmaf(xr[1], wr[1], fmaf(xr[0], wr[0], bias))));
+            if (t < n) put(t, FAST ? silu_fast(z) : silu_f(z));
         }
     } else {
         for (uint32_t t = 0; t < n; ++t) put(t, silu_f(conv_at(x, ldx, c, w, t0 + t, cv, ch) + bias));

@@ -758,7 +758,7 @@ __global__ void __launch_bounds__(STEP_THREADS, 1) delta_step_kernel(DeltaStep p
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     float *S = p.state + (size_t)h * s.dim * s.vdim;
     // Row i of the head's low-rank factors: the decay's rows, then the gate's. Warp w takes rows w, w + 16, .. in batches of
-    // eight; the first batch's weights and the state's cache lines are asked for ahead of the kernel before this one.
+    // eight; the first batch's weights and the state are asked for ahead of the kernel before this one.
     const uint32_t nrows = p.wa2 ? s.dim + s.vdim : 0u;
     uint4 fw[8];
     auto factor_load = [&](uint32_t r0, uint32_t c) {
@@ -772,7 +772,19 @@ __global__ void __launch_bounds__(STEP_THREADS, 1) delta_step_kernel(DeltaStep p
         }
     };
     factor_load(warp, lane * 8);
-    for (uint32_t i = tid; i < (s.dim * s.vdim + 31) / 32; i += STEP_THREADS) asm volatile("prefetch.global.L2 [%0];" ::"l"(S + (size_t)i * 32));
+    // (the last to write the state was the token before, several kernels ago)
+    if (!KEEP)
+        for (uint32_t i = tid; i < (s.dim * s.vdim + 31) / 32; i += STEP_THREADS) asm volatile("prefetch.global.L2 [%0];" ::"l"(S + (size_t)i * 32));
+    float keep[STEP_R][STEP_C];
+    if (KEEP) {
+#pragma unroll
+        for (int r = 0; r < STEP_R; ++r)
+#pragma unroll
+            for (int c = 0; c < STEP_C; ++c) {
+                const uint32_t row = warp + 16 * r, col = lane + 32 * c;
+                keep[r][c] = (row < s.dim && col < s.vdim) ? S[(size_t)row * s.vdim + col] : 0.0f;
+            }
+    }
     pdl_wait();
     pdl_launch();
     const uint32_t pos = *p.pos;
@@ -780,17 +792,18 @@ __global__ void __launch_bounds__(STEP_THREADS, 1) delta_step_kernel(DeltaStep p
     const ConvView cv{p.ring, 2 * s.qk + s.vd, s.taps, pos};
     for (uint32_t i = tid; i < ra8; i += STEP_THREADS) a1[i] = i < p.ra ? p.a1[i] : 0.0f;
     for (uint32_t i = tid; i < rg8; i += STEP_THREADS) g1[i] = i < p.rg ? p.g1[i] : 0.0f;
-    for (uint32_t i = tid; i < 2 * s.dim + s.vdim; i += STEP_THREADS) {
-        if (i < s.dim) sq[i] = silu_f(conv_at(p.q, 0, kh * s.dim + i, p.wq, 0, cv, kh * s.dim + i));
-        else if (i < 2 * s.dim) sk[i - s.dim] = silu_f(conv_at(p.k, 0, kh * s.dim + i - s.dim, p.wk, 0, cv, s.qk + kh * s.dim + i - s.dim));
-        else sv[i - 2 * s.dim] = silu_f(conv_at(p.v, 0, h * s.vdim + i - 2 * s.dim, p.wv, 0, cv, 2 * s.qk + h * s.vdim + i - 2 * s.dim));
+    const uint32_t slot = pos % s.taps;
+    for (uint32_t i = tid; i < 2 * s.dim + s.vdim; i += STEP_THREADS) {  // (sk follows sq)
+        const uint32_t part = i < s.dim ? 0u : (i < 2 * s.dim ? 1u : 2u), c = part < 2 ? kh * s.dim + i - part * s.dim : h * s.vdim + i - 2 * s.dim;
+        const float z = silu_f(conv_step(part == 0 ? p.q : (part == 1 ? p.k : p.v), c, part == 0 ? p.wq : (part == 1 ? p.wk : p.wv), cv, slot, part * s.qk + c));
+        (part < 2 ? sq[i] : sv[i - 2 * s.dim]) = z;
     }
     __syncthreads();
     // this token's row of the ring (nobody reads it in this step); the heads of a group store the same q and k values
     for (uint32_t i = tid; i < 2 * s.dim + s.vdim; i += STEP_THREADS) {
         const uint32_t ch = i < s.dim ? kh * s.dim + i : (i < 2 * s.dim ? s.qk + kh * s.dim + i - s.dim : 2 * s.qk + h * s.vdim + i - 2 * s.dim);
         const float x = i < s.dim ? p.q[kh * s.dim + i] : (i < 2 * s.dim ? p.k[kh * s.dim + i - s.dim] : p.v[h * s.vdim + i - 2 * s.dim]);
-        p.ring[(size_t)(pos % s.taps) * cv.channels + ch] = x;
+        p.ring[(size_t)slot * cv.channels + ch] = x;
     }
     const float decay = expf(p.a_log[h]);
     if (!p.wa2) {
@@ -816,16 +829,6 @@ __global__ void __launch_bounds__(STEP_THREADS, 1) delta_step_kernel(DeltaStep p
                 else gate[i - s.dim] = sigmoid_f(v);
             }
         }
-    }
-    float keep[STEP_R][STEP_C];
-    if (KEEP) {
-#pragma unroll
-        for (int r = 0; r < STEP_R; ++r)
-#pragma unroll
-            for (int c = 0; c < STEP_C; ++c) {
-                const uint32_t row = warp + 16 * r, col = lane + 32 * c;
-                keep[r][c] = (row < s.dim && col < s.vdim) ? S[(size_t)row * s.vdim + col] : 0.0f;
-            }
     }
     if (warp < 3) {  // |q|^2, |k|^2, k . q before the scaling
         float v = 0.0f;

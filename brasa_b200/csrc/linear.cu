@@ -15,7 +15,7 @@ __device__ __forceinline__ float activate(float v, int act) {
         v = fmaxf(v, 0.0f);
         v *= v;
     } else if (act == LINEAR_ACT_GELU_TANH) {
-        v = 0.5f * v * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * v * v, v, v)));
+        v = v / (1.0f + expf(-1.5957691216057308f * fmaf(0.044715f * v * v, v, v)));  // 0.5 (1 + tanh(u)) = 1 / (1 + exp(-2 u))
     }
     return v;
 }
@@ -177,12 +177,75 @@ __global__ void __launch_bounds__(32 * GV_WARPS, 1) linear_gemv_kernel(const __g
         place(cur);
         load(cur, q);
     }
+    // ---- the input vectors ----
+    // Up to GV_KEEP values of the residual stream per thread stay in registers, with the constants asked for ahead of the wait.
+    constexpr uint32_t GV_KEEP = 4, GV_T = 32 * GV_WARPS;
+    const bool layer_norm = gp.norm == GEMV_LAYER_NORM, keep = gp.x && !(layer_norm && gp.y) && gp.width <= GV_KEEP * GV_T;
+    float xk[GV_KEEP], yk[GV_KEEP], wk[GV_KEEP], wyk[GV_KEEP];  // layer norm: yk and wyk hold the second form's and the first's constants
+    if (keep)
+#pragma unroll
+        for (uint32_t j = 0; j < GV_KEEP; ++j) {
+            const uint32_t i = tid + GV_T * j;
+            const float *wy = layer_norm ? gp.b[0] : (gp.y ? gp.wy : nullptr);
+            wk[j] = gp.norm != GEMV_PLAIN && i < gp.width ? gp.w[0][i] : 1.0f;
+            wyk[j] = wy && i < gp.width ? wy[i] : 0.0f;
+            yk[j] = layer_norm && gp.nin > 1 && i < gp.width ? gp.w[1][i] : 0.0f;
+        }
     pdl_wait();
     pdl_launch();
-    // ---- the input vectors ----
-    for (uint32_t i = tid; i < gp.x_floats; i += 32 * GV_WARPS) xs[i] = 0.0f;  // (padding)
-    __syncthreads();
-    if (gp.x) {
+    for (uint32_t k = 0; k < gp.nin; ++k)  // padding
+        if (tid < 8 && (gp.len[k] & 7) && gp.len[k] / 8 * 8 + tid >= gp.len[k]) xs[gv_plane(gp.off[k] + gp.len[k] / 8 * 8 + tid, half)] = 0.0f;
+    if (keep) {
+        float s = 0.0f;
+#pragma unroll
+        for (uint32_t j = 0; j < GV_KEEP; ++j) {
+            const uint32_t i = tid + GV_T * j;
+            xk[j] = i < gp.width ? gp.x[i] : 0.0f;
+            if (!layer_norm) yk[j] = gp.y && i < gp.width ? gp.y[i] : 0.0f;
+        }
+        if (layer_norm) {
+#pragma unroll
+            for (uint32_t j = 0; j < GV_KEEP; ++j) s += xk[j];
+            const float mean = block_sum_1024(s, red) / (float)gp.width;
+            s = 0.0f;
+#pragma unroll
+            for (uint32_t j = 0; j < GV_KEEP; ++j) {
+                xk[j] -= mean;
+                if (tid + GV_T * j < gp.width) s = fmaf(xk[j], xk[j], s);
+            }
+            const float inv = 1.0f / sqrtf(block_sum_1024(s, red) / (float)gp.width + gp.eps);
+#pragma unroll
+            for (uint32_t j = 0; j < GV_KEEP; ++j) {
+                const uint32_t i = tid + GV_T * j;
+                if (i < gp.width) {
+                    xs[gv_plane(gp.off[0] + i, half)] = fmaf(xk[j] * inv, wk[j], wyk[j]);
+                    if (gp.nin > 1) xs[gv_plane(gp.off[1] + i, half)] = fmaf(xk[j] * inv, yk[j], gp.b[1][i]);
+                }
+            }
+        } else {
+        if (gp.y) {
+#pragma unroll
+            for (uint32_t j = 0; j < GV_KEEP; ++j) s = fmaf(yk[j], yk[j], s);
+            const float sy = 1.0f / sqrtf(block_sum_1024(s, red) / (float)gp.width + gp.eps);
+            s = 0.0f;
+#pragma unroll
+            for (uint32_t j = 0; j < GV_KEEP; ++j) {
+                const uint32_t i = tid + GV_T * j;
+                xk[j] = fmaf(yk[j] * sy, wyk[j], xk[j]);
+                if (blockIdx.x == 0 && gp.x_out && i < gp.width) gp.x_out[i] = xk[j];
+            }
+        }
+        float inv = 1.0f;
+        if (gp.norm == GEMV_RMS_NORM) {
+#pragma unroll
+            for (uint32_t j = 0; j < GV_KEEP; ++j) s = fmaf(xk[j], xk[j], s);
+            inv = 1.0f / sqrtf(block_sum_1024(s, red) / (float)gp.width + gp.eps);
+        }
+#pragma unroll
+        for (uint32_t j = 0; j < GV_KEEP; ++j)
+            if (tid + GV_T * j < gp.width) xs[gv_plane(gp.off[0] + tid + GV_T * j, half)] = xk[j] * inv * wk[j];
+        }
+    } else if (gp.x) {
         // the residual stream, with the pending sublayer's normed result added; every thread keeps to its own elements
         float s = 0.0f, sy = 0.0f;
         if (gp.y) {
@@ -220,11 +283,22 @@ __global__ void __launch_bounds__(32 * GV_WARPS, 1) linear_gemv_kernel(const __g
             }
         }
     } else {
+        // (loads go out several at a time, ahead of the stores to shared memory)
+        constexpr uint32_t AT = 4;
         for (uint32_t k = 0; k < gp.nin; ++k) {
             if (gp.gated && k == 0) {
-                for (uint32_t i = tid; i < gp.len[0]; i += 32 * GV_WARPS) {
-                    const float *g = gp.v[0] + (size_t)(i >> 5) * 64 + (i & 31);
-                    xs[gv_plane(gp.off[0] + i, half)] = silu_f(g[0]) * g[32];
+                for (uint32_t i0 = tid; i0 < gp.len[0]; i0 += AT * GV_T) {
+                    float g[AT], u[AT];
+#pragma unroll
+                    for (uint32_t j = 0; j < AT; ++j) {
+                        const uint32_t i = i0 + GV_T * j;
+                        const float *src = gp.v[0] + (size_t)(i >> 5) * 64 + (i & 31);
+                        g[j] = i < gp.len[0] ? src[0] : 0.0f;
+                        u[j] = i < gp.len[0] ? src[32] : 0.0f;
+                    }
+#pragma unroll
+                    for (uint32_t j = 0; j < AT; ++j)
+                        if (i0 + GV_T * j < gp.len[0]) xs[gv_plane(gp.off[0] + i0 + GV_T * j, half)] = silu_f(g[j]) * u[j];
                 }
             } else if (gp.parts[k]) {
                 // a warp takes parts warp, warp + 32, .. where there are many; otherwise a part is the block's
@@ -241,13 +315,33 @@ __global__ void __launch_bounds__(32 * GV_WARPS, 1) linear_gemv_kernel(const __g
                 } else {
                     for (uint32_t part = 0; part < gp.parts[k]; ++part) {
                         float s = 0.0f;
-                        for (uint32_t i = tid; i < n; i += 32 * GV_WARPS) s = fmaf(gp.v[k][part * n + i], gp.v[k][part * n + i], s);
+                        for (uint32_t i0 = tid; i0 < n; i0 += AT * GV_T) {
+                            float v[AT], w[AT];
+#pragma unroll
+                            for (uint32_t j = 0; j < AT; ++j) {
+                                const uint32_t i = i0 + GV_T * j;
+                                v[j] = i < n ? gp.v[k][part * n + i] : 0.0f;
+                                w[j] = i < n ? gp.vw[k][part * n + i] : 0.0f;
+                            }
+#pragma unroll
+                            for (uint32_t j = 0; j < AT; ++j) {
+                                if (i0 + GV_T * j < n) xs[gv_plane(gp.off[k] + part * n + i0 + GV_T * j, half)] = v[j] * w[j];
+                                s = fmaf(v[j], v[j], s);
+                            }
+                        }
                         const float inv = gp.vscale[k] / sqrtf(block_sum_1024(s, red) / (float)n + gp.eps);
-                        for (uint32_t i = tid; i < n; i += 32 * GV_WARPS) xs[gv_plane(gp.off[k] + part * n + i, half)] = gp.v[k][part * n + i] * inv * gp.vw[k][part * n + i];
+                        for (uint32_t i = tid; i < n; i += 32 * GV_WARPS) xs[gv_plane(gp.off[k] + part * n + i, half)] *= inv;
                     }
                 }
             } else {
-                for (uint32_t i = tid; i < gp.len[k]; i += 32 * GV_WARPS) xs[gv_plane(gp.off[k] + i, half)] = gp.v[k][i];
+                for (uint32_t i0 = tid; i0 < gp.len[k]; i0 += AT * GV_T) {
+                    float v[AT];
+#pragma unroll
+                    for (uint32_t j = 0; j < AT; ++j) v[j] = i0 + GV_T * j < gp.len[k] ? gp.v[k][i0 + GV_T * j] : 0.0f;
+#pragma unroll
+                    for (uint32_t j = 0; j < AT; ++j)
+                        if (i0 + GV_T * j < gp.len[k]) xs[gv_plane(gp.off[k] + i0 + GV_T * j, half)] = v[j];
+                }
             }
         }
     }
@@ -338,6 +432,88 @@ struct TcShape {
     static constexpr uint32_t NS = BN == 256 ? 4 : (BN == 128 ? 6 : 8);
     static constexpr size_t SMEM = (size_t)NS * STAGE + EPI_BYTES + 1024;
 };
+
+// One warp's 32 tokens (from tok on) of a finished accumulator, ncol columns, by way of the warp's stage of shared memory. A kind
+// of its own for each of: bias, squared relu, scale and residual; gated rows; gelu times a factor; everything else. (What a kind
+// does not have is not in its loop, whose loads and stores can then overlap.)
+enum { EPI_PLAIN, EPI_GATED, EPI_GELU_MUL, EPI_ANY };
+template <int EPI>
+__device__ __forceinline__ void tile_out(const TcProblem &p, uint32_t acc, float *stage, uint32_t row0, uint32_t ncol, uint32_t tok, int lane) {
+    const uint32_t tr = lane >> 3, tc = (lane & 7) * 4;  // this lane's row and columns of the turned block
+    const uint32_t out_rows = EPI == EPI_GATED ? p.rows / 2 : p.rows;
+    for (uint32_t c0 = 0; c0 < ncol; c0 += EPI == EPI_GATED ? 64 : 32) {
+        uint32_t v[32];
+        tc_ld32(acc + c0, v);
+        if (EPI == EPI_GATED) {
+            uint32_t u[32];
+            tc_ld32(acc + c0 + 32, u);
+#pragma unroll
+            for (int e = 0; e < 32; ++e) {
+                const float g = __uint_as_float(v[e]);
+                v[e] = __float_as_uint(__fdividef(g, 1.0f + __expf(-g)) * __uint_as_float(u[e]));
+            }
+        }
+#pragma unroll
+        for (int g = 0; g < 8; ++g)
+            *reinterpret_cast<float4 *>(stage + lane * EPI_LD + 4 * g) =
+                make_float4(__uint_as_float(v[4 * g]), __uint_as_float(v[4 * g + 1]), __uint_as_float(v[4 * g + 2]), __uint_as_float(v[4 * g + 3]));
+        __syncwarp();
+        const uint32_t r = (EPI == EPI_GATED ? (row0 + c0) / 2 : row0 + c0) + tc;
+        float bias[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) bias[e] = (EPI != EPI_GATED && EPI != EPI_GELU_MUL && p.bias && r + e < out_rows) ? p.bias[r + e] : 0.0f;
+        const bool vec = r + 4 <= out_rows && (p.ldy & 3) == 0;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const uint32_t t = tok + 4 * i + tr;
+            if (t < p.tokens && r < out_rows) {
+                const float4 a = *reinterpret_cast<const float4 *>(stage + (4 * i + tr) * EPI_LD + tc);
+                float o[4] = {a.x, a.y, a.z, a.w};
+                if (EPI == EPI_PLAIN) {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        o[e] += bias[e];
+                        if (p.act == LINEAR_ACT_RELU2) {
+                            o[e] = fmaxf(o[e], 0.0f);
+                            o[e] *= o[e];
+                        }
+                        o[e] *= p.scale;
+                    }
+                }
+                if (EPI == EPI_GELU_MUL) {
+                    const uint16_t *f = p.mul + (size_t)p.mul_ids[t] * p.ldm + r;
+                    float m[4];
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) m[e] = r + e < out_rows ? __uint_as_float((uint32_t)f[e] << 16) : 0.0f;
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) o[e] = __fdividef(o[e], 1.0f + __expf(-1.5957691216057308f * fmaf(0.044715f * o[e] * o[e], o[e], o[e]))) * m[e];
+                }
+                if (EPI == EPI_ANY) {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) o[e] = finish(o[e] + bias[e], p.act, p.scale, p.cap);
+                    if (p.mul)
+                        for (int e = 0; e < 4 && r + e < out_rows; ++e) o[e] *= mul_at(p.mul, p.ldm, p.mul_ids[t], r + e);
+                }
+                const size_t at = (size_t)t * p.ldy + r;
+                if (vec) {
+                    if (EPI != EPI_GATED && EPI != EPI_GELU_MUL && p.resid) {
+                        const float4 z = *reinterpret_cast<const float4 *>(p.resid + at);
+                        o[0] += z.x; o[1] += z.y; o[2] += z.z; o[3] += z.w;
+                    }
+                    if (p.y_bf16) *reinterpret_cast<uint2 *>(static_cast<__nv_bfloat16 *>(p.y) + at) = make_uint2(bf16_pack(o[0], o[1]), bf16_pack(o[2], o[3]));
+                    else *reinterpret_cast<float4 *>(static_cast<float *>(p.y) + at) = make_float4(o[0], o[1], o[2], o[3]);
+                } else {
+                    for (int e = 0; e < 4 && r + e < out_rows; ++e) {
+                        if (EPI != EPI_GATED && EPI != EPI_GELU_MUL && p.resid) o[e] += p.resid[at + e];
+                        if (p.y_bf16) static_cast<__nv_bfloat16 *>(p.y)[at + e] = __float2bfloat16_rn(o[e]);
+                        else static_cast<float *>(p.y)[at + e] = o[e];
+                    }
+                }
+            }
+        }
+        __syncwarp();
+    }
+}
 
 template <int BN>
 __global__ void __launch_bounds__(256, 1) linear_tc_kernel(const __grid_constant__ TcParams tp) {
@@ -439,7 +615,6 @@ __global__ void __launch_bounds__(256, 1) linear_tc_kernel(const __grid_constant
     } else if (warp >= 4) {
         const uint32_t q = warp & 3;
         float *stage = reinterpret_cast<float *>(smem + NS * STAGE) + q * 32 * EPI_LD;
-        const uint32_t tr = lane >> 3, tc = (lane & 7) * 4;  // this lane's row and columns of the turned block
         uint32_t seq = 0;
         bool ok = true;
         for (uint32_t tile = blockIdx.x; tile < tp.tiles && ok; tile += gridDim.x, ++seq) {
@@ -449,56 +624,13 @@ __global__ void __launch_bounds__(256, 1) linear_tc_kernel(const __grid_constant
             ok = __all_sync(0xffffffffu, wait(&acc_full[buf], (seq >> 1) & 1));
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const uint32_t ncol = min((uint32_t)BN, p.rows - row0);
-            const bool live = tok0 + 32 * q < p.tokens, glu = p.act == LINEAR_ACT_SWIGLU;
-            const uint32_t out_rows = glu ? p.rows / 2 : p.rows;
-            for (uint32_t c0 = 0; c0 < ncol && live; c0 += glu ? 64 : 32) {
-                uint32_t v[32];
-                tc_ld32(tmem + buf * BN + ((q * 32u) << 16) + c0, v);
-                if (glu) {
-                    uint32_t u[32];
-                    tc_ld32(tmem + buf * BN + ((q * 32u) << 16) + c0 + 32, u);
-#pragma unroll
-                    for (int e = 0; e < 32; ++e) v[e] = __float_as_uint(silu_f(__uint_as_float(v[e])) * __uint_as_float(u[e]));
-                }
-#pragma unroll
-                for (int g = 0; g < 8; ++g)
-                    *reinterpret_cast<float4 *>(stage + lane * EPI_LD + 4 * g) =
-                        make_float4(__uint_as_float(v[4 * g]), __uint_as_float(v[4 * g + 1]), __uint_as_float(v[4 * g + 2]), __uint_as_float(v[4 * g + 3]));
-                __syncwarp();
-                const uint32_t r = (glu ? (row0 + c0) / 2 : row0 + c0) + tc;
-                float bias[4];
-#pragma unroll
-                for (int e = 0; e < 4; ++e) bias[e] = (p.bias && r + e < out_rows) ? p.bias[r + e] : 0.0f;
-                const bool vec = r + 4 <= out_rows && (p.ldy & 3) == 0;
-#pragma unroll
-                for (int i = 0; i < 8; ++i) {
-                    const uint32_t tok = tok0 + 32 * q + 4 * i + tr;
-                    if (tok < p.tokens && r < out_rows) {
-                        const float4 a = *reinterpret_cast<const float4 *>(stage + (4 * i + tr) * EPI_LD + tc);
-                        float o[4] = {a.x, a.y, a.z, a.w};
-#pragma unroll
-                        for (int e = 0; e < 4; ++e) o[e] = glu ? o[e] : finish(o[e] + bias[e], p.act, p.scale, p.cap);
-                        if (p.mul)
-                            for (int e = 0; e < 4 && r + e < out_rows; ++e) o[e] *= mul_at(p.mul, p.ldm, p.mul_ids[tok], r + e);
-                        const size_t at = (size_t)tok * p.ldy + r;
-                        if (vec) {
-                            if (p.resid) {
-                                const float4 z = *reinterpret_cast<const float4 *>(p.resid + at);
-                                o[0] += z.x; o[1] += z.y; o[2] += z.z; o[3] += z.w;
-                            }
-                            if (p.y_bf16) *reinterpret_cast<uint2 *>(static_cast<__nv_bfloat16 *>(p.y) + at) = make_uint2(bf16_pack(o[0], o[1]), bf16_pack(o[2], o[3]));
-                            else *reinterpret_cast<float4 *>(static_cast<float *>(p.y) + at) = make_float4(o[0], o[1], o[2], o[3]);
-                        } else {
-                            for (int e = 0; e < 4 && r + e < out_rows; ++e) {
-                                if (p.resid) o[e] += p.resid[at + e];
-                                if (p.y_bf16) static_cast<__nv_bfloat16 *>(p.y)[at + e] = __float2bfloat16_rn(o[e]);
-                                else static_cast<float *>(p.y)[at + e] = o[e];
-                            }
-                        }
-                    }
-                }
-                __syncwarp();
+            const uint32_t ncol = min((uint32_t)BN, p.rows - row0), acc = tmem + buf * BN + ((q * 32u) << 16);
+            if (tok0 + 32 * q < p.tokens) {
+                const bool bare = !p.bias && !p.resid && p.scale == 1.0f && p.cap == 0.0f;
+                if (p.act == LINEAR_ACT_GELU_TANH && p.mul && bare) tile_out<EPI_GELU_MUL>(p, acc, stage, row0, ncol, tok0 + 32 * q, lane);
+                else if (p.act == LINEAR_ACT_SWIGLU) tile_out<EPI_GATED>(p, acc, stage, row0, ncol, tok0 + 32 * q, lane);
+                else if (p.act == LINEAR_ACT_GELU_TANH || p.cap > 0.0f || p.mul) tile_out<EPI_ANY>(p, acc, stage, row0, ncol, tok0 + 32 * q, lane);
+                else tile_out<EPI_PLAIN>(p, acc, stage, row0, ncol, tok0 + 32 * q, lane);
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             __syncwarp();
@@ -595,6 +727,7 @@ int32_t brasa_linear_launch(brasa_cmd *cmd, const LinearProblem *ps, uint32_t co
         if (q.tokens == 0 || q.rows == 0) continue;
         BRASA_REQUIRE(ctx, q.seg[0].cols > 0 && q.y && q.seg[0].x && q.seg[0].w && q.ldy >= q.out_rows(), "linear: empty or short product");
         BRASA_REQUIRE(ctx, q.act != LINEAR_ACT_SWIGLU || (q.rows % 64 == 0 && !q.bias && q.scale == 1.0f && q.cap == 0.0f), "linear: gated rows come in pairs of 32, without bias, scale and cap");
+        BRASA_REQUIRE(ctx, q.act != LINEAR_ACT_SWIGLU || (!q.mul && !q.resid), "linear: gated rows take neither a factor nor a residual");
         BRASA_REQUIRE(ctx, !q.mul || q.mul_ids, "linear: a factor's rows need token ids");
         for (int s = 0; s < 2; ++s) {
             const LinearSeg &g = q.seg[s];

@@ -1,13 +1,14 @@
 // Grouped products with bfloat16 weights (linear.cu): up to LINEAR_MAX problems in one launch, each
 //   y[t, r] = resid[t, r] + mul[ids[t], r] * softcap(scale * act(sum_c w[r, c] x[t, c] (+ sum_c w2[r, c] x2[t, c]) + bias[r]))
-// with f32 accumulation; bias, softcap(v) = cap tanh(v / cap), mul and resid are optional. Weights and activations are row-major; leading dimensions are multiples of 8 elements.
+// with f32 accumulation; bias, softcap(v) = cap tanh(v / cap), mul and resid are optional. Weights and activations are row-major;
+// leading dimensions are multiples of 8 elements.
 #pragma once
 #include "brasa_internal.h"
 
 constexpr uint32_t LINEAR_MAX = 8;
 // RELU2: relu(v)^2. GELU_TANH: 0.5 v (1 + tanh(sqrt(2 / pi) (v + 0.044715 v^3))). SWIGLU: the rows come in alternating blocks of
-// 32 gate and 32 up rows (rows a multiple of 64) and y has half as many, silu(gate) * up; many tokens only: the GEMV writes
-// both kinds of rows and the product behind it forms them from there (GemvInput::gated).
+// 32 gate and 32 up rows (rows a multiple of 64) and y has half as many, silu(gate) * up (no bias, scale, cap, mul or resid);
+// many tokens only: the GEMV writes both kinds of rows and the product behind it forms them from there (GemvInput::gated).
 enum { LINEAR_ACT_NONE = 0, LINEAR_ACT_RELU2 = 1, LINEAR_ACT_GELU_TANH = 2, LINEAR_ACT_SWIGLU = 3 };
 
 struct LinearSeg {

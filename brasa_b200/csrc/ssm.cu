@@ -7,7 +7,7 @@
 // Many tokens, bf16 mode: chunks of 64. With L_t the running sum of log a inside the chunk and S the state before it,
 //   y_t = exp(L_t) S^T C_t + sum_{s <= t} exp(L_t - L_s) dt_s (C_t . B_s) x_s + D x_t
 //   S_next = exp(L_end) S + sum_s B_s (exp(L_end - L_s) dt_s x_s)^T
-// ssm_conv_kernel: convolutions, dt, L. ssm_state_kernel: the second line through the chunks, one block per head and 32 value
+// ssm_conv_kernel: convolutions, dt, L. ssm_state_kernel: the second line through the chunks, one block per head and 16 value
 // columns, the state in the accumulators; the state before every chunk goes out as two bf16 terms (16 bits and more).
 // ssm_chunk_kernel: the first line, all chunks and heads side by side. Products on mma.sync with f32 accumulation; x, B and C are
 // bf16, every f32 factor (states, weighted inputs, decayed scores) enters as two bf16 terms. ssm_out_kernel: the norm.
@@ -70,7 +70,7 @@ __global__ void __launch_bounds__(256) ssm_conv_kernel(SsmConv p) {
         if (c == UINT32_MAX) {
             for (uint32_t t = 0; t < n; ++t) elem_store(out + (size_t)t * s.ldx, 0.0f);
         } else {
-            conv_chunk(p.x, p.ldc, c, p.w, p.bias[c], t0, n, p.cv, c, [&](uint32_t t, float v) { elem_store(out + (size_t)t * s.ldx, v); });
+            conv_chunk<sizeof(T) == 2>(p.x, p.ldc, c, p.w, p.bias[c], t0, n, p.cv, c, [&](uint32_t t, float v) { elem_store(out + (size_t)t * s.ldx, v); });
         }
         return;
     }
@@ -127,6 +127,30 @@ __device__ __forceinline__ void split2(float x0, float x1, uint32_t &hi, uint32_
 
 typedef __nv_bfloat16 bf16;
 
+// 16-byte pieces of rows of `per` of them, dealt out to a block's threads one behind the other
+template <uint32_t THREADS>
+struct Pieces {
+    uint32_t row, at, per, drow, dat;
+    __device__ __forceinline__ Pieces(uint32_t tid, uint32_t per_row) : row(tid / per_row), at(tid % per_row), per(per_row), drow(THREADS / per_row), dat(THREADS % per_row) {}
+    __device__ __forceinline__ void next() {
+        row += drow;
+        at += dat;
+        if (at >= per) {
+            at -= per;
+            ++row;
+        }
+    }
+};
+// tokens 0 .. n - 1 of a chunk from src (leading dimension ld) to dst (leading dimension ldd), zeros up to SL
+template <uint32_t THREADS>
+__device__ __forceinline__ void copy_tokens(Pieces<THREADS> p, bf16 *dst, uint32_t ldd, const bf16 *src, uint32_t ld, uint32_t n) {
+    for (; p.row < SL; p.next()) {
+        bf16 *d = dst + p.row * ldd + p.at * 8;
+        if (p.row < n) cp16(d, src + (size_t)p.row * ld + p.at * 8);
+        else *reinterpret_cast<uint4 *>(d) = make_uint4(0, 0, 0, 0);
+    }
+}
+
 struct SsmState {
     SsmShape s;
     const bf16 *xbc;
@@ -138,108 +162,94 @@ struct SsmState {
     uint32_t tokens, pos0;
 };
 
-constexpr uint32_t CB = 32;  // value columns of a block
+constexpr uint32_t CB = 16, NB = 3;  // value columns of a block, chunks on their way
 
 // TPW: 16 x 16 tiles of the state per warp
 template <int TPW>
 __global__ void __launch_bounds__(256) ssm_state_kernel(SsmState p) {
     extern __shared__ __align__(16) uint8_t sm_raw[];
     const SsmShape s = p.s;
-    const uint32_t ldb = s.np + 8, h = blockIdx.x, g = h / (s.heads / s.groups), c0 = blockIdx.y * CB, nc = min(CB, s.vp - c0);
+    const uint32_t ldb = s.np + 8, h = blockIdx.x, g = h / (s.heads / s.groups), c0 = blockIdx.y * CB;
     constexpr uint32_t ldv = CB + 8;
-    bf16 *bs = (bf16 *)sm_raw, *xs = bs + 2 * SL * ldb, *xh = xs + 2 * SL * ldv, *xl = xh + SL * ldv;
-    float *lr = (float *)(xl + SL * ldv), *dts = lr + 2 * SL;  // [2][SL] each
+    bf16 *bs = (bf16 *)sm_raw, *xs = bs + NB * SL * ldb, *xh = xs + NB * SL * ldv, *xl = xh + SL * ldv;
+    float *lr = (float *)(xl + SL * ldv), *dts = lr + NB * SL;  // [NB][SL] each
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gr = lane >> 2, q = lane & 3;
-    const uint32_t mt = s.np / 16, tiles = mt * (nc / 16), chunks = (p.tokens + SL - 1) / SL;
+    const uint32_t tiles = s.np / 16, chunks = (p.tokens + SL - 1) / SL;
+    const Pieces<256> pb(tid, s.np / 8), px(tid, CB / 8);
     pdl_wait();
     pdl_launch();
     store_ring(s, p.x, p.ldc, p.ring, p.tokens, p.pos0);
-    auto fetch = [&](uint32_t chunk) {
-        const uint32_t b = chunk & 1, t0 = chunk * SL, n = min(SL, p.tokens - t0);
-        const bf16 *src = p.xbc + (size_t)t0 * s.ldx;
-        const uint32_t bo = s.heads * s.vp + g * s.np, xo = h * s.vp + c0;
-        for (uint32_t i = tid; i < SL * (s.np / 8); i += 256) {
-            const uint32_t t = i / (s.np / 8), e = i % (s.np / 8) * 8;
-            bf16 *dst = bs + (b * SL + t) * ldb + e;
-            if (t < n) cp16(dst, src + (size_t)t * s.ldx + bo + e);
-            else *reinterpret_cast<uint4 *>(dst) = make_uint4(0, 0, 0, 0);
-        }
-        for (uint32_t i = tid; i < SL * (nc / 8); i += 256) {
-            const uint32_t t = i / (nc / 8), e = i % (nc / 8) * 8;
-            bf16 *dst = xs + (b * SL + t) * ldv + e;
-            if (t < n) cp16(dst, src + (size_t)t * s.ldx + xo + e);
-            else *reinterpret_cast<uint4 *>(dst) = make_uint4(0, 0, 0, 0);
-        }
-        if (tid < 2 * SL) {
-            const size_t at = ((size_t)chunk * s.heads + h) * SL + (tid & (SL - 1));
-            cp4((tid < SL ? lr : dts) + b * SL + (tid & (SL - 1)), (tid < SL ? p.run : p.dt) + at);
+    auto fetch = [&](uint32_t chunk) {  // (a group per chunk, empty past the end: the waits below count groups)
+        if (chunk < chunks) {
+            const uint32_t b = chunk % NB, t0 = chunk * SL, n = min(SL, p.tokens - t0);
+            const bf16 *src = p.xbc + (size_t)t0 * s.ldx;
+            copy_tokens(pb, bs + b * SL * ldb, ldb, src + s.heads * s.vp + g * s.np, s.ldx, n);
+            copy_tokens(px, xs + b * SL * ldv, ldv, src + h * s.vp + c0, s.ldx, n);
+            if (tid < 2 * SL) {
+                const size_t at = ((size_t)chunk * s.heads + h) * SL + (tid & (SL - 1));
+                cp4((tid < SL ? lr : dts) + b * SL + (tid & (SL - 1)), (tid < SL ? p.run : p.dt) + at);
+            }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     fetch(0);
-    float acc[TPW][2][4];  // tile, eight columns: rows gr and gr + 8 x columns 2 q and 2 q + 1
-    auto place = [&](int i, int j, int e, uint32_t &row, uint32_t &col) {
-        const uint32_t tile = warp + 8 * i;
-        row = tile % mt * 16 + gr + 8 * (e >> 1);
-        col = tile / mt * 16 + 8 * j + 2 * q + (e & 1);
-        return tile < tiles;
-    };
+    fetch(1);
+    // tile i of the warp: rows 16 (warp + 8 i) + gr and + 8 x columns 8 j + 2 q and + 1
+    float acc[TPW][2][4];
+    auto row_of = [&](int i, int e) { return 16 * (warp + 8 * i) + gr + 8 * (e >> 1); };
+    auto col_of = [&](int j, int e) { return c0 + 8 * j + 2 * q + (e & 1); };
 #pragma unroll
     for (int i = 0; i < TPW; ++i)
 #pragma unroll
         for (int j = 0; j < 2; ++j)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                uint32_t row, col;
-                const bool live = place(i, j, e, row, col);
-                acc[i][j][e] = (live && p.pos0 != 0 && row < s.state && c0 + col < s.vdim) ? p.state[((size_t)h * s.state + row) * s.vdim + c0 + col] : 0.0f;
-            }
+            for (int e = 0; e < 4; ++e)
+                acc[i][j][e] = (p.pos0 != 0 && row_of(i, e) < s.state && col_of(j, e) < s.vdim) ? p.state[((size_t)h * s.state + row_of(i, e)) * s.vdim + col_of(j, e)] : 0.0f;
     for (uint32_t chunk = 0; chunk < chunks; ++chunk) {
-        const uint32_t b = chunk & 1;
-        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        const uint32_t b = chunk % NB;
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
         __syncthreads();  // the chunk has arrived; everything of the chunk before has been read
-        if (chunk + 1 < chunks) fetch(chunk + 1);
+        fetch(chunk + 2);
         const float end = lr[b * SL + SL - 1];
+#pragma unroll
         for (uint32_t i = tid; i < SL * (CB / 2); i += 256) {
             const uint32_t t = i / (CB / 2), e = i % (CB / 2) * 2;
-            if (e < nc) {
-                const float w = expf(end - lr[b * SL + t]) * dts[b * SL + t];
-                const uint32_t x = *reinterpret_cast<const uint32_t *>(xs + (b * SL + t) * ldv + e);
-                uint32_t hi, lo;
-                split2(bf16_lo(x) * w, bf16_hi(x) * w, hi, lo);
-                *reinterpret_cast<uint32_t *>(xh + t * ldv + e) = hi;
-                *reinterpret_cast<uint32_t *>(xl + t * ldv + e) = lo;
-            }
+            const float w = __expf(end - lr[b * SL + t]) * dts[b * SL + t];
+            const uint32_t x = *reinterpret_cast<const uint32_t *>(xs + (b * SL + t) * ldv + e);
+            uint32_t hi, lo;
+            split2(bf16_lo(x) * w, bf16_hi(x) * w, hi, lo);
+            *reinterpret_cast<uint32_t *>(xh + t * ldv + e) = hi;
+            *reinterpret_cast<uint32_t *>(xl + t * ldv + e) = lo;
         }
-        const float fade = expf(end);
+        const float fade = __expf(end);
         bf16 *out = p.before + ((size_t)chunk * s.heads + h) * 2 * s.np * s.vp;
 #pragma unroll
         for (int i = 0; i < TPW; ++i)
             if (warp + 8 * i < tiles)
 #pragma unroll
                 for (int j = 0; j < 2; ++j) {
+                    if (chunk > 0 || p.pos0 != 0)
 #pragma unroll
-                    for (int e = 0; e < 4; e += 2) {
-                        uint32_t row, col, hi, lo;
-                        place(i, j, e, row, col);
-                        split2(acc[i][j][e], acc[i][j][e + 1], hi, lo);
-                        *reinterpret_cast<uint32_t *>(out + (size_t)row * s.vp + c0 + col) = hi;
-                        *reinterpret_cast<uint32_t *>(out + (size_t)(s.np + row) * s.vp + c0 + col) = lo;
-                    }
+                        for (int e = 0; e < 4; e += 2) {
+                            uint32_t hi, lo;
+                            split2(acc[i][j][e], acc[i][j][e + 1], hi, lo);
+                            uint32_t *dst = reinterpret_cast<uint32_t *>(out + (size_t)row_of(i, e) * s.vp + col_of(j, e));
+                            dst[0] = hi;
+                            dst[s.np * s.vp / 2] = lo;
+                        }
 #pragma unroll
                     for (int e = 0; e < 4; ++e) acc[i][j][e] *= fade;
                 }
         __syncthreads();
 #pragma unroll
         for (int i = 0; i < TPW; ++i) {
-            const uint32_t tile = warp + 8 * i;
-            if (tile >= tiles) break;
-            const uint32_t n0 = tile % mt * 16, v0 = tile / mt * 16;
+            const uint32_t n0 = 16 * (warp + 8 * i);
+            if (n0 >= s.np) break;
 #pragma unroll
             for (uint32_t k0 = 0; k0 < SL; k0 += 16) {
                 uint32_t a[4], bh[4], bl[4];
                 ldm4t(a, smem_u32(bs + (b * SL + k0 + (lane & 7) + (lane >> 4) * 8) * ldb + n0 + ((lane >> 3) & 1) * 8));
-                const uint32_t at = (k0 + (lane & 7) + ((lane >> 3) & 1) * 8) * ldv + v0 + (lane >> 4) * 8;
+                const uint32_t at = (k0 + (lane & 7) + ((lane >> 3) & 1) * 8) * ldv + (lane >> 4) * 8;
                 ldm4t(bh, smem_u32(xh + at));
                 ldm4t(bl, smem_u32(xl + at));
 #pragma unroll
@@ -255,10 +265,8 @@ __global__ void __launch_bounds__(256) ssm_state_kernel(SsmState p) {
 #pragma unroll
         for (int j = 0; j < 2; ++j)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                uint32_t row, col;
-                if (place(i, j, e, row, col) && row < s.state && c0 + col < s.vdim) p.state[((size_t)h * s.state + row) * s.vdim + c0 + col] = acc[i][j][e];
-            }
+            for (int e = 0; e < 4; ++e)
+                if (row_of(i, e) < s.state && col_of(j, e) < s.vdim) p.state[((size_t)h * s.state + row_of(i, e)) * s.vdim + col_of(j, e)] = acc[i][j][e];
 }
 
 struct SsmChunk {
@@ -271,38 +279,31 @@ struct SsmChunk {
     bool empty;  // the state before the first chunk is zero
 };
 
-// Block: one chunk of one head, warp w = tokens 16 w .. 16 w + 15. VT: 16-wide blocks of the value columns.
+// Block: one chunk of one head, warps w and w + 4 = tokens 16 w .. 16 w + 15, each half of the value columns. VT: 16-wide blocks
+// of a warp's columns, at most.
 template <int VT>
-__global__ void __launch_bounds__(128) ssm_chunk_kernel(SsmChunk p) {
+__global__ void __launch_bounds__(256, 2) ssm_chunk_kernel(SsmChunk p) {
     extern __shared__ __align__(16) uint8_t sm_raw[];
     const SsmShape s = p.s;
     const uint32_t ldb = s.np + 8, ldv = s.vp + 8, chunk = blockIdx.x, h = blockIdx.y, g = h / (s.heads / s.groups), t0 = chunk * SL, n = min(SL, p.tokens - t0);
     bf16 *cs = (bf16 *)sm_raw, *bs = cs + SL * ldb, *xs = bs + SL * ldb, *sh = xs + SL * ldv, *sl = sh + s.np * ldv;
     float *lr = (float *)(sl + s.np * ldv), *dts = lr + SL;
-    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gr = lane >> 2, q = lane & 3;
+    const uint32_t tid = threadIdx.x, lane = tid & 31, warp = (tid >> 5) & 3, gr = lane >> 2, q = lane & 3;
+    const uint32_t vt = s.vp / 16, v0 = tid < 128 ? 0u : (vt + 1) / 2, nv = tid < 128 ? (vt + 1) / 2 : vt / 2;  // this warp's blocks of value columns
     const bool inter = chunk > 0 || !p.empty;
     pdl_wait();
     pdl_launch();
     {
         const bf16 *src = p.xbc + (size_t)t0 * s.ldx;
-        const uint32_t bo = s.heads * s.vp + g * s.np, co = bo + s.groups * s.np, xo = h * s.vp;
-        auto rows = [&](bf16 *dst, uint32_t ld, uint32_t off, uint32_t cols) {
-            for (uint32_t i = tid; i < SL * (cols / 8); i += 128) {
-                const uint32_t t = i / (cols / 8), e = i % (cols / 8) * 8;
-                if (t < n) cp16(dst + t * ld + e, src + (size_t)t * s.ldx + off + e);
-                else *reinterpret_cast<uint4 *>(dst + t * ld + e) = make_uint4(0, 0, 0, 0);
-            }
-        };
-        rows(cs, ldb, co, s.np);
-        rows(bs, ldb, bo, s.np);
-        rows(xs, ldv, xo, s.vp);
-        cp4((tid < SL ? lr : dts) + (tid & (SL - 1)), (tid < SL ? p.run : p.dt) + ((size_t)chunk * s.heads + h) * SL + (tid & (SL - 1)));
+        const uint32_t bo = s.heads * s.vp + g * s.np;
+        const Pieces<256> pn(tid, s.np / 8), pv(tid, s.vp / 8);
+        copy_tokens(pn, cs, ldb, src + bo + s.groups * s.np, s.ldx, n);
+        copy_tokens(pn, bs, ldb, src + bo, s.ldx, n);
+        copy_tokens(pv, xs, ldv, src + h * s.vp, s.ldx, n);
+        if (tid < 2 * SL) cp4((tid < SL ? lr : dts) + (tid & (SL - 1)), (tid < SL ? p.run : p.dt) + ((size_t)chunk * s.heads + h) * SL + (tid & (SL - 1)));
         if (inter) {
             const bf16 *st = p.before + ((size_t)chunk * s.heads + h) * 2 * s.np * s.vp;
-            for (uint32_t i = tid; i < 2 * s.np * (s.vp / 8); i += 128) {
-                const uint32_t r = i / (s.vp / 8), e = i % (s.vp / 8) * 8;
-                cp16(sh + r * ldv + e, st + (size_t)r * s.vp + e);  // (lo rows follow the hi rows in both)
-            }
+            for (Pieces<256> r = pv; r.row < 2 * s.np; r.next()) cp16(sh + r.row * ldv + r.at * 8, st + (size_t)r.row * s.vp + r.at * 8);  // (lo rows follow the hi rows in both)
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
         asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -324,8 +325,8 @@ __global__ void __launch_bounds__(128) ssm_chunk_kernel(SsmChunk p) {
         if (inter)
 #pragma unroll
             for (int c = 0; c < VT; ++c)
-                if (16 * c < (int)s.vp) {
-                    const uint32_t at = (k0 + (lane & 7) + ((lane >> 3) & 1) * 8) * ldv + 16 * c + (lane >> 4) * 8;
+                if (c < (int)nv) {
+                    const uint32_t at = (k0 + (lane & 7) + ((lane >> 3) & 1) * 8) * ldv + 16 * (v0 + c) + (lane >> 4) * 8;
                     uint32_t bh[4], bl[4];
                     ldm4t(bh, smem_u32(sh + at));
                     ldm4t(bl, smem_u32(sl + at));
@@ -338,7 +339,7 @@ __global__ void __launch_bounds__(128) ssm_chunk_kernel(SsmChunk p) {
     }
     const float l0 = lr[row0 + gr], l1 = lr[row0 + gr + 8];
     if (inter) {
-        const float f0 = expf(l0), f1 = expf(l1);
+        const float f0 = __expf(l0), f1 = __expf(l1);
 #pragma unroll
         for (int c = 0; c < VT; ++c)
 #pragma unroll
@@ -361,16 +362,16 @@ __global__ void __launch_bounds__(128) ssm_chunk_kernel(SsmChunk p) {
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const uint32_t t = row0 + gr + 8 * (e >> 1), ss = c + (e & 1);
-                    m[e] = ss <= t ? gg[e] * expf((e >> 1 ? l1 : l0) - lr[ss]) * dts[ss] : 0.0f;
+                    m[e] = ss <= t ? gg[e] * __expf((e >> 1 ? l1 : l0) - lr[ss]) * dts[ss] : 0.0f;
                 }
                 split2(m[0], m[1], ah[2 * half], al[2 * half]);
                 split2(m[2], m[3], ah[2 * half + 1], al[2 * half + 1]);
             }
 #pragma unroll
             for (int c = 0; c < VT; ++c)
-                if (16 * c < (int)s.vp) {
+                if (c < (int)nv) {
                     uint32_t b[4];
-                    ldm4t(b, smem_u32(xs + (16 * j + (lane & 7) + ((lane >> 3) & 1) * 8) * ldv + 16 * c + (lane >> 4) * 8));
+                    ldm4t(b, smem_u32(xs + (16 * j + (lane & 7) + ((lane >> 3) & 1) * 8) * ldv + 16 * (v0 + c) + (lane >> 4) * 8));
 #pragma unroll
                     for (int k = 0; k < 2; ++k) {
                         mma_bf16(y[c][k], al, b[2 * k], b[2 * k + 1]);
@@ -386,18 +387,18 @@ __global__ void __launch_bounds__(128) ssm_chunk_kernel(SsmChunk p) {
         for (int j = 0; j < 2; ++j)
 #pragma unroll
             for (int e = 0; e < 4; e += 2) {
-                const uint32_t t = row0 + gr + 4 * e, col = 16 * c + 8 * j + 2 * q;
-                if (t >= n || col >= s.vdim) continue;
+                const uint32_t t = row0 + gr + 4 * e, col = 16 * (v0 + c) + 8 * j + 2 * q;
+                if (c >= (int)nv || t >= n || col >= s.vdim) continue;
                 const uint32_t x = *reinterpret_cast<const uint32_t *>(xs + t * ldv + col);
                 const float v0 = fmaf(D, bf16_lo(x), y[c][j][e]), v1 = fmaf(D, bf16_hi(x), y[c][j][e + 1]);
                 const float *z = p.z + (size_t)(t0 + t) * p.ldz + h * s.vdim + col;
                 float *dst = p.y + (size_t)(t0 + t) * s.inner + h * s.vdim + col;
                 if (pair) {
                     const float2 zz = *reinterpret_cast<const float2 *>(z);
-                    *reinterpret_cast<float2 *>(dst) = make_float2(v0 * silu_f(zz.x), v1 * silu_f(zz.y));
+                    *reinterpret_cast<float2 *>(dst) = make_float2(v0 * silu_fast(zz.x), v1 * silu_fast(zz.y));
                 } else {
-                    dst[0] = v0 * silu_f(z[0]);
-                    if (col + 1 < s.vdim) dst[1] = v1 * silu_f(z[1]);
+                    dst[0] = v0 * silu_fast(z[0]);
+                    if (col + 1 < s.vdim) dst[1] = v1 * silu_fast(z[1]);
                 }
             }
 }
@@ -521,10 +522,12 @@ struct SsmStep {
     const uint32_t *pos;
 };
 
-// Block: 32 value columns (lanes) of one head; warp w owns the state's rows w, w + 8, .., which are read ahead of the kernel
+constexpr uint32_t SW = 16;  // warps of a block
+
+// Block: 32 value columns (lanes) of one head; warp w owns the state's rows w, w + SW, .., which are read ahead of the kernel
 // before this one: the last to write them was the token before.
 template <int R>
-__global__ void __launch_bounds__(256) ssm_step_kernel(SsmStep p) {
+__global__ void __launch_bounds__(32 * SW) ssm_step_kernel(SsmStep p) {
     extern __shared__ __align__(16) float sm[];
     const SsmShape s = p.s;
     float *bs = sm, *cs = bs + s.state, *xs = cs + s.state, *part = xs + 32;
@@ -533,17 +536,17 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(SsmStep p) {
     float *state = p.state + (size_t)h * s.state * s.vdim + c0 + lane;
     float S[R];
 #pragma unroll
-    for (int i = 0; i < R; ++i) S[i] = (col && warp + 8 * i < s.state) ? state[(size_t)(warp + 8 * i) * s.vdim] : 0.0f;
+    for (int i = 0; i < R; ++i) S[i] = (col && warp + SW * i < s.state) ? state[(size_t)(warp + SW * i) * s.vdim] : 0.0f;
     pdl_wait();
     pdl_launch();
-    const uint32_t pos = *p.pos, nx = min(32u, s.vdim - c0);
+    const uint32_t pos = *p.pos, slot = pos % s.taps, nx = min(32u, s.vdim - c0);
     const ConvView cv{p.ring, s.channels, s.taps, pos};
     const bool keeper = h % share == 0 && blockIdx.y == 0;  // stores the group's B and C inputs (nobody reads this row in this step)
-    for (uint32_t i = tid; i < 2 * s.state + nx; i += 256) {
+    for (uint32_t i = tid; i < 2 * s.state + nx; i += 32 * SW) {
         const uint32_t c = i < s.state ? s.inner + g * s.state + i
                                        : (i < 2 * s.state ? s.inner + (s.groups + g) * s.state + i - s.state : h * s.vdim + c0 + i - 2 * s.state);
-        (i < s.state ? bs[i] : (i < 2 * s.state ? cs[i - s.state] : xs[i - 2 * s.state])) = silu_f(conv_at(p.x, 0, c, p.w, 0, cv, c) + p.bias[c]);
-        if (keeper || i >= 2 * s.state) p.ring[(size_t)(pos % s.taps) * s.channels + c] = p.x[c];
+        (i < s.state ? bs[i] : (i < 2 * s.state ? cs[i - s.state] : xs[i - 2 * s.state])) = silu_f(conv_step(p.x, c, p.w, cv, slot, c) + p.bias[c]);
+        if (keeper || i >= 2 * s.state) p.ring[(size_t)slot * s.channels + c] = p.x[c];
     }
     const float dt = softplus_f(p.dt_raw[h] + p.dt_bias[h]), f = pos == 0 ? 0.0f : expf(-expf(p.a_log[h]) * dt);
     __syncthreads();
@@ -551,7 +554,7 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(SsmStep p) {
     float y = 0.0f;
 #pragma unroll
     for (int i = 0; i < R; ++i) {
-        const uint32_t row = warp + 8 * i;
+        const uint32_t row = warp + SW * i;
         if (row < s.state) {
             S[i] = fmaf(bs[row], x, pos == 0 ? 0.0f : S[i] * f);
             y = fmaf(S[i], cs[row], y);
@@ -562,7 +565,7 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(SsmStep p) {
     __syncthreads();
     if (tid < nx) {
         y = p.D[h] * xs[tid];
-        for (uint32_t w = 0; w < 8; ++w) y += part[w * 32 + tid];
+        for (uint32_t w = 0; w < SW; ++w) y += part[w * 32 + tid];
         p.y[h * s.vdim + c0 + tid] = y * silu_f(p.z[h * s.vdim + c0 + tid]);
     }
 }
@@ -664,18 +667,18 @@ class StateSpace : public Mixer {
             const bf16 *xbc = (const bf16 *)(r.scratch + at_.xbc);
             bf16 *before = (bf16 *)(r.scratch + at_.before);
             SsmState sp{s_, xbc, f(at_.dt), f(at_.run), f(at_.c), ldc_, ring_, state_, before, r.tokens, r.pos0};
-            const size_t ssm = (size_t)(2 * SL * (s_.np + 8) + 4 * SL * (CB + 8)) * 2 + 4 * SL * 4;
-            const dim3 grid(s_.heads, (s_.vp + CB - 1) / CB);
-            auto state = s_.np <= 128 ? ssm_state_kernel<2> : ssm_state_kernel<4>;
+            const size_t ssm = (size_t)(NB * SL * (s_.np + 8) + (NB + 2) * SL * (CB + 8)) * 2 + 2 * NB * SL * 4;
+            const dim3 grid(s_.heads, s_.vp / CB);
+            auto state = s_.np <= 128 ? ssm_state_kernel<1> : ssm_state_kernel<2>;
             BRASA_TRY(brasa_smem_optin(ctx, (const void *)state, std::max<size_t>(ssm, 48 * 1024)));
             BRASA_CUDA(ctx, brasa_launch_dependent(ctx, state, grid, dim3(256), ssm, sp));
             BRASA_TRY(brasa_post_launch(r.cmd, "ssm_state"));
             SsmChunk kp{s_, xbc, before, f(at_.dt), f(at_.run), f(at_.z), d_, ldz_, f(at_.y), r.tokens, r.pos0 == 0};
             const size_t csm = (size_t)(2 * SL * (s_.np + 8) + (SL + 2 * s_.np) * (s_.vp + 8)) * 2 + 2 * SL * 4;
             BRASA_REQUIRE(ctx, csm + 1024 <= ctx->smem_optin, "state space: sizes too large");
-            auto chunk = s_.vp <= 64 ? ssm_chunk_kernel<4> : ssm_chunk_kernel<8>;
+            auto chunk = s_.vp <= 64 ? ssm_chunk_kernel<2> : ssm_chunk_kernel<4>;
             BRASA_TRY(brasa_smem_optin(ctx, (const void *)chunk, std::max<size_t>(csm, 48 * 1024)));
-            BRASA_CUDA(ctx, brasa_launch_dependent(ctx, chunk, dim3(chunks, s_.heads), dim3(128), csm, kp));
+            BRASA_CUDA(ctx, brasa_launch_dependent(ctx, chunk, dim3(chunks, s_.heads), dim3(256), csm, kp));
             BRASA_TRY(brasa_post_launch(r.cmd, "ssm_chunk"));
         } else {
             SsmScan sp{s_, r.scratch + at_.xbc, f(at_.c), f(at_.dt_raw), dt_bias_, a_log_, f(at_.z), d_, ldc_, lddt_, ldz_, ring_, state_, f(at_.y), r.tokens, r.pos0};
@@ -694,9 +697,9 @@ class StateSpace : public Mixer {
         brasa_ctx *ctx = r.cmd->ctx;
         auto f = [&](uint64_t at) { return (float *)(r.scratch + at); };
         SsmStep p{s_, f(at_.c), f(at_.dt_raw), f(at_.z), w_, bias_, dt_bias_, a_log_, d_, ring_, state_, (float *)r.out[0], r.dev_pos};
-        const size_t smem = (size_t)(2 * s_.state + 32 + 8 * 32) * 4;
-        auto kernel = s_.state <= 128 ? ssm_step_kernel<16> : (s_.state <= 256 ? ssm_step_kernel<32> : ssm_step_kernel<64>);
-        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, kernel, dim3(s_.heads, (s_.vdim + 31) / 32), dim3(256), smem, p));
+        const size_t smem = (size_t)(2 * s_.state + 32 + SW * 32) * 4;
+        auto kernel = s_.state <= 128 ? ssm_step_kernel<8> : (s_.state <= 256 ? ssm_step_kernel<16> : ssm_step_kernel<32>);
+        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, kernel, dim3(s_.heads, (s_.vdim + 31) / 32), dim3(32 * SW), smem, p));
         return brasa_post_launch(r.cmd, "ssm_step");
     }
 

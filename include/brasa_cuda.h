@@ -217,7 +217,7 @@ int32_t brasa_k_add_rms_norm(brasa_cmd *cmd, brasa_arg x, brasa_arg y, brasa_arg
 /* y[t, r] = resid[t, r] + mul[mul_ids[t], r] * softcap(scale * act(w[r, :] . x[t, :] (+ w2[r, :] . x2[t, :]) + bias[r])) with bf16
  * row-major weights; softcap(v) = cap tanh(v / cap), cap 0: none. Leading dimensions in elements, multiples of 8 (ldm: any).
  * Optional parts have buf NULL (w2: cols2 = 0). SWIGLU: the rows are alternating blocks of 32 gate and 32 up rows, y has rows / 2
- * columns silu(gate) * up (no bias, scale or cap). The ids must lie inside mul's mul_rows rows. */
+ * columns silu(gate) * up (no bias, scale, cap, mul or resid). The ids must lie inside mul's mul_rows rows. */
 enum brasa_linear_act { BRASA_ACT_NONE = 0, BRASA_ACT_RELU2 = 1 /* relu(v)^2 */, BRASA_ACT_GELU_TANH = 2, BRASA_ACT_SWIGLU = 3 };
 typedef struct brasa_linear {
     brasa_arg w, x, w2, x2, y, bias, resid; /* bias f32[rows]; resid f32[tokens][ldy], may be y */
