@@ -101,18 +101,19 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(DeltaChunk p) {
                 gh[tid] = tid < n ? expf(-a * softplus_f(p.z[(size_t)(t0 + tid) * p.ldz + h])) : 1.0f;
                 if (tid < n) p.g[(size_t)(t0 + tid) * s.heads + h] = gh[tid];
             }
-        } else
-        for (uint32_t t = warp; t < CH; t += 8)
+        } else {
+            for (uint32_t t = warp; t < CH; t += 8)
 #pragma unroll
-            for (int j = 0; j < E; ++j) {
-                const uint32_t e = lane + 32 * j;
-                float g = 1.0f;
-                if (t < n && e < s.dim) {
-                    g = expf(-a * softplus_f(p.z[(size_t)(t0 + t) * p.ldz + h * s.dim + e]));
-                    p.g[((size_t)(t0 + t) * s.heads + h) * s.dim + e] = g;
+                for (int j = 0; j < E; ++j) {
+                    const uint32_t e = lane + 32 * j;
+                    float g = 1.0f;
+                    if (t < n && e < s.dim) {
+                        g = expf(-a * softplus_f(p.z[(size_t)(t0 + t) * p.ldz + h * s.dim + e]));
+                        p.g[((size_t)(t0 + t) * s.heads + h) * s.dim + e] = g;
+                    }
+                    sg[t * D + e] = g;
                 }
-                sg[t * D + e] = g;
-            }
+        }
         if (tid < CH) beta[tid] = tid < n ? sigmoid_f(p.b[(size_t)(t0 + tid) * p.ldb + h]) : 0.0f;
     }
     __syncthreads();
@@ -714,8 +715,7 @@ __global__ void __launch_bounds__(256) delta_out_kernel(const float *o, const fl
     float ss = 0.0f;
     for (uint32_t e = lane; e < vdim; e += 32) ss = fmaf(x[e], x[e], ss);
     const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + eps);
-    for (uint32_t e = lane; e < vdim; e += 32)
-    {
+    for (uint32_t e = lane; e < vdim; e += 32) {
         const float z = gate[(size_t)t * ldg + h * vdim + e];
         elem_store(out + (size_t)t * ldo + h * vdim + e, x[e] * inv * w[e] * (SILU ? silu_f(z) : sigmoid_f(z)));
     }

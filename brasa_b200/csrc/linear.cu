@@ -223,27 +223,27 @@ __global__ void __launch_bounds__(32 * GV_WARPS, 1) linear_gemv_kernel(const __g
                 }
             }
         } else {
-        if (gp.y) {
+            if (gp.y) {
 #pragma unroll
-            for (uint32_t j = 0; j < GV_KEEP; ++j) s = fmaf(yk[j], yk[j], s);
-            const float sy = 1.0f / sqrtf(block_sum_1024(s, red) / (float)gp.width + gp.eps);
-            s = 0.0f;
+                for (uint32_t j = 0; j < GV_KEEP; ++j) s = fmaf(yk[j], yk[j], s);
+                const float sy = 1.0f / sqrtf(block_sum_1024(s, red) / (float)gp.width + gp.eps);
+                s = 0.0f;
 #pragma unroll
-            for (uint32_t j = 0; j < GV_KEEP; ++j) {
-                const uint32_t i = tid + GV_T * j;
-                xk[j] = fmaf(yk[j] * sy, wyk[j], xk[j]);
-                if (blockIdx.x == 0 && gp.x_out && i < gp.width) gp.x_out[i] = xk[j];
+                for (uint32_t j = 0; j < GV_KEEP; ++j) {
+                    const uint32_t i = tid + GV_T * j;
+                    xk[j] = fmaf(yk[j] * sy, wyk[j], xk[j]);
+                    if (blockIdx.x == 0 && gp.x_out && i < gp.width) gp.x_out[i] = xk[j];
+                }
             }
-        }
-        float inv = 1.0f;
-        if (gp.norm == GEMV_RMS_NORM) {
+            float inv = 1.0f;
+            if (gp.norm == GEMV_RMS_NORM) {
 #pragma unroll
-            for (uint32_t j = 0; j < GV_KEEP; ++j) s = fmaf(xk[j], xk[j], s);
-            inv = 1.0f / sqrtf(block_sum_1024(s, red) / (float)gp.width + gp.eps);
-        }
+                for (uint32_t j = 0; j < GV_KEEP; ++j) s = fmaf(xk[j], xk[j], s);
+                inv = 1.0f / sqrtf(block_sum_1024(s, red) / (float)gp.width + gp.eps);
+            }
 #pragma unroll
-        for (uint32_t j = 0; j < GV_KEEP; ++j)
-            if (tid + GV_T * j < gp.width) xs[gv_plane(gp.off[0] + tid + GV_T * j, half)] = xk[j] * inv * wk[j];
+            for (uint32_t j = 0; j < GV_KEEP; ++j)
+                if (tid + GV_T * j < gp.width) xs[gv_plane(gp.off[0] + tid + GV_T * j, half)] = xk[j] * inv * wk[j];
         }
     } else if (gp.x) {
         // the residual stream, with the pending sublayer's normed result added; every thread keeps to its own elements
@@ -463,6 +463,16 @@ __device__ __forceinline__ void tile_out(const TcProblem &p, uint32_t acc, float
 #pragma unroll
         for (int e = 0; e < 4; ++e) bias[e] = (EPI != EPI_GATED && EPI != EPI_GELU_MUL && p.bias && r + e < out_rows) ? p.bias[r + e] : 0.0f;
         const bool vec = r + 4 <= out_rows && (p.ldy & 3) == 0;
+        uint16_t f[8][4];  // the factors, all asked for at once
+        if (EPI == EPI_GELU_MUL) {
+            uint32_t id[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) id[i] = tok + 4 * i + tr < p.tokens ? p.mul_ids[tok + 4 * i + tr] : 0u;
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) f[i][e] = tok + 4 * i + tr < p.tokens && r + e < out_rows ? p.mul[(size_t)id[i] * p.ldm + r + e] : (uint16_t)0;
+        }
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
             const uint32_t t = tok + 4 * i + tr;
@@ -481,12 +491,9 @@ __device__ __forceinline__ void tile_out(const TcProblem &p, uint32_t acc, float
                     }
                 }
                 if (EPI == EPI_GELU_MUL) {
-                    const uint16_t *f = p.mul + (size_t)p.mul_ids[t] * p.ldm + r;
-                    float m[4];
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) m[e] = r + e < out_rows ? __uint_as_float((uint32_t)f[e] << 16) : 0.0f;
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) o[e] = __fdividef(o[e], 1.0f + __expf(-1.5957691216057308f * fmaf(0.044715f * o[e] * o[e], o[e], o[e]))) * m[e];
+                    for (int e = 0; e < 4; ++e)
+                        o[e] = __fdividef(o[e], 1.0f + __expf(-1.5957691216057308f * fmaf(0.044715f * o[e] * o[e], o[e], o[e]))) * __uint_as_float((uint32_t)f[i][e] << 16);
                 }
                 if (EPI == EPI_ANY) {
 #pragma unroll

@@ -358,46 +358,46 @@ __global__ void __launch_bounds__(288, 1) window_tc_kernel(const __grid_constant
                     }
                 }
             } else {
-            float tmax = -INFINITY;
+                float tmax = -INFINITY;
 #pragma unroll
-            for (int cc = 0; cc < 2; ++cc) {
-                uint32_t v[32];
-                tc_ld32(ts + 32 * cc, v);
-                if (free_tile) {
+                for (int cc = 0; cc < 2; ++cc) {
+                    uint32_t v[32];
+                    tc_ld32(ts + 32 * cc, v);
+                    if (free_tile) {
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) tmax = fmaxf(tmax, __uint_as_float(v[i]) * sl);
-                } else {
+                        for (int i = 0; i < 32; ++i) tmax = fmaxf(tmax, __uint_as_float(v[i]) * sl);
+                    } else {
 #pragma unroll
-                    for (int i = 0; i < 32; ++i)
-                        if (32 * cc + i <= hib && 32 * cc + i >= lob) tmax = fmaxf(tmax, __uint_as_float(v[i]) * sl);
-                }
-            }
-            pair_max[cgrp][row] = tmax;
-            asm volatile("bar.sync %0, %1;" ::"r"(1 + (warp & 3)), "r"(64) : "memory");  // the two warps that share these rows
-            tmax = fmaxf(pair_max[0][row], pair_max[1][row]);
-            if (tmax > m + SLACK || (m == -INFINITY && tmax != -INFINITY)) {
-                move = m != -INFINITY;
-                rescale = move ? ex2(m - tmax) : 1.0f;
-                l *= rescale;
-                m = tmax;
-            }
-            const float mneg = m == -INFINITY ? 0.0f : -m;
-#pragma unroll
-            for (int cc = 0; cc < 2; ++cc) {
-                uint32_t v[32];
-                tc_ld32(ts + 32 * cc, v);
-#pragma unroll
-                for (int i = 0; i < 32; i += 2) {
-                    float p0 = ex2(fmaf(__uint_as_float(v[i]), sl, mneg)), p1 = ex2(fmaf(__uint_as_float(v[i + 1]), sl, mneg));
-                    if (!free_tile) {
-                        const int c = 32 * cc + i;
-                        if (c > hib || c < lob) p0 = 0.0f;
-                        if (c + 1 > hib || c + 1 < lob) p1 = 0.0f;
+                        for (int i = 0; i < 32; ++i)
+                            if (32 * cc + i <= hib && 32 * cc + i >= lob) tmax = fmaxf(tmax, __uint_as_float(v[i]) * sl);
                     }
-                    l += p0 + p1;
-                    split_bf16(p0, p1, hi[16 * cc + i / 2], lo_[16 * cc + i / 2]);
                 }
-            }
+                pair_max[cgrp][row] = tmax;
+                asm volatile("bar.sync %0, %1;" ::"r"(1 + (warp & 3)), "r"(64) : "memory");  // the two warps that share these rows
+                tmax = fmaxf(pair_max[0][row], pair_max[1][row]);
+                if (tmax > m + SLACK || (m == -INFINITY && tmax != -INFINITY)) {
+                    move = m != -INFINITY;
+                    rescale = move ? ex2(m - tmax) : 1.0f;
+                    l *= rescale;
+                    m = tmax;
+                }
+                const float mneg = m == -INFINITY ? 0.0f : -m;
+#pragma unroll
+                for (int cc = 0; cc < 2; ++cc) {
+                    uint32_t v[32];
+                    tc_ld32(ts + 32 * cc, v);
+#pragma unroll
+                    for (int i = 0; i < 32; i += 2) {
+                        float p0 = ex2(fmaf(__uint_as_float(v[i]), sl, mneg)), p1 = ex2(fmaf(__uint_as_float(v[i + 1]), sl, mneg));
+                        if (!free_tile) {
+                            const int c = 32 * cc + i;
+                            if (c > hib || c < lob) p0 = 0.0f;
+                            if (c + 1 > hib || c + 1 < lob) p1 = 0.0f;
+                        }
+                        l += p0 + p1;
+                        split_bf16(p0, p1, hi[16 * cc + i / 2], lo_[16 * cc + i / 2]);
+                    }
+                }
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
         }
