@@ -128,7 +128,9 @@ __device__ __forceinline__ float block_sum_1024(float v, float *red) {
     return v;
 }
 
-template <int S>
+// IN: what the input is formed from.
+enum { IN_VECTORS, IN_STREAM, IN_LAYER_NORM };
+template <int S, int IN>
 __global__ void __launch_bounds__(32 * GV_WARPS, 1) linear_gemv_kernel(const __grid_constant__ GemvDevParams gp) {
     extern __shared__ __align__(16) float xs[];
     __shared__ float red[32], part[2][GV_WARPS];
@@ -180,30 +182,30 @@ __global__ void __launch_bounds__(32 * GV_WARPS, 1) linear_gemv_kernel(const __g
     // ---- the input vectors ----
     // Up to GV_KEEP values of the residual stream per thread stay in registers, with the constants asked for ahead of the wait.
     constexpr uint32_t GV_KEEP = 4, GV_T = 32 * GV_WARPS;
-    const bool layer_norm = gp.norm == GEMV_LAYER_NORM, keep = gp.x && !(layer_norm && gp.y) && gp.width <= GV_KEEP * GV_T;
-    float xk[GV_KEEP], yk[GV_KEEP], wk[GV_KEEP], wyk[GV_KEEP];  // layer norm: yk and wyk hold the second form's and the first's constants
-    if (keep)
+    constexpr bool LN = IN == IN_LAYER_NORM;
+    const bool keep = gp.width <= GV_KEEP * GV_T;
+    float xk[GV_KEEP], yk[GV_KEEP], wk[GV_KEEP], bk[GV_KEEP];
+    if (IN != IN_VECTORS && keep)
 #pragma unroll
         for (uint32_t j = 0; j < GV_KEEP; ++j) {
             const uint32_t i = tid + GV_T * j;
-            const float *wy = layer_norm ? gp.b[0] : (gp.y ? gp.wy : nullptr);
-            wk[j] = gp.norm != GEMV_PLAIN && i < gp.width ? gp.w[0][i] : 1.0f;
-            wyk[j] = wy && i < gp.width ? wy[i] : 0.0f;
-            yk[j] = layer_norm && gp.nin > 1 && i < gp.width ? gp.w[1][i] : 0.0f;
+            const float *b = LN ? gp.b[0] : (gp.y ? gp.wy : nullptr);
+            wk[j] = (LN || gp.norm == GEMV_RMS_NORM) && i < gp.width ? gp.w[0][i] : 1.0f;
+            bk[j] = b && i < gp.width ? b[i] : 0.0f;
         }
     pdl_wait();
     pdl_launch();
     for (uint32_t k = 0; k < gp.nin; ++k)  // padding
         if (tid < 8 && (gp.len[k] & 7) && gp.len[k] / 8 * 8 + tid >= gp.len[k]) xs[gv_plane(gp.off[k] + gp.len[k] / 8 * 8 + tid, half)] = 0.0f;
-    if (keep) {
+    if (IN != IN_VECTORS && keep) {
         float s = 0.0f;
 #pragma unroll
         for (uint32_t j = 0; j < GV_KEEP; ++j) {
             const uint32_t i = tid + GV_T * j;
             xk[j] = i < gp.width ? gp.x[i] : 0.0f;
-            if (!layer_norm) yk[j] = gp.y && i < gp.width ? gp.y[i] : 0.0f;
+            yk[j] = !LN && gp.y && i < gp.width ? gp.y[i] : 0.0f;
         }
-        if (layer_norm) {
+        if (LN) {
 #pragma unroll
             for (uint32_t j = 0; j < GV_KEEP; ++j) s += xk[j];
             const float mean = block_sum_1024(s, red) / (float)gp.width;
@@ -218,8 +220,8 @@ __global__ void __launch_bounds__(32 * GV_WARPS, 1) linear_gemv_kernel(const __g
             for (uint32_t j = 0; j < GV_KEEP; ++j) {
                 const uint32_t i = tid + GV_T * j;
                 if (i < gp.width) {
-                    xs[gv_plane(gp.off[0] + i, half)] = fmaf(xk[j] * inv, wk[j], wyk[j]);
-                    if (gp.nin > 1) xs[gv_plane(gp.off[1] + i, half)] = fmaf(xk[j] * inv, yk[j], gp.b[1][i]);
+                    xs[gv_plane(gp.off[0] + i, half)] = fmaf(xk[j] * inv, wk[j], bk[j]);
+                    if (gp.nin > 1) xs[gv_plane(gp.off[1] + i, half)] = fmaf(xk[j] * inv, gp.w[1][i], gp.b[1][i]);
                 }
             }
         } else {
@@ -231,7 +233,7 @@ __global__ void __launch_bounds__(32 * GV_WARPS, 1) linear_gemv_kernel(const __g
 #pragma unroll
                 for (uint32_t j = 0; j < GV_KEEP; ++j) {
                     const uint32_t i = tid + GV_T * j;
-                    xk[j] = fmaf(yk[j] * sy, wyk[j], xk[j]);
+                    xk[j] = fmaf(yk[j] * sy, bk[j], xk[j]);
                     if (blockIdx.x == 0 && gp.x_out && i < gp.width) gp.x_out[i] = xk[j];
                 }
             }
@@ -245,42 +247,39 @@ __global__ void __launch_bounds__(32 * GV_WARPS, 1) linear_gemv_kernel(const __g
             for (uint32_t j = 0; j < GV_KEEP; ++j)
                 if (tid + GV_T * j < gp.width) xs[gv_plane(gp.off[0] + tid + GV_T * j, half)] = xk[j] * inv * wk[j];
         }
-    } else if (gp.x) {
-        // the residual stream, with the pending sublayer's normed result added; every thread keeps to its own elements
+    } else if (IN != IN_VECTORS) {
+        // a wider stream: its values in shared memory meanwhile; every thread keeps to its own elements
         float s = 0.0f, sy = 0.0f;
-        if (gp.y) {
-            for (uint32_t i = tid; i < gp.width; i += 32 * GV_WARPS) s = fmaf(gp.y[i], gp.y[i], s);
+        if (!LN && gp.y) {
+            for (uint32_t i = tid; i < gp.width; i += GV_T) s = fmaf(gp.y[i], gp.y[i], s);
             sy = 1.0f / sqrtf(block_sum_1024(s, red) / (float)gp.width + gp.eps);
         }
         s = 0.0f;
-        for (uint32_t i = tid; i < gp.width; i += 32 * GV_WARPS) {
+        for (uint32_t i = tid; i < gp.width; i += GV_T) {
             float v = gp.x[i];
-            if (gp.y) {
+            if (!LN && gp.y) {
                 v = fmaf(gp.y[i] * sy, gp.wy[i], v);
                 if (blockIdx.x == 0 && gp.x_out) gp.x_out[i] = v;
             }
             xs[gv_plane(gp.off[0] + i, half)] = v;
-            s += gp.norm == GEMV_LAYER_NORM ? v : v * v;
+            s += LN ? v : v * v;
         }
-        if (gp.norm == GEMV_LAYER_NORM) {
+        if (LN) {
             const float mean = block_sum_1024(s, red) / (float)gp.width;
             s = 0.0f;
-            for (uint32_t i = tid; i < gp.width; i += 32 * GV_WARPS) {
+            for (uint32_t i = tid; i < gp.width; i += GV_T) {
                 const float d = xs[gv_plane(gp.off[0] + i, half)] - mean;
                 s = fmaf(d, d, s);
             }
             const float inv = 1.0f / sqrtf(block_sum_1024(s, red) / (float)gp.width + gp.eps);
-            for (uint32_t i = tid; i < gp.width; i += 32 * GV_WARPS) {
+            for (uint32_t i = tid; i < gp.width; i += GV_T) {
                 const float z = (xs[gv_plane(gp.off[0] + i, half)] - mean) * inv;
                 xs[gv_plane(gp.off[0] + i, half)] = fmaf(z, gp.w[0][i], gp.b[0][i]);
                 if (gp.nin > 1) xs[gv_plane(gp.off[1] + i, half)] = fmaf(z, gp.w[1][i], gp.b[1][i]);
             }
         } else if (gp.norm == GEMV_RMS_NORM) {
             const float inv = 1.0f / sqrtf(block_sum_1024(s, red) / (float)gp.width + gp.eps);
-            for (uint32_t i = tid; i < gp.width; i += 32 * GV_WARPS) {
-                const uint32_t at = gv_plane(gp.off[0] + i, half);
-                xs[at] = xs[at] * inv * gp.w[0][i];
-            }
+            for (uint32_t i = tid; i < gp.width; i += GV_T) xs[gv_plane(gp.off[0] + i, half)] *= inv * gp.w[0][i];
         }
     } else {
         // (loads go out several at a time, ahead of the stores to shared memory)
@@ -330,7 +329,7 @@ __global__ void __launch_bounds__(32 * GV_WARPS, 1) linear_gemv_kernel(const __g
                             }
                         }
                         const float inv = gp.vscale[k] / sqrtf(block_sum_1024(s, red) / (float)n + gp.eps);
-                        for (uint32_t i = tid; i < n; i += 32 * GV_WARPS) xs[gv_plane(gp.off[k] + part * n + i, half)] *= inv;
+                        for (uint32_t i = tid; i < n; i += GV_T) xs[gv_plane(gp.off[k] + part * n + i, half)] *= inv;
                     }
                 }
             } else {
@@ -775,7 +774,7 @@ int32_t brasa_linear_gemv_launch(brasa_cmd *cmd, const GemvInput &in, const Gemv
     GemvDevParams g;
     memset(&g, 0, sizeof g);
     auto up8 = [](uint32_t v) { return (v + 7) / 8 * 8; };
-    BRASA_REQUIRE(ctx, !in.y || (in.x && in.wy && in.x_out != in.x), "gemv: a pending sum needs its weights and a place of its own");
+    BRASA_REQUIRE(ctx, !in.y || (in.x && in.wy && in.x_out != in.x && in.norm != GEMV_LAYER_NORM), "gemv: a pending sum needs its weights, a place of its own and no layer norm");
     g.x = in.x;
     g.y = in.y;
     g.wy = in.wy;
@@ -848,18 +847,16 @@ int32_t brasa_linear_gemv_launch(brasa_cmd *cmd, const GemvInput &in, const Gemv
         }
     }
     const uint32_t grid = std::min<uint32_t>((uint32_t)ctx->sm_count, (rows * best + GV_WARPS - 1) / GV_WARPS);
-#define GEMV_LAUNCH(S)                                                                                                           \
-    do {                                                                                                                         \
-        BRASA_TRY(brasa_smem_optin(ctx, (const void *)linear_gemv_kernel<S>, std::max<size_t>(smem, 48 * 1024)));                \
-        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, linear_gemv_kernel<S>, dim3(grid), dim3(32 * GV_WARPS), smem, g));           \
-    } while (0)
-    switch (best) {
-    case 1: GEMV_LAUNCH(1); break;
-    case 2: GEMV_LAUNCH(2); break;
-    case 4: GEMV_LAUNCH(4); break;
-    default: GEMV_LAUNCH(8); break;
-    }
-#undef GEMV_LAUNCH
+    const int form = !in.x ? IN_VECTORS : (in.norm == GEMV_LAYER_NORM ? IN_LAYER_NORM : IN_STREAM);
+    auto launch = [&](void (*kernel)(GemvDevParams)) -> int32_t {
+        BRASA_TRY(brasa_smem_optin(ctx, (const void *)kernel, std::max<size_t>(smem, 48 * 1024)));
+        BRASA_CUDA(ctx, brasa_launch_dependent(ctx, kernel, dim3(grid), dim3(32 * GV_WARPS), smem, g));
+        return BRASA_OK;
+    };
+#define GEMV_KERNELS(S) {linear_gemv_kernel<S, IN_VECTORS>, linear_gemv_kernel<S, IN_STREAM>, linear_gemv_kernel<S, IN_LAYER_NORM>}
+    static void (*const kernels[4][3])(GemvDevParams) = {GEMV_KERNELS(1), GEMV_KERNELS(2), GEMV_KERNELS(4), GEMV_KERNELS(8)};
+#undef GEMV_KERNELS
+    BRASA_TRY(launch(kernels[best == 1 ? 0 : (best == 2 ? 1 : (best == 4 ? 2 : 3))][form]));
     return brasa_post_launch(cmd, "linear_gemv");
 }
 

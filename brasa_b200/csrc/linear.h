@@ -37,9 +37,9 @@ struct LinearProblem {
 int32_t brasa_linear_launch(brasa_cmd *cmd, const LinearProblem *p, uint32_t n, bool x_f32);
 
 // One token (vectors in f32; y f32): the weights stream once through all SMs. The input of every problem is a slice of the
-// block's input vector, which the kernel forms itself. Either from the residual stream x: plus y / rms(y) * wy where y is
-// given (a sublayer's normed result; the sum also goes to x_out, which must not be x), then one or two affine forms of its
-// layer norm, its RMS norm times w[0], or as it is. Or from up to two vectors one behind the other, each as it is, in equal
+// block's input vector, which the kernel forms itself. Either from the residual stream x: one or two affine forms of its layer
+// norm; or x plus y / rms(y) * wy where y is given (a sublayer's normed result; the sum also goes to x_out, which must not be
+// x), as the RMS norm times w[0] or as it is. Or from up to two vectors one behind the other, each as it is, in equal
 // parts over their root mean squares, or silu(gate) * up out of alternating blocks of 32. The kernel is a programmatic
 // dependent of the kernel before it.
 enum GemvNorm { GEMV_LAYER_NORM, GEMV_RMS_NORM, GEMV_PLAIN };

@@ -224,6 +224,20 @@ def test_prompts_portions_and_decoding(ctx, folders, name, dtype):
     m.free()
 
 
+@pytest.mark.parametrize("width", [4100, 6004])
+def test_wide_stream(ctx, tmp_path, width):
+    """A residual stream wider than the single-token product keeps in registers, and than a norm's block does."""
+    cfg = config(width, 40, [(parallel(attn(2, 1, 16, 8, 9, 8), ssm(2, 8, 16, 1, 2, 3)), 24), (delta(1, 1, 8, 8, 2), None)])
+    w = G.random_weights(cfg, 0)
+    D.write_model(tmp_path, cfg, w)
+    ids = tokens(cfg, 24)
+    for dtype in DTYPES:
+        m = load(ctx, tmp_path, dtype, ctx_len=32, max_tokens=32, rows=32)
+        for sizes in ([24], [1], [10, 1, 1]):
+            assert agree(portions(m, ids, sizes), cfg, w, ids, dtype), (dtype, sizes)
+        m.free()
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("name", ["ragged", "ones"])
 def test_first_tokens(ctx, folders, name, dtype):
